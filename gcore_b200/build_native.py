@@ -32,6 +32,13 @@ NVCC_FLAGS = [
     "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=hidden",
     "--expt-relaxed-constexpr",
 ]
+# sources of models that promise 32-bit arithmetic where they say so: compiled without the approximate math functions
+EXACT_MATH = {"matrix_memory", "matrix_memory_chunk", "sandwich_norm", "window_attention", "window_prefill"}
+# sources one served architecture needs: ``ensure_kernels`` builds only these when the full library is not there
+KERNEL_SETS = {
+    "nafitar": ("comm", "elementwise", "gemm_skinny", "gemm_tcgen05", "gemm_wide", "matrix_memory", "matrix_memory_chunk",
+                "sample_filtered", "sandwich_norm", "vocab", "window_attention", "window_prefill"),
+}
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-Wall", "-pthread"]
 
 
@@ -61,13 +68,31 @@ def _run(cmd, verbose):
     return r
 
 
-def build_kernels(force=False, verbose=False, ptxas_info=False) -> Path:
-    srcs = sorted(OPS_SRC.glob("*.cu"))
-    hdrs = sorted(list(OPS_SRC.glob("*.cuh")) + list(OPS_SRC.glob("*.h")))
-    stamp = BUILD / "kernels.sha"
+def _stamp(lib: Path) -> Path:
+    return lib.with_suffix(".stamp")   # beside the library, so that a copied tree keeps both
+
+
+def _fresh(lib: Path, digest: str) -> bool:
+    st = _stamp(lib)
+    return lib.exists() and st.exists() and st.read_text() == digest
+
+
+def _headers():
+    return sorted(list(OPS_SRC.glob("*.cuh")) + list(OPS_SRC.glob("*.h")))
+
+
+def _set_sources(name):
+    return [OPS_SRC / f"{stem}.cu" for stem in KERNEL_SETS[name] if (OPS_SRC / f"{stem}.cu").exists()]
+
+
+def build_kernels(force=False, verbose=False, ptxas_info=False, only=None) -> Path:
+    """The kernel library of all sources, or with ``only`` (a key of ``KERNEL_SETS``) the library of that set."""
+    srcs = _set_sources(only) if only else sorted(OPS_SRC.glob("*.cu"))
+    target = KERNEL_LIB.with_name(f"_gk_kernels_{only}.so") if only else KERNEL_LIB
+    hdrs = _headers()
     dig = _digest(srcs + hdrs)
-    if not force and KERNEL_LIB.exists() and stamp.exists() and stamp.read_text() == dig:
-        return KERNEL_LIB
+    if not force and _fresh(target, dig):
+        return target
     BUILD.mkdir(exist_ok=True)
     nvcc = _nvcc()
     hdr_dig = _digest(hdrs)
@@ -75,10 +100,10 @@ def build_kernels(force=False, verbose=False, ptxas_info=False) -> Path:
     def compile_one(src: Path) -> Path:
         obj = BUILD / (src.stem + ".o")
         ostamp = BUILD / (src.stem + ".sha")
-        d = hashlib.sha256(src.read_bytes() + hdr_dig.encode()).hexdigest()
+        flags = [f for f in NVCC_FLAGS if not (f == "--use_fast_math" and src.stem in EXACT_MATH)]
+        d = hashlib.sha256(src.read_bytes() + hdr_dig.encode() + " ".join(flags).encode()).hexdigest()
         if not force and obj.exists() and ostamp.exists() and ostamp.read_text() == d:
             return obj
-        flags = list(NVCC_FLAGS)
         if ptxas_info:
             flags += ["-Xptxas", "-v"]
         r = _run([nvcc, *flags, "-I", OPS_SRC, "-c", src, "-o", obj], verbose)
@@ -89,23 +114,42 @@ def build_kernels(force=False, verbose=False, ptxas_info=False) -> Path:
 
     with ThreadPoolExecutor(max_workers=min(8, os.cpu_count() or 2)) as ex:
         objs = list(ex.map(compile_one, srcs))
-    _run([nvcc, "-shared", "-o", KERNEL_LIB, *objs, "-lcudart"], verbose)
-    stamp.write_text(dig)
-    return KERNEL_LIB
+    _link([nvcc, "-shared"], objs, ["-lcudart"], target, dig, verbose)
+    return target
+
+
+def _link(cmd, inputs, libs, target: Path, digest: str, verbose):
+    """Links beside the target and moves into place, so that an interrupted build leaves no half-written library."""
+    part = target.with_name(f".{target.stem}.{os.getpid()}.part")
+    _run([*cmd, "-o", part, *inputs, *libs], verbose)
+    os.replace(part, target)
+    _stamp(target).write_text(digest)
 
 
 def build_runtime(force=False, verbose=False) -> Path:
     srcs = sorted(RT_SRC.glob("*.cpp"))
     hdrs = sorted(RT_SRC.glob("*.h"))
-    stamp = BUILD / "runtime.sha"
     dig = _digest(srcs + hdrs)
-    if not force and RUNTIME_LIB.exists() and stamp.exists() and stamp.read_text() == dig:
+    if not force and _fresh(RUNTIME_LIB, dig):
         return RUNTIME_LIB
     BUILD.mkdir(exist_ok=True)
     cxx = os.environ.get("CXX", "g++")
-    _run([cxx, *CXX_FLAGS, "-shared", "-o", RUNTIME_LIB, *srcs], verbose)
-    stamp.write_text(dig)
+    _link([cxx, *CXX_FLAGS, "-shared"], srcs, [], RUNTIME_LIB, dig, verbose)
     return RUNTIME_LIB
+
+
+def ensure_kernels(name: str) -> Path:
+    """Kernel library that serves architecture ``name``: the full one when it is up to date, else the library of the
+    architecture's own set, built now if need be.  Also brings the host runtime up to date.  Safe to call from several
+    processes of one checkout."""
+    import fcntl
+    BUILD.mkdir(exist_ok=True)
+    with open(BUILD / ".lock", "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        build_runtime()
+        if _fresh(KERNEL_LIB, _digest(sorted(OPS_SRC.glob("*.cu")) + _headers())):
+            return KERNEL_LIB
+        return build_kernels(only=name)
 
 
 def build_all(force=False, verbose=False, ptxas_info=False):

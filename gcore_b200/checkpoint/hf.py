@@ -130,6 +130,29 @@ def read_hf_dir(path: str) -> Dict[str, torch.Tensor]:
     return out
 
 
+def read_model_config(path: str):
+    """``ModelConfig`` of a checkpoint folder (its ``config.json``), or None without one."""
+    from ..models.config import from_hf_config
+    file = os.path.join(path, "config.json")
+    if not os.path.isfile(file):
+        return None
+    with open(file) as fh:
+        return from_hf_config(json.load(fh))
+
+
+def load_serving_model(path: str, device, dtype: Optional[str] = None):
+    """Model of a checkpoint folder as the rollout engine serves it, without a training engine around it: decoders that
+    are described by a layer plan.  Returns ``(ModelConfig, module)``."""
+    from dataclasses import replace
+    from ..models.plan_decoder import PlanDecoder
+    cfg = read_model_config(path)
+    if cfg is None or cfg.layer_plan is None:
+        raise ValueError(f"{path} does not hold a model that is served without a training engine")
+    if dtype is not None:
+        cfg = replace(cfg, dtype=dtype)
+    return cfg, PlanDecoder(cfg, device).load_tensors(read_hf_dir(path))
+
+
 def load_hf(engine, path: str):
     """Loads full HF weights into this rank's shards and refreshes the optimizer's master copy."""
     tensors = read_hf_dir(path)

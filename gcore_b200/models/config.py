@@ -6,6 +6,8 @@ from __future__ import annotations
 from dataclasses import dataclass, field, fields
 from typing import Tuple, Any, Dict, List, Optional
 
+from .layer_plan import LayerPlan, nafitar_plan
+
 
 @dataclass
 class ModelConfig:
@@ -66,6 +68,9 @@ class ModelConfig:
     mtp_num_layers: int = 0
     mtp_loss_scaling_factor: float = 0.1
     fp8_base_weights: bool = False  # frozen e4m3 base with 128x128 block scales
+    # decoders described layer by layer (mixers side by side, looped layers, norms before and after each sublayer,
+    # learned positions); None for the uniform families above.  Such models are served, not trained.
+    layer_plan: Optional[LayerPlan] = None
 
     def __post_init__(self):
         if self.head_dim is None:
@@ -106,6 +111,8 @@ class ModelConfig:
 
     def num_parameters(self, include_embedding=True) -> int:
         h, L = self.hidden_size, self.num_layers
+        if self.layer_plan is not None:
+            return self._plan_parameters(include_embedding)
         if self.use_mla:
             attn = (h * self.q_lora_rank + self.q_lora_rank * self.num_attention_heads * self.qk_head_dim
                     if self.q_lora_rank else h * self.num_attention_heads * self.qk_head_dim)
@@ -128,6 +135,17 @@ class ModelConfig:
             total += self.vocab_size * h * (1 if self.tie_word_embeddings else 2)
         return total
 
+    def _plan_parameters(self, include_embedding: bool) -> int:
+        h, total = self.hidden_size, self.hidden_size * (1 + self.layer_plan.loop_times)
+        for sp in self.layer_plan.layers:
+            a, m = sp.attention, sp.memory
+            total += (2 * a.heads + a.kv_heads) * a.dim * h + (a.heads + a.kv_heads) * a.dim
+            total += m.heads * (2 * m.dim + 3 * m.vdim + 2) * h + m.heads * (m.vdim + 2)
+            total += (4 if not sp.ffn else 6) * h + 3 * sp.ffn * h
+        if include_embedding:
+            total += (2 * self.vocab_size + self.max_position_embeddings) * h
+        return total
+
     def active_parameters(self) -> int:
         if not self.is_moe:
             return self.num_parameters()
@@ -144,7 +162,7 @@ class ModelConfig:
 
 
 MODEL_ARCH = ("llama", "llama4", "qwen2", "qwen2_5_vl", "qwen3", "qwen3_moe", "qwen3_vl", "qwen3_vl_moe", "qwen2_moe",
-              "qwen2_vl", "deepseek_v3", "mistral", "gemma3_text", "seed_oss", "gpt_oss")
+              "qwen2_vl", "deepseek_v3", "mistral", "gemma3_text", "seed_oss", "gpt_oss", "nafitar")
 
 PRESETS: Dict[str, Dict[str, Any]] = {
     # tiny Llama-style decoder
@@ -178,8 +196,30 @@ def get_preset(name: str, **overrides) -> ModelConfig:
     return ModelConfig(**d)
 
 
+def from_nafitar_config(conf: Dict[str, Any], dtype: str = "bfloat16") -> ModelConfig:
+    """Maps a Nafitar ``config.json`` (``architecture``, ``layers``, ``loop``, ``norm``, ``vocab``, ``width``,
+    ``max_positions``)."""
+    plan = nafitar_plan(conf)
+    a = plan.layers[0].attention
+    return ModelConfig(arch="nafitar", num_layers=len(plan.layers), hidden_size=conf["width"],
+                       num_attention_heads=a.heads, num_kv_heads=a.kv_heads, head_dim=a.dim,
+                       ffn_hidden_size=plan.layers[0].ffn, vocab_size=conf["vocab"],
+                       rms_norm_eps=float(conf["norm"]["eps"]), max_position_embeddings=conf["max_positions"],
+                       qkv_bias=True, dtype=dtype, layer_plan=plan)
+
+
+# architectures whose config.json names them in ``architecture``: reader of that file
+ARCH_READERS = {"nafitar": from_nafitar_config}
+
+
 def from_hf_config(hf: Dict[str, Any]) -> ModelConfig:
-    """Maps a HuggingFace config dict (llama / qwen2 / qwen3 / qwen3_moe / deepseek_v3 / mistral / gpt_oss)."""
+    """Maps a checkpoint's config dict: HuggingFace keys (llama / qwen2 / qwen3 / qwen3_moe / deepseek_v3 / mistral /
+    gpt_oss) or, when the file names its ``architecture``, the reader registered for it."""
+    if "architecture" in hf:
+        reader = ARCH_READERS.get(str(hf["architecture"]).lower())
+        if reader is None:
+            raise ValueError(f"unknown architecture {hf['architecture']!r} (known: {sorted(ARCH_READERS)})")
+        return reader(hf)
     mt = hf.get("model_type", "llama")
     kw: Dict[str, Any] = dict(
         arch={"qwen2": "qwen2", "qwen3": "qwen3", "qwen3_moe": "qwen3_moe", "deepseek_v3": "deepseek_v3",

@@ -42,10 +42,21 @@ def use_native(t: torch.Tensor | None = None) -> bool:
     return True
 
 
+_LIBRARY = "_gk_kernels.so"
+
+
+def use_library(path):
+    """Selects the kernel library ``kernels()`` loads (one built for a single architecture's kernels, say); before the
+    first kernel call."""
+    global _LIBRARY
+    assert _KERNELS is None or _LIBRARY == Path(path).name, "a kernel library is loaded already"
+    _LIBRARY = Path(path).name
+
+
 def kernels() -> ctypes.CDLL:
     global _KERNELS
     if _KERNELS is None:
-        path = _HERE / "_gk_kernels.so"
+        path = _HERE / _LIBRARY
         if not path.exists():
             raise RuntimeError(
                 f"{path} is missing: run `python -m gcore_b200.build_native` (the GPU path does not fall back "
@@ -202,6 +213,16 @@ def _declare_kernels(lib: ctypes.CDLL):
     d("gk_mla_decode_scratch", [I, I, I, I, ctypes.POINTER(L)], None)
     d("gk_mla_decode_supported", [I, I])
     d("gk_mla_set_target_ctas", [I], None)
+    d("gk_sandwich_norm", [I, I, P, P, F, P])
+    d("gk_swiglu_f32", [P, P, L, I, P])
+    d("gk_append_keys", [P, L, L, I, P, P, I, P])
+    d("gk_window_attn", [I, P, L, P, P, P, P, P, P, P, P, F, P])
+    d("gk_shared_kv_decode", [P, L, P, P, P, P, P, P, P, P, F, P])
+    d("gk_shared_kv_decode_scratch", [I, I, I, I], L)
+    d("gk_shared_decode_set_target_ctas", [I], None)
+    d("gk_window_prefill", [P, L, P, P, P, P, P, P, P, F, P, P])
+    d("gk_matrix_memory_scan", [I, P, L, P, F, F, P])
+    d("gk_memory_output", [I, P, P, L, P, P, P, F, P])
     d("gk_attn_fwd", [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, I, P, P])
     d("gk_attn_bwd", [P, P, P, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, I, P, P])
     d("gk_attn_bwd_dv", [P, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, I, P, P])

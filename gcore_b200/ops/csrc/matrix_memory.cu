@@ -1,0 +1,278 @@
+// Matrix memory (mLSTM): per head S_t = e^(f + m - m') S + e^(i - m') k v^T, n likewise with k alone, running maximum
+// m' = max(f + m, i), output S^T q / (max(|n . q|, e^-m') + 1e-6).  All of it is 32-bit; q, k, v arrive in the storage
+// type of the projection.
+//   * matrix_memory_scan_kernel  token by token with the state slice in registers: decoding (one token per request, the
+//                                gate projections fused in) and the true 32-bit path for prompt portions;
+//   * memory_output_kernel       per-head RMS norm, gain and sigmoid output gate.
+// bf16 prompt portions run the chunkwise kernel in matrix_memory_chunk.cu.
+//
+// State layout per layer run: S [slots, heads, dim, vdim], n [slots, heads, slices, dim], m [slots, heads, slices]: a head's
+// value columns are cut into slices of 64 that different CTAs own, and each keeps its own copy of n and m, so no CTA
+// reads what another one writes.
+#include "host_utils.h"
+#include <cuda_bf16.h>
+#include <type_traits>
+
+namespace gk {
+
+constexpr int MM_SLICE = 64;
+constexpr int MM_THREADS = 256;
+
+__device__ __forceinline__ float mm_f(float v) { return v; }
+__device__ __forceinline__ float mm_f(__nv_bfloat16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ float4 mm_ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 mm_ld4(const __nv_bfloat16* p) {
+  const uint2 r = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void mm_st4(float* p, float a, float b, float c, float d) {
+  *reinterpret_cast<float4*>(p) = make_float4(a, b, c, d);
+}
+__device__ __forceinline__ void mm_st4(__nv_bfloat16* p, float a, float b, float c, float d) {
+  __nv_bfloat162 x = __floats2bfloat162_rn(a, b), y = __floats2bfloat162_rn(c, d);
+  uint2 r;
+  r.x = *reinterpret_cast<uint32_t*>(&x);
+  r.y = *reinterpret_cast<uint32_t*>(&y);
+  *reinterpret_cast<uint2*>(p) = r;
+}
+__device__ __forceinline__ float mm_logsigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
+
+template <typename T>
+struct ScanParams {
+  const T* proj;           // packed projection rows
+  long long ld;
+  int q_off, k_off, v_off;
+  const T* h;              // [rows, width] mixer input, with gate_w: the gate projections are computed here
+  const T* gate_w;         // [2 * heads, width]: input gates, then forget gates
+  const float* gates;      // or: [rows, 2 * heads] projected gates without bias
+  const float* gate_b;     // [2 * heads]
+  const int* cu;           // [n + 1] first row of every segment, or null: one row per segment
+  const int* first_pos;    // position of every segment's first token (0: the state starts at zero)
+  const int* slots;        // state slot per segment; negative: inactive (zero output, no state touched)
+  float* S;
+  float* n;
+  float* m;
+  float* out;              // [rows, heads, vdim] 32-bit
+  int width, heads, dim, vdim, slices;
+  float cap, q_scale;
+};
+
+// grid (heads * slices, segments).  Thread (warp w, lane): rows rg, rg + 16, ... with rg = 2 w + lane / 16; columns
+// 4 * (lane % 16) .. + 3 of the slice.  R = rows per thread.
+template <typename T, int R>
+__global__ void __launch_bounds__(MM_THREADS) matrix_memory_scan_kernel(const ScanParams<T> p) {
+  __shared__ float sq[2][16 * R], sk[2][16 * R];
+  __shared__ float red[2][8][MM_SLICE + 4];
+  __shared__ float gred[2][8];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int head = blockIdx.x / p.slices, slice = blockIdx.x % p.slices, seg = blockIdx.y;
+  const int r_beg = p.cu ? p.cu[seg] : seg, r_end = p.cu ? p.cu[seg + 1] : seg + 1;
+  const int slot = p.slots[seg];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int rg = warp * 2 + (lane >> 4), c0 = (lane & 15) * 4;
+  const int col = slice * MM_SLICE + c0;                 // vdim is a multiple of 4
+  const bool live = col < p.vdim;
+  if (slot < 0) {
+    for (int r = r_beg; r < r_end; ++r)
+      if (tid < MM_SLICE && slice * MM_SLICE + tid < p.vdim)
+        p.out[(static_cast<long long>(r) * p.heads + head) * p.vdim + slice * MM_SLICE + tid] = 0.f;
+    return;
+  }
+  const long long sh = static_cast<long long>(slot) * p.heads + head;
+  float* Sg = p.S + sh * p.dim * p.vdim + col;
+  float* ng = p.n + (sh * p.slices + slice) * p.dim;
+  float* mg = p.m + sh * p.slices + slice;
+  const bool fresh = p.first_pos[seg] == 0;
+  float4 S[R];
+  float n[R];
+  float m = fresh ? 0.f : *mg;
+#pragma unroll
+  for (int j = 0; j < R; ++j) {
+    const int r = rg + 16 * j;
+    S[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+    n[j] = 0.f;
+    if (!fresh && r < p.dim) {
+      if (live) S[j] = *reinterpret_cast<const float4*>(Sg + static_cast<long long>(r) * p.vdim);
+      n[j] = ng[r];
+    }
+  }
+  const float bi = p.gate_b[head], bf = p.gate_b[p.heads + head];
+  for (int row = r_beg, it = 0; row < r_end; ++row, ++it) {
+    const int buf = it & 1;
+    const T* pr = p.proj + row * p.ld;
+    for (int d = tid; d < 16 * R; d += MM_THREADS) {
+      sq[buf][d] = d < p.dim ? mm_f(pr[p.q_off + static_cast<long long>(head) * p.dim + d]) * p.q_scale : 0.f;
+      sk[buf][d] = d < p.dim ? mm_f(pr[p.k_off + static_cast<long long>(head) * p.dim + d]) : 0.f;
+    }
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (live) v = mm_ld4(pr + p.v_off + static_cast<long long>(head) * p.vdim + col);
+    float gi, gf;
+    if (p.gates) {
+      gi = p.gates[static_cast<long long>(row) * 2 * p.heads + head];
+      gf = p.gates[static_cast<long long>(row) * 2 * p.heads + p.heads + head];
+    } else {
+      const T* hr = p.h + static_cast<long long>(row) * p.width;
+      const T* wi = p.gate_w + static_cast<long long>(head) * p.width;
+      const T* wf = p.gate_w + static_cast<long long>(p.heads + head) * p.width;
+      float a = 0.f, b = 0.f;
+      for (int d = tid * 4; d < p.width; d += MM_THREADS * 4) {
+        const float4 x = mm_ld4(hr + d), u = mm_ld4(wi + d), w = mm_ld4(wf + d);
+        a += x.x * u.x + x.y * u.y + x.z * u.z + x.w * u.w;
+        b += x.x * w.x + x.y * w.y + x.z * w.z + x.w * w.w;
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        a += __shfl_xor_sync(0xffffffff, a, o);
+        b += __shfl_xor_sync(0xffffffff, b, o);
+      }
+      if (lane == 0) { gred[0][warp] = a; gred[1][warp] = b; }
+      __syncthreads();
+      gi = gf = 0.f;
+#pragma unroll
+      for (int w = 0; w < 8; ++w) { gi += gred[0][w]; gf += gred[1][w]; }
+    }
+    __syncthreads();
+    gi = p.cap * tanhf((gi + bi) / p.cap);
+    gf = mm_logsigmoid(p.cap * tanhf((gf + bf) / p.cap));
+    const float mn = fmaxf(gf + m, gi);
+    const float keep = expf(gf + m - mn), put = expf(gi - mn);
+    m = mn;
+    float a0 = 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f, nq = 0.f;
+#pragma unroll
+    for (int j = 0; j < R; ++j) {
+      const float q = sq[buf][rg + 16 * j], k = sk[buf][rg + 16 * j] * put;
+      n[j] = keep * n[j] + k;
+      nq += n[j] * q;
+      S[j].x = keep * S[j].x + k * v.x; a0 += S[j].x * q;
+      S[j].y = keep * S[j].y + k * v.y; a1 += S[j].y * q;
+      S[j].z = keep * S[j].z + k * v.z; a2 += S[j].z * q;
+      S[j].w = keep * S[j].w + k * v.w; a3 += S[j].w * q;
+    }
+    a0 += __shfl_xor_sync(0xffffffff, a0, 16);
+    a1 += __shfl_xor_sync(0xffffffff, a1, 16);
+    a2 += __shfl_xor_sync(0xffffffff, a2, 16);
+    a3 += __shfl_xor_sync(0xffffffff, a3, 16);
+    nq += __shfl_xor_sync(0xffffffff, nq, 16);
+    if (lane < 16) {
+      *reinterpret_cast<float4*>(&red[buf][warp][c0]) = make_float4(a0, a1, a2, a3);
+      if (lane == 0) red[buf][warp][MM_SLICE] = nq;
+    }
+    __syncthreads();
+    if (tid < MM_SLICE && slice * MM_SLICE + tid < p.vdim) {
+      float o = 0.f, d = 0.f;
+#pragma unroll
+      for (int w = 0; w < 8; ++w) { o += red[buf][w][tid]; d += red[buf][w][MM_SLICE]; }
+      p.out[(static_cast<long long>(row) * p.heads + head) * p.vdim + slice * MM_SLICE + tid] =
+          o / (fmaxf(fabsf(d), expf(-m)) + 1e-6f);
+    }
+  }
+  if (r_end > r_beg) {
+#pragma unroll
+    for (int j = 0; j < R; ++j) {
+      const int r = rg + 16 * j;
+      if (r < p.dim) {
+        if (live) *reinterpret_cast<float4*>(Sg + static_cast<long long>(r) * p.vdim) = S[j];
+        if (c0 == 0) ng[r] = n[j];
+      }
+    }
+    if (tid == 0) *mg = m;
+  }
+}
+
+// y = o / rms(o over the head's true size) * gain * sigmoid(g).  One warp per (row, head).
+template <typename T>
+__global__ void __launch_bounds__(256) memory_output_kernel(const float* __restrict__ o, const T* __restrict__ proj,
+                                                            long long ld, int g_off, const float* __restrict__ gain,
+                                                            T* __restrict__ y, int rows, int heads, int vdim,
+                                                            int vdim_true, float eps) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long long item = static_cast<long long>(blockIdx.x) * 8 + warp;
+  if (item >= static_cast<long long>(rows) * heads) return;
+  const long long row = item / heads;
+  const int head = static_cast<int>(item - row * heads);
+  const float* src = o + item * vdim;
+  float ss = 0.f;
+  for (int c = lane * 4; c < vdim; c += 128) {
+    const float4 v = *reinterpret_cast<const float4*>(src + c);
+    ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+  }
+#pragma unroll
+  for (int s = 16; s > 0; s >>= 1) ss += __shfl_xor_sync(0xffffffff, ss, s);
+  const float r = 1.f / sqrtf(ss / vdim_true + eps);
+  for (int c = lane * 4; c < vdim; c += 128) {
+    const float4 v = *reinterpret_cast<const float4*>(src + c);
+    const float4 w = *reinterpret_cast<const float4*>(gain + head * vdim + c);
+    const float4 g = mm_ld4(proj + row * ld + g_off + static_cast<long long>(head) * vdim + c);
+    mm_st4(y + item * vdim + c, v.x * r * w.x / (1.f + expf(-g.x)), v.y * r * w.y / (1.f + expf(-g.y)),
+           v.z * r * w.z / (1.f + expf(-g.z)), v.w * r * w.w / (1.f + expf(-g.w)));
+  }
+}
+
+template <typename T>
+int launch_scan(const ScanParams<T>& p, int segments, cudaStream_t st) {
+  const dim3 grid(p.heads * p.slices, segments);
+  if (p.dim <= 32) launch_k(matrix_memory_scan_kernel<T, 2>, grid, dim3(MM_THREADS), 0, st, p);
+  else if (p.dim <= 64) launch_k(matrix_memory_scan_kernel<T, 4>, grid, dim3(MM_THREADS), 0, st, p);
+  else if (p.dim <= 128) launch_k(matrix_memory_scan_kernel<T, 8>, grid, dim3(MM_THREADS), 0, st, p);
+  else if (p.dim <= 256) launch_k(matrix_memory_scan_kernel<T, 16>, grid, dim3(MM_THREADS), 0, st, p);
+  else if (p.dim <= 512) launch_k(matrix_memory_scan_kernel<T, 32>, grid, dim3(MM_THREADS), 0, st, p);
+  else return -2;
+  return launch_status();
+}
+
+}  // namespace gk
+
+using namespace gk;
+
+// ptrs: {proj, h, gate_w, gates, gate_b, cu, first_pos, slots, S, n, m, out}
+// dims: {segments, q_off, k_off, v_off, width, heads, dim, vdim}
+GK_EXPORT int gk_matrix_memory_scan(int is_fp32, void* const* ptrs, long long ld, const int* dims, float cap,
+                                    float q_scale, void* stream) {
+  if (dims[0] == 0) return 0;
+  if (dims[7] % 4 || ld % 4 || dims[3] % 4 || (!ptrs[3] && dims[4] % 4)) return -1;
+  auto fill = [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    ScanParams<T> p;
+    p.proj = static_cast<const T*>(ptrs[0]);
+    p.ld = ld;
+    p.h = static_cast<const T*>(ptrs[1]);
+    p.gate_w = static_cast<const T*>(ptrs[2]);
+    p.gates = static_cast<const float*>(ptrs[3]);
+    p.gate_b = static_cast<const float*>(ptrs[4]);
+    p.cu = static_cast<const int*>(ptrs[5]);
+    p.first_pos = static_cast<const int*>(ptrs[6]);
+    p.slots = static_cast<const int*>(ptrs[7]);
+    p.S = static_cast<float*>(ptrs[8]);
+    p.n = static_cast<float*>(ptrs[9]);
+    p.m = static_cast<float*>(ptrs[10]);
+    p.out = static_cast<float*>(ptrs[11]);
+    p.q_off = dims[1]; p.k_off = dims[2]; p.v_off = dims[3];
+    p.width = dims[4]; p.heads = dims[5]; p.dim = dims[6]; p.vdim = dims[7];
+    p.slices = (p.vdim + MM_SLICE - 1) / MM_SLICE;
+    p.cap = cap; p.q_scale = q_scale;
+    return launch_scan<T>(p, dims[0], reinterpret_cast<cudaStream_t>(stream));
+  };
+  return is_fp32 ? fill(static_cast<float*>(nullptr)) : fill(static_cast<__nv_bfloat16*>(nullptr));
+}
+
+// dims: {rows, heads, vdim, vdim_true, g_off}
+GK_EXPORT int gk_memory_output(int is_fp32, const float* o, const void* proj, long long ld, const float* gain, void* y,
+                               const int* dims, float eps, void* stream) {
+  const long long items = static_cast<long long>(dims[0]) * dims[1];
+  if (items == 0) return 0;
+  if (dims[2] % 4 || ld % 4 || dims[4] % 4) return -1;
+  const dim3 grid(static_cast<unsigned>((items + 7) / 8));
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  if (is_fp32)
+    launch_k(memory_output_kernel<float>, grid, dim3(256), 0, st, o, static_cast<const float*>(proj), ld, dims[4], gain,
+             static_cast<float*>(y), dims[0], dims[1], dims[2], dims[3], eps);
+  else
+    launch_k(memory_output_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, o, static_cast<const __nv_bfloat16*>(proj), ld,
+             dims[4], gain, static_cast<__nv_bfloat16*>(y), dims[0], dims[1], dims[2], dims[3], eps);
+  return launch_status();
+}

@@ -20,6 +20,7 @@ import torch
 from . import _lib
 
 _SCRATCH: dict = {}
+_RETIRED: list = []   # outgrown scratch buffers: captured graphs may still hold their addresses
 LAUNCHES = {"gemm": 0}
 
 
@@ -27,8 +28,10 @@ def _scratch(device, ws_floats: int, counters: int):
     key = (device.index,)
     ws, cnt = _SCRATCH.get(key, (None, None))
     if ws is None or ws.numel() < ws_floats:
+        _RETIRED.append(ws)
         ws = torch.empty(max(ws_floats, 1 << 20), dtype=torch.float32, device=device)
     if cnt is None or cnt.numel() < counters:
+        _RETIRED.append(cnt)
         cnt = torch.zeros(max(counters, 4096), dtype=torch.int32, device=device)
     _SCRATCH[key] = (ws, cnt)
     return ws, cnt
@@ -269,12 +272,25 @@ def _skinny_plan(T: int, tiles: int, kb: int, K: int):
     return plan
 
 
+def _linear_f32(x, w, bias, out):
+    """32-bit models: the library's true fp32 product (never TF32)."""
+    tf32 = torch.backends.cuda.matmul.allow_tf32
+    torch.backends.cuda.matmul.allow_tf32 = False
+    try:
+        y = torch.matmul(x, w.t(), out=out)
+    finally:
+        torch.backends.cuda.matmul.allow_tf32 = tf32
+    return y if bias is None else y.add_(bias)
+
+
 def linear_forward(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None,
                    out: torch.Tensor | None = None, out_dtype=None) -> torch.Tensor:
     """``y[T,N] = x[T,K] @ w[N,K]^T + bias``.  Few tokens (decode) run swap-AB + split-K so the weight streams
     from HBM exactly once with every SM busy."""
     T, K = x.shape
     N = w.shape[0]
+    if x.is_cuda and x.dtype == torch.float32:
+        return _linear_f32(x, w, bias, out)
     if _lib.use_native(x) and T <= 128 and N >= 256:
         bn = 32 if T <= 32 else (64 if T <= 64 else 128)
         tiles = (N + 127) // 128

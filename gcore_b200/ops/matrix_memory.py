@@ -1,0 +1,121 @@
+"""Recurrent matrix memory (mLSTM) over the rows of a serving step (``csrc/matrix_memory.cu``,
+``csrc/matrix_memory_chunk.cu``).  CPU tensors run the plain PyTorch definition."""
+from __future__ import annotations
+
+import ctypes
+from dataclasses import dataclass
+
+import torch
+
+from . import _lib
+from .gemm import linear_forward
+from .rows import StepRows
+
+LAUNCHES = {"matrix_memory": 0}
+SLICE = 64        # value columns per state slice (csrc/matrix_memory.cu: MM_SLICE)
+MAX_KEY_DIM = 512
+
+
+def padded_key_dim(dim: int) -> int:
+    if dim > MAX_KEY_DIM:
+        raise ValueError(f"matrix-memory keys of {dim} are not supported (at most {MAX_KEY_DIM})")
+    return (dim + 15) // 16 * 16
+
+
+def padded_value_dim(vdim: int) -> int:
+    return (vdim + 15) // 16 * 16
+
+
+@dataclass
+class MemoryState:
+    """State of one layer run for every request slot; a request's first token finds it as zeros whatever it holds."""
+    S: torch.Tensor   # [slots, heads, dim, vdim]
+    n: torch.Tensor   # [slots, heads, slices, dim]
+    m: torch.Tensor   # [slots, heads, slices]
+
+    @classmethod
+    def allocate(cls, slots, heads, dim, vdim, device):
+        ns = (vdim + SLICE - 1) // SLICE
+        z = dict(dtype=torch.float32, device=device)
+        return cls(torch.zeros(slots, heads, dim, vdim, **z), torch.zeros(slots, heads, ns, dim, **z),
+                   torch.zeros(slots, heads, ns, **z))
+
+    @staticmethod
+    def bytes_per_slot(heads, dim, vdim):
+        return 4 * heads * (dim * vdim + ((vdim + SLICE - 1) // SLICE) * (dim + 1))
+
+    def copy_slots(self, src, dst):
+        for t in (self.S, self.n, self.m):
+            t[dst] = t[src]
+
+
+def _ref(proj, offs, gates, gate_b, cap, q_scale, heads, dim, vdim, rows: StepRows, st: MemoryState):
+    q_off, k_off, v_off = offs
+    T = proj.shape[0]
+    out = torch.zeros(T, heads, vdim)
+    g = gates + gate_b
+    gi = cap * torch.tanh(g[:, :heads] / cap)
+    gf = torch.nn.functional.logsigmoid(cap * torch.tanh(g[:, heads:] / cap))
+    for t in range(T):
+        s, slot = int(rows.row_seq[t]), int(rows.states[rows.row_seq[t]])
+        if slot < 0:
+            continue
+        zero = int(rows.pos[t]) == 0
+        S, n, m = (torch.zeros_like(x) if zero else x for x in (st.S[slot], st.n[slot, :, 0], st.m[slot, :, 0]))
+        q = proj[t, q_off:q_off + heads * dim].view(heads, dim).float() * q_scale
+        k = proj[t, k_off:k_off + heads * dim].view(heads, dim).float()
+        v = proj[t, v_off:v_off + heads * vdim].view(heads, vdim).float()
+        mn = torch.maximum(gf[t] + m, gi[t])
+        keep, put = torch.exp(gf[t] + m - mn), torch.exp(gi[t] - mn)
+        S = keep[:, None, None] * S + put[:, None, None] * k[:, :, None] * v[:, None, :]
+        n = keep[:, None] * n + put[:, None] * k
+        den = torch.maximum((n * q).sum(-1).abs(), torch.exp(-mn)) + 1e-6
+        out[t] = torch.einsum("hdv,hd->hv", S, q) / den[:, None]
+        st.S[slot], st.n[slot], st.m[slot] = S, n[:, None].expand_as(st.n[slot]), mn[:, None].expand_as(st.m[slot])
+    return out
+
+
+def _scan(proj, offs, h, gate_w, gates, gate_b, cap, q_scale, heads, dim, vdim, cu, first_pos, slots, st, out):
+    ptrs = (ctypes.c_void_p * 12)(*[t.data_ptr() if t is not None else None for t in
+                                    (proj, h, gate_w, gates, gate_b, cu, first_pos, slots, st.S, st.n, st.m, out)])
+    dims = (ctypes.c_int * 8)(slots.numel(), *offs, h.shape[1] if h is not None else 0, heads, dim, vdim)
+    LAUNCHES["matrix_memory"] += 1
+    _lib.check(_lib.kernels().gk_matrix_memory_scan(int(proj.dtype == torch.float32), ptrs, proj.stride(0), dims,
+                                                    float(cap), float(q_scale), _lib.stream_ptr()), "matrix_memory_scan")
+
+
+def _output(o, proj, g_off, gain, vdim_true, eps):
+    T, heads, vdim = o.shape
+    if not o.is_cuda:
+        y = o * torch.rsqrt(o.pow(2).sum(-1, keepdim=True) / vdim_true + eps)
+        g = torch.sigmoid(proj[:, g_off:g_off + heads * vdim].float())
+        return (y.reshape(T, -1) * gain * g).to(proj.dtype)
+    y = torch.empty(T, heads * vdim, dtype=proj.dtype, device=proj.device)
+    dims = (ctypes.c_int * 5)(T, heads, vdim, vdim_true, g_off)
+    LAUNCHES["matrix_memory"] += 1
+    _lib.check(_lib.kernels().gk_memory_output(int(proj.dtype == torch.float32), _lib.ptr(o), _lib.ptr(proj),
+                                               proj.stride(0), _lib.ptr(gain), _lib.ptr(y), dims, float(eps),
+                                               _lib.stream_ptr()), "memory_output")
+    return y
+
+
+def matrix_memory(proj, q_off: int, k_off: int, v_off: int, g_off: int, h, gate_w, gate_b, cap: float, q_scale: float,
+                  heads: int, dim: int, vdim: int, vdim_true: int, rows: StepRows, state: MemoryState, gain, eps: float):
+    """Runs every row of the step through its request's memory and returns the gated, head-normed output
+    [T, heads * vdim].  ``proj``: packed projections; ``h`` [T, width]: the mixer's input, which the 32-bit gate
+    projections ``gate_w`` [2 * heads, width] read."""
+    T, P = proj.shape[0], rows.portion_rows
+    offs = (q_off, k_off, v_off)
+    if not proj.is_cuda:
+        gates = h.float() @ gate_w.float().t()
+        o = _ref(proj, offs, gates, gate_b, cap, q_scale, heads, dim, vdim, rows, state)
+        return _output(o, proj, g_off, gain, vdim_true, eps)
+    o = torch.empty(T, heads, vdim, dtype=torch.float32, device=proj.device)
+    n = rows.n_portions
+    common = (gate_b, cap, q_scale, heads, dim, vdim)
+    if P:
+        gates = linear_forward(h[:P], gate_w, out_dtype=torch.float32)
+        _scan(proj, offs, None, None, gates, *common, rows.cu, rows.first_pos, rows.states[:n], state, o)
+    if T > P:
+        _scan(proj[P:], offs, h[P:], gate_w, None, *common, None, rows.first_pos[n:], rows.states[n:], state, o[P:])
+    return _output(o, proj, g_off, gain, vdim_true, eps)

@@ -1,0 +1,109 @@
+"""Sliding-window attention with a linear distance penalty on a paged cache whose rows are key and value at once
+(``csrc/window_attention.cu``, ``csrc/window_prefill.cu``).  CPU tensors run the plain PyTorch definition."""
+from __future__ import annotations
+
+import ctypes
+from typing import Dict
+
+import torch
+
+from . import _lib
+from .rows import StepRows
+
+LAUNCHES = {"window_attention": 0}
+MAX_HEAD_DIM = 512
+_SCRATCH: Dict[tuple, torch.Tensor] = {}
+
+
+def padded_head_dim(dim: int) -> int:
+    """Head size the kernels store: the tensor-core kernels are built for 64 and 128, larger heads run the general
+    kernel (zero columns change neither scores nor outputs)."""
+    if dim > MAX_HEAD_DIM:
+        raise ValueError(f"attention heads of {dim} are not supported (at most {MAX_HEAD_DIM})")
+    return 64 if dim <= 64 else 128 if dim <= 128 else (dim + 7) // 8 * 8
+
+
+def _ref(proj, q_off, k_off, H, G, D, rows, cache, slopes, scale, window):
+    bs = cache.shape[1]
+    out = torch.zeros(proj.shape[0], H, D, dtype=proj.dtype)
+    flat = cache.view(-1, G, D)
+    live = rows.slots >= 0
+    flat[rows.slots[live].long()] = proj[live, k_off:k_off + G * D].view(-1, G, D)
+    for t in range(proj.shape[0]):
+        if rows.slots[t] < 0:
+            continue
+        i = int(rows.pos[t])
+        j = torch.arange(max(0, i - window + 1), i + 1)
+        slots = rows.tables[rows.row_seq[t], j // bs].long() * bs + j % bs
+        k = flat[slots].float().repeat_interleave(H // G, 1)                       # [n, H, D]
+        s = torch.einsum("hd,nhd->hn", proj[t, q_off:q_off + H * D].view(H, D).float(), k) * scale
+        p = torch.softmax(s - slopes[:, None] * (i - j).float()[None], -1)
+        out[t] = torch.einsum("hn,nhd->hd", p, k).to(proj.dtype)
+    return out.view(-1, H * D)
+
+
+def _decode_scratch(device, floats: int):
+    # one buffer per size class, never replaced: captured graphs keep the address
+    n = 1 << max(20, (floats - 1).bit_length())
+    buf = _SCRATCH.get((device.index, n))
+    if buf is None:
+        buf = _SCRATCH[device.index, n] = torch.empty(n, dtype=torch.float32, device=device)
+    return buf
+
+
+def append_keys(proj, k_off, n, slots, cache):
+    """Copies ``n`` key elements at column ``k_off`` of every row to its cache slot."""
+    es = proj.element_size()
+    LAUNCHES["window_attention"] += 1
+    _lib.check(_lib.kernels().gk_append_keys(_lib.ptr(proj), proj.stride(0) * es, k_off * es, n * es, _lib.ptr(slots),
+                                             _lib.ptr(cache), slots.numel(), _lib.stream_ptr()), "append_keys")
+
+
+def _general(q, q_ld, cache, rows: StepRows, lo, hi, slopes, out, H, G, D, window, scale):
+    dims = (ctypes.c_int * 7)(hi - lo, H, G, D, window, cache.shape[1], rows.tables.shape[1])
+    LAUNCHES["window_attention"] += 1
+    _lib.check(_lib.kernels().gk_window_attn(
+        int(q.dtype == torch.float32), _lib.ptr(q), q_ld, _lib.ptr(cache), _lib.ptr(rows.tables),
+        _lib.ptr(rows.row_seq[lo:hi]), _lib.ptr(rows.pos[lo:hi]), _lib.ptr(rows.slots[lo:hi]), _lib.ptr(slopes),
+        _lib.ptr(out), dims, float(scale), _lib.stream_ptr()), "window_attn")
+
+
+def window_attention(proj, q_off: int, k_off: int, heads: int, kv_heads: int, dim: int, rows: StepRows, cache, slopes,
+                     scale: float, window: int):
+    """``proj`` [T, ld]: packed projections with the queries at ``q_off`` and the keys at ``k_off``.  Stores the new keys
+    in ``cache`` [blocks, block_size, kv_heads, dim] and returns the attention output [T, heads * dim]."""
+    H, G, D = heads, kv_heads, dim
+    if not proj.is_cuda:
+        return _ref(proj, q_off, k_off, H, G, D, rows, cache, slopes, scale, window)
+    T, P, bs = proj.shape[0], rows.portion_rows, cache.shape[1]
+    out = torch.empty(T, H * D, dtype=proj.dtype, device=proj.device)
+    lib, bf16 = _lib.kernels(), proj.dtype == torch.bfloat16
+    tiled = bf16 and D in (64, 128)
+    if not tiled:
+        append_keys(proj, k_off, G * D, rows.slots, cache)
+        _general(proj[:, q_off:], proj.stride(0), cache, rows, 0, T, slopes, out, H, G, D, window, scale)
+        return out
+    if P:
+        append_keys(proj[:P], k_off, G * D, rows.slots[:P], cache)
+        if bs in (8, 16, 32) or bs % 64 == 0:
+            dims = (ctypes.c_int * 12)(rows.n_portions, P, H, G, D, window, bs, rows.tables.shape[1], rows.max_portion,
+                                       q_off, cache.shape[0], 0)
+            LAUNCHES["window_attention"] += 1
+            _lib.check(lib.gk_window_prefill(_lib.ptr(proj), proj.stride(0), _lib.ptr(cache), _lib.ptr(rows.tables),
+                                             _lib.ptr(rows.cu), _lib.ptr(rows.first_pos), _lib.ptr(slopes),
+                                             _lib.ptr(out), dims, float(scale), _lib.ptr(_lib.err_flag(proj.device)),
+                                             _lib.stream_ptr()), "window_prefill")
+        else:
+            _general(proj[:, q_off:], proj.stride(0), cache, rows, 0, P, slopes, out, H, G, D, window, scale)
+    if T > P:
+        B = T - P
+        ptab = rows.tables[rows.n_portions:]
+        span = min(window, rows.max_ctx)
+        scratch = _decode_scratch(proj.device, int(lib.gk_shared_kv_decode_scratch(B, H, D, span)))
+        dims = (ctypes.c_int * 10)(B, H, G, D, window, bs, rows.tables.shape[1], rows.max_ctx, q_off, k_off)
+        LAUNCHES["window_attention"] += 1
+        _lib.check(lib.gk_shared_kv_decode(_lib.ptr(proj[P:]), proj.stride(0), _lib.ptr(cache), _lib.ptr(ptab),
+                                           _lib.ptr(rows.ctx), _lib.ptr(rows.slots[P:]), _lib.ptr(slopes),
+                                           _lib.ptr(out[P:]), _lib.ptr(scratch), dims, float(scale),
+                                           _lib.stream_ptr()), "shared_kv_decode")
+    return out

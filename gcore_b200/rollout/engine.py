@@ -31,9 +31,11 @@ import torch.distributed as dist
 
 from ..core import parallel_state as ps
 from ..models.config import ModelConfig
+from ..models.plan_decoder import PlanDecoder
 from ..ops import _lib, fused
 from ..ops.attention import flash_attn_varlen, kv_append_rope, mla_paged_decode, paged_decode_append
 from ..ops.gemm import linear_forward
+from ..ops.rows import StepRows
 from ..ops.vocab import apply_top_k_top_p, sample, sample_filtered
 from ..utils import io_counters
 
@@ -71,7 +73,7 @@ class Request:
 class _Sched:
     """ctypes face of the C++ scheduler / block manager (``runtime/csrc/scheduler.cpp``)."""
 
-    def __init__(self, num_blocks, block_size, max_running, max_prefill_tokens):
+    def __init__(self, num_blocks, block_size, max_running, max_prefill_tokens, state_slots=0):
         self.lib = _lib.runtime()
         L = self.lib
         L.gkrt_sched_create.restype = ctypes.c_void_p
@@ -93,10 +95,16 @@ class _Sched:
                                          ctypes.POINTER(ctypes.c_int), ctypes.c_int, ctypes.POINTER(ctypes.c_int)],
              ctypes.c_int),
             ("gkrt_sched_stats", [ctypes.c_void_p, ctypes.POINTER(ctypes.c_int64)], None),
+            ("gkrt_sched_set_states", [ctypes.c_void_p, ctypes.c_int], None),
+            ("gkrt_sched_open", [ctypes.c_void_p, ctypes.c_int64], ctypes.c_int),
+            ("gkrt_sched_states", [ctypes.c_void_p, ctypes.POINTER(ctypes.c_int64), ctypes.c_int,
+                                   ctypes.POINTER(ctypes.c_int)], ctypes.c_int),
         ):
             f = getattr(L, fn)
             f.argtypes, f.restype = args, res
         self.h = L.gkrt_sched_create(num_blocks, block_size, max_running, max_prefill_tokens)
+        if state_slots:
+            L.gkrt_sched_set_states(self.h, state_slots)
 
     def __del__(self):
         try:
@@ -106,6 +114,17 @@ class _Sched:
 
     def add(self, rid, prompt_len, max_new):
         return self.lib.gkrt_sched_add(self.h, rid, prompt_len, max_new)
+
+    def open(self, rid):
+        """Admits a request whose tokens come in portions the caller chooses."""
+        return self.lib.gkrt_sched_open(self.h, rid)
+
+    def states(self, rids):
+        n = len(rids)
+        out = (ctypes.c_int * max(n, 1))()
+        rc = self.lib.gkrt_sched_states(self.h, (ctypes.c_int64 * max(n, 1))(*rids), n, out)
+        assert rc == 0
+        return list(out[:n])
 
     def fork(self, parent, child, max_new):
         a, b = ctypes.c_int(), ctypes.c_int()
@@ -151,8 +170,9 @@ class _Sched:
 
 
 def _count_launches() -> int:
-    from ..ops import attention, gemm, optim, rl, vocab
-    return sum(sum(m.LAUNCHES.values()) for m in (attention, fused, gemm, optim, rl, vocab))
+    from ..ops import attention, gemm, matrix_memory, optim, rl, sandwich, vocab, window_attention
+    return sum(sum(m.LAUNCHES.values()) for m in (attention, fused, gemm, matrix_memory, optim, rl, sandwich, vocab,
+                                                  window_attention))
 
 
 class LayerWeights:
@@ -168,6 +188,7 @@ class RolloutWeights:
     def __init__(self):
         self.layers: List[LayerWeights] = []
         self.embed = self.final_ln = self.head = None
+        self.plan: Optional[PlanDecoder] = None   # decoder described by a layer plan: the module itself serves
 
     @staticmethod
     def _serving_module(module, clone: bool):
@@ -192,6 +213,10 @@ class RolloutWeights:
         f = (lambda t: t.detach().clone()) if clone else (lambda t: t.detach())
         w = cls()
         model = getattr(model, "language_model", model)  # vision-language wrapper: the decoder is what serves
+        if isinstance(model, PlanDecoder):
+            w.plan = cls._serving_module(model, clone)
+            w.embed, w.final_ln, w.head = w.plan.embed.detach(), w.plan.final_gain.detach(), w.plan.head.detach()
+            return w
         w.embed = f(model.embedding.word_embeddings.weight)
         w.final_ln = f(model.decoder.final_layernorm.weight)
         w.head = f(model.output_weight())
@@ -237,6 +262,9 @@ class RolloutWeights:
         return w
 
     def tensors(self):
+        if self.plan is not None:
+            yield from self.plan.parameters()
+            return
         for t in (self.embed, self.final_ln, self.head):
             yield t
         for lw in self.layers:
@@ -264,6 +292,14 @@ class InferEngine:
         self.D = cfg.head_dim
         self.mla_dim = (cfg.kv_lora_rank + cfg.qk_rope_head_dim) if getattr(cfg, "use_mla", False) else 0
         self._mla_abs: Dict[int, list] = {}   # id(attention module) -> [absorbed up-projection, stale]
+        self.plan = weights.plan
+        if self.plan is not None:
+            if tp_size != 1:
+                raise ValueError("layer-plan decoders are served without tensor parallelism")
+            if max_model_len > cfg.max_position_embeddings:
+                raise ValueError(f"max_model_len {max_model_len} exceeds the model's {cfg.max_position_embeddings} "
+                                 "positions")
+        self.memory: list = []                # recurrent state of every layer run (layer-plan decoders)
         self.vocab_local = weights.head.shape[0]
         self.vocab_start = self.vocab_local * (dist.get_rank(tp_group) if (tp_group is not None and tp_size > 1) else 0)
         # the library (eager) backend launches its decode ops one by one (its GPU path has no host synchronisation, so
@@ -296,6 +332,7 @@ class InferEngine:
         self.v_cache: List[torch.Tensor] = []
         self.sched: Optional[_Sched] = None
         self.requests: Dict[int, Request] = {}
+        self._open: Dict[int, int] = {}       # requests of ``step``: tokens run so far
         self._next_rid = 0
         self._graphs: Dict[int, tuple] = {}
         self._state = None
@@ -307,6 +344,9 @@ class InferEngine:
 
     # ------------------------------------------------------------------ memory
     def _kv_bytes_per_block(self):
+        if self.plan is not None:
+            es = self.w.embed.element_size()
+            return sum(math.prod(self.plan.layers[r.layer].cache_shape()) for r in self.cfg.layer_plan.runs) * self.bs * es
         if self.mla_dim:
             return len(self.w.layers) * self.bs * self.mla_dim * 2
         return 2 * len(self.w.layers) * self.bs * self.hk * self.D * 2
@@ -319,13 +359,22 @@ class InferEngine:
                 need = self.max_running * self.max_blocks + 8
                 if self.device.type == "cuda":
                     free, total = torch.cuda.mem_get_info(self.device)
+                    if self.plan is not None:
+                        free -= self.max_running * sum(self.plan.layers[r.layer].state_bytes()
+                                                       for r in self.cfg.layer_plan.runs)
                     budget = int(free * self.gpu_memory_utilization)
                     n = max(min(need, budget // self._kv_bytes_per_block()), self.max_blocks + 1)
                 else:
                     n = need
             self.num_blocks = n
             dt = self.w.embed.dtype
-            if self.mla_dim:
+            if self.plan is not None:
+                # per layer run: one cached row serves as key and value, and one recurrent state per request slot
+                per_run = [self.plan.layers[r.layer] for r in self.cfg.layer_plan.runs]
+                self.k_cache = [torch.zeros(n, self.bs, *ly.cache_shape(), dtype=dt, device=self.device) for ly in per_run]
+                self.v_cache = []
+                self.memory = [ly.new_state(self.max_running, self.device) for ly in per_run]
+            elif self.mla_dim:
                 # latent cache: one row of (kv_lora + rope) values per token, shared by all heads; block ``n`` is a
                 # sink for the rows of inactive batch slots
                 self.k_cache = [torch.zeros(n + 1, self.bs, 1, self.mla_dim, dtype=dt, device=self.device)
@@ -336,7 +385,8 @@ class InferEngine:
                                 for _ in self.w.layers]
                 self.v_cache = [torch.zeros(n, self.bs, self.hk, self.D, dtype=dt, device=self.device)
                                 for _ in self.w.layers]
-            self.sched = _Sched(n, self.bs, self.max_running, self.max_prefill_tokens)
+            self.sched = _Sched(n, self.bs, self.max_running, self.max_prefill_tokens,
+                                self.max_running if self.plan is not None else 0)
             self.asleep["kv_cache"] = False
             self._graphs.clear()
         if "weights" in tags:
@@ -347,7 +397,7 @@ class InferEngine:
         if "kv_cache" in tags and not self.asleep["kv_cache"]:
             self._graphs.clear()
             self._state = None
-            self.k_cache, self.v_cache = [], []
+            self.k_cache, self.v_cache, self.memory = [], [], []
             self.sched = None
             self.asleep["kv_cache"] = True
             if self.device.type == "cuda":
@@ -402,6 +452,7 @@ class InferEngine:
         if self.sched is not None:
             self.sched.abort_all()
         self.requests.clear()
+        self._open.clear()
 
     def abort_all_requests(self):
         self.flush_cache()
@@ -568,9 +619,18 @@ class InferEngine:
         cfg = self.cfg
         B = st["tokens"].numel()
         pos = st["pos"]
-        blk = st["block_table"].gather(1, (pos // self.bs).long()[:, None]).squeeze(1)
-        slots = torch.where(st["active"], blk * self.bs + pos % self.bs, torch.full_like(pos, -1))
-        ctx = torch.where(st["active"], pos + 1, torch.zeros_like(pos))
+        blk = st["block_table"].gather(1, (pos // self.bs).long()[:, None].clamp_max(self.max_blocks - 1)).squeeze(1)
+        # a request at its length limit has no cache behind it: the rest of the interval is discarded, nothing is stored
+        live = st["active"] & (pos < st["limit"])
+        slots = torch.where(live, blk * self.bs + pos % self.bs, torch.full_like(pos, -1))
+        ctx = torch.where(live, pos + 1, torch.zeros_like(pos))
+        if self.plan is not None:
+            rows = StepRows(tokens=st["tokens"], pos=pos, slots=slots, tables=st["block_table"],
+                            states=torch.where(live, st["state"], torch.full_like(pos, -1)), first_pos=pos, cu=None,
+                            ctx=ctx, row_seq=st["row_seq"], n_portions=0, portion_rows=0, max_portion=0,
+                            max_ctx=self.max_model_len)
+            self._finish_decode(self.plan(rows, self.k_cache, self.memory), st)
+            return
         x = self._embed(st["tokens"])
         res = None
         if self.mla_dim:
@@ -601,9 +661,12 @@ class InferEngine:
             h, res = self._reduce_norm(self._lin(o.view(B, self.hq * self.D), lw, "o_w"), lw.ln2, res, self.tp > 1)
             x, pending = self._mlp(lw, h, reduce=False)
         hl, _ = self._reduce_norm(x, self.w.final_ln, res, pending)
+        self._finish_decode(hl, st)
+
+    def _finish_decode(self, hl, st):
+        """Samples the next token of every row and advances the batch state."""
         self._sample_into(hl, st)
-        # state advance
-        st["pos"].add_(st["active"].to(pos.dtype))
+        st["pos"].add_(st["active"].to(st["pos"].dtype))
         st["steps"].add_(1)
         st["ring_idx"].add_(1)
 
@@ -738,6 +801,9 @@ class InferEngine:
             tokens=torch.zeros(B, dtype=torch.int64, device=dev), pos=torch.zeros(B, dtype=torch.int32, device=dev),
             active=torch.zeros(B, dtype=torch.bool, device=dev),
             block_table=torch.zeros(B, self.max_blocks, dtype=torch.int32, device=dev),
+            limit=torch.zeros(B, dtype=torch.int32, device=dev),   # positions below it have cache reserved
+            state=torch.full((B,), -1, dtype=torch.int32, device=dev),
+            row_seq=torch.arange(B, dtype=torch.int32, device=dev),
             seeds=torch.zeros(B, dtype=torch.int64, device=dev), steps=torch.zeros(B, dtype=torch.int32, device=dev),
             ring_tok=torch.zeros(R, B, dtype=torch.int64, device=dev),
             ring_lp=torch.zeros(R, B, dtype=torch.float32, device=dev),
@@ -787,6 +853,121 @@ class InferEngine:
         g[0].replay()
         self.stats["graph_replays"] += 1
 
+    # ------------------------------------------------------------------ portions (layer-plan decoders)
+    def _step_rows(self, entries):
+        """Packs ``entries`` = [(rid, first position, tokens)] into one batch: portions of two and more tokens first,
+        single tokens behind them.  Returns the rows and, per entry, the row of its first token."""
+        order = sorted(range(len(entries)), key=lambda e: len(entries[e][2]) == 1)      # stable
+        rids = [entries[e][0] for e in order]
+        first = [entries[e][1] for e in order]
+        lens = [len(entries[e][2]) for e in order]
+        n_port = sum(l > 1 for l in lens)
+        n, T, port_rows = len(order), sum(lens), sum(l for l in lens if l > 1)
+        bt, _ = self.sched.tables(rids, self.max_blocks)
+        lens_t = torch.tensor(lens)
+        cu = torch.zeros(n + 1, dtype=torch.int32)
+        cu[1:] = lens_t.cumsum(0)
+        row_seq = torch.repeat_interleave(torch.arange(n, dtype=torch.int32), lens_t)
+        first_t = torch.tensor(first, dtype=torch.int32)
+        pos = torch.arange(T, dtype=torch.int32) - (cu[:-1] - first_t)[row_seq.long()]
+        slots = bt[row_seq.long(), (pos // self.bs).long()] * self.bs + pos % self.bs
+        ctx = (first_t + 1)[n_port:]
+        parts = [torch.tensor([t for e in order for t in entries[e][2]], dtype=torch.int32), pos, slots.to(torch.int32),
+                 torch.tensor(self.sched.states(rids), dtype=torch.int32), first_t, cu[:n_port + 1], ctx, row_seq,
+                 bt.reshape(-1)]
+        packed = torch.cat(parts)
+        if self.device.type == "cuda":
+            packed = packed.pin_memory()
+        io_counters.add_h2d(io_counters.tensor_bytes(packed))
+        tok, pos, slots, states, first_d, cu_d, ctx, row_seq, tables = packed.to(self.device, non_blocking=True).split(
+            [p.numel() for p in parts])
+        rows = StepRows(tokens=tok.long(), pos=pos, slots=slots, tables=tables.view(n, self.max_blocks), states=states,
+                        first_pos=first_d, cu=cu_d, ctx=ctx, row_seq=row_seq, n_portions=n_port, portion_rows=port_rows,
+                        max_portion=max(lens[:n_port], default=0), max_ctx=max((f + 1 for f in first[n_port:]), default=1))
+        base = [0] * n
+        for k, e in enumerate(order):
+            base[e] = int(cu[k])
+        return rows, base
+
+    @torch.no_grad()
+    def _run_portions(self, entries, want):
+        """Runs one batch of portions from the cache and state that earlier steps left and returns the final-normed
+        hidden states of the wanted rows (``want[e]``: places among entry e's tokens), in entry order."""
+        rows, base = self._step_rows(entries)
+        x = self.plan(rows, self.k_cache, self.memory, final=False)
+        picked = [b + w for b, ws in zip(base, want) for w in ws]
+        if not picked:
+            return None
+        return self.plan.final_rows(x, torch.tensor(picked, dtype=torch.int64, device=self.device))
+
+    def _prefill_portions(self, pre: List[Request]):
+        """Prompts through the model in steps of at most ``max_prefill_tokens`` rows; last-token hidden of every one."""
+        hidden: Dict[int, torch.Tensor] = {}
+        todo = [(r, 0) for r in pre]
+        while todo:
+            budget, batch, rest = self.max_prefill_tokens, [], []
+            for r, done in todo:
+                take = min(budget, len(r.prompt) - done)
+                if take:
+                    batch.append((r, done, take))
+                    budget -= take
+                if done + take < len(r.prompt):
+                    rest.append((r, done + take))
+            ends = [d + t == len(r.prompt) for r, d, t in batch]
+            h = self._run_portions([(r.rid, d, r.prompt[d:d + t]) for r, d, t in batch],
+                                   [[t - 1] if e else [] for (_, _, t), e in zip(batch, ends)])
+            for k, r in enumerate(b[0] for b, e in zip(batch, ends) if e):
+                hidden[r.rid] = h[k:k + 1]
+            todo = rest
+        return torch.cat([hidden[r.rid] for r in pre])
+
+    def open_request(self) -> int:
+        """Admits a request whose tokens the caller brings with ``step``; returns its id."""
+        if self.plan is None:
+            raise NotImplementedError("step-wise serving is built for layer-plan decoders")
+        if self.asleep["kv_cache"]:
+            self.wake_up(("kv_cache",))
+        rid = self._next_rid
+        if self.sched.open(rid) != 0:
+            raise RuntimeError("no free request slot: raise max_running_requests")
+        self._next_rid += 1
+        self._open[rid] = 0
+        return rid
+
+    def close_request(self, rid: int):
+        """Gives back what the request holds in the cache and the state."""
+        self.sched.finish(rid)
+        del self._open[rid]
+
+    @torch.no_grad()
+    def step(self, entries: Sequence[tuple], want: Optional[Sequence[Sequence[int]]] = None):
+        """One batch of ``(request id, next tokens)``: portions of prompts beside single decoded tokens.  Returns the
+        32-bit logits of the wanted places of every entry, in entry order ([wanted, vocab]; None if nothing is)."""
+        want = want if want is not None else [[] for _ in entries]
+        batch = []
+        if len({rid for rid, _ in entries}) != len(entries):
+            raise ValueError("a request appears twice in one step")
+        for (rid, tokens), ws in zip(entries, want):
+            done = self._open[rid]
+            if not tokens or not (0 <= min(tokens) and max(tokens) < self.cfg.vocab_size):
+                raise ValueError(f"request {rid}: tokens are empty or outside [0, {self.cfg.vocab_size})")
+            if done + len(tokens) > self.max_model_len:
+                raise ValueError(f"request {rid} outgrows max_model_len {self.max_model_len}")
+            if any(not 0 <= w < len(tokens) for w in ws):
+                raise ValueError(f"request {rid}: a wanted place lies outside its tokens")
+            batch.append((rid, done, list(tokens)))
+        if not batch:
+            return None
+        for rid, _, tokens in batch:
+            if self.sched.reserve(rid, len(tokens)) != 0:
+                raise RuntimeError("KV cache exhausted: raise num_kv_blocks")
+        h = self._run_portions(batch, want)
+        for rid, done, tokens in batch:
+            self.sched.advance(rid, len(tokens))
+            self._open[rid] = done + len(tokens)
+        self.stats["prefill_tokens"] += sum(len(t) for _, _, t in batch)
+        return None if h is None else linear_forward(h, self.w.head, out_dtype=torch.float32)
+
     # ------------------------------------------------------------------ public generate
     @torch.no_grad()
     def generate(self, prompts: Sequence[Sequence[int]], params: SamplingParams, n: int = 1,
@@ -812,6 +993,11 @@ class InferEngine:
             if len(p) and not (0 <= min(p) and max(p) < vocab):
                 # checked on the host: an id outside the embedding table would otherwise trip a device-side assert
                 raise ValueError(f"prompt {i} holds token ids outside [0, {vocab})")
+            if self.plan is not None and (not len(p) or len(p) + params.max_new_tokens > self.max_model_len):
+                raise ValueError(f"prompt {i}: {len(p)} + {params.max_new_tokens} tokens do not fit max_model_len "
+                                 f"{self.max_model_len}")
+        if self.plan is not None and image_embeds is not None:
+            raise ValueError("image prompts are not supported by layer-plan decoders")
         for i, p in enumerate(prompts):
             for j in range(n):
                 rid = self._next_rid
@@ -846,9 +1032,12 @@ class InferEngine:
         host_seed = torch.zeros(B, dtype=torch.int64)
         host_step = torch.zeros(B, dtype=torch.int32)
         host_bt = torch.zeros(B, self.max_blocks, dtype=torch.int32)
+        host_limit = torch.zeros(B, dtype=torch.int32)
+        host_state = torch.full((B,), -1, dtype=torch.int32)
         if dev.type == "cuda":
-            host_tok, host_pos, host_active, host_seed, host_step, host_bt = (
-                t.pin_memory() for t in (host_tok, host_pos, host_active, host_seed, host_step, host_bt))
+            host_tok, host_pos, host_active, host_seed, host_step, host_bt, host_limit, host_state = (
+                t.pin_memory() for t in (host_tok, host_pos, host_active, host_seed, host_step, host_bt, host_limit,
+                                         host_state))
         # numpy views: scalar writes through a tensor cost microseconds each, and there are hundreds per interval
         n_tok, n_pos, n_active, n_seed, n_step = (t.numpy() for t in (host_tok, host_pos, host_active, host_seed,
                                                                       host_step))
@@ -869,6 +1058,8 @@ class InferEngine:
             n_active[s] = True
             n_seed[s] = r.seed
             n_step[s] = 1
+            host_limit[s] = len(r.prompt) + params.max_new_tokens
+            host_state[s] = self.sched.states([r.rid])[0]
             if "seen" in st:   # the slot's table restarts from this request's prompt and first token
                 st["seen"][s].zero_()
                 st["seen"][s, torch.tensor(list(r.prompt) + [first_tok], dtype=torch.int64, device=dev)] = True
@@ -884,8 +1075,10 @@ class InferEngine:
                               torch.full((1,), -1, dtype=torch.int32, device=dev))
             if pre_ids:
                 pre = [self.requests[i] for i in pre_ids]
-                toks = torch.tensor([t for r in pre for t in r.prompt], dtype=torch.int64)
                 lens = [len(r.prompt) for r in pre]
+                hl = self._prefill_portions(pre) if self.plan is not None else None
+            if pre_ids and self.plan is None:
+                toks = torch.tensor([t for r in pre for t in r.prompt], dtype=torch.int64)
                 cu = torch.tensor([0] + list(torch.tensor(lens).cumsum(0)), dtype=torch.int32)
                 pos = torch.cat([torch.arange(l, dtype=torch.int32) for l in lens])
                 bt, _ = self.sched.tables(pre_ids, self.max_blocks)
@@ -914,7 +1107,8 @@ class InferEngine:
                 hl = self._prefill(toks.to(dev, non_blocking=True), pos.to(dev, non_blocking=True),
                                    cu.to(dev, non_blocking=True), max(lens), slots.to(dev, non_blocking=True),
                                    embed_rows)
-                self.stats["prefill_tokens"] += int(toks.numel())
+            if pre_ids:
+                self.stats["prefill_tokens"] += sum(lens)
                 for r in pre:
                     self.sched.commit(r.rid, True)
                 # the first token of a prompt's samples all come from the same last-position hidden state
@@ -951,9 +1145,13 @@ class InferEngine:
                 if copies:
                     src = torch.tensor([a for a, _ in copies], device=dev)
                     dst = torch.tensor([b for _, b in copies], device=dev)
-                    for li in range(len(self.w.layers)):
-                        self.k_cache[li][dst] = self.k_cache[li][src]
-                        self.v_cache[li][dst] = self.v_cache[li][src]
+                    for c in self.k_cache + self.v_cache:
+                        c[dst] = c[src]
+                if self.plan is not None and len(owners) > len(pre):
+                    pairs = [(r.rid, c.rid) for r in pre for c in children.get(r.rid, [])]
+                    s_src, s_dst = (torch.tensor(self.sched.states([p[k] for p in pairs]), device=dev) for k in (0, 1))
+                    for state in self.memory:
+                        state.copy_slots(s_src, s_dst)
                 for c in owners:
                     place(c, *first[c.rid])
             if self.ep_group is not None:
@@ -984,14 +1182,17 @@ class InferEngine:
                 interval = max(interval, min(left, self.max_sync_interval))
             for s, r in list(slot_req.items()):
                 remaining = params.max_new_tokens - len(r.out_tokens)
-                self.sched.reserve(r.rid, min(interval, remaining) + 1)
+                if self.sched.reserve(r.rid, min(interval, remaining) + 1) != 0:
+                    raise RuntimeError("KV cache exhausted while decoding: raise num_kv_blocks or lower "
+                                       "max_running_requests")
             rids = [slot_req[s].rid if s in slot_req else -1 for s in range(B)]
             live = [s for s in range(B) if s in slot_req]
             bt, _ = self.sched.tables([rids[s] for s in live], self.max_blocks)
             host_bt.zero_()
             host_bt[torch.tensor(live)] = bt
             for k, src in (("tokens", host_tok), ("pos", host_pos), ("active", host_active), ("seeds", host_seed),
-                           ("steps", host_step), ("block_table", host_bt)):
+                           ("steps", host_step), ("block_table", host_bt), ("limit", host_limit),
+                           ("state", host_state)):
                 st[k].copy_(src, non_blocking=True)
                 io_counters.add_h2d(io_counters.tensor_bytes(src))
             st["ring_idx"].zero_()

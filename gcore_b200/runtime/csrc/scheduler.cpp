@@ -25,6 +25,7 @@ struct Request {
   bool prefilled = false;
   bool finished = false;
   int64_t arrival;
+  int state = -1;         // recurrent-state slot (models with recurrent mixers)
   std::vector<int> blocks;
 };
 
@@ -32,6 +33,8 @@ struct Scheduler {
   int num_blocks, block_size, max_running, max_prefill_tokens;
   std::vector<int> free_list;
   std::vector<int> refcnt;
+  bool has_states = false;
+  std::vector<int> free_states;
   std::unordered_map<int64_t, Request> reqs;
   std::deque<int64_t> waiting;
   std::vector<int64_t> running;
@@ -57,6 +60,16 @@ struct Scheduler {
     }
     r.blocks.clear();
     r.cached_tokens = 0;
+    if (r.state >= 0) free_states.push_back(r.state);
+    r.state = -1;
+  }
+  // A request that runs holds one state slot from admission to release.
+  bool take_state(Request& r) {
+    if (!has_states || r.state >= 0) return true;
+    if (free_states.empty()) return false;
+    r.state = free_states.back();
+    free_states.pop_back();
+    return true;
   }
 };
 
@@ -72,6 +85,14 @@ RT_EXPORT void* gkrt_sched_create(int num_blocks, int block_size, int max_runnin
   s->free_list.reserve(num_blocks);
   for (int b = num_blocks - 1; b >= 0; --b) s->free_list.push_back(b);
   return s;
+}
+
+// Requests of models with recurrent mixers also hold one of `n` state slots while they run.
+RT_EXPORT void gkrt_sched_set_states(void* h, int n) {
+  auto* s = static_cast<Scheduler*>(h);
+  s->has_states = true;
+  s->free_states.clear();
+  for (int i = n - 1; i >= 0; --i) s->free_states.push_back(i);
 }
 
 RT_EXPORT void gkrt_sched_destroy(void* h) { delete static_cast<Scheduler*>(h); }
@@ -103,6 +124,7 @@ RT_EXPORT int gkrt_sched_fork(void* h, int64_t parent, int64_t child, int max_ne
   const int full = shared_tokens / s->block_size;
   const bool partial = shared_tokens % s->block_size != 0;
   if (partial && s->free_list.empty()) return -1;
+  if (s->has_states && s->free_states.empty()) return -1;
   Request c;
   c.id = child;
   c.prompt_len = p.prompt_len;
@@ -122,8 +144,37 @@ RT_EXPORT int gkrt_sched_fork(void* h, int64_t parent, int64_t child, int max_ne
     *copy_src = p.blocks[full];
     *copy_dst = b;
   }
+  s->take_state(c);
   s->running.push_back(child);
   s->reqs.emplace(child, std::move(c));
+  return 0;
+}
+
+// Admits a request whose tokens the caller brings in portions of its own choosing (gkrt_sched_reserve before and
+// gkrt_sched_advance after each).  Returns 0, -1 for a known id, -3 when no run or state slot is free.
+RT_EXPORT int gkrt_sched_open(void* h, int64_t id) {
+  auto* s = static_cast<Scheduler*>(h);
+  if (s->reqs.count(id)) return -1;
+  if (static_cast<int>(s->running.size()) >= s->max_running) return -3;
+  Request r;
+  r.id = id;
+  r.prompt_len = r.max_new = 0;
+  r.prefilled = true;
+  r.arrival = s->clock++;
+  if (!s->take_state(r)) return -3;
+  s->running.push_back(id);
+  s->reqs.emplace(id, std::move(r));
+  return 0;
+}
+
+// State slots of a batch of requests (-1: none).
+RT_EXPORT int gkrt_sched_states(void* h, const int64_t* ids, int n, int* out) {
+  auto* s = static_cast<Scheduler*>(h);
+  for (int i = 0; i < n; ++i) {
+    auto it = s->reqs.find(ids[i]);
+    if (it == s->reqs.end()) return -1;
+    out[i] = it->second.state;
+  }
   return 0;
 }
 
@@ -172,6 +223,7 @@ RT_EXPORT int gkrt_sched_step(void* h, int64_t* prefill_ids, int cap_prefill, in
     // keep one block of head-room per running request so decode does not immediately preempt
     const int need = s->blocks_needed(r.prompt_len + 1);
     if (static_cast<int>(s->free_list.size()) < need + static_cast<int>(s->running.size())) break;
+    if (!s->take_state(r)) break;
     s->alloc(r, r.prompt_len + 1);
     budget -= r.prompt_len;
     prefill_ids[(*n_prefill)++] = r.id;
