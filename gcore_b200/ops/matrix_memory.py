@@ -14,6 +14,8 @@ from .rows import StepRows
 LAUNCHES = {"matrix_memory": 0}
 SLICE = 64        # value columns per state slice (csrc/matrix_memory.cu: MM_SLICE)
 MAX_KEY_DIM = 512
+CHUNK_MAX_KEY_DIM = 256   # keys the chunkwise tensor-core kernel takes
+SCAN_MAX_TOKENS = 8       # portions up to here run token by token
 
 
 def padded_key_dim(dim: int) -> int:
@@ -84,6 +86,17 @@ def _scan(proj, offs, h, gate_w, gates, gate_b, cap, q_scale, heads, dim, vdim, 
                                                     float(cap), float(q_scale), _lib.stream_ptr()), "matrix_memory_scan")
 
 
+def _chunk(proj, offs, gates, gate_b, cap, q_scale, heads, dim, vdim, rows: StepRows, st, out):
+    n = rows.n_portions
+    states = rows.states[:n]
+    ptrs = (ctypes.c_void_p * 11)(*[t.data_ptr() for t in (proj, gates, gate_b, rows.cu, rows.first_pos, states, st.S, st.n,
+                                                           st.m, out, _lib.err_flag(proj.device))])
+    dims = (ctypes.c_int * 8)(n, rows.portion_rows, *offs, heads, dim, vdim)
+    LAUNCHES["matrix_memory"] += 1
+    _lib.check(_lib.kernels().gk_matrix_memory_chunk(ptrs, proj.stride(0), dims, float(cap), float(q_scale),
+                                                     _lib.stream_ptr()), "matrix_memory_chunk")
+
+
 def _output(o, proj, g_off, gain, vdim_true, eps):
     T, heads, vdim = o.shape
     if not o.is_cuda:
@@ -115,7 +128,10 @@ def matrix_memory(proj, q_off: int, k_off: int, v_off: int, g_off: int, h, gate_
     common = (gate_b, cap, q_scale, heads, dim, vdim)
     if P:
         gates = linear_forward(h[:P], gate_w, out_dtype=torch.float32)
-        _scan(proj, offs, None, None, gates, *common, rows.cu, rows.first_pos, rows.states[:n], state, o)
+        if proj.dtype == torch.bfloat16 and dim <= CHUNK_MAX_KEY_DIM and rows.max_portion > SCAN_MAX_TOKENS:
+            _chunk(proj, offs, gates, *common, rows, state, o)
+        else:
+            _scan(proj, offs, None, None, gates, *common, rows.cu, rows.first_pos, rows.states[:n], state, o)
     if T > P:
         _scan(proj[P:], offs, h[P:], gate_w, None, *common, None, rows.first_pos[n:], rows.states[n:], state, o[P:])
     return _output(o, proj, g_off, gain, vdim_true, eps)

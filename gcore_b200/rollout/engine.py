@@ -833,6 +833,8 @@ class InferEngine:
         if g is None or g[1] is not st:
             # warm up once eagerly on a side stream (allocates scratch, configures kernels), then capture
             keep = {k: v.clone() for k, v in st.items() if isinstance(v, torch.Tensor)}
+            if self.plan is not None:
+                st["active"].zero_()   # recurrent state, unlike a cache row, must not see the step twice
             s = torch.cuda.Stream()
             s.wait_stream(torch.cuda.current_stream())
             with torch.cuda.stream(s):
