@@ -270,7 +270,12 @@ def main():
                     help="1: the frozen reference model lives in pinned host memory outside its forward pass (its "
                     "upload runs on a side stream under the old-policy pass); default: on at 1 GPU, where the whole "
                     "model's optimizer state shares the GPU with the activations")
+    ap.add_argument("--serve", nargs="*", default=None, metavar="SIZE",
+                    help="instead of the recipe: prefill and decode throughput of layer-plan decoders beside the closest "
+                    "dense model, kernel by kernel (sizes: see gcore_b200/tools/serve_bench.py; default all); one JSON line")
     args = ap.parse_args()
+    if args.serve is not None:
+        return serve_bench(args)
     for k, v in CONFIGS[args.config].items():
         if k != "kind" and getattr(args, k, None) is None:
             setattr(args, k, v)
@@ -439,6 +444,20 @@ def main():
     if world > 1:
         dist.barrier()
         dist.destroy_process_group()
+    return 0
+
+
+def serve_bench(args):
+    """``--serve``: one GPU, clocks sampled while it runs."""
+    import torch
+    from gcore_b200.tools import serve_bench as sb
+    torch.cuda.set_device(0)
+    clocks = ClockSampler(0, period_s=0.2)
+    clocks.start()
+    clocks.mark()
+    out = sb.run(args.serve or None)
+    out["clocks"] = clocks.stop()
+    print(json.dumps({"metric": "serve_prefill_decode_tokens_per_s", **out}))
     return 0
 
 

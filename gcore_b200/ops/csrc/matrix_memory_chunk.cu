@@ -348,7 +348,7 @@ matrix_memory_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
       ok = mbar_wait(&g_full[buf], (c >> 1) & 1, p.err, ERR_WAIT_MISC);
       if (!ok) break;
       const float m0 = gs[3 * MC_L], g_end = gs[MC_L + MC_L - 1];
-      const float decay = exp2f((m0 - g_end) * MC_LOG2E);
+      const float decay = ex2((m0 - g_end) * MC_LOG2E);
 #pragma unroll
       for (int h = 0; h < NH; ++h) {
         // ---- state -> operand of q S (undecayed); its decayed value goes back to tensor memory for the update
@@ -399,7 +399,7 @@ matrix_memory_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
           // ---- weighted values (token r, 32 columns) and key weights
           ok = mbar_wait(v_full, c & 1, p.err, ERR_WAIT_FULL);
           if (!ok) break;
-          const float wt = exp2f((gs[r] - g_end) * MC_LOG2E);
+          const float wt = ex2((gs[r] - g_end) * MC_LOG2E);
           const uint8_t* src = smem + McSmem::V + r * 128;
           uint8_t* dst = smem + McSmem::VW + r * 128;
 #pragma unroll
@@ -445,7 +445,7 @@ matrix_memory_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
           const float av[8] = {a0.x, a0.y, a0.z, a0.w, a1.x, a1.y, a1.z, a1.w};
 #pragma unroll
           for (int e = 0; e < 8; ++e) {
-            const float d = s0 + e <= r ? exp2f((av[e] - g) * MC_LOG2E) * p.q_scale : 0.f;
+            const float d = s0 + e <= r ? ex2((av[e] - g) * MC_LOG2E) * p.q_scale : 0.f;
             v[e] = s0 + e <= r ? __uint_as_float(w[u * 8 + e]) * d : 0.f;
             rs += v[e];
           }
@@ -464,7 +464,7 @@ matrix_memory_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
       if (!ok) break;
       tc_fence_after();
       {
-        const float inter = exp2f((m0 - g) * MC_LOG2E) * p.q_scale;
+        const float inter = ex2((m0 - g) * MC_LOG2E) * p.q_scale;
         uint32_t qn[16], oi[32], oa[32];
         tmem_ld16(lane_addr + MC_T_QN, qn);
         tmem_ld32(lane_addr + MC_T_OI + half * 32, oi);
@@ -472,7 +472,7 @@ matrix_memory_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
         tmem_ld_wait();
         const float den = inter * (__uint_as_float(qn[0]) + __uint_as_float(qn[1])) + rsum[buf * 2 * MC_L + r] +
                           rsum[(buf * 2 + 1) * MC_L + r];
-        const float inv = 1.f / (fmaxf(fabsf(den), exp2f(-gs[2 * MC_L + r] * MC_LOG2E)) + 1e-6f);
+        const float inv = 1.f / (fmaxf(fabsf(den), ex2(-gs[2 * MC_L + r] * MC_LOG2E)) + 1e-6f);
         const int t = c * MC_L + r;
         if (t < len) {
           float* dst = p.out + (static_cast<long long>(r_beg + t) * p.heads + head) * p.vdim + col0;

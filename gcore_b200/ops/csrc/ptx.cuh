@@ -246,6 +246,14 @@ __host__ __device__ constexpr uint32_t make_idesc(int m, int n, int a_fmt, int b
          (static_cast<uint32_t>(m >> 4) << 24);       // M / 16
 }
 
+// 2^x on the special-function unit, results below 2^-126 flushed to zero (kernels compiled without the approximate math
+// functions use it where a softmax or decay weight feeds a bf16 tensor-core operand anyway).
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
 __device__ __forceinline__ float bf16_bits_to_float(uint16_t b) {
   return __uint_as_float(static_cast<uint32_t>(b) << 16);
 }

@@ -8,6 +8,7 @@
 //                             splits, append of the new key fused in.
 // Probabilities stay 32-bit: where they feed a tensor core they are split into two bf16 terms (high part + remainder).
 // Prompt portions in bf16 run the tcgen05 kernel in window_prefill.cu.
+#include "ptx.cuh"
 #include "host_utils.h"
 #include <cuda_bf16.h>
 #include <float.h>
@@ -137,7 +138,9 @@ inline int& shared_decode_target_ctas() {
 }
 
 // grid (request, kv head x blocks of 16 query heads, split).  q / k: rows of the packed projection.
-template <int D>
+// ONE8: groups of up to 8 heads.  Rows 8-15 of the probability tile then carry the remainder terms of rows 0-7, so one
+// product serves both terms, and the halves of the output tile are added at the end.
+template <int D, bool ONE8>
 __global__ void __launch_bounds__(SD_WARPS * 32, 3) shared_kv_decode_kernel(
     const __nv_bfloat16* __restrict__ proj, long long ld, int q_off, int k_off, __nv_bfloat16* __restrict__ cache,
     const int* __restrict__ tables, int max_blocks, const int* __restrict__ ctx_len, const int* __restrict__ new_slots,
@@ -250,11 +253,12 @@ __global__ void __launch_bounds__(SD_WARPS * 32, 3) shared_kv_decode_kernel(
           wa_mma(sc[j], qa[2 * kp + 1], kb[2], kb[3]);
         }
       }
+      constexpr int HV = ONE8 ? 1 : 2;     // row halves that hold scores
       float mx[2] = {-FLT_MAX, -FLT_MAX};
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
+        for (int e = 0; e < 2 * HV; ++e) {
           const int ti = j * 8 + cq + (e & 1), half = e >> 1;
           const float v = ti < nt ? sc[j][e] * sl2 - slope[half] * static_cast<float>(len - 1 - (tok0 + ti)) : -FLT_MAX;
           sc[j][e] = v;
@@ -263,14 +267,15 @@ __global__ void __launch_bounds__(SD_WARPS * 32, 3) shared_kv_decode_kernel(
       }
       float resc[2];
 #pragma unroll
-      for (int u = 0; u < 2; ++u) {
+      for (int u = 0; u < HV; ++u) {
         mx[u] = fmaxf(mx[u], __shfl_xor_sync(0xffffffff, mx[u], 1));
         mx[u] = fmaxf(mx[u], __shfl_xor_sync(0xffffffff, mx[u], 2));
         const float mn = fmaxf(m_run[u], mx[u]);
-        resc[u] = exp2f(m_run[u] - mn);
+        resc[u] = ex2(m_run[u] - mn);
         m_run[u] = mn;
         l_run[u] *= resc[u];
       }
+      if (ONE8) resc[1] = resc[0];
 #pragma unroll
       for (int j = 0; j < NC; ++j) { o[j][0] *= resc[0]; o[j][1] *= resc[0]; o[j][2] *= resc[1]; o[j][3] *= resc[1]; }
       uint32_t ph[2][4], pl[2][4];
@@ -278,14 +283,18 @@ __global__ void __launch_bounds__(SD_WARPS * 32, 3) shared_kv_decode_kernel(
       for (int j = 0; j < 4; ++j) {
         float pv[4];
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          pv[e] = sc[j][e] == -FLT_MAX ? 0.f : exp2f(sc[j][e] - m_run[e >> 1]);
+        for (int e = 0; e < 2 * HV; ++e) {
+          pv[e] = sc[j][e] == -FLT_MAX ? 0.f : ex2(sc[j][e] - m_run[e >> 1]);
           l_run[e >> 1] += pv[e];
         }
         ph[j >> 1][(j & 1) * 2] = wa_pack(pv[0], pv[1]);
-        ph[j >> 1][(j & 1) * 2 + 1] = wa_pack(pv[2], pv[3]);
-        pl[j >> 1][(j & 1) * 2] = wa_pack(wa_rest(pv[0]), wa_rest(pv[1]));
-        pl[j >> 1][(j & 1) * 2 + 1] = wa_pack(wa_rest(pv[2]), wa_rest(pv[3]));
+        if (ONE8) {
+          ph[j >> 1][(j & 1) * 2 + 1] = wa_pack(wa_rest(pv[0]), wa_rest(pv[1]));
+        } else {
+          ph[j >> 1][(j & 1) * 2 + 1] = wa_pack(pv[2], pv[3]);
+          pl[j >> 1][(j & 1) * 2] = wa_pack(wa_rest(pv[0]), wa_rest(pv[1]));
+          pl[j >> 1][(j & 1) * 2 + 1] = wa_pack(wa_rest(pv[2]), wa_rest(pv[3]));
+        }
       }
 #pragma unroll
       for (int kk = 0; kk < 2; ++kk) {
@@ -296,8 +305,10 @@ __global__ void __launch_bounds__(SD_WARPS * 32, 3) shared_kv_decode_kernel(
           wa_ldsm_x4_t(vb, ts + row * RB + ((ch ^ (row & SWZ)) << 4));
           wa_mma(o[2 * np], ph[kk], vb[0], vb[1]);
           wa_mma(o[2 * np + 1], ph[kk], vb[2], vb[3]);
-          wa_mma(o[2 * np], pl[kk], vb[0], vb[1]);
-          wa_mma(o[2 * np + 1], pl[kk], vb[2], vb[3]);
+          if (!ONE8) {
+            wa_mma(o[2 * np], pl[kk], vb[0], vb[1]);
+            wa_mma(o[2 * np + 1], pl[kk], vb[2], vb[3]);
+          }
         }
       }
       __syncwarp();   // every lane is done with the tile before it is refilled
@@ -313,12 +324,17 @@ __global__ void __launch_bounds__(SD_WARPS * 32, 3) shared_kv_decode_kernel(
   float* o_all = reinterpret_cast<float*>(sd_dyn);   // [warp][16][D]
   if ((lane & 3) == 0) {
     m_all[warp][r0] = m_run[0]; l_all[warp][r0] = l_run[0];
-    m_all[warp][r0 + 8] = m_run[1]; l_all[warp][r0 + 8] = l_run[1];
+    if (!ONE8) { m_all[warp][r0 + 8] = m_run[1]; l_all[warp][r0 + 8] = l_run[1]; }
   }
 #pragma unroll
   for (int j = 0; j < NC; ++j) {
-    *reinterpret_cast<float2*>(o_all + (warp * SD_ROWS + r0) * D + j * 8 + cq) = make_float2(o[j][0], o[j][1]);
-    *reinterpret_cast<float2*>(o_all + (warp * SD_ROWS + r0 + 8) * D + j * 8 + cq) = make_float2(o[j][2], o[j][3]);
+    if (ONE8) {
+      *reinterpret_cast<float2*>(o_all + (warp * SD_ROWS + r0) * D + j * 8 + cq) =
+          make_float2(o[j][0] + o[j][2], o[j][1] + o[j][3]);
+    } else {
+      *reinterpret_cast<float2*>(o_all + (warp * SD_ROWS + r0) * D + j * 8 + cq) = make_float2(o[j][0], o[j][1]);
+      *reinterpret_cast<float2*>(o_all + (warp * SD_ROWS + r0 + 8) * D + j * 8 + cq) = make_float2(o[j][2], o[j][3]);
+    }
   }
   __syncthreads();
   for (int i = tid; i < nh * D; i += SD_WARPS * 32) {
@@ -329,7 +345,7 @@ __global__ void __launch_bounds__(SD_WARPS * 32, 3) shared_kv_decode_kernel(
     float acc = 0.f, ls = 0.f;
 #pragma unroll
     for (int w = 0; w < SD_WARPS; ++w) {
-      const float f = m_all[w][r] == -FLT_MAX ? 0.f : exp2f(m_all[w][r] - mm);
+      const float f = m_all[w][r] == -FLT_MAX ? 0.f : ex2(m_all[w][r] - mm);
       acc += o_all[(w * SD_ROWS + r) * D + d] * f;
       ls += l_all[w][r] * f;
     }
@@ -359,7 +375,7 @@ __global__ void shared_kv_combine_kernel(const float* __restrict__ scratch, cons
   float l = 0.f, acc = 0.f;
   for (int s = 0; s < ns; ++s) {
     const float ms = base[s * (D + 2) + D];
-    const float w = ms == -FLT_MAX ? 0.f : exp2f(ms - m);
+    const float w = ms == -FLT_MAX ? 0.f : ex2(ms - m);
     l += base[s * (D + 2) + D + 1] * w;
     acc += base[s * (D + 2) + d] * w;
   }
@@ -391,8 +407,8 @@ inline void shared_decode_splits(int B, int yblocks, int span, int* nsplit, int*
   *split_tokens = st;
 }
 
-template <int D>
-int launch_shared_decode(const void* proj, long long ld, int q_off, int k_off, void* cache, const int* tables,
+template <int D, bool ONE8>
+int launch_shared_decode_impl(const void* proj, long long ld, int q_off, int k_off, void* cache, const int* tables,
                          int max_blocks, const int* ctx, const int* new_slots, const float* slopes, void* out,
                          float* scratch, int B, int H, int G, int block_size, int window, int max_ctx, float scale,
                          cudaStream_t st) {
@@ -400,14 +416,14 @@ int launch_shared_decode(const void* proj, long long ld, int q_off, int k_off, v
   static_assert(SMEM >= SD_WARPS * SD_ROWS * D * 4, "the merge fits the key tiles");
   static bool configured = false;
   if (!configured) {
-    cudaFuncSetAttribute(shared_kv_decode_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
+    cudaFuncSetAttribute(shared_kv_decode_kernel<D, ONE8>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
     configured = true;
   }
   const int grp = H / G, yb = G * ((grp + SD_ROWS - 1) / SD_ROWS);
   int nsplit, split_tokens;
   shared_decode_splits(B, yb, window < max_ctx ? window : max_ctx, &nsplit, &split_tokens);
   if (nsplit > 1 && !scratch) return -2;
-  launch_k(shared_kv_decode_kernel<D>, dim3(B, yb, nsplit), dim3(SD_WARPS * 32), SMEM, st,
+  launch_k(shared_kv_decode_kernel<D, ONE8>, dim3(B, yb, nsplit), dim3(SD_WARPS * 32), SMEM, st,
            static_cast<const __nv_bfloat16*>(proj), ld, q_off, k_off, static_cast<__nv_bfloat16*>(cache), tables,
            max_blocks, ctx, new_slots, slopes, static_cast<__nv_bfloat16*>(out), scratch, H, G, block_size, window, scale,
            nsplit, split_tokens);
@@ -415,6 +431,11 @@ int launch_shared_decode(const void* proj, long long ld, int q_off, int k_off, v
     launch_k(shared_kv_combine_kernel<D>, dim3(B, H), dim3(D), 0, st, static_cast<const float*>(scratch), ctx, window,
              static_cast<__nv_bfloat16*>(out), H, nsplit, split_tokens);
   return launch_status();
+}
+
+template <int D, typename... A>
+int launch_shared_decode(bool one8, A... a) {
+  return one8 ? launch_shared_decode_impl<D, true>(a...) : launch_shared_decode_impl<D, false>(a...);
 }
 
 }  // namespace gk
@@ -464,10 +485,10 @@ GK_EXPORT int gk_shared_kv_decode(const void* proj, long long ld, void* cache, c
   if (B == 0) return 0;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   if (D == 64)
-    return launch_shared_decode<64>(proj, ld, dims[8], dims[9], cache, tables, dims[6], ctx, new_slots, slopes, out,
+    return launch_shared_decode<64>(H / G <= 8, proj, ld, dims[8], dims[9], cache, tables, dims[6], ctx, new_slots, slopes, out,
                                     scratch, B, H, G, dims[5], dims[4], dims[7], scale, st);
   if (D == 128)
-    return launch_shared_decode<128>(proj, ld, dims[8], dims[9], cache, tables, dims[6], ctx, new_slots, slopes, out,
+    return launch_shared_decode<128>(H / G <= 8, proj, ld, dims[8], dims[9], cache, tables, dims[6], ctx, new_slots, slopes, out,
                                      scratch, B, H, G, dims[5], dims[4], dims[7], scale, st);
   return -4;
 }

@@ -236,11 +236,11 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
       const bool grow = (m == -FLT_MAX) ? (m_cand != -FLT_MAX) : (m_cand > m + 8.f);
       const float m_new = grow ? m_cand : m;
       const float m_use = m_new == -FLT_MAX ? 0.f : m_new;
-      const float corr = grow ? exp2f(m - m_use) : 1.f;
+      const float corr = grow ? ex2(m - m_use) : 1.f;
       float ps = 0.f;
 #pragma unroll
       for (int j = 0; j < WP_BN; ++j) {
-        const float e = exp2f(sv[j] - m_use);   // masked scores underflow to exactly 0
+        const float e = ex2(sv[j] - m_use);   // masked scores underflow to exactly 0
         sv[j] = e;
         ps += e;
       }
