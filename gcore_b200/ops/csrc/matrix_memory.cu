@@ -62,7 +62,7 @@ struct ScanParams {
 // grid (heads * slices, segments).  Thread (warp w, lane): rows rg, rg + 16, ... with rg = 2 w + lane / 16; columns
 // 4 * (lane % 16) .. + 3 of the slice.  R = rows per thread.
 template <typename T, int R>
-__global__ void __launch_bounds__(MM_THREADS) matrix_memory_scan_kernel(const ScanParams<T> p) {
+__global__ void __launch_bounds__(MM_THREADS, R <= 8 ? 3 : R <= 16 ? 2 : 1) matrix_memory_scan_kernel(const ScanParams<T> p) {
   __shared__ float sq[2][16 * R], sk[2][16 * R];
   __shared__ float red[2][8][MM_SLICE + 4];
   __shared__ float gred[2][8];

@@ -12,8 +12,11 @@
 //               column half = warp >> 2)
 //   warp 8      TMA producer        warp 9  MMA issuer        warp 10  gates of the next chunk (scan over 128 tokens)
 //
-// TMEM columns (512): scores [0,128), inter-chunk output [128,192), intra-chunk output [192,256), state [256,256+64*NH),
-// normaliser [384,384+16*NH), q . n [416,432).
+// The elementwise warps turn the state into the next chunk's operand before they wait for the current chunk's output, so
+// the tensor core is fed while they finish it; inter-chunk outputs therefore alternate between two buffers.
+//
+// TMEM columns (512): scores [0,128), inter-chunk output 2 x 64 at 128, intra-chunk output [256,320), state 64 * NH at 320,
+// normaliser 16 * NH at 448, q . n 2 x 16 at 480.
 #include "ptx.cuh"
 #include "host_utils.h"
 
@@ -25,7 +28,7 @@ constexpr int MC_SLICE = 64;       // value columns per CTA (= MM_SLICE of matri
 constexpr int MC_THREADS = 352;
 constexpr int MC_EW = 256;         // elementwise threads
 constexpr float MC_LOG2E = 1.4426950408889634f;
-constexpr uint32_t MC_T_S = 0, MC_T_OI = 128, MC_T_OA = 192, MC_T_ST = 256, MC_T_N = 384, MC_T_QN = 416;
+constexpr uint32_t MC_T_S = 0, MC_T_OI = 128, MC_T_OA = 256, MC_T_ST = 320, MC_T_N = 448, MC_T_QN = 480;
 
 struct McSmem {
   static constexpr int Q = 0;                    // [2 chunks of 64 dims][128 rows][128 B]
@@ -183,6 +186,7 @@ matrix_memory_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
     const uint32_t aN = smem_u32(smem + McSmem::N), aW = smem_u32(smem + McSmem::W);
     bool ok = true;
     for (int c = 0; c < chunks && ok; ++c) {
+      const uint32_t t_oi = tmem + MC_T_OI + (c & 1) * 64, t_qn = tmem + MC_T_QN + (c & 1) * 16;
       for (int h = 0; h < NH && ok; ++h) {
         const int it = c * NH + h;
         ok = mbar_wait(qk_full, it & 1, p.err, ERR_WAIT_FULL);
@@ -205,9 +209,9 @@ matrix_memory_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
 #pragma unroll
           for (int k4 = 0; k4 < 8; ++k4) {
             const uint64_t a = make_smem_desc_sw128(aQ + (k4 >> 2) * 16384 + (k4 & 3) * 32, 16, 1024);
-            umma_f16(tmem + MC_T_OI, a, make_smem_desc_sw128(aST + k4 * 2048, 16384, 1024), id_o, (h > 0 || k4 > 0) ? 1u : 0u);
-            umma_f16(tmem + MC_T_OI, a, make_smem_desc_sw128(aST + 16384 + k4 * 2048, 16384, 1024), id_o, 1u);
-            umma_f16(tmem + MC_T_QN, a, make_smem_desc_sw128(aN + (k4 >> 2) * 2048 + (k4 & 3) * 32, 16, 1024), id_qn,
+            umma_f16(t_oi, a, make_smem_desc_sw128(aST + k4 * 2048, 16384, 1024), id_o, (h > 0 || k4 > 0) ? 1u : 0u);
+            umma_f16(t_oi, a, make_smem_desc_sw128(aST + 16384 + k4 * 2048, 16384, 1024), id_o, 1u);
+            umma_f16(t_qn, a, make_smem_desc_sw128(aN + (k4 >> 2) * 2048 + (k4 & 3) * 32, 16, 1024), id_qn,
                      (h > 0 || k4 > 0) ? 1u : 0u);
           }
         }
@@ -341,89 +345,96 @@ matrix_memory_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
       }
     }
     tmem_st_wait();
-    bool ok = true;
+    // state -> operand of q S (undecayed); its decayed value goes back to tensor memory for the update
+    auto state_operand = [&](int c, int h) -> bool {
+      const int it = c * NH + h;
+      if (h == 0 && !mbar_wait(&g_full[c & 1], (c >> 1) & 1, p.err, ERR_WAIT_MISC)) return false;
+      if (it > 0) {
+        if (!mbar_wait(upd_done, (it - 1) & 1, p.err, ERR_WAIT_MISC)) return false;
+        tc_fence_after();
+      }
+      const float* gs = gates_s + (c & 1) * McSmem::GATE_FLOATS;
+      const float decay = ex2((gs[3 * MC_L] - gs[MC_L + MC_L - 1]) * MC_LOG2E);
+      {
+        uint32_t w[32];
+        const uint32_t ta = lane_addr + MC_T_ST + h * 64 + half * 32;
+        tmem_ld32(ta, w);
+        tmem_ld_wait();
+        uint8_t* dst = smem + McSmem::ST + r * 128;
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+          float v[8];
+          uint4 hi, lo;
+#pragma unroll
+          for (int e = 0; e < 8; ++e) {
+            v[e] = __uint_as_float(w[u * 8 + e]);
+            w[u * 8 + e] = __float_as_uint(v[e] * decay);
+          }
+          mc_split8(v, hi, lo);
+          const int o = ((half * 4 + u) ^ (r & 7)) << 4;
+          *reinterpret_cast<uint4*>(dst + o) = hi;
+          *reinterpret_cast<uint4*>(dst + 16384 + o) = lo;
+        }
+        tmem_st32(ta, w);
+        if (half == 0) {
+          uint32_t nv[16];
+          tmem_ld16(lane_addr + MC_T_N + h * 16, nv);
+          tmem_ld_wait();
+          const float nn = __uint_as_float(nv[0]) + __uint_as_float(nv[1]);
+          mc_put_row01(smem + McSmem::N, r, nn);
+#pragma unroll
+          for (int j = 0; j < 16; ++j) nv[j] = 0;
+          nv[0] = __float_as_uint(nn * decay);
+          tmem_st16(lane_addr + MC_T_N + h * 16, nv);
+        }
+        tmem_st_wait();
+      }
+      fence_proxy_async();
+      tc_fence_before();
+      mbar_arrive(sop_ready);
+      return true;
+    };
+    // weighted values (token r, 32 columns) and key weights
+    auto weighted_values = [&](int c) -> bool {
+      if (!mbar_wait(v_full, c & 1, p.err, ERR_WAIT_FULL)) return false;
+      const float* gs = gates_s + (c & 1) * McSmem::GATE_FLOATS;
+      const float wt = ex2((gs[r] - gs[MC_L + MC_L - 1]) * MC_LOG2E);
+      const uint8_t* src = smem + McSmem::V + r * 128;
+      uint8_t* dst = smem + McSmem::VW + r * 128;
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        const int o = ((half * 4 + u) ^ (r & 7)) << 4;
+        const uint4 x = *reinterpret_cast<const uint4*>(src + o);
+        const uint32_t xs[4] = {x.x, x.y, x.z, x.w};
+        float v[8];
+        uint4 hi, lo;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          v[2 * e] = bf16_bits_to_float(static_cast<uint16_t>(xs[e] & 0xffff)) * wt;
+          v[2 * e + 1] = bf16_bits_to_float(static_cast<uint16_t>(xs[e] >> 16)) * wt;
+        }
+        mc_split8(v, hi, lo);
+        *reinterpret_cast<uint4*>(dst + o) = hi;
+        *reinterpret_cast<uint4*>(dst + 16384 + o) = lo;
+      }
+      if (half == 0) mc_put_row01(smem + McSmem::W, r, wt);
+      fence_proxy_async();
+      mbar_arrive(vw_ready);
+      return true;
+    };
+    // what a chunk needs from the elementwise warps behind its first state operand
+    auto rest_of_operands = [&](int c) -> bool {
+      bool fine = weighted_values(c);
+#pragma unroll
+      for (int h = 1; h < NH; ++h) fine = fine && state_operand(c, h);
+      return fine;
+    };
+    const float log_qs = log2f(p.q_scale);
+    bool ok = state_operand(0, 0) && rest_of_operands(0);
     for (int c = 0; c < chunks && ok; ++c) {
       const int buf = c & 1;
       const float* gs = gates_s + buf * McSmem::GATE_FLOATS;
-      ok = mbar_wait(&g_full[buf], (c >> 1) & 1, p.err, ERR_WAIT_MISC);
-      if (!ok) break;
-      const float m0 = gs[3 * MC_L], g_end = gs[MC_L + MC_L - 1];
-      const float decay = ex2((m0 - g_end) * MC_LOG2E);
-#pragma unroll
-      for (int h = 0; h < NH; ++h) {
-        // ---- state -> operand of q S (undecayed); its decayed value goes back to tensor memory for the update
-        const int it = c * NH + h;
-        if (it > 0) {
-          ok = mbar_wait(upd_done, (it - 1) & 1, p.err, ERR_WAIT_MISC);
-          if (!ok) break;
-          tc_fence_after();
-        }
-        {
-          uint32_t w[32];
-          const uint32_t ta = lane_addr + MC_T_ST + h * 64 + half * 32;
-          tmem_ld32(ta, w);
-          tmem_ld_wait();
-          uint8_t* dst = smem + McSmem::ST + r * 128;
-#pragma unroll
-          for (int u = 0; u < 4; ++u) {
-            float v[8];
-            uint4 hi, lo;
-#pragma unroll
-            for (int e = 0; e < 8; ++e) {
-              v[e] = __uint_as_float(w[u * 8 + e]);
-              w[u * 8 + e] = __float_as_uint(v[e] * decay);
-            }
-            mc_split8(v, hi, lo);
-            const int o = ((half * 4 + u) ^ (r & 7)) << 4;
-            *reinterpret_cast<uint4*>(dst + o) = hi;
-            *reinterpret_cast<uint4*>(dst + 16384 + o) = lo;
-          }
-          tmem_st32(ta, w);
-          if (half == 0) {
-            uint32_t nv[16];
-            tmem_ld16(lane_addr + MC_T_N + h * 16, nv);
-            tmem_ld_wait();
-            const float nn = __uint_as_float(nv[0]) + __uint_as_float(nv[1]);
-            mc_put_row01(smem + McSmem::N, r, nn);
-#pragma unroll
-            for (int j = 0; j < 16; ++j) nv[j] = 0;
-            nv[0] = __float_as_uint(nn * decay);
-            tmem_st16(lane_addr + MC_T_N + h * 16, nv);
-          }
-          tmem_st_wait();
-        }
-        fence_proxy_async();
-        tc_fence_before();
-        mbar_arrive(sop_ready);
-        if (h == 0) {
-          // ---- weighted values (token r, 32 columns) and key weights
-          ok = mbar_wait(v_full, c & 1, p.err, ERR_WAIT_FULL);
-          if (!ok) break;
-          const float wt = ex2((gs[r] - g_end) * MC_LOG2E);
-          const uint8_t* src = smem + McSmem::V + r * 128;
-          uint8_t* dst = smem + McSmem::VW + r * 128;
-#pragma unroll
-          for (int u = 0; u < 4; ++u) {
-            const int o = ((half * 4 + u) ^ (r & 7)) << 4;
-            const uint4 x = *reinterpret_cast<const uint4*>(src + o);
-            const uint32_t xs[4] = {x.x, x.y, x.z, x.w};
-            float v[8];
-            uint4 hi, lo;
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-              v[2 * e] = bf16_bits_to_float(static_cast<uint16_t>(xs[e] & 0xffff)) * wt;
-              v[2 * e + 1] = bf16_bits_to_float(static_cast<uint16_t>(xs[e] >> 16)) * wt;
-            }
-            mc_split8(v, hi, lo);
-            *reinterpret_cast<uint4*>(dst + o) = hi;
-            *reinterpret_cast<uint4*>(dst + 16384 + o) = lo;
-          }
-          if (half == 0) mc_put_row01(smem + McSmem::W, r, wt);
-          fence_proxy_async();
-          mbar_arrive(vw_ready);
-        }
-      }
-      if (!ok) break;
+      const float m0 = gs[3 * MC_L];
       // ---- decayed scores: token r against 64 keys
       const float g = gs[MC_L + r];
       ok = mbar_wait(s_full, c & 1, p.err, ERR_WAIT_TMEM_FULL);
@@ -445,8 +456,8 @@ matrix_memory_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
           const float av[8] = {a0.x, a0.y, a0.z, a0.w, a1.x, a1.y, a1.z, a1.w};
 #pragma unroll
           for (int e = 0; e < 8; ++e) {
-            const float d = s0 + e <= r ? ex2((av[e] - g) * MC_LOG2E) * p.q_scale : 0.f;
-            v[e] = s0 + e <= r ? __uint_as_float(w[u * 8 + e]) * d : 0.f;
+            const float x2 = fmaf(av[e] - g, MC_LOG2E, log_qs);
+            v[e] = __uint_as_float(w[u * 8 + e]) * ex2(s0 + e <= r ? x2 : -1e30f);
             rs += v[e];
           }
           mc_split8(v, hi, lo);
@@ -459,6 +470,10 @@ matrix_memory_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
       fence_proxy_async();
       tc_fence_before();
       mbar_arrive(p_ready);
+      if (NH > 1 && c + 1 < chunks) {
+        ok = state_operand(c + 1, 0);
+        if (!ok) break;
+      }
       // ---- output
       ok = mbar_wait(p_ready, c & 1, p.err, ERR_WAIT_MISC) && mbar_wait(o_done, c & 1, p.err, ERR_WAIT_TMEM_FULL);
       if (!ok) break;
@@ -466,30 +481,39 @@ matrix_memory_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
       {
         const float inter = ex2((m0 - g) * MC_LOG2E) * p.q_scale;
         uint32_t qn[16], oi[32], oa[32];
-        tmem_ld16(lane_addr + MC_T_QN, qn);
-        tmem_ld32(lane_addr + MC_T_OI + half * 32, oi);
+        tmem_ld16(lane_addr + MC_T_QN + buf * 16, qn);
+        tmem_ld32(lane_addr + MC_T_OI + buf * 64 + half * 32, oi);
         tmem_ld32(lane_addr + MC_T_OA + half * 32, oa);
         tmem_ld_wait();
         const float den = inter * (__uint_as_float(qn[0]) + __uint_as_float(qn[1])) + rsum[buf * 2 * MC_L + r] +
                           rsum[(buf * 2 + 1) * MC_L + r];
         const float inv = 1.f / (fmaxf(fabsf(den), ex2(-gs[2 * MC_L + r] * MC_LOG2E)) + 1e-6f);
-        const int t = c * MC_L + r;
-        if (t < len) {
-          float* dst = p.out + (static_cast<long long>(r_beg + t) * p.heads + head) * p.vdim + col0;
+        // a warp's 32 x 32 outputs change hands in shared memory (the scores' buffer is free now), so that its stores
+        // are whole 128-byte lines; 16-byte unit u of row r sits at unit u ^ (r & 7)
+        uint8_t* stage = smem + McSmem::P + warp * 4096;
 #pragma unroll
-          for (int j = 0; j < 32; j += 4) {
-            if (col0 + j < p.vdim) {
-              *reinterpret_cast<float4*>(dst + j) =
-                  make_float4((inter * __uint_as_float(oi[j]) + __uint_as_float(oa[j])) * inv,
-                              (inter * __uint_as_float(oi[j + 1]) + __uint_as_float(oa[j + 1])) * inv,
-                              (inter * __uint_as_float(oi[j + 2]) + __uint_as_float(oa[j + 2])) * inv,
-                              (inter * __uint_as_float(oi[j + 3]) + __uint_as_float(oa[j + 3])) * inv);
-            }
-          }
+        for (int u = 0; u < 8; ++u) {
+          *reinterpret_cast<float4*>(stage + lane * 128 + ((u ^ (lane & 7)) << 4)) =
+              make_float4((inter * __uint_as_float(oi[4 * u]) + __uint_as_float(oa[4 * u])) * inv,
+                          (inter * __uint_as_float(oi[4 * u + 1]) + __uint_as_float(oa[4 * u + 1])) * inv,
+                          (inter * __uint_as_float(oi[4 * u + 2]) + __uint_as_float(oa[4 * u + 2])) * inv,
+                          (inter * __uint_as_float(oi[4 * u + 3]) + __uint_as_float(oa[4 * u + 3])) * inv);
         }
+        __syncwarp();
+        const int u = lane & 7, t0 = c * MC_L + quad * 32;
+        float* dst = p.out + (static_cast<long long>(r_beg + t0) * p.heads + head) * p.vdim + col0 + u * 4;
+#pragma unroll
+        for (int x = 0; x < 8; ++x) {
+          const int rr = x * 4 + (lane >> 3);
+          const float4 v = *reinterpret_cast<const float4*>(stage + rr * 128 + ((u ^ (rr & 7)) << 4));
+          if (t0 + rr < len && col0 + u * 4 < p.vdim)
+            *reinterpret_cast<float4*>(dst + static_cast<long long>(rr) * p.heads * p.vdim) = v;
+        }
+        __syncwarp();
       }
       tc_fence_before();
       mbar_arrive(&g_empty[buf]);
+      if (c + 1 < chunks) ok = (NH > 1 || state_operand(c + 1, 0)) && rest_of_operands(c + 1);
     }
     if (ok) {
       ok = mbar_wait(upd_done, (chunks * NH - 1) & 1, p.err, ERR_WAIT_MISC);
