@@ -221,7 +221,7 @@ def _declare_kernels(lib: ctypes.CDLL):
     d("gk_shared_kv_decode_scratch", [I, I, I, I], L)
     d("gk_shared_decode_set_target_ctas", [I], None)
     d("gk_window_prefill", [P, L, P, P, P, P, P, P, P, F, P, P])
-    d("gk_matrix_memory_scan", [I, P, L, P, F, F, P])
+    d("gk_matrix_memory_scan", [I, P, L, P, F, F, F, P])
     d("gk_matrix_memory_chunk", [P, L, P, F, F, P])
     d("gk_memory_output", [I, P, P, L, P, P, P, F, P])
     d("gk_attn_fwd", [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, I, P, P])

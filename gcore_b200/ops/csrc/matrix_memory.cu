@@ -3,7 +3,9 @@
 // type of the projection.
 //   * matrix_memory_scan_kernel  token by token with the state slice in registers: decoding (one token per request, the
 //                                gate projections fused in) and the true 32-bit path for prompt portions;
-//   * memory_output_kernel       per-head RMS norm, gain and sigmoid output gate.
+//                                One token per request with at most 8 slices: the slices of a head form a cluster, share
+//                                their sums of squares through distributed shared memory and write the finished output;
+//   * memory_output_kernel       per-head RMS norm, gain and sigmoid output gate behind every other case.
 // bf16 prompt portions run the chunkwise kernel in matrix_memory_chunk.cu.
 //
 // State layout per layer run: S [slots, heads, dim, vdim], n [slots, heads, slices, dim], m [slots, heads, slices]: a head's
@@ -54,18 +56,35 @@ struct ScanParams {
   float* S;
   float* n;
   float* m;
-  float* out;              // [rows, heads, vdim] 32-bit
+  float* out;              // [rows, heads, vdim] 32-bit (unless the output is finished here)
+  T* y;                    // FINISH: [rows, heads * vdim] normed and gated output
+  const float* gain;       // FINISH: [heads * vdim]
+  int g_off, vdim_true;    // FINISH
+  float eps;               // FINISH
   int width, heads, dim, vdim, slices;
   float cap, q_scale;
 };
 
+__device__ __forceinline__ void mm_cluster_arrive() { asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory"); }
+__device__ __forceinline__ void mm_cluster_wait() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
+__device__ __forceinline__ void mm_store_remote(const float* local, uint32_t cta, float v) {
+  const uint32_t a = static_cast<uint32_t>(__cvta_generic_to_shared(local));
+  uint32_t r;
+  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(r) : "r"(a), "r"(cta));
+  asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(r), "f"(v) : "memory");
+}
+__device__ __forceinline__ void mm_st1(float* p, float v) { *p = v; }
+__device__ __forceinline__ void mm_st1(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
+
 // grid (heads * slices, segments).  Thread (warp w, lane): rows rg, rg + 16, ... with rg = 2 w + lane / 16; columns
 // 4 * (lane % 16) .. + 3 of the slice.  R = rows per thread.
-template <typename T, int R>
+template <typename T, int R, bool FINISH>
 __global__ void __launch_bounds__(MM_THREADS, R <= 8 ? 3 : R <= 16 ? 2 : 1) matrix_memory_scan_kernel(const ScanParams<T> p) {
   __shared__ float sq[2][16 * R], sk[2][16 * R];
   __shared__ float red[2][8][MM_SLICE + 4];
   __shared__ float gred[2][8];
+  __shared__ float peer_ss[8];      // FINISH: sum of squares of every slice of the head
+  __shared__ float warp_ss[2];
   pdl_launch_dependents();
   pdl_wait();
   const int head = blockIdx.x / p.slices, slice = blockIdx.x % p.slices, seg = blockIdx.y;
@@ -77,10 +96,14 @@ __global__ void __launch_bounds__(MM_THREADS, R <= 8 ? 3 : R <= 16 ? 2 : 1) matr
   const bool live = col < p.vdim;
   if (slot < 0) {
     for (int r = r_beg; r < r_end; ++r)
-      if (tid < MM_SLICE && slice * MM_SLICE + tid < p.vdim)
-        p.out[(static_cast<long long>(r) * p.heads + head) * p.vdim + slice * MM_SLICE + tid] = 0.f;
-    return;
+      if (tid < MM_SLICE && slice * MM_SLICE + tid < p.vdim) {
+        const long long at = (static_cast<long long>(r) * p.heads + head) * p.vdim + slice * MM_SLICE + tid;
+        if (FINISH) mm_st1(p.y + at, 0.f);
+        else p.out[at] = 0.f;
+      }
+    return;      // uniform over the slices of the head
   }
+  if (FINISH) mm_cluster_arrive();
   const long long sh = static_cast<long long>(slot) * p.heads + head;
   float* Sg = p.S + sh * p.dim * p.vdim + col;
   float* ng = p.n + (sh * p.slices + slice) * p.dim;
@@ -99,6 +122,17 @@ __global__ void __launch_bounds__(MM_THREADS, R <= 8 ? 3 : R <= 16 ? 2 : 1) matr
       n[j] = ng[r];
     }
   }
+  auto store_state = [&]() {
+#pragma unroll
+    for (int j = 0; j < R; ++j) {
+      const int r = rg + 16 * j;
+      if (r < p.dim) {
+        if (live) *reinterpret_cast<float4*>(Sg + static_cast<long long>(r) * p.vdim) = S[j];
+        if (c0 == 0) ng[r] = n[j];
+      }
+    }
+    if (tid == 0) *mg = m;
+  };
   const float bi = p.gate_b[head], bf = p.gate_b[p.heads + head];
   for (int row = r_beg, it = 0; row < r_end; ++row, ++it) {
     const int buf = it & 1;
@@ -151,6 +185,7 @@ __global__ void __launch_bounds__(MM_THREADS, R <= 8 ? 3 : R <= 16 ? 2 : 1) matr
       S[j].z = keep * S[j].z + k * v.z; a2 += S[j].z * q;
       S[j].w = keep * S[j].w + k * v.w; a3 += S[j].w * q;
     }
+    if (FINISH) store_state();   // on its way while the slices exchange their sums
     a0 += __shfl_xor_sync(0xffffffff, a0, 16);
     a1 += __shfl_xor_sync(0xffffffff, a1, 16);
     a2 += __shfl_xor_sync(0xffffffff, a2, 16);
@@ -161,25 +196,42 @@ __global__ void __launch_bounds__(MM_THREADS, R <= 8 ? 3 : R <= 16 ? 2 : 1) matr
       if (lane == 0) red[buf][warp][MM_SLICE] = nq;
     }
     __syncthreads();
-    if (tid < MM_SLICE && slice * MM_SLICE + tid < p.vdim) {
-      float o = 0.f, d = 0.f;
+    float o = 0.f;
+    const int oc = slice * MM_SLICE + tid;
+    const bool mine = tid < MM_SLICE && oc < p.vdim;
+    if (mine) {
+      float d = 0.f;
 #pragma unroll
       for (int w = 0; w < 8; ++w) { o += red[buf][w][tid]; d += red[buf][w][MM_SLICE]; }
-      p.out[(static_cast<long long>(row) * p.heads + head) * p.vdim + slice * MM_SLICE + tid] =
-          o / (fmaxf(fabsf(d), expf(-m)) + 1e-6f);
+      o = o / (fmaxf(fabsf(d), expf(-m)) + 1e-6f);
+      if (!FINISH) p.out[(static_cast<long long>(row) * p.heads + head) * p.vdim + oc] = o;
     }
-  }
-  if (r_end > r_beg) {
+    if (FINISH) {   // one row per segment
+      float gate = 0.f, gain = 0.f;
+      if (mine) {
+        gate = mm_f(pr[p.g_off + static_cast<long long>(head) * p.vdim + oc]);
+        gain = p.gain[head * p.vdim + oc];
+      }
+      if (warp < 2) {
+        float ss = o * o;
 #pragma unroll
-    for (int j = 0; j < R; ++j) {
-      const int r = rg + 16 * j;
-      if (r < p.dim) {
-        if (live) *reinterpret_cast<float4*>(Sg + static_cast<long long>(r) * p.vdim) = S[j];
-        if (c0 == 0) ng[r] = n[j];
+        for (int x = 16; x > 0; x >>= 1) ss += __shfl_xor_sync(0xffffffff, ss, x);
+        if (lane == 0) warp_ss[warp] = ss;
+      }
+      __syncthreads();
+      mm_cluster_wait();                       // every slice has started: its shared memory may be written
+      if (tid < p.slices) mm_store_remote(&peer_ss[slice], tid, warp_ss[0] + warp_ss[1]);
+      mm_cluster_arrive();
+      mm_cluster_wait();
+      if (mine) {
+        float ss = 0.f;
+        for (int x = 0; x < p.slices; ++x) ss += peer_ss[x];
+        const float r = 1.f / sqrtf(ss / p.vdim_true + p.eps);
+        mm_st1(p.y + (static_cast<long long>(row) * p.heads + head) * p.vdim + oc, o * r * gain / (1.f + expf(-gate)));
       }
     }
-    if (tid == 0) *mg = m;
   }
+  if (!FINISH && r_end > r_beg) store_state();
 }
 
 // y = o / rms(o over the head's true size) * gain * sigmoid(g).  One warp per (row, head).
@@ -213,28 +265,55 @@ __global__ void __launch_bounds__(256) memory_output_kernel(const float* __restr
   }
 }
 
+template <typename T, int R>
+int launch_scan_r(const ScanParams<T>& p, int segments, cudaStream_t st) {
+  const dim3 grid(p.heads * p.slices, segments);
+  if (!p.y) {
+    launch_k(matrix_memory_scan_kernel<T, R, false>, grid, dim3(MM_THREADS), 0, st, p);
+    return launch_status();
+  }
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = grid;
+  cfg.blockDim = dim3(MM_THREADS);
+  cfg.stream = st;
+  cudaLaunchAttribute attr[2];
+  attr[0].id = cudaLaunchAttributeClusterDimension;
+  attr[0].val.clusterDim.x = p.slices;
+  attr[0].val.clusterDim.y = 1;
+  attr[0].val.clusterDim.z = 1;
+  attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[1].val.programmaticStreamSerializationAllowed = pdl_flag() ? 1 : 0;
+  cfg.attrs = attr;
+  cfg.numAttrs = 2;
+  if (cudaLaunchKernelEx(&cfg, matrix_memory_scan_kernel<T, R, true>, p) != cudaSuccess) {
+    const int rc = launch_status();
+    return rc ? rc : -7;
+  }
+  return launch_status();
+}
+
 template <typename T>
 int launch_scan(const ScanParams<T>& p, int segments, cudaStream_t st) {
-  const dim3 grid(p.heads * p.slices, segments);
-  if (p.dim <= 32) launch_k(matrix_memory_scan_kernel<T, 2>, grid, dim3(MM_THREADS), 0, st, p);
-  else if (p.dim <= 64) launch_k(matrix_memory_scan_kernel<T, 4>, grid, dim3(MM_THREADS), 0, st, p);
-  else if (p.dim <= 128) launch_k(matrix_memory_scan_kernel<T, 8>, grid, dim3(MM_THREADS), 0, st, p);
-  else if (p.dim <= 256) launch_k(matrix_memory_scan_kernel<T, 16>, grid, dim3(MM_THREADS), 0, st, p);
-  else if (p.dim <= 512) launch_k(matrix_memory_scan_kernel<T, 32>, grid, dim3(MM_THREADS), 0, st, p);
-  else return -2;
-  return launch_status();
+  if (p.dim <= 32) return launch_scan_r<T, 2>(p, segments, st);
+  if (p.dim <= 64) return launch_scan_r<T, 4>(p, segments, st);
+  if (p.dim <= 128) return launch_scan_r<T, 8>(p, segments, st);
+  if (p.dim <= 256) return launch_scan_r<T, 16>(p, segments, st);
+  if (p.dim <= 512) return launch_scan_r<T, 32>(p, segments, st);
+  return -2;
 }
 
 }  // namespace gk
 
 using namespace gk;
 
-// ptrs: {proj, h, gate_w, gates, gate_b, cu, first_pos, slots, S, n, m, out}
-// dims: {segments, q_off, k_off, v_off, width, heads, dim, vdim}
+// ptrs: {proj, h, gate_w, gates, gate_b, cu, first_pos, slots, S, n, m, out, y, gain}; y (finished output, one row per
+// segment, at most 512 value columns) replaces out.
+// dims: {segments, q_off, k_off, v_off, width, heads, dim, vdim, g_off, vdim_true}
 GK_EXPORT int gk_matrix_memory_scan(int is_fp32, void* const* ptrs, long long ld, const int* dims, float cap,
-                                    float q_scale, void* stream) {
+                                    float q_scale, float eps, void* stream) {
   if (dims[0] == 0) return 0;
   if (dims[7] % 4 || ld % 4 || dims[3] % 4 || (!ptrs[3] && dims[4] % 4)) return -1;
+  if (ptrs[12] && (ptrs[5] || dims[7] > 8 * MM_SLICE || !ptrs[13])) return -3;
   auto fill = [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
     ScanParams<T> p;
@@ -251,6 +330,9 @@ GK_EXPORT int gk_matrix_memory_scan(int is_fp32, void* const* ptrs, long long ld
     p.n = static_cast<float*>(ptrs[9]);
     p.m = static_cast<float*>(ptrs[10]);
     p.out = static_cast<float*>(ptrs[11]);
+    p.y = static_cast<T*>(ptrs[12]);
+    p.gain = static_cast<const float*>(ptrs[13]);
+    p.g_off = dims[8]; p.vdim_true = dims[9]; p.eps = eps;
     p.q_off = dims[1]; p.k_off = dims[2]; p.v_off = dims[3];
     p.width = dims[4]; p.heads = dims[5]; p.dim = dims[6]; p.vdim = dims[7];
     p.slices = (p.vdim + MM_SLICE - 1) / MM_SLICE;

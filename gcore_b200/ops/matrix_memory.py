@@ -16,6 +16,8 @@ SLICE = 64        # value columns per state slice (csrc/matrix_memory.cu: MM_SLI
 MAX_KEY_DIM = 512
 CHUNK_MAX_KEY_DIM = 256   # keys the chunkwise tensor-core kernel takes
 SCAN_MAX_TOKENS = 8       # portions up to here run token by token
+FINISH_SLICES = 8         # slices of a head a single-token step can finish in one launch (a cluster)
+FINISH_CTAS = 400         # ... and does up to this grid: larger ones stream faster as independent CTAs + output kernel
 
 
 def padded_key_dim(dim: int) -> int:
@@ -77,13 +79,17 @@ def _ref(proj, offs, gates, gate_b, cap, q_scale, heads, dim, vdim, rows: StepRo
     return out
 
 
-def _scan(proj, offs, h, gate_w, gates, gate_b, cap, q_scale, heads, dim, vdim, cu, first_pos, slots, st, out):
-    ptrs = (ctypes.c_void_p * 12)(*[t.data_ptr() if t is not None else None for t in
-                                    (proj, h, gate_w, gates, gate_b, cu, first_pos, slots, st.S, st.n, st.m, out)])
-    dims = (ctypes.c_int * 8)(slots.numel(), *offs, h.shape[1] if h is not None else 0, heads, dim, vdim)
+def _scan(proj, offs, h, gate_w, gates, gate_b, cap, q_scale, heads, dim, vdim, cu, first_pos, slots, st, out=None,
+          finish=None):
+    """Token by token.  ``finish`` = (y, gain, g_off, vdim_true, eps): the normed, gated output in place of ``out``."""
+    y, gain, g_off, vdim_true, eps = finish if finish is not None else (None, None, 0, vdim, 0.0)
+    ptrs = (ctypes.c_void_p * 14)(*[t.data_ptr() if t is not None else None for t in
+                                    (proj, h, gate_w, gates, gate_b, cu, first_pos, slots, st.S, st.n, st.m, out, y, gain)])
+    dims = (ctypes.c_int * 10)(slots.numel(), *offs, h.shape[1] if h is not None else 0, heads, dim, vdim, g_off, vdim_true)
     LAUNCHES["matrix_memory"] += 1
     _lib.check(_lib.kernels().gk_matrix_memory_scan(int(proj.dtype == torch.float32), ptrs, proj.stride(0), dims,
-                                                    float(cap), float(q_scale), _lib.stream_ptr()), "matrix_memory_scan")
+                                                    float(cap), float(q_scale), float(eps), _lib.stream_ptr()),
+               "matrix_memory_scan")
 
 
 def _chunk(proj, offs, gates, gate_b, cap, q_scale, heads, dim, vdim, rows: StepRows, st, out):
@@ -97,13 +103,12 @@ def _chunk(proj, offs, gates, gate_b, cap, q_scale, heads, dim, vdim, rows: Step
                                                      _lib.stream_ptr()), "matrix_memory_chunk")
 
 
-def _output(o, proj, g_off, gain, vdim_true, eps):
+def _output(o, proj, g_off, gain, vdim_true, eps, y=None):
     T, heads, vdim = o.shape
     if not o.is_cuda:
-        y = o * torch.rsqrt(o.pow(2).sum(-1, keepdim=True) / vdim_true + eps)
+        n = o * torch.rsqrt(o.pow(2).sum(-1, keepdim=True) / vdim_true + eps)
         g = torch.sigmoid(proj[:, g_off:g_off + heads * vdim].float())
-        return (y.reshape(T, -1) * gain * g).to(proj.dtype)
-    y = torch.empty(T, heads * vdim, dtype=proj.dtype, device=proj.device)
+        return (n.reshape(T, -1) * gain * g).to(proj.dtype)
     dims = (ctypes.c_int * 5)(T, heads, vdim, vdim_true, g_off)
     LAUNCHES["matrix_memory"] += 1
     _lib.check(_lib.kernels().gk_memory_output(int(proj.dtype == torch.float32), _lib.ptr(o), _lib.ptr(proj),
@@ -123,15 +128,24 @@ def matrix_memory(proj, q_off: int, k_off: int, v_off: int, g_off: int, h, gate_
         gates = h.float() @ gate_w.float().t()
         o = _ref(proj, offs, gates, gate_b, cap, q_scale, heads, dim, vdim, rows, state)
         return _output(o, proj, g_off, gain, vdim_true, eps)
-    o = torch.empty(T, heads, vdim, dtype=torch.float32, device=proj.device)
+    y = torch.empty(T, heads * vdim, dtype=proj.dtype, device=proj.device)
     n = rows.n_portions
     common = (gate_b, cap, q_scale, heads, dim, vdim)
     if P:
+        o = torch.empty(P, heads, vdim, dtype=torch.float32, device=proj.device)
         gates = linear_forward(h[:P], gate_w, out_dtype=torch.float32)
         if proj.dtype == torch.bfloat16 and dim <= CHUNK_MAX_KEY_DIM and rows.max_portion > SCAN_MAX_TOKENS:
             _chunk(proj, offs, gates, *common, rows, state, o)
         else:
             _scan(proj, offs, None, None, gates, *common, rows.cu, rows.first_pos, rows.states[:n], state, o)
+        _output(o, proj, g_off, gain, vdim_true, eps, y)
     if T > P:
-        _scan(proj[P:], offs, h[P:], gate_w, None, *common, None, rows.first_pos[n:], rows.states[n:], state, o[P:])
-    return _output(o, proj, g_off, gain, vdim_true, eps)
+        single = (proj[P:], offs, h[P:], gate_w, None, *common, None, rows.first_pos[n:], rows.states[n:], state)
+        slices = (vdim + SLICE - 1) // SLICE
+        if slices <= FINISH_SLICES and slices * heads * (T - P) <= FINISH_CTAS:
+            _scan(*single, finish=(y[P:], gain, g_off, vdim_true, eps))
+        else:
+            o = torch.empty(T - P, heads, vdim, dtype=torch.float32, device=proj.device)
+            _scan(*single, o)
+            _output(o, proj[P:], g_off, gain, vdim_true, eps, y[P:])
+    return y

@@ -209,10 +209,10 @@ def kernel_table(s, prompts, length, B, ctx, bs=64):
     fl = T * s["mh"] * (4.0 * s["mk"] * s["mv"] + 128.0 * (s["mk"] + s["mv"]))
     table.append(("prefill", "matrix_memory_chunk", t,
                   ideal(T * s["mh"] * ((2 * s["mk"] + s["mv"]) * 2 + s["mv"] * 4), fl), None, None, None))
-    gain = torch.ones(s["mh"] * s["mv"], device=dev)
-    t = graph_us([lambda p=p: mm._output(o, p, off[5], gain, s["mv"], 1e-6) for p in projs])
+    gain, y = torch.ones(s["mh"] * s["mv"], device=dev), torch.empty(T, s["mh"] * s["mv"], **bf)
+    t = graph_us([lambda p=p: mm._output(o, p, off[5], gain, s["mv"], 1e-6, y) for p in projs])
     table.append(("prefill", "memory_output", t, ideal(T * s["mh"] * s["mv"] * 8), None, None, None))
-    del projs, o
+    del projs, o, y
     # ---- residual steps
     for phase, n, cp in (("prefill", T, 2), ("decode", B, 16)):
         xs = [torch.randn(n, width, device=dev) for _ in range(cp)]
@@ -250,7 +250,7 @@ def kernel_table(s, prompts, length, B, ctx, bs=64):
     run = lambda st: mm.matrix_memory(proj, *off[2:6], h, gw, gate_b, 15.0, s["mk"] ** -0.5, s["mh"], s["mk"], s["mv"],
                                       s["mv"], rows, st, gain, 1e-6)
     t = graph_us([lambda st=st: run(st) for st in sts])
-    table.append(("decode", "matrix_memory step (scan + output)", t, ideal(2 * B * s["mh"] * s["mk"] * s["mv"] * 4), None, None,
+    table.append(("decode", "matrix_memory step", t, ideal(2 * B * s["mh"] * s["mk"] * s["mv"] * 4), None, None,
                   None))
     return table
 
