@@ -272,5 +272,7 @@ def build_model_config(arch_or_preset: str, overrides: Optional[Dict[str, Any]] 
         return get_preset(arch_or_preset, **overrides)
     if "hf_config" in overrides:
         return from_hf_config(overrides.pop("hf_config"))
+    if arch_or_preset in ARCH_READERS and overrides.get("layer_plan") is None:
+        raise ValueError(f"{arch_or_preset} needs its config.json: pass it as model_config.hf_config")
     overrides.setdefault("arch", arch_or_preset)
     return ModelConfig(**overrides)

@@ -401,6 +401,8 @@ class GPTModel(nn.Module):
                  pre_process: bool = True, post_process: bool = True, layer_range=None, recompute: str = "none",
                  device=None, value_head: bool = False):
         super().__init__()
+        if cfg.layer_plan is not None:
+            raise ValueError(f"{cfg.arch} is described by a layer plan: it is served (models/plan_decoder.py), not trained")
         self.cfg = cfg
         self.tp_size, self.ep_size = tp_size, ep_size
         self.sequence_parallel = sequence_parallel and tp_size > 1

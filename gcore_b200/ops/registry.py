@@ -44,13 +44,15 @@ def resolve(name: str, impl: Optional[str] = None) -> Callable:
 
 
 def _populate():
-    from . import attention, fused, gemm, optim, quant, rl, vocab
+    from . import attention, fused, gemm, matrix_memory, optim, quant, rl, sandwich, vocab, window_attention
     for mod, names in ((gemm, ("gemm", "grouped_gemm", "grouped_wgrad", "linear")),
                        (fused, ("rmsnorm", "rope", "swiglu")),
                        (attention, ("flash_attn_varlen", "flash_attn_qkvpacked", "paged_decode", "kv_append_rope")),
                        (vocab, ("linear_logprob_entropy", "sample")),
                        (optim, ("adam_step", "sumsq", "axpy_cast")),
                        (quant, ("quant_act_1x128", "quant_weight_128x128", "quant_fp4_1x32", "gemm_fp8_blockscaled")),
+                       (sandwich, ("embed_rows", "add_sublayer", "norm_rows")),
+                       (window_attention, ("window_attention",)), (matrix_memory, ("matrix_memory",)),
                        (rl, ("fused_grpo_loss", "gae"))):
         for n in names:
             fn = getattr(mod, n, None)

@@ -292,7 +292,6 @@ class InferEngine:
         self.D = cfg.head_dim
         self.mla_dim = (cfg.kv_lora_rank + cfg.qk_rope_head_dim) if getattr(cfg, "use_mla", False) else 0
         self._mla_abs: Dict[int, list] = {}   # id(attention module) -> [absorbed up-projection, stale]
-        self.plan = weights.plan
         if self.plan is not None:
             if tp_size != 1:
                 raise ValueError("layer-plan decoders are served without tensor parallelism")
@@ -341,6 +340,11 @@ class InferEngine:
         self.record_routed_experts = False
         self._peer_ar = None
         self.weight_scales: dict = {}  # name -> fp32 128x128 block scales when weights are held in e4m3
+
+    @property
+    def plan(self) -> Optional[PlanDecoder]:
+        """The decoder module when the model is described by a layer plan, else None."""
+        return self.w.plan if self.w is not None else None
 
     # ------------------------------------------------------------------ memory
     def _kv_bytes_per_block(self):
@@ -417,6 +421,11 @@ class InferEngine:
         copied into the bucket and from the bucket into the engine's own storage - the byte traffic of the reference's
         export -> flattened bucket -> engine ``load_weights`` hand-over on one GPU
         (gpatch_v4/client/update_weight_factory.py:271-379)."""
+        if isinstance(model, PlanDecoder):   # serving-only module: its copy is the engine's own storage
+            self.w = RolloutWeights.from_model(model, clone=True)
+            self.owns_weights, self.asleep["weights"] = True, False
+            self._graphs.clear()
+            return sum(t.numel() * t.element_size() for t in self.w.tensors())
         w = RolloutWeights.from_model(model, clone=False)
         own = RolloutWeights.from_model(model, clone=False)
         stage = torch.empty(bucket_mb << 20, dtype=torch.uint8, device=self.device)
@@ -481,6 +490,8 @@ class InferEngine:
         128; called after each weight hand-over when the engine serves in fp8 (the reference's fp8 rollout:
         gpatch_v4/generation_backend/sglang_model_specific/sglang_weight_update_dsv4.py:267-321)."""
         from ..ops.quant import quant_weight_128x128
+        if self.plan is not None:
+            raise NotImplementedError("layer-plan decoders are served in bfloat16 or float32")
         self.fp8_enabled = True
         for lw in self.w.layers:
             lw.fp8 = {}

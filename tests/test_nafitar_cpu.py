@@ -63,6 +63,36 @@ def test_serving_copy_owns_its_weights():
     assert all(a.data_ptr() != b.data_ptr() and torch.equal(a, b) for a, b in zip(shared.tensors(), own.tensors()))
 
 
+def test_registered_and_served_only():
+    from gcore_b200 import build_native
+    from gcore_b200.models.config import build_model_config
+    from gcore_b200.models.gpt import GPTModel
+    from gcore_b200.ops import registry
+    c = nu.uneven_conf(positions=32)
+    assert build_model_config("nafitar", {"hf_config": c}).layer_plan == from_hf_config(c).layer_plan
+    with pytest.raises(ValueError, match="config.json"):
+        build_model_config("nafitar")
+    with pytest.raises(ValueError, match="served"):
+        GPTModel(from_hf_config(c))
+    eng = nu.make_engine(c, oracle.random_weights(c), max_model_len=32)
+    with pytest.raises(NotImplementedError):
+        eng.quantize_weights_fp8()
+    assert {"window_attention", "matrix_memory", "add_sublayer"} <= set(registry.available())
+    assert all((build_native.OPS_SRC / f"{s}.cu").exists() for s in build_native.KERNEL_SETS["nafitar"])
+
+
+def test_new_weights_replace_the_old_ones():
+    c = nu.uneven_conf(positions=64)
+    Wa, Wb = oracle.random_weights(c, seed=1), oracle.random_weights(c, seed=2)
+    eng = nu.make_engine(c, Wa, max_model_len=64)
+    other = PlanDecoder(eng.cfg).load_tensors(Wb)
+    seq = nu.tokens(20, 75, 1)
+    eng.update_weights(RolloutWeights.from_model(other))
+    nu.assert_close(nu.run_alone(eng, seq, [20]), oracle.forward(Wb, c, seq))
+    eng.load_weights_from(PlanDecoder(eng.cfg).load_tensors(Wa))
+    nu.assert_close(nu.run_alone(eng, seq, [20]), oracle.forward(Wa, c, seq))
+
+
 # --------------------------------------------------------------------------------------------------------- plain oracle
 def test_plain_window_and_distance_penalty_by_hand():
     """One head, keys that are all alike except one: the window keeps exactly ``size`` tokens."""

@@ -325,3 +325,13 @@ def test_trace_replay_through_the_executable_entry(tmp_path):
         got = torch.from_numpy(np.fromfile(tmp_path / f"{n}.f32", "<f4").reshape(-1, c["vocab"]).copy())
         nu.assert_close(got, want)
     assert eng.get_load()["free_blocks"] == eng.num_blocks
+
+
+def test_serving_benchmark_runs_on_a_small_size():
+    from gcore_b200.tools import serve_bench as sb
+    s = dict(width=256, heads=4, kv=2, dim=128, window=100, mh=2, mk=64, mv=128, ff=512, layers=2)
+    for kind in ("nafitar", "dense"):
+        eng = sb.build(kind, s, 512, 4)
+        assert sb.prefill_step(eng, 2, 130, 2) > 0 and sb.decode_step(eng, 4, 200, 2) > 0
+    table = sb.kernel_table(s, 2, 130, 4, 200)
+    assert {r[0] for r in table} == {"prefill", "decode"} and all(r[2] > 0 for r in table)
