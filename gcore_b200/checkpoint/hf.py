@@ -144,13 +144,13 @@ def load_serving_model(path: str, device, dtype: Optional[str] = None):
     """Model of a checkpoint folder as the rollout engine serves it, without a training engine around it: decoders that
     are described by a layer plan.  Returns ``(ModelConfig, module)``."""
     from dataclasses import replace
-    from ..models.plan_decoder import PlanDecoder
+    from ..models.plan_decoder import build_decoder
     cfg = read_model_config(path)
     if cfg is None or cfg.layer_plan is None:
         raise ValueError(f"{path} does not hold a model that is served without a training engine")
     if dtype is not None:
         cfg = replace(cfg, dtype=dtype)
-    return cfg, PlanDecoder(cfg, device).load_tensors(read_hf_dir(path))
+    return cfg, build_decoder(cfg, device).load_tensors(read_hf_dir(path))
 
 
 def load_hf(engine, path: str):

@@ -6,7 +6,8 @@ from __future__ import annotations
 from dataclasses import dataclass, field, fields
 from typing import Tuple, Any, Dict, List, Optional
 
-from .layer_plan import LayerPlan, nafitar_plan
+from .layer_plan import (DenseSpec, ExpertsSpec, LatentAttentionSpec, LayerPlan, ParallelLayerSpec, kedesun_plan,
+                         nafitar_plan)
 
 
 @dataclass
@@ -68,8 +69,8 @@ class ModelConfig:
     mtp_num_layers: int = 0
     mtp_loss_scaling_factor: float = 0.1
     fp8_base_weights: bool = False  # frozen e4m3 base with 128x128 block scales
-    # decoders described layer by layer (mixers side by side, looped layers, norms before and after each sublayer,
-    # learned positions); None for the uniform families above.  Such models are served, not trained.
+    # decoders described layer by layer (other mixers per layer, looped layers, another residual stream); None for the
+    # uniform families above.  Such models are served, not trained.
     layer_plan: Optional[LayerPlan] = None
 
     def __post_init__(self):
@@ -137,14 +138,32 @@ class ModelConfig:
 
     def _plan_parameters(self, include_embedding: bool) -> int:
         h, total = self.hidden_size, self.hidden_size * (1 + self.layer_plan.loop_times)
-        for sp in self.layer_plan.layers:
+        for i, sp in enumerate(self.layer_plan.layers):
+            if isinstance(sp, ParallelLayerSpec):
+                total += self._parallel_layer_parameters(sp, i)
+                continue
             a, m = sp.attention, sp.memory
             total += (2 * a.heads + a.kv_heads) * a.dim * h + (a.heads + a.kv_heads) * a.dim
             total += m.heads * (2 * m.dim + 3 * m.vdim + 2) * h + m.heads * (m.vdim + 2)
             total += (4 if not sp.ffn else 6) * h + 3 * sp.ffn * h
         if include_embedding:
-            total += (2 * self.vocab_size + self.max_position_embeddings) * h
+            total += self.vocab_size * h if self.tie_word_embeddings else \
+                (2 * self.vocab_size + self.max_position_embeddings) * h
         return total
+
+    def _parallel_layer_parameters(self, sp: ParallelLayerSpec, index: int) -> int:
+        h, m, f = self.hidden_size, sp.mixer, sp.ffn
+        n = h + index + 2                       # norm, depth average
+        if isinstance(m, LatentAttentionSpec):
+            n += m.heads * (m.dim + m.rot_dim + m.vdim + 1) * h + (m.kv_rank + m.rot_dim) * h
+            n += m.kv_rank * (1 + m.heads * (m.dim + m.vdim))
+        else:
+            n += m.heads * (2 * m.dim + 3 * m.vdim) * h
+        if isinstance(f, DenseSpec):
+            n += 3 * f.ff * h
+        elif isinstance(f, ExpertsSpec):
+            n += f.experts * (2 * f.ff * h + h + 1) + ((2 * f.shared_ff + 1) * h if f.shared_ff else 0)
+        return n
 
     def active_parameters(self) -> int:
         if not self.is_moe:
@@ -162,7 +181,8 @@ class ModelConfig:
 
 
 MODEL_ARCH = ("llama", "llama4", "qwen2", "qwen2_5_vl", "qwen3", "qwen3_moe", "qwen3_vl", "qwen3_vl_moe", "qwen2_moe",
-              "qwen2_vl", "deepseek_v3", "mistral", "gemma3_text", "seed_oss", "gpt_oss", "nafitar")
+              "qwen2_vl", "deepseek_v3", "mistral", "gemma3_text", "seed_oss", "gpt_oss", "nafitar",
+              "kedesun")
 
 PRESETS: Dict[str, Dict[str, Any]] = {
     # tiny Llama-style decoder
@@ -208,8 +228,24 @@ def from_nafitar_config(conf: Dict[str, Any], dtype: str = "bfloat16") -> ModelC
                        qkv_bias=True, dtype=dtype, layer_plan=plan)
 
 
+# rotary positions only: a position enters the rotation as a 32-bit float, exact below this bound
+ROTARY_POSITIONS = 1 << 24
+
+
+def from_kedesun_config(conf: Dict[str, Any], dtype: str = "bfloat16") -> ModelConfig:
+    """Maps a Kedesun ``config.json`` (``architecture``, ``layers``, ``norm``, ``vocab``, ``width``)."""
+    plan = kedesun_plan(conf)
+    m = plan.layers[0].mixer
+    ffn = next((sp.ffn for sp in plan.layers if isinstance(sp.ffn, DenseSpec)), None)
+    moe = next((sp.ffn for sp in plan.layers if isinstance(sp.ffn, ExpertsSpec)), None)
+    return ModelConfig(arch="kedesun", num_layers=len(plan.layers), hidden_size=conf["width"], num_attention_heads=m.heads,
+                       num_kv_heads=m.heads, head_dim=m.dim, ffn_hidden_size=ffn.ff if ffn else moe.ff if moe else 0,
+                       vocab_size=conf["vocab"], rms_norm_eps=float(conf["norm"]["eps"]), tie_word_embeddings=True,
+                       max_position_embeddings=ROTARY_POSITIONS, dtype=dtype, layer_plan=plan)
+
+
 # architectures whose config.json names them in ``architecture``: reader of that file
-ARCH_READERS = {"nafitar": from_nafitar_config}
+ARCH_READERS = {"nafitar": from_nafitar_config, "kedesun": from_kedesun_config}
 
 
 def from_hf_config(hf: Dict[str, Any]) -> ModelConfig:

@@ -1,0 +1,273 @@
+"""Serving modules of layer-plan decoders whose layers run one mixer and one feed-forward side by side on the same normed
+input and hand on a weighted average over depth (Kedesun).
+
+Because both sublayers read the same input and are summed, a layer has two projections only: one into
+``[mixer columns | feed-forward columns]`` and one out of ``[mixer output | feed-forward activation]``, whose product is the
+sum of the two.  Routed experts are added to it, still in expert order, by the residual step.
+
+Every block of columns is a multiple of 8 wide and heads are padded with zero rows to the sizes the kernels store; zero
+padding changes no score, state or output, and means are taken over the true sizes."""
+from __future__ import annotations
+
+import math
+
+import torch
+import torch.nn as nn
+
+from ..ops import depth, latent_attention as la, matrix_memory as mm, moe, sandwich
+from ..ops.gemm import linear_forward
+from .config import ModelConfig
+from .layer_plan import DenseSpec, ExpertsSpec, LatentAttentionSpec, ParallelLayerSpec, RetentionSpec
+from .plan_decoder import CheckpointTensors, PlanDecoder, _buf, _up, put, put_heads
+
+
+def _columns(*sizes):
+    """Offsets of consecutive blocks and their total."""
+    at, n = [], 0
+    for s in sizes:
+        at.append(n)
+        n += s
+    return at, n
+
+
+class LatentAttentionMixer(nn.Module):
+    def __init__(self, spec: LatentAttentionSpec, width: int, eps: float, dtype, device):
+        super().__init__()
+        self.spec, self.width = spec, width
+        rank, rot = la.cached_row(spec.kv_rank, spec.rot_dim)
+        dim, vdim = _up(spec.dim, 8), _up(spec.vdim, 8)
+        (q, down, gate), self.columns = _columns(spec.heads * (dim + rot), rank + rot, _up(spec.heads, 8))
+        self.layout = la.LatentLayout(q=q, down=down, gate=gate, heads=spec.heads, dim=dim, vdim=vdim, rank=spec.kv_rank,
+                                      row_rank=rank, rot=spec.rot_dim, row_rot=rot, scale=spec.scale,
+                                      magnitude=spec.rot.magnitude(), eps=eps)
+        self.out_columns = spec.heads * vdim
+        self.gain = _buf(torch.zeros(spec.kv_rank, dtype=torch.float32, device=device))
+        self.freq = _buf(torch.tensor(spec.rot.frequencies(), dtype=torch.float32, device=device))
+        self.up_kv = _buf(torch.zeros(spec.heads * (dim + vdim), rank, dtype=dtype, device=device))
+
+    def cache_shape(self):
+        return 1, self.layout.row
+
+    def new_state(self, slots, device):
+        return None
+
+    def state_bytes(self):
+        return 0
+
+    def load(self, take, p: str, rows, out):
+        s, ly, W = self.spec, self.layout, self.width
+        H, d, r, C = s.heads, s.dim, s.rot_dim, s.kv_rank
+        q = take(p + "q", H * (d + r), W).view(H, d + r, W)
+        dst = rows[ly.q:ly.q + H * (ly.dim + ly.row_rot)].view(H, ly.dim + ly.row_rot, -1)
+        put(dst, q[:, :d])
+        put(dst[:, ly.dim:], q[:, d:])
+        down = take(p + "dkv", C + r, W)
+        put(rows[ly.down:], down[:C])
+        put(rows[ly.down + ly.row_rank:], down[C:])
+        put(rows[ly.gate:], take(p + "g", H, W))
+        put(self.gain, take(p + "dkv.norm", C).float())
+        put_heads(self.up_kv[:H * ly.dim], take(p + "uk", H * d, C), H, d, ly.dim)
+        put_heads(self.up_kv[H * ly.dim:], take(p + "uv", H * s.vdim, C), H, s.vdim, ly.vdim)
+        put(out.view(out.shape[0], H, ly.vdim), take(p + "o", W, H * s.vdim).view(W, H, s.vdim))
+
+    def forward(self, proj, rows, cache, state, out):
+        la.latent_attention(proj, self.layout, self.gain, self.freq, self.up_kv, rows, cache, out)
+
+
+class RetentionMixer(nn.Module):
+    def __init__(self, spec: RetentionSpec, width: int, eps: float, dtype, device):
+        super().__init__()
+        self.spec, self.width, self.eps = spec, width, eps
+        self.dim, self.vdim = mm.padded_key_dim(spec.dim), mm.padded_value_dim(spec.vdim)
+        H = spec.heads
+        self.at, self.columns = _columns(H * self.dim, H * self.dim, H * self.vdim, H * self.vdim)
+        self.out_columns = H * self.vdim
+        self.decay = _buf(torch.tensor(spec.decay, dtype=torch.float32, device=device))
+
+    def cache_shape(self):
+        return None
+
+    def new_state(self, slots, device):
+        return mm.MemoryState.allocate(slots, self.spec.heads, self.dim, self.vdim, device, gated=False)
+
+    def state_bytes(self):
+        return mm.MemoryState.bytes_per_slot(self.spec.heads, self.dim, self.vdim, gated=False)
+
+    def load(self, take, p: str, rows, out):
+        s, W, H = self.spec, self.width, self.spec.heads
+        for at, nm, dim, pad in zip(self.at, "qkvg", (s.dim, s.dim, s.vdim, s.vdim), (self.dim, self.dim, self.vdim, self.vdim)):
+            put_heads(rows[at:at + H * pad], take(p + nm, H * dim, W), H, dim, pad)
+        put(out.view(out.shape[0], H, self.vdim), take(p + "o", W, H * s.vdim).view(W, H, s.vdim))
+
+    def forward(self, proj, rows, cache, state, out):
+        s = self.spec
+        mm.retention(proj, *self.at, self.decay, s.dim ** -0.5, s.heads, self.dim, self.vdim, s.vdim, rows, state, self.eps, out)
+
+
+class DenseFeedForward(nn.Module):
+    def __init__(self, spec: DenseSpec, width: int, width_pad: int, dtype, device):
+        super().__init__()
+        self.spec, self.width, self.ff = spec, width, _up(spec.ff, 8)
+        self.columns, self.out_columns = 2 * self.ff, self.ff
+
+    def load(self, take, p: str, rows, out):
+        f, W = self.spec.ff, self.width
+        put(rows, take(p + "gate", f, W))
+        put(rows[self.ff:], take(p + "up", f, W))
+        put(out, take(p + "down", W, f))
+
+    def forward(self, h, proj, out, counts):
+        moe.activate(moe.SILU_GATE, proj, self.ff, self.ff, out)
+        return None
+
+
+class ExpertFeedForward(nn.Module):
+    """The shared expert is part of the layer's two projections; routed experts run on the grouped GEMM."""
+
+    def __init__(self, spec: ExpertsSpec, width: int, width_pad: int, dtype, device):
+        super().__init__()
+        if spec.experts > moe.MAX_EXPERTS or spec.top > moe.MAX_TOP:
+            raise ValueError(f"at most {moe.MAX_EXPERTS} experts and {moe.MAX_TOP} choices are supported")
+        self.spec, self.width = spec, width
+        self.ff, self.shared = _up(spec.ff, 8), _up(spec.shared_ff, 8)
+        self.columns = self.out_columns = self.shared
+        act = dict(dtype=dtype, device=device)
+        E = spec.experts
+        self.router = _buf(torch.zeros(E + (1 if self.shared else 0), width_pad, **act))   # + the shared expert's gate
+        self.correction = _buf(torch.zeros(E, dtype=torch.float32, device=device))
+        self.up = _buf(torch.zeros(E, self.ff, width_pad, **act))
+        self.down = _buf(torch.zeros(E, width_pad, self.ff, **act))
+
+    def load(self, take, p: str, rows, out):
+        s, W = self.spec, self.width
+        put(self.router, take(p + "router", s.experts, W))
+        put(self.correction, take(p + "correction", s.experts).float())
+        for e in range(s.experts):
+            put(self.up[e], take(f"{p}e{e}.up", s.ff, W))
+            put(self.down[e], take(f"{p}e{e}.down", W, s.ff))
+        if self.shared:
+            put(rows, take(p + "shared.up", s.shared_ff, W))
+            put(out, take(p + "shared.down", W, s.shared_ff))
+            put(self.router[s.experts:], take(p + "shared.sg", 1, W))
+
+    def forward(self, h, proj, out, counts):
+        s = self.spec
+        logits = linear_forward(h, self.router, out_dtype=torch.float32)
+        if self.shared:
+            moe.activate(moe.RELU2, proj, self.shared, 0, out, row_logit=logits[:, s.experts])
+        return moe.routed_experts(h, logits, s.top, self.correction, self.up, self.down, counts)
+
+
+class ParallelLayer(nn.Module):
+    """One layer's weights and its forward over the rows of a step."""
+
+    def __init__(self, index: int, spec: ParallelLayerSpec, width: int, width_pad: int, eps: float, dtype, device):
+        super().__init__()
+        self.index, self.width = index, width
+        mixer = LatentAttentionMixer if isinstance(spec.mixer, LatentAttentionSpec) else RetentionMixer
+        self.mixer = mixer(spec.mixer, width, eps, dtype, device)
+        self.ffn = None
+        if spec.ffn is not None:
+            ffn = ExpertFeedForward if isinstance(spec.ffn, ExpertsSpec) else DenseFeedForward
+            self.ffn = ffn(spec.ffn, width, width_pad, dtype, device)
+        self.experts = spec.ffn.experts if isinstance(spec.ffn, ExpertsSpec) else 0
+        n, k = self.mixer.columns, self.mixer.out_columns
+        if self.ffn is not None:
+            n, k = n + self.ffn.columns, k + self.ffn.out_columns
+        self.in_proj = _buf(torch.zeros(n, width_pad, dtype=dtype, device=device))
+        self.out_proj = _buf(torch.zeros(width_pad, k, dtype=dtype, device=device))
+        self.pre = _buf(torch.zeros(width_pad, dtype=torch.float32, device=device))
+        self.avg = _buf(torch.zeros(index + 2, dtype=torch.float32, device=device))
+
+    def cache_shape(self):
+        return self.mixer.cache_shape()
+
+    def new_state(self, slots, device):
+        return self.mixer.new_state(slots, device)
+
+    def state_bytes(self):
+        return self.mixer.state_bytes()
+
+    def load(self, take, p: str):
+        put(self.pre, take(p + "norm1", self.width).float())
+        put(self.avg, take(p + "dwa", self.index + 2).float())
+        n, k = self.mixer.columns, self.mixer.out_columns
+        self.mixer.load(take, p + "mix.", self.in_proj[:n], self.out_proj[:, :k])
+        if self.ffn is not None:
+            self.ffn.load(take, p + "mlp.", self.in_proj[n:], self.out_proj[:, k:])
+
+    def forward(self, h, rows, cache, state, counts):
+        """``h``: normed input.  Returns the layer's summed update and the routed experts' part of it (or None)."""
+        proj = linear_forward(h, self.in_proj)
+        act = torch.empty(h.shape[0], self.out_proj.shape[1], dtype=h.dtype, device=h.device)
+        n, k = self.mixer.columns, self.mixer.out_columns
+        self.mixer(proj, rows, cache, state, act[:, :k])
+        routed = self.ffn(h, proj[:, n:], act[:, k:], counts) if self.ffn is not None else None
+        return linear_forward(act, self.out_proj), routed
+
+
+class ParallelDecoder(PlanDecoder):
+    """Output matrix = embedding table."""
+
+    def __init__(self, cfg: ModelConfig, device=None):
+        if cfg.layer_plan.loop_times:
+            raise ValueError("a weighted average over depth and looped layers do not go together")
+        super().__init__(cfg, device)
+
+    @property
+    def output_weight(self):
+        return self.embed
+
+    def make_layer(self, index, spec, device):
+        return ParallelLayer(index, spec, self.width, self.width_pad, self.cfg.rms_norm_eps, self.dtype, device)
+
+    @torch.no_grad()
+    def load_tensors(self, tensors):
+        """Fills the module from a Kedesun checkpoint's tensors (``embed``, ``l<i>.norm1``, ``l<i>.mix.q`` ...,
+        ``l<i>.mlp.e<j>.up`` ..., ``l<i>.dwa``, ``final.norm``); every tensor must be there with its configured shape and
+        none may be left over."""
+        take = CheckpointTensors(tensors)
+        put(self.embed, take("embed", self.cfg.vocab_size, self.width))
+        put(self.final_gain, take("final.norm", self.width).float())
+        for i, layer in enumerate(self.layers):
+            layer.load(take, f"l{i}.")
+        take.done()
+        return self
+
+    @torch.no_grad()
+    def randomize(self, seed: int = 0):
+        """Random weights of the right scale (benchmarks); padding is not kept apart."""
+        g = torch.Generator(device=self.embed.device).manual_seed(seed)
+        for name, p in self.named_parameters():
+            leaf = name.rsplit(".", 1)[-1]
+            if leaf in ("freq", "decay"):
+                continue
+            if leaf == "avg":
+                p.fill_(0.3 / p.numel())
+                p[-1] = 0.7
+            elif leaf == "correction":
+                p.normal_(0.0, 0.01, generator=g)
+            elif p.dim() == 1:
+                p.fill_(1.0)
+            else:
+                p.normal_(0.0, 1.0 if name == "embed" else 1.0 / math.sqrt(p.shape[-1]), generator=g)
+        return self
+
+    def forward(self, rows, caches, states, final=True, record=None):
+        L, eps, W, T = len(self.layers), self.cfg.rms_norm_eps, self.width, rows.tokens.numel()
+        f32 = dict(dtype=torch.float32, device=self.embed.device)
+        history = torch.empty(L, T, self.width_pad, **f32)
+        x = torch.empty(T, self.width_pad, **f32)
+        experts = [ly.experts for ly in self.layers]
+        counts = None
+        if any(experts):     # cleared once per step for all layers
+            counts = torch.zeros(L, max(experts), dtype=torch.int32, device=self.embed.device)
+        _, _, h = sandwich.embed_rows(rows.tokens, rows.pos, self.embed, None, self.layers[0].pre, W, eps, x=history[0])
+        for i, layer in enumerate(self.layers):
+            y, routed = layer(h, rows, caches[i], states[i], counts[i, :experts[i]] if experts[i] else None)
+            last = i + 1 == L
+            gain = (self.final_gain if final else None) if last else self.layers[i + 1].pre
+            h = depth.add_layer(history, i + 1, x if i else history[0], y, layer.avg, W, eps, x, gain, routed, keep=not last)
+            if record is not None:
+                record.append(x.clone())
+        return h if final else x

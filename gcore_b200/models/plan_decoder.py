@@ -1,6 +1,10 @@
-"""Serving module of decoders that are described by a layer plan (``models/layer_plan.py``): the weights of every layer
-in the layout the kernels read, and the layer itself as a sequence of framework ops.  The cache, the recurrent state, the
-scheduler and the loop over layer runs belong to the rollout engine.
+"""Serving modules of decoders that are described by a layer plan (``models/layer_plan.py``): the weights of every layer
+in the layout the kernels read, and the layer itself as a sequence of framework ops.  The cache, the recurrent state and
+the scheduler belong to the rollout engine.
+
+``PlanDecoder`` is what the engine talks to: per layer the cache and state it needs, and one forward over the rows of a
+step.  Subclasses supply the layers and the residual stream; ``build_decoder`` picks one by the plan.  ``SandwichDecoder``
+here: mixers side by side, norms before and after each sublayer, looped layers.
 
 Layout against the checkpoint:
   * one input projection per layer, rows ``[left q | left k | right q | right k | right v | right g]``, each block's heads
@@ -21,7 +25,7 @@ from ..ops import sandwich
 from ..ops import window_attention as wa
 from ..ops.gemm import linear_forward
 from .config import ModelConfig
-from .layer_plan import LayerSpec
+from .layer_plan import LayerSpec, ParallelLayerSpec
 
 
 def _up(n: int, m: int) -> int:
@@ -30,6 +34,35 @@ def _up(n: int, m: int) -> int:
 
 def _buf(t: torch.Tensor) -> nn.Parameter:
     return nn.Parameter(t, requires_grad=False)
+
+
+def put(dst: torch.Tensor, t: torch.Tensor):
+    """Copies ``t`` into the leading corner of ``dst``."""
+    dst[tuple(slice(0, s) for s in t.shape)].copy_(t)
+
+
+def put_heads(dst: torch.Tensor, t: torch.Tensor, heads: int, dim: int, pad: int):
+    """[heads * dim, ...] -> rows of heads padded to ``pad``."""
+    put(dst.view(heads, pad, *dst.shape[1:]), t.view(heads, dim, *t.shape[1:]))
+
+
+class CheckpointTensors:
+    """Tensors of a checkpoint, taken one by one: each must be there with its configured shape, none may be left over."""
+
+    def __init__(self, tensors: Dict[str, torch.Tensor]):
+        self.left = dict(tensors)
+
+    def __call__(self, name: str, *shape: int) -> torch.Tensor:
+        if name not in self.left:
+            raise KeyError(f"checkpoint lacks '{name}'")
+        t = self.left.pop(name)
+        if tuple(t.shape) != shape:
+            raise ValueError(f"'{name}' has shape {tuple(t.shape)}, the configuration says {shape}")
+        return t
+
+    def done(self):
+        if self.left:
+            raise ValueError(f"checkpoint tensors without a place in the model: {sorted(self.left)[:8]}")
 
 
 class PlanLayer(nn.Module):
@@ -98,22 +131,70 @@ class PlanLayer(nn.Module):
 
 
 class PlanDecoder(nn.Module):
+    """Base of the decoders a layer plan describes: embedding, layers, final norm, output matrix, and the interface of the
+    rollout engine."""
+
     def __init__(self, cfg: ModelConfig, device=None):
         super().__init__()
-        self.cfg, plan = cfg, cfg.layer_plan
-        dtype = {"bfloat16": torch.bfloat16, "float32": torch.float32}.get(cfg.dtype)
-        if dtype is None:
+        self.cfg = cfg
+        self.dtype = {"bfloat16": torch.bfloat16, "float32": torch.float32}.get(cfg.dtype)
+        if self.dtype is None:
             raise ValueError(f"layer-plan decoders run in bfloat16 or float32, not {cfg.dtype}")
         self.width, self.width_pad = cfg.hidden_size, _up(cfg.hidden_size, 8)
-        act = dict(dtype=dtype, device=device)
-        f32 = dict(dtype=torch.float32, device=device)
-        self.embed = _buf(torch.zeros(cfg.vocab_size, self.width_pad, **act))
+        self.embed = _buf(torch.zeros(cfg.vocab_size, self.width_pad, dtype=self.dtype, device=device))
+        self.layers = nn.ModuleList([self.make_layer(i, sp, device) for i, sp in enumerate(cfg.layer_plan.layers)])
+        self.final_gain = _buf(torch.zeros(self.width_pad, dtype=torch.float32, device=device))
+
+    @property
+    def output_weight(self) -> torch.Tensor:
+        """[vocab, width] matrix of the logits."""
+        raise NotImplementedError
+
+    def make_layer(self, index: int, spec, device) -> nn.Module:
+        raise NotImplementedError
+
+    def forward(self, rows, caches, states, final: bool = True, record: Optional[list] = None):
+        """All layer runs over the rows of one step.  ``caches`` / ``states``: one per layer run.  Returns the
+        final-normed hidden states of all rows, or with ``final=False`` the 32-bit residual in front of the final norm
+        (``final_rows`` then norms the rows that are wanted).  ``record`` collects the residual after every run."""
+        raise NotImplementedError
+
+    def final_rows(self, x, rows=None):
+        return sandwich.norm_rows(x, self.final_gain, self.width, self.cfg.rms_norm_eps, self.embed.dtype, rows)
+
+    # ---- what the engine allocates for every layer run
+    def new_caches(self, blocks: int, block_size: int, device) -> list:
+        """Paged cache of every run: one row per token serves as key and value; None for runs without one."""
+        shapes = [self.layers[r.layer].cache_shape() for r in self.cfg.layer_plan.runs]
+        return [torch.zeros(blocks, block_size, *s, dtype=self.dtype, device=device) if s else None for s in shapes]
+
+    def new_states(self, slots: int, device) -> list:
+        """Recurrent state of every run, one per request slot; None for runs without one."""
+        return [self.layers[r.layer].new_state(slots, device) for r in self.cfg.layer_plan.runs]
+
+    def cache_bytes_per_token(self) -> int:
+        shapes = [self.layers[r.layer].cache_shape() for r in self.cfg.layer_plan.runs]
+        return sum(math.prod(s) for s in shapes if s) * self.embed.element_size()
+
+    def state_bytes_per_slot(self) -> int:
+        return sum(self.layers[r.layer].state_bytes() for r in self.cfg.layer_plan.runs)
+
+
+class SandwichDecoder(PlanDecoder):
+    def __init__(self, cfg: ModelConfig, device=None):
+        super().__init__(cfg, device)
+        plan, f32 = cfg.layer_plan, dict(dtype=torch.float32, device=device)
+        act = dict(dtype=self.dtype, device=device)
         self.pos_table = _buf(torch.zeros(cfg.max_position_embeddings, self.width_pad, **act))
         self.loop_step = _buf(torch.zeros(plan.loop_times, self.width_pad, **f32)) if plan.loop_times else None
-        self.layers = nn.ModuleList([PlanLayer(sp, self.width, self.width_pad, cfg.rms_norm_eps, dtype, device)
-                                     for sp in plan.layers])
-        self.final_gain = _buf(torch.zeros(self.width_pad, **f32))
         self.head = _buf(torch.zeros(cfg.vocab_size, self.width_pad, **act))
+
+    @property
+    def output_weight(self):
+        return self.head
+
+    def make_layer(self, index, spec, device):
+        return PlanLayer(spec, self.width, self.width_pad, self.cfg.rms_norm_eps, self.dtype, device)
 
     # ------------------------------------------------------------------ checkpoint
     @torch.no_grad()
@@ -121,23 +202,7 @@ class PlanDecoder(nn.Module):
         """Fills the module from a Nafitar checkpoint's tensors (``embed``, ``pos``, ``loop.step``, ``l<i>.norm1``,
         ``l<i>.mix.left.q`` ..., ``final.norm``, ``head``); every tensor must be there with its configured shape and
         none may be left over."""
-        left = dict(tensors)
-
-        def take(name, *shape):
-            if name not in left:
-                raise KeyError(f"checkpoint lacks '{name}'")
-            t = left.pop(name)
-            if tuple(t.shape) != shape:
-                raise ValueError(f"'{name}' has shape {tuple(t.shape)}, the configuration says {shape}")
-            return t
-
-        def put(dst, t):
-            dst[tuple(slice(0, s) for s in t.shape)].copy_(t)
-
-        def heads_rows(dst, t, heads, dim, pad):       # [heads * dim, ...] -> rows of heads padded to ``pad``
-            put(dst.view(heads, pad, *dst.shape[1:]), t.view(heads, dim, *t.shape[1:]))
-
-        W = self.width
+        take, W = CheckpointTensors(tensors), self.width
         put(self.embed, take("embed", self.cfg.vocab_size, W))
         put(self.pos_table, take("pos", self.cfg.max_position_embeddings, W))
         put(self.head, take("head", self.cfg.vocab_size, W))
@@ -152,15 +217,15 @@ class PlanDecoder(nn.Module):
             for key, nm, n, dim, pad in (("q", "left.q", a.heads, a.dim, D), ("k", "left.k", a.kv_heads, a.dim, D),
                                          ("mq", "right.q", m.heads, m.dim, dk), ("mk", "right.k", m.heads, m.dim, dk),
                                          ("mv", "right.v", m.heads, m.vdim, dv), ("mg", "right.g", m.heads, m.vdim, dv)):
-                heads_rows(ly.in_proj[o[key]:o[key] + n * pad], take(p + "mix." + nm, n * dim, W), n, dim, pad)
+                put_heads(ly.in_proj[o[key]:o[key] + n * pad], take(p + "mix." + nm, n * dim, W), n, dim, pad)
                 if key in ("q", "k"):
-                    heads_rows(ly.in_bias[o[key]:o[key] + n * pad], take(p + f"mix.{nm}.b", n * dim), n, dim, pad)
+                    put_heads(ly.in_bias[o[key]:o[key] + n * pad], take(p + f"mix.{nm}.b", n * dim), n, dim, pad)
             for r, nm in enumerate(("right.i", "right.f")):
                 put(ly.gate_w[r * m.heads:(r + 1) * m.heads], take(p + "mix." + nm, m.heads, W))
                 put(ly.gate_b[r * m.heads:(r + 1) * m.heads], take(p + f"mix.{nm}.b", m.heads).float())
             for dst, nm, n, dim, pad in ((ly.att_out, "left.o", a.heads, a.dim, D), (ly.mem_out, "right.o", m.heads, m.vdim, dv)):
                 put(dst.view(dst.shape[0], n, pad), take(p + "mix." + nm, W, n * dim).view(W, n, dim))
-            heads_rows(ly.mem_gain, take(p + "mix.right.norm", m.heads * m.vdim).float(), m.heads, m.vdim, dv)
+            put_heads(ly.mem_gain, take(p + "mix.right.norm", m.heads * m.vdim).float(), m.heads, m.vdim, dv)
             put(ly.gain_att, take(p + "mix.left.out", W).float())
             put(ly.gain_mem, take(p + "mix.right.out", W).float())
             if ly.spec.ffn:
@@ -170,8 +235,7 @@ class PlanDecoder(nn.Module):
                 put(ly.fc1[:f], take(p + "mlp.gate", f, W))
                 put(ly.fc1[ly.ffn_pad:ly.ffn_pad + f], take(p + "mlp.up", f, W))
                 put(ly.fc2, take(p + "mlp.down", W, f))
-        if left:
-            raise ValueError(f"checkpoint tensors without a place in the model: {sorted(left)[:8]}")
+        take.done()
         return self
 
     @torch.no_grad()
@@ -190,9 +254,6 @@ class PlanDecoder(nn.Module):
 
     # ------------------------------------------------------------------ forward
     def forward(self, rows, caches, states, final: bool = True, record: Optional[list] = None):
-        """All layer runs over the rows of one step.  ``caches`` / ``states``: one per layer run.  Returns the
-        final-normed hidden states of all rows, or with ``final=False`` the 32-bit residual in front of the final norm
-        (``final_rows`` then norms the rows that are wanted).  ``record`` collects the residual after every run."""
         plan, eps = self.cfg.layer_plan, self.cfg.rms_norm_eps
         runs = plan.runs
         opens = [r.opens_pass for r in runs] + [None]
@@ -216,5 +277,9 @@ class PlanDecoder(nn.Module):
                 h = sandwich.norm_rows(x, gain, self.width, eps, self.embed.dtype)
         return h if final else x
 
-    def final_rows(self, x, rows=None):
-        return sandwich.norm_rows(x, self.final_gain, self.width, self.cfg.rms_norm_eps, self.embed.dtype, rows)
+
+def build_decoder(cfg: ModelConfig, device=None) -> PlanDecoder:
+    """The serving module of a layer-plan configuration."""
+    from .parallel_decoder import ParallelDecoder
+    cls = ParallelDecoder if isinstance(cfg.layer_plan.layers[0], ParallelLayerSpec) else SandwichDecoder
+    return cls(cfg, device)

@@ -14,6 +14,11 @@
 // With one CTA per SM the four softmax warps (one per scheduler) left every pipe under 35 % busy (ncu): the kernel was
 // bound by the latency of each warp's dependent chain, so the tile is 64 keys wide and two CTAs interleave on an SM.
 // P is written as bf16 into a 128-byte-swizzled K-major shared tile and consumed as the A operand of P V.
+//
+// LAT instances serve latent attention over prompt portions: the last 64-wide chunk of queries and keys is a rotated part
+// that comes from matrices of its own (the key's is shared by all heads), heads narrower than the tile are zero-filled by
+// the loads, probabilities enter P V as two bf16 terms (rounded value and remainder, 16 significant bits), and the output
+// is scaled by a sigmoid gate per (token, head).
 #include "ptx.cuh"
 #include "host_utils.h"
 #include <float.h>
@@ -36,15 +41,21 @@ struct FaParams {
   int causal, window;
   float scale;
   int* err;
+  const __nv_bfloat16* gate;   // LAT: [Tq, Hq] logits, gate_ld apart, or null
+  long long gate_ld;
+  int dv;                      // LAT: value columns in use (a multiple of 8)
 };
 
 // DQK = head dim of queries and keys, DV = head dim of values and of the output (equal except for multi-head latent
 // attention expanded to per-head keys: 128 + 64 rotary dims against 128-wide values).
-template <int DQK, int DV>
-__global__ void __launch_bounds__(FA_THREADS, 2)
+template <int DQK, int DV, bool LAT>
+__global__ void __launch_bounds__(FA_THREADS, LAT ? 1 : 2)
 attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
-                const __grid_constant__ CUtensorMap tmV, FaParams p) {
+                const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmQr,
+                const __grid_constant__ CUtensorMap tmKr, FaParams p) {
   constexpr int NCH = DQK / 64;            // 64-element (128-byte) chunks along the query / key head dim
+  constexpr int NPLAIN = LAT ? NCH - 1 : NCH;
+  constexpr int TERMS = LAT ? 2 : 1;       // bf16 terms of a probability
   constexpr int NCHV = DV / 64;
   constexpr int TILE_BYTES = 128 * DQK * 2;    // the Q tile
   constexpr int K_BYTES = FA_BN * DQK * 2;     // one K tile
@@ -59,7 +70,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
   uint8_t* sK = sQ + TILE_BYTES;    // 2 stages
   uint8_t* sV = sK + 2 * K_BYTES;   // 2 stages
   uint8_t* sP = sV + 2 * V_BYTES;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(sP + P_BYTES);
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sP + TERMS * P_BYTES);
   uint64_t* q_full = bars;         // 1
   uint64_t* k_full = bars + 1;     // 2
   uint64_t* v_full = bars + 3;     // 2
@@ -111,6 +122,10 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     prefetch_tmap(&tmQ);
     prefetch_tmap(&tmK);
     prefetch_tmap(&tmV);
+    if (LAT) {
+      prefetch_tmap(&tmQr);
+      prefetch_tmap(&tmKr);
+    }
   }
   if (warp == 5) {
     tmem_alloc(tmem_holder, 256);
@@ -128,7 +143,8 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       if (lane == 0) {
         mbar_expect_tx(q_full, TILE_BYTES);
 #pragma unroll
-        for (int c = 0; c < NCH; ++c) tma_load_3d(sQ + c * 16384, &tmQ, q_full, c * 64, h, q_beg + q0);
+        for (int c = 0; c < NPLAIN; ++c) tma_load_3d(sQ + c * 16384, &tmQ, q_full, c * 64, h, q_beg + q0);
+        if (LAT) tma_load_3d(sQ + NPLAIN * 16384, &tmQr, q_full, 0, h, q_beg + q0);
       }
       __syncwarp();
       bool ok = true;
@@ -141,7 +157,8 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
           const int krow = k_beg + (j_beg + it) * FA_BN;
           mbar_expect_tx(&k_full[s], K_BYTES);
 #pragma unroll
-          for (int c = 0; c < NCH; ++c) tma_load_3d(sK + s * K_BYTES + c * KV_CHUNK, &tmK, &k_full[s], c * 64, hk, krow);
+          for (int c = 0; c < NPLAIN; ++c) tma_load_3d(sK + s * K_BYTES + c * KV_CHUNK, &tmK, &k_full[s], c * 64, hk, krow);
+          if (LAT) tma_load_3d(sK + s * K_BYTES + NPLAIN * KV_CHUNK, &tmKr, &k_full[s], 0, 0, krow);
           mbar_expect_tx(&v_full[s], V_BYTES);
 #pragma unroll
           for (int c = 0; c < NCHV; ++c) tma_load_3d(sV + s * V_BYTES + c * KV_CHUNK, &tmV, &v_full[s], c * 64, hk, krow);
@@ -189,10 +206,13 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       if (lane == 0) {
         const uint32_t pa = smem_u32(sP), va = smem_u32(sV + s * V_BYTES);
 #pragma unroll
-        for (int k4 = 0; k4 < FA_BN / 16; ++k4) {
-          const uint64_t adesc = make_smem_desc_sw128(pa + (k4 >> 2) * 16384 + (k4 & 3) * 32, 16, 1024);
-          const uint64_t bdesc = make_smem_desc_sw128(va + k4 * 2048, KV_CHUNK, 1024);
-          umma_f16(tmem_o, adesc, bdesc, idesc_pv, (it > 0 || k4 > 0) ? 1u : 0u);
+        for (int term = 0; term < TERMS; ++term) {
+#pragma unroll
+          for (int k4 = 0; k4 < FA_BN / 16; ++k4) {
+            const uint64_t adesc = make_smem_desc_sw128(pa + term * P_BYTES + (k4 >> 2) * 16384 + (k4 & 3) * 32, 16, 1024);
+            const uint64_t bdesc = make_smem_desc_sw128(va + k4 * 2048, KV_CHUNK, 1024);
+            umma_f16(tmem_o, adesc, bdesc, idesc_pv, (it > 0 || term > 0 || k4 > 0) ? 1u : 0u);
+          }
         }
         umma_commit(&kv_empty[s]);
         umma_commit(pv_done);
@@ -292,6 +312,15 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
           w.z = pack_bf16x2(sv[c * 64 + u * 8 + 4], sv[c * 64 + u * 8 + 5]);
           w.w = pack_bf16x2(sv[c * 64 + u * 8 + 6], sv[c * 64 + u * 8 + 7]);
           *reinterpret_cast<uint4*>(rowp + ((u ^ (row & 7)) << 4)) = w;
+          if (LAT) {
+            const uint32_t hi[4] = {w.x, w.y, w.z, w.w};
+            uint32_t lo[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+              lo[e] = pack_bf16x2(sv[c * 64 + u * 8 + 2 * e] - bf16_bits_to_float(static_cast<uint16_t>(hi[e] & 0xffff)),
+                                  sv[c * 64 + u * 8 + 2 * e + 1] - bf16_bits_to_float(static_cast<uint16_t>(hi[e] >> 16)));
+            *reinterpret_cast<uint4*>(rowp + P_BYTES + ((u ^ (row & 7)) << 4)) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+          }
         }
       }
       fence_proxy_async();
@@ -306,9 +335,11 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
     if (ok) {
       const float m_use = m == -FLT_MAX ? 0.f : m;
       if (p.sinks) l += exp2f(p.sinks[h] * 1.4426950408889634f - m_use);
-      const float inv = l > 0.f ? 1.f / l : 0.f;
+      float inv = l > 0.f ? 1.f / l : 0.f;
       const bool valid = qi < lq;
-      __nv_bfloat16* orow = p.out + static_cast<long long>(q_beg + qi) * p.o_stride_t + static_cast<long long>(h) * DV;
+      if (LAT && p.gate && valid)
+        inv /= 1.f + exp2f(-1.4426950408889634f * __bfloat162float(p.gate[static_cast<long long>(q_beg + qi) * p.gate_ld + h]));
+      __nv_bfloat16* orow = p.out + static_cast<long long>(q_beg + qi) * p.o_stride_t + static_cast<long long>(h) * (LAT ? p.dv : DV);
 #pragma unroll
       for (int c = 0; c < DV / 32; ++c) {
         uint32_t r[32];
@@ -322,6 +353,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
         if (valid) {
 #pragma unroll
           for (int j = 0; j < 4; ++j) {
+            if (LAT && c * 32 + j * 8 >= p.dv) break;
             uint4 w;
             w.x = pack_bf16x2(__uint_as_float(r[8 * j + 0]) * inv, __uint_as_float(r[8 * j + 1]) * inv);
             w.y = pack_bf16x2(__uint_as_float(r[8 * j + 2]) * inv, __uint_as_float(r[8 * j + 3]) * inv);
@@ -346,21 +378,21 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
   }
 }
 
-template <int DQK, int DV>
-int launch_fa(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const FaParams& p, dim3 grid,
-              cudaStream_t st) {
-  // 112 KB at 128 / 128 (two CTAs per SM), 144 KB at 192 / 128 (one)
-  constexpr int SMEM = 128 * DQK * 2 + 2 * FA_BN * DQK * 2 + 2 * FA_BN * DV * 2 + 128 * FA_BN * 2 + 256;
+template <int DQK, int DV, bool LAT = false>
+int launch_fa(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& tqr,
+              const CUtensorMap& tkr, const FaParams& p, dim3 grid, cudaStream_t st) {
+  // 112 KB at 128 / 128 (two CTAs per SM), 144 KB at 192 / 128 (one); LAT: 16 KB more
+  constexpr int SMEM = 128 * DQK * 2 + 2 * FA_BN * DQK * 2 + 2 * FA_BN * DV * 2 + (LAT ? 2 : 1) * 128 * FA_BN * 2 + 256;
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(attn_fwd_kernel<DQK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
+    cudaError_t e = cudaFuncSetAttribute(attn_fwd_kernel<DQK, DV, LAT>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
     if (e != cudaSuccess) return static_cast<int>(e);
     // the whole L1 / shared array as shared memory, so that two CTAs fit
-    cudaFuncSetAttribute(attn_fwd_kernel<DQK, DV>, cudaFuncAttributePreferredSharedMemoryCarveout,
+    cudaFuncSetAttribute(attn_fwd_kernel<DQK, DV, LAT>, cudaFuncAttributePreferredSharedMemoryCarveout,
                          cudaSharedmemCarveoutMaxShared);
     configured = true;
   }
-  attn_fwd_kernel<DQK, DV><<<grid, FA_THREADS, SMEM, st>>>(tq, tk, tv, p);
+  attn_fwd_kernel<DQK, DV, LAT><<<grid, FA_THREADS, SMEM, st>>>(tq, tk, tv, tqr, tkr, p);
   return launch_status();
 }
 
@@ -392,9 +424,55 @@ GK_EXPORT int gk_attn_fwd(const void* q, const void* k, const void* v, void* out
   p.lse = lse; p.tq_total = Tq;
   p.Hq = Hq; p.Hk = Hk; p.causal = causal; p.window = window; p.scale = scale;
   p.err = reinterpret_cast<int*>(se[1]);
+  p.gate = nullptr; p.gate_ld = 0; p.dv = Dv;
   dim3 grid((max_q + FA_BM - 1) / FA_BM, Hq, B);
   cudaStream_t st = reinterpret_cast<cudaStream_t>(se[0]);
-  if (D == 192) return launch_fa<192, 128>(tq, tk, tv, p, grid, st);
-  if (D == 128) return launch_fa<128, 128>(tq, tk, tv, p, grid, st);
-  return launch_fa<64, 64>(tq, tk, tv, p, grid, st);
+  if (D == 192) return launch_fa<192, 128>(tq, tk, tv, tq, tk, p, grid, st);
+  if (D == 128) return launch_fa<128, 128>(tq, tk, tv, tq, tk, p, grid, st);
+  return launch_fa<64, 64>(tq, tk, tv, tq, tk, p, grid, st);
+}
+
+// 1 when a kernel is built for heads of `dim` unrotated, `rot` rotated and `vdim` value dimensions
+GK_EXPORT int gk_latent_prefill_supported(int dim, int rot, int vdim) {
+  return dim >= 1 && dim <= 128 && rot >= 1 && rot <= 64 && vdim >= 1 && vdim <= 128;
+}
+
+// Latent attention over prompt portions whose context lies expanded and contiguous: query i of portion b sees the keys
+// 0 .. lk - lq + i of its context.  q [Tq rows, q_ld]: head h has `dim` unrotated columns at q_off + h * q_hs and `rot`
+// rotated ones behind them; kv [Tk rows, kv_ld]: head h has its `dim` key columns at h * dim and `vdim` value columns at
+// H * dim + h * vdim; kr [Tk rows, kr_ld]: the rotated key part of all heads; gate [Tq rows, gate_ld]: one logit per head.
+// All widths, offsets and strides are multiples of 8 elements.
+// ptrs: {q, kv, kr, gate, out, cu_q, cu_k, err};  lds: {q_ld, kv_ld, kr_ld, gate_ld, out_ld}
+// dims: {portions, Tq, Tk, H, dim, rot, vdim, q_hs, max_q}
+GK_EXPORT int gk_latent_prefill(void* const* ptrs, const long long* lds, const int* dims, float scale, void* stream) {
+  const int B = dims[0], Tq = dims[1], Tk = dims[2], H = dims[3], dim = dims[4], rot = dims[5], vdim = dims[6];
+  if (!gk_latent_prefill_supported(dim, rot, vdim)) return -1;
+  if (dim % 8 || rot % 8 || vdim % 8 || dims[7] % 8 || lds[0] % 8 || lds[1] % 8 || lds[2] % 8 || lds[4] % 8) return -2;
+  if (B == 0 || Tq == 0) return 0;
+  const __nv_bfloat16 *q = static_cast<const __nv_bfloat16*>(ptrs[0]), *kv = static_cast<const __nv_bfloat16*>(ptrs[1]),
+                      *kr = static_cast<const __nv_bfloat16*>(ptrs[2]);
+  if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(kv) | reinterpret_cast<uintptr_t>(kr) |
+       reinterpret_cast<uintptr_t>(ptrs[4])) & 15)
+    return -2;
+  CUtensorMap tq, tqr, tk, tkr, tv;
+  if (make_tmap_3d(&tq, q, 2, Tq, H, dim, lds[0], dims[7], FA_BM, 1, 64, true)) return -3;
+  if (make_tmap_3d(&tqr, q + dim, 2, Tq, H, rot, lds[0], dims[7], FA_BM, 1, 64, true)) return -4;
+  if (make_tmap_3d(&tk, kv, 2, Tk, H, dim, lds[1], dim, FA_BN, 1, 64, true)) return -5;
+  if (make_tmap_3d(&tv, kv + static_cast<long long>(H) * dim, 2, Tk, H, vdim, lds[1], vdim, FA_BN, 1, 64, true)) return -6;
+  if (make_tmap_3d(&tkr, kr, 2, Tk, 1, rot, lds[2], rot, FA_BN, 1, 64, true)) return -7;
+  FaParams p;
+  p.cu_q = static_cast<const int*>(ptrs[5]); p.cu_k = static_cast<const int*>(ptrs[6]); p.sinks = nullptr;
+  p.out = static_cast<__nv_bfloat16*>(ptrs[4]);
+  p.o_stride_t = lds[4];
+  p.lse = nullptr; p.tq_total = Tq;
+  p.Hq = H; p.Hk = H; p.causal = 1; p.window = 0; p.scale = scale;
+  p.err = static_cast<int*>(ptrs[7]);
+  p.gate = static_cast<const __nv_bfloat16*>(ptrs[3]); p.gate_ld = lds[3]; p.dv = vdim;
+  const dim3 grid((dims[8] + FA_BM - 1) / FA_BM, H, B);
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  if (dim <= 64)
+    return vdim <= 64 ? launch_fa<128, 64, true>(tq, tk, tv, tqr, tkr, p, grid, st)
+                      : launch_fa<128, 128, true>(tq, tk, tv, tqr, tkr, p, grid, st);
+  return vdim <= 64 ? launch_fa<192, 64, true>(tq, tk, tv, tqr, tkr, p, grid, st)
+                    : launch_fa<192, 128, true>(tq, tk, tv, tqr, tkr, p, grid, st);
 }

@@ -1,0 +1,151 @@
+// Steps around the latent-attention kernels of served decoders (attention_fwd.cu for prompt portions, mla_decode.cu for
+// single tokens, window_attention.cu for 32-bit models and other sizes).  A cached row is [latent, normed | key part rotated
+// at its position], both padded with zeros; it serves every head.
+//   * latent_prep_kernel    a packed projection row -> its cache row (norm of the latent in 32-bit, rotation), the queries'
+//                           rotated parts in place, and a copy of the cache row in the portion's contiguous context;
+//   * latent_gather_kernel  cache rows of the tokens in front of a portion -> the portion's contiguous context.
+// The rotation pairs dimension 2i with 2i + 1; angle and rotation are 32-bit.
+#include "host_utils.h"
+#include "row_ops.cuh"
+#include <type_traits>
+
+namespace gk {
+
+constexpr int LP_THREADS = 128;
+constexpr int LP_MAX_ROT = 256;
+
+__device__ __forceinline__ float lp_f(float v) { return v; }
+__device__ __forceinline__ float lp_f(__nv_bfloat16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ void lp_st(float* p, float v) { *p = v; }
+__device__ __forceinline__ void lp_st(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
+
+template <typename T>
+struct LatentPrepParams {
+  T* proj;                 // packed projection rows
+  long long ld;
+  int q_off, q_hs;         // head h: unrotated columns at q_off + h * q_hs, rotated ones `q_rot` behind
+  int q_rot;
+  int d_off;               // latent columns, then the shared key part at d_off + CV
+  const float* gain;       // [C]
+  const float* freq;       // [rot / 2]
+  const int* pos;
+  const int* slots;        // cache slot of every row; negative: not stored
+  T* cache;                // rows of CV + DR
+  T* context;              // [context rows, CV + DR] or null
+  const int* row_seq;      // with context: portion of every row
+  const int* cu_ctx;       //   first context row of every portion
+  int rows, context_rows;  //   rows that belong to portions (they come first)
+  int H, C, CV, rot, DR;
+  float eps, magnitude;
+};
+
+// One CTA per row.
+template <typename T>
+__global__ void __launch_bounds__(LP_THREADS) latent_prep_kernel(const LatentPrepParams<T> p) {
+  __shared__ float red[64];
+  __shared__ float s_cos[LP_MAX_ROT / 2], s_sin[LP_MAX_ROT / 2];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int row = blockIdx.x, tid = threadIdx.x, half = p.rot >> 1;
+  T* pr = p.proj + row * p.ld;
+  const int pos = p.pos[row], slot = p.slots[row];
+  for (int i = tid; i < half; i += LP_THREADS) {
+    float s, c;
+    sincosf(static_cast<float>(pos) * p.freq[i], &s, &c);
+    s_cos[i] = c * p.magnitude;
+    s_sin[i] = s * p.magnitude;
+  }
+  float ss = 0.f;
+  for (int c = tid; c < p.C; c += LP_THREADS) {
+    const float v = lp_f(pr[p.d_off + c]);
+    ss += v * v;
+  }
+  const float r = 1.f / sqrtf(block_sum2(ss, 0.f, red).x / p.C + p.eps);      // also orders the angles for all threads
+  const int width = p.CV + p.DR;
+  T* dst = slot >= 0 ? p.cache + static_cast<long long>(slot) * width : nullptr;
+  T* ctx = p.context && row < p.context_rows
+               ? p.context + (static_cast<long long>(p.cu_ctx[p.row_seq[row]]) + pos) * width : nullptr;
+  for (int c = tid; c < width; c += LP_THREADS) {
+    float v = 0.f;
+    if (c < p.C) {
+      v = lp_f(pr[p.d_off + c]) * r * p.gain[c];
+    } else if (c >= p.CV && c - p.CV < p.rot) {
+      const int i = (c - p.CV) >> 1;
+      const float a = lp_f(pr[p.d_off + p.CV + 2 * i]), b = lp_f(pr[p.d_off + p.CV + 2 * i + 1]);
+      v = (c - p.CV) & 1 ? b * s_cos[i] + a * s_sin[i] : a * s_cos[i] - b * s_sin[i];
+    }
+    if (dst) lp_st(dst + c, v);
+    if (ctx) lp_st(ctx + c, v);
+  }
+  for (int i = tid; i < p.H * half; i += LP_THREADS) {
+    const int h = i / half, j = i - h * half;
+    T* q = pr + p.q_off + static_cast<long long>(h) * p.q_hs + p.q_rot + 2 * j;
+    const float a = lp_f(q[0]), b = lp_f(q[1]);
+    lp_st(q, a * s_cos[j] - b * s_sin[j]);
+    lp_st(q + 1, b * s_cos[j] + a * s_sin[j]);
+  }
+}
+
+// grid (row groups, portions); one warp per cached row, rows of `vec` 16-byte units
+__global__ void __launch_bounds__(256) latent_gather_kernel(const uint4* __restrict__ cache, const int* __restrict__ tables,
+                                                            int max_blocks, int block_size,
+                                                            const int* __restrict__ first_pos,
+                                                            const int* __restrict__ cu_ctx, uint4* __restrict__ context,
+                                                            int vec) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int b = blockIdx.y, n = first_pos[b], lane = threadIdx.x & 31;
+  const int* table = tables + static_cast<long long>(b) * max_blocks;
+  uint4* out = context + static_cast<long long>(cu_ctx[b]) * vec;
+  for (int j = blockIdx.x * 8 + (threadIdx.x >> 5); j < n; j += gridDim.x * 8) {
+    const uint4* src = cache + (static_cast<long long>(table[j / block_size]) * block_size + j % block_size) * vec;
+    uint4* dst = out + static_cast<long long>(j) * vec;
+    for (int c = lane; c < vec; c += 32) dst[c] = src[c];
+  }
+}
+
+}  // namespace gk
+
+using namespace gk;
+
+// ptrs: {proj, gain, freq, pos, slots, cache, context, row_seq, cu_ctx}; context null: single tokens only
+// dims: {rows, context_rows, q_off, q_hs, q_rot, d_off, H, C, CV, rot, DR}
+GK_EXPORT int gk_latent_prep(int is_fp32, void* const* ptrs, long long ld, const int* dims, float eps, float magnitude,
+                             void* stream) {
+  if (dims[0] == 0) return 0;
+  if (dims[9] % 2 || dims[9] > LP_MAX_ROT || dims[9] > dims[10] || dims[7] > dims[8] || dims[7] < 1) return -1;
+  if (ptrs[6] && (!ptrs[7] || !ptrs[8])) return -2;
+  auto fill = [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    LatentPrepParams<T> p;
+    p.proj = static_cast<T*>(ptrs[0]);
+    p.ld = ld;
+    p.gain = static_cast<const float*>(ptrs[1]);
+    p.freq = static_cast<const float*>(ptrs[2]);
+    p.pos = static_cast<const int*>(ptrs[3]);
+    p.slots = static_cast<const int*>(ptrs[4]);
+    p.cache = static_cast<T*>(ptrs[5]);
+    p.context = static_cast<T*>(ptrs[6]);
+    p.row_seq = static_cast<const int*>(ptrs[7]);
+    p.cu_ctx = static_cast<const int*>(ptrs[8]);
+    p.rows = dims[0]; p.context_rows = dims[1]; p.q_off = dims[2]; p.q_hs = dims[3]; p.q_rot = dims[4]; p.d_off = dims[5];
+    p.H = dims[6]; p.C = dims[7]; p.CV = dims[8]; p.rot = dims[9]; p.DR = dims[10];
+    p.eps = eps; p.magnitude = magnitude;
+    launch_k(latent_prep_kernel<T>, dim3(dims[0]), dim3(LP_THREADS), 0, reinterpret_cast<cudaStream_t>(stream), p);
+    return launch_status();
+  };
+  return is_fp32 ? fill(static_cast<float*>(nullptr)) : fill(static_cast<__nv_bfloat16*>(nullptr));
+}
+
+// Rows 0 .. first_pos[b] - 1 of every portion's request from the paged cache to its context.
+GK_EXPORT int gk_latent_gather(const void* cache, const int* tables, const int* first_pos, const int* cu_ctx, void* context,
+                               int portions, int max_blocks, int block_size, int row_bytes, int max_first, void* stream) {
+  if (row_bytes % 16) return -1;
+  if (portions == 0 || max_first == 0) return 0;
+  int blocks = (max_first + 7) / 8;
+  if (blocks > sm_count() * 4) blocks = sm_count() * 4;
+  launch_k(latent_gather_kernel, dim3(blocks, portions), dim3(256), 0, reinterpret_cast<cudaStream_t>(stream),
+           static_cast<const uint4*>(cache), tables, max_blocks, block_size, first_pos, cu_ctx, static_cast<uint4*>(context),
+           row_bytes / 16);
+  return launch_status();
+}

@@ -8,6 +8,9 @@
 //   * memory_output_kernel       per-head RMS norm, gain and sigmoid output gate behind every other case.
 // bf16 prompt portions run the chunkwise kernel in matrix_memory_chunk.cu.
 //
+// Retention is the same recurrence with constant gates and without normaliser and maximum: S_t = decay S + k v^T, output
+// S^T q, normed per head without a gain and gated by a silu.  The RET instances of the kernels compute it.
+//
 // State layout per layer run: S [slots, heads, dim, vdim], n [slots, heads, slices, dim], m [slots, heads, slices]: a head's
 // value columns are cut into slices of 64 that different CTAs own, and each keeps its own copy of n and m, so no CTA
 // reads what another one writes.
@@ -59,8 +62,10 @@ struct ScanParams {
   float* out;              // [rows, heads, vdim] 32-bit (unless the output is finished here)
   T* y;                    // FINISH: [rows, heads * vdim] normed and gated output
   const float* gain;       // FINISH: [heads * vdim]
+  long long y_ld;          // FINISH: elements between rows of y
   int g_off, vdim_true;    // FINISH
   float eps;               // FINISH
+  const float* decay;      // RET: [heads]; gates, n and m are absent
   int width, heads, dim, vdim, slices;
   float cap, q_scale;
 };
@@ -76,9 +81,11 @@ __device__ __forceinline__ void mm_store_remote(const float* local, uint32_t cta
 __device__ __forceinline__ void mm_st1(float* p, float v) { *p = v; }
 __device__ __forceinline__ void mm_st1(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
 
+__device__ __forceinline__ float mm_gate(float g, bool silu) { return (silu ? g : 1.f) / (1.f + expf(-g)); }
+
 // grid (heads * slices, segments).  Thread (warp w, lane): rows rg, rg + 16, ... with rg = 2 w + lane / 16; columns
 // 4 * (lane % 16) .. + 3 of the slice.  R = rows per thread.
-template <typename T, int R, bool FINISH>
+template <typename T, int R, bool FINISH, bool RET>
 __global__ void __launch_bounds__(MM_THREADS, R <= 8 ? 3 : R <= 16 ? 2 : 1) matrix_memory_scan_kernel(const ScanParams<T> p) {
   __shared__ float sq[2][16 * R], sk[2][16 * R];
   __shared__ float red[2][8][MM_SLICE + 4];
@@ -98,7 +105,7 @@ __global__ void __launch_bounds__(MM_THREADS, R <= 8 ? 3 : R <= 16 ? 2 : 1) matr
     for (int r = r_beg; r < r_end; ++r)
       if (tid < MM_SLICE && slice * MM_SLICE + tid < p.vdim) {
         const long long at = (static_cast<long long>(r) * p.heads + head) * p.vdim + slice * MM_SLICE + tid;
-        if (FINISH) mm_st1(p.y + at, 0.f);
+        if (FINISH) mm_st1(p.y + r * p.y_ld + static_cast<long long>(head) * p.vdim + slice * MM_SLICE + tid, 0.f);
         else p.out[at] = 0.f;
       }
     return;      // uniform over the slices of the head
@@ -106,12 +113,12 @@ __global__ void __launch_bounds__(MM_THREADS, R <= 8 ? 3 : R <= 16 ? 2 : 1) matr
   if (FINISH) mm_cluster_arrive();
   const long long sh = static_cast<long long>(slot) * p.heads + head;
   float* Sg = p.S + sh * p.dim * p.vdim + col;
-  float* ng = p.n + (sh * p.slices + slice) * p.dim;
-  float* mg = p.m + sh * p.slices + slice;
+  float* ng = RET ? nullptr : p.n + (sh * p.slices + slice) * p.dim;
+  float* mg = RET ? nullptr : p.m + sh * p.slices + slice;
   const bool fresh = p.first_pos[seg] == 0;
   float4 S[R];
   float n[R];
-  float m = fresh ? 0.f : *mg;
+  float m = RET || fresh ? 0.f : *mg;
 #pragma unroll
   for (int j = 0; j < R; ++j) {
     const int r = rg + 16 * j;
@@ -119,7 +126,7 @@ __global__ void __launch_bounds__(MM_THREADS, R <= 8 ? 3 : R <= 16 ? 2 : 1) matr
     n[j] = 0.f;
     if (!fresh && r < p.dim) {
       if (live) S[j] = *reinterpret_cast<const float4*>(Sg + static_cast<long long>(r) * p.vdim);
-      n[j] = ng[r];
+      if (!RET) n[j] = ng[r];
     }
   }
   auto store_state = [&]() {
@@ -128,12 +135,13 @@ __global__ void __launch_bounds__(MM_THREADS, R <= 8 ? 3 : R <= 16 ? 2 : 1) matr
       const int r = rg + 16 * j;
       if (r < p.dim) {
         if (live) *reinterpret_cast<float4*>(Sg + static_cast<long long>(r) * p.vdim) = S[j];
-        if (c0 == 0) ng[r] = n[j];
+        if (!RET && c0 == 0) ng[r] = n[j];
       }
     }
-    if (tid == 0) *mg = m;
+    if (!RET && tid == 0) *mg = m;
   };
-  const float bi = p.gate_b[head], bf = p.gate_b[p.heads + head];
+  const float bi = RET ? 0.f : p.gate_b[head], bf = RET ? 0.f : p.gate_b[p.heads + head];
+  const float decay = RET ? p.decay[head] : 0.f;
   for (int row = r_beg, it = 0; row < r_end; ++row, ++it) {
     const int buf = it & 1;
     const T* pr = p.proj + row * p.ld;
@@ -143,8 +151,9 @@ __global__ void __launch_bounds__(MM_THREADS, R <= 8 ? 3 : R <= 16 ? 2 : 1) matr
     }
     float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
     if (live) v = mm_ld4(pr + p.v_off + static_cast<long long>(head) * p.vdim + col);
-    float gi, gf;
-    if (p.gates) {
+    float gi = 0.f, gf = 0.f;
+    if (RET) {
+    } else if (p.gates) {
       gi = p.gates[static_cast<long long>(row) * 2 * p.heads + head];
       gf = p.gates[static_cast<long long>(row) * 2 * p.heads + p.heads + head];
     } else {
@@ -169,17 +178,23 @@ __global__ void __launch_bounds__(MM_THREADS, R <= 8 ? 3 : R <= 16 ? 2 : 1) matr
       for (int w = 0; w < 8; ++w) { gi += gred[0][w]; gf += gred[1][w]; }
     }
     __syncthreads();
-    gi = p.cap * tanhf((gi + bi) / p.cap);
-    gf = mm_logsigmoid(p.cap * tanhf((gf + bf) / p.cap));
-    const float mn = fmaxf(gf + m, gi);
-    const float keep = expf(gf + m - mn), put = expf(gi - mn);
-    m = mn;
+    float keep = decay, put = 1.f;
+    if (!RET) {
+      gi = p.cap * tanhf((gi + bi) / p.cap);
+      gf = mm_logsigmoid(p.cap * tanhf((gf + bf) / p.cap));
+      const float mn = fmaxf(gf + m, gi);
+      keep = expf(gf + m - mn);
+      put = expf(gi - mn);
+      m = mn;
+    }
     float a0 = 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f, nq = 0.f;
 #pragma unroll
     for (int j = 0; j < R; ++j) {
       const float q = sq[buf][rg + 16 * j], k = sk[buf][rg + 16 * j] * put;
-      n[j] = keep * n[j] + k;
-      nq += n[j] * q;
+      if (!RET) {
+        n[j] = keep * n[j] + k;
+        nq += n[j] * q;
+      }
       S[j].x = keep * S[j].x + k * v.x; a0 += S[j].x * q;
       S[j].y = keep * S[j].y + k * v.y; a1 += S[j].y * q;
       S[j].z = keep * S[j].z + k * v.z; a2 += S[j].z * q;
@@ -190,10 +205,10 @@ __global__ void __launch_bounds__(MM_THREADS, R <= 8 ? 3 : R <= 16 ? 2 : 1) matr
     a1 += __shfl_xor_sync(0xffffffff, a1, 16);
     a2 += __shfl_xor_sync(0xffffffff, a2, 16);
     a3 += __shfl_xor_sync(0xffffffff, a3, 16);
-    nq += __shfl_xor_sync(0xffffffff, nq, 16);
+    if (!RET) nq += __shfl_xor_sync(0xffffffff, nq, 16);
     if (lane < 16) {
       *reinterpret_cast<float4*>(&red[buf][warp][c0]) = make_float4(a0, a1, a2, a3);
-      if (lane == 0) red[buf][warp][MM_SLICE] = nq;
+      if (!RET && lane == 0) red[buf][warp][MM_SLICE] = nq;
     }
     __syncthreads();
     float o = 0.f;
@@ -202,15 +217,18 @@ __global__ void __launch_bounds__(MM_THREADS, R <= 8 ? 3 : R <= 16 ? 2 : 1) matr
     if (mine) {
       float d = 0.f;
 #pragma unroll
-      for (int w = 0; w < 8; ++w) { o += red[buf][w][tid]; d += red[buf][w][MM_SLICE]; }
-      o = o / (fmaxf(fabsf(d), expf(-m)) + 1e-6f);
+      for (int w = 0; w < 8; ++w) {
+        o += red[buf][w][tid];
+        if (!RET) d += red[buf][w][MM_SLICE];
+      }
+      if (!RET) o = o / (fmaxf(fabsf(d), expf(-m)) + 1e-6f);
       if (!FINISH) p.out[(static_cast<long long>(row) * p.heads + head) * p.vdim + oc] = o;
     }
     if (FINISH) {   // one row per segment
-      float gate = 0.f, gain = 0.f;
+      float gate = 0.f, gain = 1.f;
       if (mine) {
         gate = mm_f(pr[p.g_off + static_cast<long long>(head) * p.vdim + oc]);
-        gain = p.gain[head * p.vdim + oc];
+        if (!RET) gain = p.gain[head * p.vdim + oc];
       }
       if (warp < 2) {
         float ss = o * o;
@@ -227,18 +245,19 @@ __global__ void __launch_bounds__(MM_THREADS, R <= 8 ? 3 : R <= 16 ? 2 : 1) matr
         float ss = 0.f;
         for (int x = 0; x < p.slices; ++x) ss += peer_ss[x];
         const float r = 1.f / sqrtf(ss / p.vdim_true + p.eps);
-        mm_st1(p.y + (static_cast<long long>(row) * p.heads + head) * p.vdim + oc, o * r * gain / (1.f + expf(-gate)));
+        mm_st1(p.y + row * p.y_ld + static_cast<long long>(head) * p.vdim + oc, o * r * gain * mm_gate(gate, RET));
       }
     }
   }
   if (!FINISH && r_end > r_beg) store_state();
 }
 
-// y = o / rms(o over the head's true size) * gain * sigmoid(g).  One warp per (row, head).
+// y = o / rms(o over the head's true size) * gain * sigmoid(g), or without a gain: ... * silu(g).  One warp per
+// (row, head).
 template <typename T>
 __global__ void __launch_bounds__(256) memory_output_kernel(const float* __restrict__ o, const T* __restrict__ proj,
                                                             long long ld, int g_off, const float* __restrict__ gain,
-                                                            T* __restrict__ y, int rows, int heads, int vdim,
+                                                            T* __restrict__ y, long long y_ld, int rows, int heads, int vdim,
                                                             int vdim_true, float eps) {
   pdl_launch_dependents();
   pdl_wait();
@@ -258,18 +277,18 @@ __global__ void __launch_bounds__(256) memory_output_kernel(const float* __restr
   const float r = 1.f / sqrtf(ss / vdim_true + eps);
   for (int c = lane * 4; c < vdim; c += 128) {
     const float4 v = *reinterpret_cast<const float4*>(src + c);
-    const float4 w = *reinterpret_cast<const float4*>(gain + head * vdim + c);
     const float4 g = mm_ld4(proj + row * ld + g_off + static_cast<long long>(head) * vdim + c);
-    mm_st4(y + item * vdim + c, v.x * r * w.x / (1.f + expf(-g.x)), v.y * r * w.y / (1.f + expf(-g.y)),
-           v.z * r * w.z / (1.f + expf(-g.z)), v.w * r * w.w / (1.f + expf(-g.w)));
+    const float4 w = gain ? *reinterpret_cast<const float4*>(gain + head * vdim + c) : g;
+    mm_st4(y + row * y_ld + static_cast<long long>(head) * vdim + c, v.x * r * w.x / (1.f + expf(-g.x)),
+           v.y * r * w.y / (1.f + expf(-g.y)), v.z * r * w.z / (1.f + expf(-g.z)), v.w * r * w.w / (1.f + expf(-g.w)));
   }
 }
 
-template <typename T, int R>
+template <typename T, int R, bool RET>
 int launch_scan_r(const ScanParams<T>& p, int segments, cudaStream_t st) {
   const dim3 grid(p.heads * p.slices, segments);
   if (!p.y) {
-    launch_k(matrix_memory_scan_kernel<T, R, false>, grid, dim3(MM_THREADS), 0, st, p);
+    launch_k(matrix_memory_scan_kernel<T, R, false, RET>, grid, dim3(MM_THREADS), 0, st, p);
     return launch_status();
   }
   cudaLaunchConfig_t cfg = {};
@@ -285,20 +304,20 @@ int launch_scan_r(const ScanParams<T>& p, int segments, cudaStream_t st) {
   attr[1].val.programmaticStreamSerializationAllowed = pdl_flag() ? 1 : 0;
   cfg.attrs = attr;
   cfg.numAttrs = 2;
-  if (cudaLaunchKernelEx(&cfg, matrix_memory_scan_kernel<T, R, true>, p) != cudaSuccess) {
+  if (cudaLaunchKernelEx(&cfg, matrix_memory_scan_kernel<T, R, true, RET>, p) != cudaSuccess) {
     const int rc = launch_status();
     return rc ? rc : -7;
   }
   return launch_status();
 }
 
-template <typename T>
+template <typename T, bool RET>
 int launch_scan(const ScanParams<T>& p, int segments, cudaStream_t st) {
-  if (p.dim <= 32) return launch_scan_r<T, 2>(p, segments, st);
-  if (p.dim <= 64) return launch_scan_r<T, 4>(p, segments, st);
-  if (p.dim <= 128) return launch_scan_r<T, 8>(p, segments, st);
-  if (p.dim <= 256) return launch_scan_r<T, 16>(p, segments, st);
-  if (p.dim <= 512) return launch_scan_r<T, 32>(p, segments, st);
+  if (p.dim <= 32) return launch_scan_r<T, 2, RET>(p, segments, st);
+  if (p.dim <= 64) return launch_scan_r<T, 4, RET>(p, segments, st);
+  if (p.dim <= 128) return launch_scan_r<T, 8, RET>(p, segments, st);
+  if (p.dim <= 256) return launch_scan_r<T, 16, RET>(p, segments, st);
+  if (p.dim <= 512) return launch_scan_r<T, 32, RET>(p, segments, st);
   return -2;
 }
 
@@ -306,14 +325,16 @@ int launch_scan(const ScanParams<T>& p, int segments, cudaStream_t st) {
 
 using namespace gk;
 
-// ptrs: {proj, h, gate_w, gates, gate_b, cu, first_pos, slots, S, n, m, out, y, gain}; y (finished output, one row per
-// segment, at most 512 value columns) replaces out.
+// ptrs: {proj, h, gate_w, gates, gate_b, cu, first_pos, slots, S, n, m, out, y, gain, decay}; y (finished output, one row
+// per segment, at most 512 value columns, rows y_ld apart) replaces out; decay (retention) replaces h to gate_b, n, m, gain.
 // dims: {segments, q_off, k_off, v_off, width, heads, dim, vdim, g_off, vdim_true}
-GK_EXPORT int gk_matrix_memory_scan(int is_fp32, void* const* ptrs, long long ld, const int* dims, float cap,
+GK_EXPORT int gk_matrix_memory_scan(int is_fp32, void* const* ptrs, long long ld, long long y_ld, const int* dims, float cap,
                                     float q_scale, float eps, void* stream) {
   if (dims[0] == 0) return 0;
-  if (dims[7] % 4 || ld % 4 || dims[3] % 4 || (!ptrs[3] && dims[4] % 4)) return -1;
-  if (ptrs[12] && (ptrs[5] || dims[7] > 8 * MM_SLICE || !ptrs[13])) return -3;
+  const bool ret = ptrs[14] != nullptr;
+  if (dims[7] % 4 || ld % 4 || dims[3] % 4 || (!ret && !ptrs[3] && dims[4] % 4)) return -1;
+  if (ptrs[12] && (ptrs[5] || dims[7] > 8 * MM_SLICE || (!ret && !ptrs[13]))) return -3;
+  if (!ret && (!ptrs[4] || !ptrs[9] || !ptrs[10])) return -4;
   auto fill = [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
     ScanParams<T> p;
@@ -332,29 +353,31 @@ GK_EXPORT int gk_matrix_memory_scan(int is_fp32, void* const* ptrs, long long ld
     p.out = static_cast<float*>(ptrs[11]);
     p.y = static_cast<T*>(ptrs[12]);
     p.gain = static_cast<const float*>(ptrs[13]);
-    p.g_off = dims[8]; p.vdim_true = dims[9]; p.eps = eps;
+    p.decay = static_cast<const float*>(ptrs[14]);
+    p.g_off = dims[8]; p.vdim_true = dims[9]; p.eps = eps; p.y_ld = y_ld;
     p.q_off = dims[1]; p.k_off = dims[2]; p.v_off = dims[3];
     p.width = dims[4]; p.heads = dims[5]; p.dim = dims[6]; p.vdim = dims[7];
     p.slices = (p.vdim + MM_SLICE - 1) / MM_SLICE;
     p.cap = cap; p.q_scale = q_scale;
-    return launch_scan<T>(p, dims[0], reinterpret_cast<cudaStream_t>(stream));
+    cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+    return ret ? launch_scan<T, true>(p, dims[0], st) : launch_scan<T, false>(p, dims[0], st);
   };
   return is_fp32 ? fill(static_cast<float*>(nullptr)) : fill(static_cast<__nv_bfloat16*>(nullptr));
 }
 
-// dims: {rows, heads, vdim, vdim_true, g_off}
+// gain null: no gain, silu in place of the sigmoid.  dims: {rows, heads, vdim, vdim_true, g_off}
 GK_EXPORT int gk_memory_output(int is_fp32, const float* o, const void* proj, long long ld, const float* gain, void* y,
-                               const int* dims, float eps, void* stream) {
+                               long long y_ld, const int* dims, float eps, void* stream) {
   const long long items = static_cast<long long>(dims[0]) * dims[1];
   if (items == 0) return 0;
-  if (dims[2] % 4 || ld % 4 || dims[4] % 4) return -1;
+  if (dims[2] % 4 || ld % 4 || y_ld % 4 || dims[4] % 4) return -1;
   const dim3 grid(static_cast<unsigned>((items + 7) / 8));
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   if (is_fp32)
     launch_k(memory_output_kernel<float>, grid, dim3(256), 0, st, o, static_cast<const float*>(proj), ld, dims[4], gain,
-             static_cast<float*>(y), dims[0], dims[1], dims[2], dims[3], eps);
+             static_cast<float*>(y), y_ld, dims[0], dims[1], dims[2], dims[3], eps);
   else
     launch_k(memory_output_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, o, static_cast<const __nv_bfloat16*>(proj), ld,
-             dims[4], gain, static_cast<__nv_bfloat16*>(y), dims[0], dims[1], dims[2], dims[3], eps);
+             dims[4], gain, static_cast<__nv_bfloat16*>(y), y_ld, dims[0], dims[1], dims[2], dims[3], eps);
   return launch_status();
 }

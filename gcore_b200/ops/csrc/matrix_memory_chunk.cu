@@ -7,6 +7,9 @@
 // product reads as bf16 - the decayed scores, the state, the weighted values - enters it as two bf16 terms (rounded
 // value and remainder); the state itself stays in tensor memory in 32-bit from chunk to chunk.
 //
+// Retention (RET) is the case of constant gates, f = log(decay) and i = 0, without normaliser, maximum and denominator:
+// a_s = -s log(decay), g_t = -t log(decay), and the state enters as if m_0 were log(decay).
+//
 // One CTA = one head of one portion and a slice of 64 value columns.  Keys of more than 128 dims are taken in halves.
 //   warps 0-7   elementwise work: state -> operand, weighted values, decayed scores, output (lane quadrant = warp & 3,
 //               column half = warp >> 2)
@@ -59,6 +62,7 @@ struct McParams {
   float* out;              // [rows, heads, vdim]
   int heads, dim, vdim, slices;
   float cap, q_scale;
+  const float* decay;      // RET: [heads]; gates, gate_b, n and m are absent
   int* err;
 };
 
@@ -84,7 +88,7 @@ __device__ __forceinline__ void mc_put_row01(uint8_t* base, int e, float v) {
   *reinterpret_cast<uint16_t*>(c + 128 + ((u ^ 1) << 4)) = static_cast<uint16_t>(l);
 }
 
-template <int NH>
+template <int NH, bool RET>
 __global__ void __launch_bounds__(MC_THREADS, 1)
 matrix_memory_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                            const __grid_constant__ CUtensorMap tmV, McParams p) {
@@ -111,8 +115,8 @@ matrix_memory_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
   const int chunks = (len + MC_L - 1) / MC_L;
   const bool fresh = p.first_pos[seg] == 0;
   const long long sh = static_cast<long long>(slot) * p.heads + head;
-  float* ng = p.n + (sh * p.slices + slice) * p.dim;
-  float* mg = p.m + sh * p.slices + slice;
+  float* ng = RET ? nullptr : p.n + (sh * p.slices + slice) * p.dim;
+  float* mg = RET ? nullptr : p.m + sh * p.slices + slice;
 
   if (tid == 0) {
     mbar_init(qk_full, 1);
@@ -211,8 +215,9 @@ matrix_memory_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
             const uint64_t a = make_smem_desc_sw128(aQ + (k4 >> 2) * 16384 + (k4 & 3) * 32, 16, 1024);
             umma_f16(t_oi, a, make_smem_desc_sw128(aST + k4 * 2048, 16384, 1024), id_o, (h > 0 || k4 > 0) ? 1u : 0u);
             umma_f16(t_oi, a, make_smem_desc_sw128(aST + 16384 + k4 * 2048, 16384, 1024), id_o, 1u);
-            umma_f16(t_qn, a, make_smem_desc_sw128(aN + (k4 >> 2) * 2048 + (k4 & 3) * 32, 16, 1024), id_qn,
-                     (h > 0 || k4 > 0) ? 1u : 0u);
+            if (!RET)
+              umma_f16(t_qn, a, make_smem_desc_sw128(aN + (k4 >> 2) * 2048 + (k4 & 3) * 32, 16, 1024), id_qn,
+                       (h > 0 || k4 > 0) ? 1u : 0u);
           }
         }
         __syncwarp();
@@ -227,7 +232,8 @@ matrix_memory_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
             const uint64_t a = make_smem_desc_sw128(aK + k4 * 2048, 16384, 1024);
             umma_f16(tmem + MC_T_ST + h * 64, a, make_smem_desc_sw128(aVW + k4 * 2048, 16384, 1024), id_up, 1u);
             umma_f16(tmem + MC_T_ST + h * 64, a, make_smem_desc_sw128(aVW + 16384 + k4 * 2048, 16384, 1024), id_up, 1u);
-            umma_f16(tmem + MC_T_N + h * 16, a, make_smem_desc_sw128(aW + (k4 >> 2) * 2048 + (k4 & 3) * 32, 16, 1024), id_un, 1u);
+            if (!RET)
+              umma_f16(tmem + MC_T_N + h * 16, a, make_smem_desc_sw128(aW + (k4 >> 2) * 2048 + (k4 & 3) * 32, 16, 1024), id_un, 1u);
           }
           umma_commit(upd_done);
           umma_commit(qk_empty);
@@ -254,14 +260,27 @@ matrix_memory_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
     }
   } else if (warp == 10) {
     // ------------------------------------------------------------------ gates: a, g, m of every token of a chunk
-    const float bi = p.gate_b[head], bf = p.gate_b[p.heads + head];
-    float m0 = fresh ? 0.f : *mg;
+    const float bi = RET ? 0.f : p.gate_b[head], bf = RET ? 0.f : p.gate_b[p.heads + head];
+    const float log_decay = RET ? fmaxf(logf(p.decay[head]), -80.f) : 0.f;
+    float m0 = RET ? log_decay : fresh ? 0.f : *mg;
     bool ok = true;
     for (int c = 0; c < chunks; ++c) {
       const int buf = c & 1;
       ok = mbar_wait(&g_empty[buf], ((c >> 1) & 1) ^ 1, p.err, ERR_WAIT_EMPTY);
       if (!ok) break;
       float* gs = gates_s + buf * McSmem::GATE_FLOATS;
+      if (RET) {
+        const int last = len - c * MC_L - 1 < MC_L - 1 ? len - c * MC_L - 1 : MC_L - 1;   // newest token of the chunk
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const int t = lane * 4 + j;
+          gs[t] = t <= last ? -static_cast<float>(t) * log_decay : -1e30f;
+          gs[MC_L + t] = -static_cast<float>(t < last ? t : last) * log_decay;
+        }
+        if (lane == 0) gs[3 * MC_L] = m0;
+        mbar_arrive(&g_full[buf]);
+        continue;
+      }
       float gi[4], b[4];
       float sum = 0.f;
 #pragma unroll
@@ -314,7 +333,7 @@ matrix_memory_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
       m0 = __shfl_sync(0xffffffff, mt, 31);
       mbar_arrive(&g_full[buf]);
     }
-    if (ok && lane == 0) *mg = m0;
+    if (!RET && ok && lane == 0) *mg = m0;
   } else {
     // ------------------------------------------------------------------ elementwise warps
     const int quad = warp & 3, half = warp >> 2;
@@ -336,7 +355,7 @@ matrix_memory_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
         w[j + 2] = __float_as_uint(v.z); w[j + 3] = __float_as_uint(v.w);
       }
       tmem_st32(lane_addr + MC_T_ST + h * 64 + half * 32, w);
-      if (half == 0) {
+      if (!RET && half == 0) {
         uint32_t nv[16];
 #pragma unroll
         for (int j = 0; j < 16; ++j) nv[j] = 0;
@@ -376,7 +395,7 @@ matrix_memory_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
           *reinterpret_cast<uint4*>(dst + 16384 + o) = lo;
         }
         tmem_st32(ta, w);
-        if (half == 0) {
+        if (!RET && half == 0) {
           uint32_t nv[16];
           tmem_ld16(lane_addr + MC_T_N + h * 16, nv);
           tmem_ld_wait();
@@ -417,7 +436,7 @@ matrix_memory_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
         *reinterpret_cast<uint4*>(dst + o) = hi;
         *reinterpret_cast<uint4*>(dst + 16384 + o) = lo;
       }
-      if (half == 0) mc_put_row01(smem + McSmem::W, r, wt);
+      if (!RET && half == 0) mc_put_row01(smem + McSmem::W, r, wt);
       fence_proxy_async();
       mbar_arrive(vw_ready);
       return true;
@@ -458,7 +477,7 @@ matrix_memory_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
           for (int e = 0; e < 8; ++e) {
             const float x2 = fmaf(av[e] - g, MC_LOG2E, log_qs);
             v[e] = __uint_as_float(w[u * 8 + e]) * ex2(s0 + e <= r ? x2 : -1e30f);
-            rs += v[e];
+            if (!RET) rs += v[e];
           }
           mc_split8(v, hi, lo);
           const int o = ((x * 4 + u) ^ (r & 7)) << 4;
@@ -466,7 +485,7 @@ matrix_memory_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
           *reinterpret_cast<uint4*>(prow + 32768 + o) = lo;
         }
       }
-      rsum[(buf * 2 + half) * MC_L + r] = rs;
+      if (!RET) rsum[(buf * 2 + half) * MC_L + r] = rs;
       fence_proxy_async();
       tc_fence_before();
       mbar_arrive(p_ready);
@@ -481,13 +500,16 @@ matrix_memory_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
       {
         const float inter = ex2((m0 - g) * MC_LOG2E) * p.q_scale;
         uint32_t qn[16], oi[32], oa[32];
-        tmem_ld16(lane_addr + MC_T_QN + buf * 16, qn);
+        if (!RET) tmem_ld16(lane_addr + MC_T_QN + buf * 16, qn);
         tmem_ld32(lane_addr + MC_T_OI + buf * 64 + half * 32, oi);
         tmem_ld32(lane_addr + MC_T_OA + half * 32, oa);
         tmem_ld_wait();
-        const float den = inter * (__uint_as_float(qn[0]) + __uint_as_float(qn[1])) + rsum[buf * 2 * MC_L + r] +
-                          rsum[(buf * 2 + 1) * MC_L + r];
-        const float inv = 1.f / (fmaxf(fabsf(den), ex2(-gs[2 * MC_L + r] * MC_LOG2E)) + 1e-6f);
+        float inv = 1.f;
+        if (!RET) {
+          const float den = inter * (__uint_as_float(qn[0]) + __uint_as_float(qn[1])) + rsum[buf * 2 * MC_L + r] +
+                            rsum[(buf * 2 + 1) * MC_L + r];
+          inv = 1.f / (fmaxf(fabsf(den), ex2(-gs[2 * MC_L + r] * MC_LOG2E)) + 1e-6f);
+        }
         // a warp's 32 x 32 outputs change hands in shared memory (the scores' buffer is free now), so that its stores
         // are whole 128-byte lines; 16-byte unit u of row r sits at unit u ^ (r & 7)
         uint8_t* stage = smem + McSmem::P + warp * 4096;
@@ -524,7 +546,7 @@ matrix_memory_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
           const int d = h * MC_DH + r;
           uint32_t w[32], nv[16];
           tmem_ld32(lane_addr + MC_T_ST + h * 64 + half * 32, w);
-          tmem_ld16(lane_addr + MC_T_N + h * 16, nv);
+          if (!RET) tmem_ld16(lane_addr + MC_T_N + h * 16, nv);
           tmem_ld_wait();
           if (d < p.dim) {
             float* dst = p.S + (sh * p.dim + d) * p.vdim + col0;
@@ -535,7 +557,7 @@ matrix_memory_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
                                                                   __uint_as_float(w[j + 2]), __uint_as_float(w[j + 3]));
               }
             }
-            if (half == 0) ng[d] = __uint_as_float(nv[0]) + __uint_as_float(nv[1]);
+            if (!RET && half == 0) ng[d] = __uint_as_float(nv[0]) + __uint_as_float(nv[1]);
           }
         }
       }
@@ -550,17 +572,17 @@ matrix_memory_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
   }
 }
 
-template <int NH>
+template <int NH, bool RET>
 int launch_mc(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const McParams& p, int portions,
               cudaStream_t st) {
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(matrix_memory_chunk_kernel<NH>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    cudaError_t e = cudaFuncSetAttribute(matrix_memory_chunk_kernel<NH, RET>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          McSmem::BYTES);
     if (e != cudaSuccess) return static_cast<int>(e);
     configured = true;
   }
-  launch_k(matrix_memory_chunk_kernel<NH>, dim3(p.heads * p.slices, portions), dim3(MC_THREADS), McSmem::BYTES, st, tq, tk,
+  launch_k(matrix_memory_chunk_kernel<NH, RET>, dim3(p.heads * p.slices, portions), dim3(MC_THREADS), McSmem::BYTES, st, tq, tk,
            tv, p);
   return launch_status();
 }
@@ -570,7 +592,7 @@ int launch_mc(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& t
 using namespace gk;
 
 // bf16 prompt portions, keys of at most 256 dims (a multiple of 8), values a multiple of 8 wide.
-// ptrs: {proj, gates, gate_b, cu, first_pos, slots, S, n, m, out, err}
+// ptrs: {proj, gates, gate_b, cu, first_pos, slots, S, n, m, out, err, decay}; decay (retention) replaces gates, gate_b, n, m
 // dims: {portions, rows, q_off, k_off, v_off, heads, dim, vdim}
 GK_EXPORT int gk_matrix_memory_chunk(void* const* ptrs, long long ld, const int* dims, float cap, float q_scale,
                                      void* stream) {
@@ -594,8 +616,11 @@ GK_EXPORT int gk_matrix_memory_chunk(void* const* ptrs, long long ld, const int*
   p.m = static_cast<float*>(ptrs[8]);
   p.out = static_cast<float*>(ptrs[9]);
   p.err = static_cast<int*>(ptrs[10]);
+  p.decay = static_cast<const float*>(ptrs[11]);
+  if (!p.decay && (!p.gates || !p.gate_b || !p.n || !p.m)) return -6;
   p.heads = heads; p.dim = dim; p.vdim = vdim; p.slices = (vdim + MC_SLICE - 1) / MC_SLICE;
   p.cap = cap; p.q_scale = q_scale;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
-  return dim <= MC_DH ? launch_mc<1>(tq, tk, tv, p, n, st) : launch_mc<2>(tq, tk, tv, p, n, st);
+  if (p.decay) return dim <= MC_DH ? launch_mc<1, true>(tq, tk, tv, p, n, st) : launch_mc<2, true>(tq, tk, tv, p, n, st);
+  return dim <= MC_DH ? launch_mc<1, false>(tq, tk, tv, p, n, st) : launch_mc<2, false>(tq, tk, tv, p, n, st);
 }

@@ -13,6 +13,8 @@
 //     and multiplies the probabilities, re-packed in registers as an A operand, with its quarter of the value columns.
 //     (Evaluating each exponential once and passing P through shared memory costs a third barrier per tile and
 //     measured 5 % slower: the kernel is bound by issue latency at two warps per scheduler, not by the exponentials.)
+// SPLIT instances keep the probabilities at 16 significant bits (two bf16 terms, rounded value and remainder), and any
+// instance can scale the output by a sigmoid gate per (request, head).
 // Stands in for the latent decode kernels the reference reaches through its serving engines and its own
 // gpatch_v4/models/deepseek_v4/kernel/flash_mla_wrapper.py:56-160.
 #include "host_utils.h"
@@ -79,14 +81,20 @@ __device__ __forceinline__ uint32_t pack2(float lo, float hi) {
   return *reinterpret_cast<uint32_t*>(&v);
 }
 
+__device__ __forceinline__ float rest(float v) { return v - __bfloat162float(__float2bfloat16(v)); }
+__device__ __forceinline__ float gate_of(const __nv_bfloat16* gate, long long gate_ld, int b, int h) {
+  return gate ? 1.f / (1.f + __expf(-__bfloat162float(gate[b * gate_ld + h]))) : 1.f;
+}
+
 // q_lat [B, H, CV] and q_rope [B, H, DR] and out [B, H, CV] are addressed through (batch, head) strides in elements,
 // so the batched projections around the kernel can keep their head-major layout.
-template <int CV, int DR>
+template <int CV, int DR, bool SPLIT>
 __global__ void __launch_bounds__(THREADS, 2) mla_paged_decode_kernel(
     const __nv_bfloat16* __restrict__ q_lat, long long qs_b, long long qs_h, const __nv_bfloat16* __restrict__ q_rope,
     long long rs_b, long long rs_h, const __nv_bfloat16* __restrict__ cache, const int* __restrict__ block_table,
     int max_blocks, const int* __restrict__ ctx_len, __nv_bfloat16* __restrict__ out, long long os_b, long long os_h,
-    float* __restrict__ scratch, int H, int block_size, float scale, int nsplit, int split_tokens) {
+    float* __restrict__ scratch, int H, int block_size, float scale, int nsplit, int split_tokens,
+    const __nv_bfloat16* __restrict__ gate, long long gate_ld) {
   using G = Geo<CV, DR>;
   extern __shared__ __align__(128) uint8_t mla_smem[];
   uint8_t* sq = mla_smem;
@@ -243,7 +251,7 @@ __global__ void __launch_bounds__(THREADS, 2) mla_paged_decode_kernel(
 #pragma unroll
       for (int j = 0; j < G::NT; ++j) { o[j][0] *= resc[0]; o[j][1] *= resc[0]; o[j][2] *= resc[1]; o[j][3] *= resc[1]; }
     }
-    uint32_t pa[2][4];
+    uint32_t pa[2][4], pr[2][4];
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       float p[4];
@@ -255,6 +263,10 @@ __global__ void __launch_bounds__(THREADS, 2) mla_paged_decode_kernel(
       // A fragment of k-step j / 2: {rows lo cols lo, rows hi cols lo, rows lo cols hi, rows hi cols hi}
       pa[j >> 1][(j & 1) * 2] = pack2(p[0], p[1]);
       pa[j >> 1][(j & 1) * 2 + 1] = pack2(p[2], p[3]);
+      if (SPLIT) {
+        pr[j >> 1][(j & 1) * 2] = pack2(rest(p[0]), rest(p[1]));
+        pr[j >> 1][(j & 1) * 2 + 1] = pack2(rest(p[2]), rest(p[3]));
+      }
     }
 
     // ---- O += P V on this warp's quarter of the value columns: 2 k-steps of 16 tokens
@@ -268,6 +280,10 @@ __global__ void __launch_bounds__(THREADS, 2) mla_paged_decode_kernel(
         ldsm_x4_trans(vb, tb + swz(row, ch, G::ROW_BYTES));
         mma_16816(o[2 * np], pa[kk], vb[0], vb[1]);
         mma_16816(o[2 * np + 1], pa[kk], vb[2], vb[3]);
+        if (SPLIT) {
+          mma_16816(o[2 * np], pr[kk], vb[0], vb[1]);
+          mma_16816(o[2 * np + 1], pr[kk], vb[2], vb[3]);
+        }
       }
     }
   }
@@ -283,7 +299,7 @@ __global__ void __launch_bounds__(THREADS, 2) mla_paged_decode_kernel(
     if (head >= H) continue;
     const int col0 = warp * G::COLS_PER_WARP + cq;
     if (nsplit == 1) {
-      const float inv = l_run[h] > 0.f ? 1.f / l_run[h] : 0.f;
+      const float inv = l_run[h] > 0.f ? gate_of(gate, gate_ld, b, head) / l_run[h] : 0.f;
       __nv_bfloat16* dst = out + b * os_b + head * os_h + col0;
 #pragma unroll
       for (int j = 0; j < G::NT; ++j) {
@@ -304,7 +320,8 @@ __global__ void __launch_bounds__(THREADS, 2) mla_paged_decode_kernel(
 // Merges the live KV splits of one (request, head): scratch rows are [CV values | running max | running sum].
 __global__ void mla_decode_combine_kernel(const float* __restrict__ scratch, const int* __restrict__ ctx_len,
                                           __nv_bfloat16* __restrict__ out, long long os_b, long long os_h, int H,
-                                          int CV, int nsplit_total, int split_tokens) {
+                                          int CV, int nsplit_total, int split_tokens,
+                                          const __nv_bfloat16* __restrict__ gate, long long gate_ld) {
   pdl_launch_dependents();
   pdl_wait();
   const int b = blockIdx.x, h = blockIdx.y;
@@ -319,7 +336,7 @@ __global__ void mla_decode_combine_kernel(const float* __restrict__ scratch, con
     const float ms = base[s * (CV + 2) + CV];
     l += base[s * (CV + 2) + CV + 1] * (ms == -FLT_MAX ? 0.f : __expf(ms - m));
   }
-  const float inv = l > 0.f ? 1.f / l : 0.f;
+  const float inv = l > 0.f ? gate_of(gate, gate_ld, b, h) / l : 0.f;
   for (int d = threadIdx.x; d < CV; d += blockDim.x) {
     float acc = 0.f;
     for (int s = 0; s < nsplit; ++s) {
@@ -347,21 +364,22 @@ static void plan(int B, int H, int max_ctx, int* nsplit, int* split_tokens) {
   *split_tokens = st;
 }
 
-template <int CV, int DR>
+template <int CV, int DR, bool SPLIT>
 static int launch(const void* q_lat, long long qs_b, long long qs_h, const void* q_rope, long long rs_b,
                   long long rs_h, const void* cache, const int* block_table, int max_blocks, const int* ctx_len,
                   void* out, long long os_b, long long os_h, float* scratch, int B, int H, int block_size, float scale,
-                  int nsplit, int split_tokens, cudaStream_t st) {
+                  int nsplit, int split_tokens, const __nv_bfloat16* gate, long long gate_ld, cudaStream_t st) {
   using G = Geo<CV, DR>;
   static bool configured = false;
   if (!configured) {
-    cudaFuncSetAttribute(mla_paged_decode_kernel<CV, DR>, cudaFuncAttributeMaxDynamicSharedMemorySize, G::SMEM);
+    cudaFuncSetAttribute(mla_paged_decode_kernel<CV, DR, SPLIT>, cudaFuncAttributeMaxDynamicSharedMemorySize, G::SMEM);
     configured = true;
   }
-  launch_k(mla_paged_decode_kernel<CV, DR>, dim3(B, (H + HEADS - 1) / HEADS, nsplit), dim3(THREADS), G::SMEM, st,
+  launch_k(mla_paged_decode_kernel<CV, DR, SPLIT>, dim3(B, (H + HEADS - 1) / HEADS, nsplit), dim3(THREADS), G::SMEM, st,
            reinterpret_cast<const __nv_bfloat16*>(q_lat), qs_b, qs_h, reinterpret_cast<const __nv_bfloat16*>(q_rope),
            rs_b, rs_h, reinterpret_cast<const __nv_bfloat16*>(cache), block_table, max_blocks, ctx_len,
-           reinterpret_cast<__nv_bfloat16*>(out), os_b, os_h, scratch, H, block_size, scale, nsplit, split_tokens);
+           reinterpret_cast<__nv_bfloat16*>(out), os_b, os_h, scratch, H, block_size, scale, nsplit, split_tokens, gate,
+           gate_ld);
   return 0;
 }
 
@@ -382,28 +400,48 @@ GK_EXPORT void gk_mla_decode_scratch(int B, int H, int CV, int max_ctx, long lon
   *floats = ns > 1 ? static_cast<long long>(B) * H * ns * (CV + 2) : 0;
 }
 
-// max_ctx bounds every ctx_len[b]; strides are in elements and must be multiples of 8 (16-byte query loads).
-GK_EXPORT int gk_mla_paged_decode(const void* q_lat, long long qs_b, long long qs_h, const void* q_rope,
-                                  long long rs_b, long long rs_h, const void* cache, const int* block_table,
-                                  const int* ctx_len, void* out, long long os_b, long long os_h, float* scratch,
-                                  int B, int H, int CV, int DR, int block_size, int max_blocks, int max_ctx,
-                                  float scale, void* stream) {
+static int decode(const void* q_lat, long long qs_b, long long qs_h, const void* q_rope, long long rs_b, long long rs_h,
+                  const void* cache, const int* block_table, const int* ctx_len, void* out, long long os_b, long long os_h,
+                  float* scratch, int B, int H, int CV, int DR, int block_size, int max_blocks, int max_ctx, float scale,
+                  bool split, const __nv_bfloat16* gate, long long gate_ld, cudaStream_t st) {
   if (!gk_mla_decode_supported(CV, DR)) return -1;
   if ((qs_b | qs_h | rs_b | rs_h) % 8 || (os_b | os_h) % 2) return -3;
   if (B == 0 || H == 0) return 0;
   int nsplit, split_tokens;
   plan(B, H, max_ctx, &nsplit, &split_tokens);
   if (nsplit > 1 && !scratch) return -2;
-  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
 #define GK_MLA_ARGS q_lat, qs_b, qs_h, q_rope, rs_b, rs_h, cache, block_table, max_blocks, ctx_len, out, os_b, os_h, \
-                    scratch, B, H, block_size, scale, nsplit, split_tokens, st
-  if (CV == 512) launch<512, 64>(GK_MLA_ARGS);
-  else if (CV == 256) launch<256, 64>(GK_MLA_ARGS);
-  else launch<128, 32>(GK_MLA_ARGS);
+                    scratch, B, H, block_size, scale, nsplit, split_tokens, gate, gate_ld, st
+#define GK_MLA_LAUNCH(cv, dr) (split ? launch<cv, dr, true>(GK_MLA_ARGS) : launch<cv, dr, false>(GK_MLA_ARGS))
+  if (CV == 512) GK_MLA_LAUNCH(512, 64);
+  else if (CV == 256) GK_MLA_LAUNCH(256, 64);
+  else GK_MLA_LAUNCH(128, 32);
+#undef GK_MLA_LAUNCH
 #undef GK_MLA_ARGS
   if (nsplit > 1) {
     launch_k(mla_decode_combine_kernel, dim3(B, H), dim3(128), 0, st, static_cast<const float*>(scratch), ctx_len,
-             reinterpret_cast<__nv_bfloat16*>(out), os_b, os_h, H, CV, nsplit, split_tokens);
+             reinterpret_cast<__nv_bfloat16*>(out), os_b, os_h, H, CV, nsplit, split_tokens, gate, gate_ld);
   }
   return launch_status();
+}
+
+// max_ctx bounds every ctx_len[b]; strides are in elements and must be multiples of 8 (16-byte query loads).
+GK_EXPORT int gk_mla_paged_decode(const void* q_lat, long long qs_b, long long qs_h, const void* q_rope,
+                                  long long rs_b, long long rs_h, const void* cache, const int* block_table,
+                                  const int* ctx_len, void* out, long long os_b, long long os_h, float* scratch,
+                                  int B, int H, int CV, int DR, int block_size, int max_blocks, int max_ctx,
+                                  float scale, void* stream) {
+  return decode(q_lat, qs_b, qs_h, q_rope, rs_b, rs_h, cache, block_table, ctx_len, out, os_b, os_h, scratch, B, H, CV, DR,
+                block_size, max_blocks, max_ctx, scale, false, nullptr, 0, reinterpret_cast<cudaStream_t>(stream));
+}
+
+// The same with 32-bit-like probabilities (two bf16 terms) and a gate: logits [B, gate_ld], one per head, or null.
+GK_EXPORT int gk_mla_paged_decode_gated(const void* q_lat, long long qs_b, long long qs_h, const void* q_rope,
+                                        long long rs_b, long long rs_h, const void* cache, const int* block_table,
+                                        const int* ctx_len, void* out, long long os_b, long long os_h, float* scratch,
+                                        int B, int H, int CV, int DR, int block_size, int max_blocks, int max_ctx,
+                                        float scale, const void* gate, long long gate_ld, void* stream) {
+  return decode(q_lat, qs_b, qs_h, q_rope, rs_b, rs_h, cache, block_table, ctx_len, out, os_b, os_h, scratch, B, H, CV, DR,
+                block_size, max_blocks, max_ctx, scale, true, static_cast<const __nv_bfloat16*>(gate), gate_ld,
+                reinterpret_cast<cudaStream_t>(stream));
 }

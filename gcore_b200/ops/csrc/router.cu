@@ -26,6 +26,9 @@ struct RouterParams {
   int E, K, G, topk_group;
   int sigmoid, norm;
   float scale;
+  long long ld;             // floats between the logits of two tokens
+  int* counts;              // [E] or null: tokens of every expert, added to what is there
+  int* place;               // [T, K] with counts: the choice's place among its expert's tokens
 };
 
 __device__ __forceinline__ void warp_argmax(float& v, int& i) {
@@ -41,22 +44,24 @@ template <int VPT>
 __global__ void __launch_bounds__(256) router_fwd_kernel(RouterParams p) {
   const long long t = (blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x) >> 5;
   const int lane = threadIdx.x & 31;
+  gk::pdl_launch_dependents();
+  gk::pdl_wait();
   if (t >= p.T) return;
-  const float* row = p.logits + t * p.E;
+  const float* row = p.logits + t * p.ld;
   float sc[VPT], sel[VPT];
-  // ---- scores
+  // ---- scores (lanes past the last expert hold none)
   if (p.sigmoid) {
 #pragma unroll
-    for (int i = 0; i < VPT; ++i) sc[i] = 1.f / (1.f + __expf(-row[lane + 32 * i]));
+    for (int i = 0; i < VPT; ++i) sc[i] = lane + 32 * i < p.E ? 1.f / (1.f + expf(-row[lane + 32 * i])) : 0.f;
   } else {
     float m = -FLT_MAX;
 #pragma unroll
-    for (int i = 0; i < VPT; ++i) { sc[i] = row[lane + 32 * i]; m = fmaxf(m, sc[i]); }
+    for (int i = 0; i < VPT; ++i) { sc[i] = lane + 32 * i < p.E ? row[lane + 32 * i] : -FLT_MAX; m = fmaxf(m, sc[i]); }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
     float s = 0.f;
 #pragma unroll
-    for (int i = 0; i < VPT; ++i) { sc[i] = __expf(sc[i] - m); s += sc[i]; }
+    for (int i = 0; i < VPT; ++i) { sc[i] = lane + 32 * i < p.E ? expf(sc[i] - m) : 0.f; s += sc[i]; }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
     const float inv = 1.f / s;
@@ -83,7 +88,8 @@ __global__ void __launch_bounds__(256) router_fwd_kernel(RouterParams p) {
     }
   } else {
 #pragma unroll
-    for (int i = 0; i < VPT; ++i) sel[i] = sc[i] + (p.bias ? p.bias[lane + 32 * i] : 0.f);
+    for (int i = 0; i < VPT; ++i)
+      sel[i] = lane + 32 * i < p.E ? sc[i] + (p.bias ? p.bias[lane + 32 * i] : 0.f) : -FLT_MAX;
     if (p.G > 1) {
       // group score = sum of the two best selection scores inside the group
       const int gs = p.E / p.G;
@@ -165,6 +171,7 @@ __global__ void __launch_bounds__(256) router_fwd_kernel(RouterParams p) {
       if (k == lane) { wv = chosen_w[k]; iv = chosen_i[k]; }
     out_idx[lane] = iv;
     out_w[lane] = wv / denom * p.scale;
+    if (p.counts) p.place[t * p.K + lane] = atomicAdd(p.counts + iv, 1);
   }
 }
 
@@ -187,7 +194,7 @@ __global__ void __launch_bounds__(256) router_bwd_kernel(RouterBwdParams p) {
   float sc[VPT], g[VPT];
   if (p.sigmoid) {
 #pragma unroll
-    for (int i = 0; i < VPT; ++i) sc[i] = 1.f / (1.f + __expf(-row[lane + 32 * i]));
+    for (int i = 0; i < VPT; ++i) sc[i] = 1.f / (1.f + expf(-row[lane + 32 * i]));
   } else {
     float m = -FLT_MAX;
 #pragma unroll
@@ -196,7 +203,7 @@ __global__ void __launch_bounds__(256) router_bwd_kernel(RouterBwdParams p) {
     for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
     float s = 0.f;
 #pragma unroll
-    for (int i = 0; i < VPT; ++i) { sc[i] = __expf(sc[i] - m); s += sc[i]; }
+    for (int i = 0; i < VPT; ++i) { sc[i] = expf(sc[i] - m); s += sc[i]; }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
     const float inv = 1.f / s;
@@ -251,36 +258,52 @@ __global__ void __launch_bounds__(256) router_bwd_kernel(RouterBwdParams p) {
 
 template <typename P, typename F>
 int dispatch_vpt(int E, const P& p, F launch) {
-  switch (E / 32) {
-    case 1: return launch(std::integral_constant<int, 1>{});
-    case 2: return launch(std::integral_constant<int, 2>{});
-    case 4: return launch(std::integral_constant<int, 4>{});
-    case 8: return launch(std::integral_constant<int, 8>{});
-    case 16: return launch(std::integral_constant<int, 16>{});
-    default: return -2;
-  }
+  if (E <= 32) return launch(std::integral_constant<int, 1>{});
+  if (E <= 64) return launch(std::integral_constant<int, 2>{});
+  if (E <= 128) return launch(std::integral_constant<int, 4>{});
+  if (E <= 256) return launch(std::integral_constant<int, 8>{});
+  if (E <= 512) return launch(std::integral_constant<int, 16>{});
+  return -2;
 }
 
 }  // namespace gkr
 
 using namespace gkr;
 
-// E in {32, 64, 128, 256, 512}; K <= 16; G <= 8 and E % G == 0.  Returns -2 for an expert count without a kernel.
+static int router_launch(const RouterParams& p, cudaStream_t st) {
+  if (p.E < 1 || p.K < 1 || p.K > MAX_K || p.K > p.E || p.G < 1 || p.G > MAX_G || p.E % p.G ||
+      (p.G > 1 && (p.topk_group < 1 || p.topk_group > p.G)))
+    return -1;
+  const unsigned blocks = static_cast<unsigned>((p.T + 7) / 8);
+  return dispatch_vpt(p.E, p, [&](auto v) {
+    gk::launch_k(router_fwd_kernel<decltype(v)::value>, dim3(blocks), dim3(256), 0, st, p);
+    return gk::launch_status();
+  });
+}
+
+// E <= 512; K <= 16; G <= 8 and E % G == 0.  Returns -2 for an expert count without a kernel.
 GK_EXPORT int gk_router_fwd(const float* logits, const float* bias, const long long* replay, long long* idx, float* w,
                             long long T, int E, int K, int G, int topk_group, int sigmoid, int norm, float scale,
                             void* stream) {
   if (T <= 0) return 0;
-  if (E % 32 || K < 1 || K > MAX_K || K > E || G < 1 || G > MAX_G || E % G || (G > 1 && (topk_group < 1 || topk_group > G)))
-    return -1;
   RouterParams p;
   p.logits = logits; p.bias = bias; p.replay = replay; p.idx = idx; p.w = w; p.T = T; p.E = E; p.K = K; p.G = G;
   p.topk_group = topk_group; p.sigmoid = sigmoid; p.norm = norm; p.scale = scale;
-  const unsigned blocks = static_cast<unsigned>((T + 7) / 8);
-  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
-  return dispatch_vpt(E, p, [&](auto v) {
-    router_fwd_kernel<decltype(v)::value><<<blocks, 256, 0, st>>>(p);
-    return gk::launch_status();
-  });
+  p.ld = E; p.counts = nullptr; p.place = nullptr;
+  return router_launch(p, reinterpret_cast<cudaStream_t>(stream));
+}
+
+// Routing of served models: logits rows `ld` floats apart, and the dispatch bookkeeping in the same launch (counts [E],
+// cleared by the caller, and every choice's place [T, K] among its expert's tokens; the places' order is not fixed).
+GK_EXPORT int gk_router_dispatch(const float* logits, long long ld, const float* bias, long long* idx, float* w, int* counts,
+                                 int* place, long long T, int E, int K, int sigmoid, int norm, float scale, void* stream) {
+  if (T <= 0) return 0;
+  if (ld < E || !counts || !place) return -1;
+  RouterParams p;
+  p.logits = logits; p.bias = bias; p.replay = nullptr; p.idx = idx; p.w = w; p.T = T; p.E = E; p.K = K; p.G = 1;
+  p.topk_group = 1; p.sigmoid = sigmoid; p.norm = norm; p.scale = scale;
+  p.ld = ld; p.counts = counts; p.place = place;
+  return router_launch(p, reinterpret_cast<cudaStream_t>(stream));
 }
 
 GK_EXPORT int gk_router_bwd(const float* logits, const long long* idx, const float* dw, float* dlogits, long long T,

@@ -2,10 +2,10 @@
 // one launch takes a sublayer's output to the next sublayer's input,
 //     x <- x + post_norm(y) [+ embedding output] [+ step vector];   h <- pre_norm(x)
 // where y is one tensor, or half the sum of two mixers' outputs each normalised with a gain of its own, and the first
-// launch of a forward pass builds x from the token and position tables instead.  Norm gains are 32-bit; "one-plus"
+// launch of a forward pass builds x from the token table (and the position table of models that have one) instead.  Norm gains are 32-bit; "one-plus"
 // gains are stored as (1 + w) by the loader, so every norm here is x / sqrt(mean(x^2) + eps) * gain.
 #include "host_utils.h"
-#include <cuda_bf16.h>
+#include "row_ops.cuh"
 #include <type_traits>
 
 namespace gk {
@@ -17,7 +17,7 @@ struct SandwichParams {
   const long long* tokens;   // SRC_EMBED
   const int* pos;            // SRC_EMBED
   const T* embed;            // [vocab, H]
-  const T* pos_table;        // [max positions, H]
+  const T* pos_table;        // [max positions, H], or null: tokens alone
   int vocab, max_pos;
   const T* ya;               // SRC_ONE / SRC_PAIR: [rows, H]
   const T* yb;               // SRC_PAIR
@@ -35,44 +35,6 @@ struct SandwichParams {
   float eps;
 };
 
-__device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
-__device__ __forceinline__ float4 ld4(const __nv_bfloat16* p) {
-  const uint2 r = *reinterpret_cast<const uint2*>(p);
-  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.x));
-  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.y));
-  return make_float4(a.x, a.y, b.x, b.y);
-}
-__device__ __forceinline__ void st4(float* p, const float4& v) { *reinterpret_cast<float4*>(p) = v; }
-__device__ __forceinline__ void st4(__nv_bfloat16* p, const float4& v) {
-  __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
-  uint2 r;
-  r.x = *reinterpret_cast<uint32_t*>(&a);
-  r.y = *reinterpret_cast<uint32_t*>(&b);
-  *reinterpret_cast<uint2*>(p) = r;
-}
-__device__ __forceinline__ float sq4(const float4& v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
-
-// Two block-wide sums at once; `red` holds 64 floats.
-__device__ __forceinline__ float2 block_sum2(float a, float b, float* red) {
-  const int lane = threadIdx.x & 31, w = threadIdx.x >> 5, nw = blockDim.x >> 5;
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) {
-    a += __shfl_xor_sync(0xffffffff, a, o);
-    b += __shfl_xor_sync(0xffffffff, b, o);
-  }
-  __syncthreads();
-  if (lane == 0) { red[w] = a; red[32 + w] = b; }
-  __syncthreads();
-  a = lane < nw ? red[lane] : 0.f;
-  b = lane < nw ? red[32 + lane] : 0.f;
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) {
-    a += __shfl_xor_sync(0xffffffff, a, o);
-    b += __shfl_xor_sync(0xffffffff, b, o);
-  }
-  return make_float2(a, b);
-}
-
 // One CTA per row; thread i owns the float4 groups i, i + blockDim, ... (NV of them).
 template <typename T, int SRC, int NV>
 __global__ void __launch_bounds__(256) sandwich_norm_kernel(const SandwichParams<T> p) {
@@ -87,7 +49,7 @@ __global__ void __launch_bounds__(256) sandwich_norm_kernel(const SandwichParams
   long long xoff = off;
   if (SRC == SRC_EMBED) {
     long long tok = p.tokens[row];
-    int ps = p.pos[row];
+    int ps = p.pos_table ? p.pos[row] : 0;
     tok = tok < 0 ? 0 : (tok >= p.vocab ? p.vocab - 1 : tok);      // ids are checked on the host
     ps = ps < 0 ? 0 : (ps >= p.max_pos ? p.max_pos - 1 : ps);
 #pragma unroll
@@ -95,8 +57,11 @@ __global__ void __launch_bounds__(256) sandwich_norm_kernel(const SandwichParams
       const int i = threadIdx.x + v * blockDim.x;
       m[v] = make_float4(0.f, 0.f, 0.f, 0.f);
       if (i < nv) {
-        const float4 a = ld4(p.embed + tok * p.H + i * 4), b = ld4(p.pos_table + static_cast<long long>(ps) * p.H + i * 4);
-        m[v] = make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w);
+        m[v] = ld4(p.embed + tok * p.H + i * 4);
+        if (p.pos_table) {
+          const float4 b = ld4(p.pos_table + static_cast<long long>(ps) * p.H + i * 4);
+          m[v].x += b.x; m[v].y += b.y; m[v].z += b.z; m[v].w += b.w;
+        }
         if (p.x_first) st4(p.x_first + off + i * 4, m[v]);
       }
     }

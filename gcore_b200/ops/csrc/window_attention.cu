@@ -2,7 +2,9 @@
 // penalty, score = (q . k) * scale - slope_h * (i - j), on a paged cache that holds one row per (token, kv head).
 //   * append_keys_kernel      copies the new keys of a packed projection into their cache slots;
 //   * window_attn_kernel      any row (prompt portion or decoded token), any head size, 32-bit or bf16 storage, one warp
-//                             per (row, head): the true 32-bit path and the sizes the tensor-core kernels do not cover;
+//                             per (row, head): the true 32-bit path and the sizes the tensor-core kernels do not cover.
+//                             The value may be the first columns of the key row only, and window, penalty and an output
+//                             gate are optional, so absorbed latent attention runs on it too;
 //   * shared_kv_decode_kernel one new token per request, bf16, head sizes 64 and 128: mma.sync tiles with the query heads
 //                             of a group as rows (a group is far below the 64-row minimum of a tcgen05 instruction), KV
 //                             splits, append of the new key fused in.
@@ -37,14 +39,16 @@ __global__ void append_keys_kernel(const uint4* __restrict__ proj, long long ld_
 }
 
 constexpr int WA_WARPS = 8;
-constexpr int WA_MAX_D = 512;
+constexpr int WA_MAX_D = 1024;
 
-// One warp per (row, query head).  slots[row] < 0 marks an inactive row (zero output).
-template <typename T>
+// One warp per (row, query head).  slots[row] < 0 marks an inactive row (zero output).  D: key columns, DV <= D: value
+// columns (DV <= 32 * NR); window 0: unlimited; slopes, gate (one logit per row and head, rows gate_ld apart): or null.
+template <typename T, int NR>
 __global__ void __launch_bounds__(WA_WARPS * 32) window_attn_kernel(
     const T* __restrict__ q, long long q_ld, const T* __restrict__ cache, const int* __restrict__ tables, int max_blocks,
     int block_size, const int* __restrict__ row_seq, const int* __restrict__ pos, const int* __restrict__ slots,
-    const float* __restrict__ slopes, T* __restrict__ out, int rows, int H, int G, int D, int window, float scale) {
+    const float* __restrict__ slopes, const T* __restrict__ gate, long long gate_ld, T* __restrict__ out, int rows, int H,
+    int G, int D, int DV, int window, float scale) {
   extern __shared__ float wa_q[];
   pdl_launch_dependents();
   pdl_wait();
@@ -52,10 +56,10 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attn_kernel(
   const long long item = static_cast<long long>(blockIdx.x) * WA_WARPS + warp;
   if (item >= static_cast<long long>(rows) * H) return;
   const int row = static_cast<int>(item / H), h = static_cast<int>(item - static_cast<long long>(row) * H);
-  T* orow = out + (static_cast<long long>(row) * H + h) * D;
-  float acc[WA_MAX_D / 32];
+  T* orow = out + (static_cast<long long>(row) * H + h) * DV;
+  float acc[NR];
 #pragma unroll
-  for (int r = 0; r < WA_MAX_D / 32; ++r) acc[r] = 0.f;
+  for (int r = 0; r < NR; ++r) acc[r] = 0.f;
   float m = -FLT_MAX, l = 0.f;
   if (slots[row] >= 0) {
     float* sq = wa_q + warp * D;
@@ -64,8 +68,8 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attn_kernel(
     __syncwarp();
     const int g = h / (H / G), i = pos[row];
     const int* table = tables + static_cast<long long>(row_seq[row]) * max_blocks;
-    const float slope = slopes[h];
-    int j0 = i - window + 1;
+    const float slope = slopes ? slopes[h] : 0.f;
+    int j0 = window > 0 ? i - window + 1 : 0;
     if (j0 < 0) j0 = 0;
     for (int base = j0; base <= i; base += 32) {
       const int j = base + lane;
@@ -89,22 +93,23 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attn_kernel(
       m = mn;
       l = l * c + p;
 #pragma unroll
-      for (int r = 0; r < WA_MAX_D / 32; ++r) acc[r] *= c;
+      for (int r = 0; r < NR; ++r) acc[r] *= c;
       for (int t = 0; t < nt; ++t) {
         const float pt = __shfl_sync(0xffffffff, p, t);
         const T* kr = cache + __shfl_sync(0xffffffff, koff, t);
 #pragma unroll
-        for (int r = 0; r < WA_MAX_D / 32; ++r)
-          if (r * 32 + lane < D) acc[r] = fmaf(pt, wa_f(kr[r * 32 + lane]), acc[r]);
+        for (int r = 0; r < NR; ++r)
+          if (r * 32 + lane < DV) acc[r] = fmaf(pt, wa_f(kr[r * 32 + lane]), acc[r]);
       }
     }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffff, l, o);
   }
-  const float inv = l > 0.f ? 1.f / l : 0.f;
+  float inv = l > 0.f ? 1.f / l : 0.f;
+  if (gate) inv /= 1.f + expf(-wa_f(gate[row * gate_ld + h]));
 #pragma unroll
-  for (int r = 0; r < WA_MAX_D / 32; ++r)
-    if (r * 32 + lane < D) wa_st(orow + r * 32 + lane, acc[r] * inv);
+  for (int r = 0; r < NR; ++r)
+    if (r * 32 + lane < DV) wa_st(orow + r * 32 + lane, acc[r] * inv);
 }
 
 // ---------------------------------------------------------------------------------------------------- bf16 decode
@@ -382,15 +387,33 @@ __global__ void shared_kv_combine_kernel(const float* __restrict__ scratch, cons
   out[(static_cast<long long>(b) * H + h) * D + d] = __float2bfloat16(l > 0.f ? acc / l : 0.f);
 }
 
-template <typename T>
-int launch_window_attn(const void* q, long long q_ld, const void* cache, const int* tables, int max_blocks, int block_size,
-                       const int* row_seq, const int* pos, const int* slots, const float* slopes, void* out, int rows,
-                       int H, int G, int D, int window, float scale, cudaStream_t st) {
-  const long long items = static_cast<long long>(rows) * H;
-  launch_k(window_attn_kernel<T>, dim3(static_cast<unsigned>((items + WA_WARPS - 1) / WA_WARPS)), dim3(WA_WARPS * 32),
-           WA_WARPS * D * sizeof(float), st, static_cast<const T*>(q), q_ld, static_cast<const T*>(cache), tables,
-           max_blocks, block_size, row_seq, pos, slots, slopes, static_cast<T*>(out), rows, H, G, D, window, scale);
+struct WindowAttnArgs {
+  const void* q;
+  long long q_ld;
+  const void* cache;
+  const int *tables, *row_seq, *pos, *slots;
+  const float* slopes;
+  const void* gate;
+  long long gate_ld;
+  void* out;
+  int rows, H, G, D, DV, window, block_size, max_blocks;
+  float scale;
+};
+
+template <typename T, int NR>
+int launch_window_attn(const WindowAttnArgs& a, cudaStream_t st) {
+  const long long items = static_cast<long long>(a.rows) * a.H;
+  launch_k(window_attn_kernel<T, NR>, dim3(static_cast<unsigned>((items + WA_WARPS - 1) / WA_WARPS)), dim3(WA_WARPS * 32),
+           WA_WARPS * a.D * sizeof(float), st, static_cast<const T*>(a.q), a.q_ld, static_cast<const T*>(a.cache), a.tables,
+           a.max_blocks, a.block_size, a.row_seq, a.pos, a.slots, a.slopes, static_cast<const T*>(a.gate), a.gate_ld,
+           static_cast<T*>(a.out), a.rows, a.H, a.G, a.D, a.DV, a.window, a.scale);
   return launch_status();
+}
+
+inline int window_attn(bool f32, const WindowAttnArgs& a, cudaStream_t st) {
+  if (a.DV <= 128) return f32 ? launch_window_attn<float, 4>(a, st) : launch_window_attn<__nv_bfloat16, 4>(a, st);
+  if (a.DV <= 512) return f32 ? launch_window_attn<float, 16>(a, st) : launch_window_attn<__nv_bfloat16, 16>(a, st);
+  return f32 ? launch_window_attn<float, 32>(a, st) : launch_window_attn<__nv_bfloat16, 32>(a, st);
 }
 
 // Splits the window so that the grid about fills the GPU once, never finer than 128 tokens.
@@ -456,16 +479,21 @@ GK_EXPORT int gk_append_keys(const void* proj, long long ld_bytes, long long off
   return launch_status();
 }
 
-// dims: {rows, H, G, D, window, block_size, max_blocks}
-GK_EXPORT int gk_window_attn(int is_fp32, const void* q, long long q_ld, const void* cache, const int* tables,
-                             const int* row_seq, const int* pos, const int* slots, const float* slopes, void* out,
-                             const int* dims, float scale, void* stream) {
-  const int rows = dims[0], H = dims[1], G = dims[2], D = dims[3];
-  if (H % G || D > WA_MAX_D || D < 1 || dims[4] < 1) return -1;
-  if (rows == 0) return 0;
-  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
-  auto f = is_fp32 ? launch_window_attn<float> : launch_window_attn<__nv_bfloat16>;
-  return f(q, q_ld, cache, tables, dims[6], dims[5], row_seq, pos, slots, slopes, out, rows, H, G, D, dims[4], scale, st);
+// ptrs: {q, cache, tables, row_seq, pos, slots, slopes, gate, out}; slopes, gate: or null
+// dims: {rows, H, G, D, DV, window, block_size, max_blocks}; window 0: unlimited
+GK_EXPORT int gk_window_attn(int is_fp32, void* const* ptrs, long long q_ld, long long gate_ld, const int* dims, float scale,
+                             void* stream) {
+  WindowAttnArgs a;
+  a.q = ptrs[0]; a.q_ld = q_ld; a.cache = ptrs[1];
+  a.tables = static_cast<const int*>(ptrs[2]); a.row_seq = static_cast<const int*>(ptrs[3]);
+  a.pos = static_cast<const int*>(ptrs[4]); a.slots = static_cast<const int*>(ptrs[5]);
+  a.slopes = static_cast<const float*>(ptrs[6]);
+  a.gate = ptrs[7]; a.gate_ld = gate_ld; a.out = ptrs[8];
+  a.rows = dims[0]; a.H = dims[1]; a.G = dims[2]; a.D = dims[3]; a.DV = dims[4]; a.window = dims[5];
+  a.block_size = dims[6]; a.max_blocks = dims[7]; a.scale = scale;
+  if (a.G < 1 || a.H % a.G || a.D > WA_MAX_D || a.DV < 1 || a.DV > a.D || a.window < 0) return -1;
+  if (a.rows == 0) return 0;
+  return window_attn(is_fp32 != 0, a, reinterpret_cast<cudaStream_t>(stream));
 }
 
 GK_EXPORT void gk_shared_decode_set_target_ctas(int n) { shared_decode_target_ctas() = n > 0 ? n : 444; }

@@ -1,9 +1,10 @@
-"""Recurrent matrix memory (mLSTM) over the rows of a serving step (``csrc/matrix_memory.cu``,
-``csrc/matrix_memory_chunk.cu``).  CPU tensors run the plain PyTorch definition."""
+"""Recurrent matrix memories over the rows of a serving step (``csrc/matrix_memory.cu``, ``csrc/matrix_memory_chunk.cu``): the
+gated memory of an mLSTM, and retention, whose decay is fixed per head.  CPU tensors run the plain PyTorch definition."""
 from __future__ import annotations
 
 import ctypes
 from dataclasses import dataclass
+from typing import Optional
 
 import torch
 
@@ -33,24 +34,25 @@ def padded_value_dim(vdim: int) -> int:
 @dataclass
 class MemoryState:
     """State of one layer run for every request slot; a request's first token finds it as zeros whatever it holds."""
-    S: torch.Tensor   # [slots, heads, dim, vdim]
-    n: torch.Tensor   # [slots, heads, slices, dim]
-    m: torch.Tensor   # [slots, heads, slices]
+    S: torch.Tensor                     # [slots, heads, dim, vdim]
+    n: Optional[torch.Tensor] = None    # [slots, heads, slices, dim]   (retention has no normaliser and maximum)
+    m: Optional[torch.Tensor] = None    # [slots, heads, slices]
 
     @classmethod
-    def allocate(cls, slots, heads, dim, vdim, device):
+    def allocate(cls, slots, heads, dim, vdim, device, gated=True):
         ns = (vdim + SLICE - 1) // SLICE
         z = dict(dtype=torch.float32, device=device)
-        return cls(torch.zeros(slots, heads, dim, vdim, **z), torch.zeros(slots, heads, ns, dim, **z),
-                   torch.zeros(slots, heads, ns, **z))
+        S = torch.zeros(slots, heads, dim, vdim, **z)
+        return cls(S, torch.zeros(slots, heads, ns, dim, **z), torch.zeros(slots, heads, ns, **z)) if gated else cls(S)
 
     @staticmethod
-    def bytes_per_slot(heads, dim, vdim):
-        return 4 * heads * (dim * vdim + ((vdim + SLICE - 1) // SLICE) * (dim + 1))
+    def bytes_per_slot(heads, dim, vdim, gated=True):
+        return 4 * heads * (dim * vdim + (((vdim + SLICE - 1) // SLICE) * (dim + 1) if gated else 0))
 
     def copy_slots(self, src, dst):
         for t in (self.S, self.n, self.m):
-            t[dst] = t[src]
+            if t is not None:
+                t[dst] = t[src]
 
 
 def _ref(proj, offs, gates, gate_b, cap, q_scale, heads, dim, vdim, rows: StepRows, st: MemoryState):
@@ -80,23 +82,26 @@ def _ref(proj, offs, gates, gate_b, cap, q_scale, heads, dim, vdim, rows: StepRo
 
 
 def _scan(proj, offs, h, gate_w, gates, gate_b, cap, q_scale, heads, dim, vdim, cu, first_pos, slots, st, out=None,
-          finish=None):
+          finish=None, decay=None):
     """Token by token.  ``finish`` = (y, gain, g_off, vdim_true, eps): the normed, gated output in place of ``out``."""
     y, gain, g_off, vdim_true, eps = finish if finish is not None else (None, None, 0, vdim, 0.0)
-    ptrs = (ctypes.c_void_p * 14)(*[t.data_ptr() if t is not None else None for t in
-                                    (proj, h, gate_w, gates, gate_b, cu, first_pos, slots, st.S, st.n, st.m, out, y, gain)])
+    ptrs = (ctypes.c_void_p * 15)(*[t.data_ptr() if t is not None else None for t in
+                                    (proj, h, gate_w, gates, gate_b, cu, first_pos, slots, st.S, st.n, st.m, out, y, gain,
+                                     decay)])
     dims = (ctypes.c_int * 10)(slots.numel(), *offs, h.shape[1] if h is not None else 0, heads, dim, vdim, g_off, vdim_true)
     LAUNCHES["matrix_memory"] += 1
-    _lib.check(_lib.kernels().gk_matrix_memory_scan(int(proj.dtype == torch.float32), ptrs, proj.stride(0), dims,
-                                                    float(cap), float(q_scale), float(eps), _lib.stream_ptr()),
+    _lib.check(_lib.kernels().gk_matrix_memory_scan(int(proj.dtype == torch.float32), ptrs, proj.stride(0),
+                                                    y.stride(0) if y is not None else 0, dims, float(cap), float(q_scale), float(eps), _lib.stream_ptr()),
                "matrix_memory_scan")
 
 
-def _chunk(proj, offs, gates, gate_b, cap, q_scale, heads, dim, vdim, rows: StepRows, st, out):
+def _chunk(proj, offs, gates, gate_b, cap, q_scale, heads, dim, vdim, rows: StepRows, st, out,
+           decay=None):
     n = rows.n_portions
     states = rows.states[:n]
-    ptrs = (ctypes.c_void_p * 11)(*[t.data_ptr() for t in (proj, gates, gate_b, rows.cu, rows.first_pos, states, st.S, st.n,
-                                                           st.m, out, _lib.err_flag(proj.device))])
+    ptrs = (ctypes.c_void_p * 12)(*[t.data_ptr() if t is not None else None for t in
+                                    (proj, gates, gate_b, rows.cu, rows.first_pos, states, st.S, st.n, st.m, out,
+                                     _lib.err_flag(proj.device), decay)])
     dims = (ctypes.c_int * 8)(n, rows.portion_rows, *offs, heads, dim, vdim)
     LAUNCHES["matrix_memory"] += 1
     _lib.check(_lib.kernels().gk_matrix_memory_chunk(ptrs, proj.stride(0), dims, float(cap), float(q_scale),
@@ -106,14 +111,14 @@ def _chunk(proj, offs, gates, gate_b, cap, q_scale, heads, dim, vdim, rows: Step
 def _output(o, proj, g_off, gain, vdim_true, eps, y=None):
     T, heads, vdim = o.shape
     if not o.is_cuda:
-        n = o * torch.rsqrt(o.pow(2).sum(-1, keepdim=True) / vdim_true + eps)
-        g = torch.sigmoid(proj[:, g_off:g_off + heads * vdim].float())
-        return (n.reshape(T, -1) * gain * g).to(proj.dtype)
+        n = (o * torch.rsqrt(o.pow(2).sum(-1, keepdim=True) / vdim_true + eps)).reshape(T, -1)
+        z = proj[:, g_off:g_off + heads * vdim].float()
+        return (n * gain * torch.sigmoid(z) if gain is not None else n * torch.nn.functional.silu(z)).to(proj.dtype)
     dims = (ctypes.c_int * 5)(T, heads, vdim, vdim_true, g_off)
     LAUNCHES["matrix_memory"] += 1
     _lib.check(_lib.kernels().gk_memory_output(int(proj.dtype == torch.float32), _lib.ptr(o), _lib.ptr(proj),
-                                               proj.stride(0), _lib.ptr(gain), _lib.ptr(y), dims, float(eps),
-                                               _lib.stream_ptr()), "memory_output")
+                                               proj.stride(0), _lib.ptr(gain), _lib.ptr(y), y.stride(0), dims,
+                                               float(eps), _lib.stream_ptr()), "memory_output")
     return y
 
 
@@ -148,4 +153,53 @@ def matrix_memory(proj, q_off: int, k_off: int, v_off: int, g_off: int, h, gate_
             o = torch.empty(T - P, heads, vdim, dtype=torch.float32, device=proj.device)
             _scan(*single, o)
             _output(o, proj[P:], g_off, gain, vdim_true, eps, y[P:])
+    return y
+
+
+def _retention_ref(proj, offs, decay, q_scale, heads, dim, vdim, rows: StepRows, st: MemoryState):
+    q_off, k_off, v_off = offs
+    T = proj.shape[0]
+    out = torch.zeros(T, heads, vdim)
+    for t in range(T):
+        slot = int(rows.states[rows.row_seq[t]])
+        if slot < 0:
+            continue
+        S = torch.zeros_like(st.S[slot]) if int(rows.pos[t]) == 0 else st.S[slot]
+        q = proj[t, q_off:q_off + heads * dim].view(heads, dim).float() * q_scale
+        k = proj[t, k_off:k_off + heads * dim].view(heads, dim).float()
+        v = proj[t, v_off:v_off + heads * vdim].view(heads, vdim).float()
+        st.S[slot] = decay[:, None, None] * S + k[:, :, None] * v[:, None, :]
+        out[t] = torch.einsum("hdv,hd->hv", st.S[slot], q)
+    return out
+
+
+def retention(proj, q_off: int, k_off: int, v_off: int, g_off: int, decay, q_scale: float, heads: int, dim: int, vdim: int,
+              vdim_true: int, rows: StepRows, state: MemoryState, eps: float, y):
+    """Retention over the rows of a step: ``S <- decay_h S + k v^T``, head output ``S^T q * q_scale`` divided by its root
+    mean square (over ``vdim_true`` columns) and multiplied by ``silu(g)``, written to ``y`` [T, heads * vdim] (any row
+    stride).  ``decay``: [heads] 32-bit."""
+    T, P, n = proj.shape[0], rows.portion_rows, rows.n_portions
+    offs = (q_off, k_off, v_off)
+    if not proj.is_cuda:
+        o = _retention_ref(proj, offs, decay, q_scale, heads, dim, vdim, rows, state)
+        y.copy_(_output(o, proj, g_off, None, vdim_true, eps))
+        return y
+    common = (None, None, 0.0, q_scale, heads, dim, vdim)
+    f32 = dict(dtype=torch.float32, device=proj.device)
+    if P:
+        o = torch.empty(P, heads, vdim, **f32)
+        if proj.dtype == torch.bfloat16 and dim <= CHUNK_MAX_KEY_DIM and rows.max_portion > SCAN_MAX_TOKENS:
+            _chunk(proj, offs, *common, rows, state, o, decay)
+        else:
+            _scan(proj, offs, None, None, *common, rows.cu, rows.first_pos, rows.states[:n], state, o, decay=decay)
+        _output(o, proj, g_off, None, vdim_true, eps, y[:P])
+    if T > P:
+        single = (proj[P:], offs, None, None, *common, None, rows.first_pos[n:], rows.states[n:], state)
+        slices = (vdim + SLICE - 1) // SLICE
+        if slices <= FINISH_SLICES and slices * heads * (T - P) <= FINISH_CTAS:
+            _scan(*single, finish=(y[P:], None, g_off, vdim_true, eps), decay=decay)
+        else:
+            o = torch.empty(T - P, heads, vdim, **f32)
+            _scan(*single, o, decay=decay)
+            _output(o, proj[P:], g_off, None, vdim_true, eps, y[P:])
     return y

@@ -23,6 +23,9 @@ class StepRows:
     portion_rows: int             # rows that belong to portions; the rest are single tokens
     max_portion: int              # longest portion
     max_ctx: int                  # bound on every context length (fixes launch shapes)
+    cu_ctx: Optional[torch.Tensor] = None   # [n_portions + 1] int32 offsets of the portions' whole contexts, laid end to end
+    ctx_rows: int = 0                       # their total length
+    max_first: int = 0                      # longest context in front of a portion
 
     @property
     def n_single(self) -> int:

@@ -31,19 +31,23 @@ def _launch(src, like, x, n_rows, width, eps, vocab=0, max_pos=0, **t):
                                                _lib.stream_ptr()), "sandwich_norm")
 
 
-def embed_rows(tokens, pos, embed, pos_table, gain_pre, width, eps, step=None, keep_first=False):
+def embed_rows(tokens, pos, embed, pos_table, gain_pre, width, eps, step=None, keep_first=False, x=None):
     """``x = embed[token] + pos_table[pos]`` (kept as ``first`` when asked), ``+ step``; returns ``(x, first, h)`` with
-    ``h`` the normed input of the first sublayer.  ``tokens`` int64, ``pos`` int32."""
+    ``h`` the normed input of the first sublayer.  ``tokens`` int64, ``pos`` int32; ``pos_table`` None: tokens alone; ``x``: where the
+    stream goes."""
     T, H = tokens.numel(), embed.shape[1]
     if not embed.is_cuda:
-        first = embed[tokens].float() + pos_table[pos.long()].float()
-        x = first + step if step is not None else first.clone()
+        first = embed[tokens].float()
+        if pos_table is not None:
+            first = first + pos_table[pos.long()].float()
+        first_x = first + step if step is not None else first.clone()
+        x = first_x if x is None else x.copy_(first_x)
         return x, (first if keep_first else None), (_rms(x, width, eps) * gain_pre).to(embed.dtype)
-    x = torch.empty(T, H, dtype=torch.float32, device=embed.device)
+    x = torch.empty(T, H, dtype=torch.float32, device=embed.device) if x is None else x
     first = torch.empty_like(x) if keep_first else None
     h = torch.empty(T, H, dtype=embed.dtype, device=embed.device)
-    _launch(_EMBED, embed.dtype, x, T, width, eps, embed.shape[0], pos_table.shape[0], tokens=tokens, pos=pos,
-            embed=embed, pos_table=pos_table, x_first=first, step=step, gain_pre=gain_pre, h=h)
+    _launch(_EMBED, embed.dtype, x, T, width, eps, embed.shape[0], 0 if pos_table is None else pos_table.shape[0],
+            tokens=tokens, pos=pos, embed=embed, pos_table=pos_table, x_first=first, step=step, gain_pre=gain_pre, h=h)
     return x, first, h
 
 

@@ -59,13 +59,17 @@ def append_keys(proj, k_off, n, slots, cache):
                                              _lib.ptr(cache), slots.numel(), _lib.stream_ptr()), "append_keys")
 
 
-def _general(q, q_ld, cache, rows: StepRows, lo, hi, slopes, out, H, G, D, window, scale):
-    dims = (ctypes.c_int * 7)(hi - lo, H, G, D, window, cache.shape[1], rows.tables.shape[1])
+def general_attention(q, q_ld, cache, rows: StepRows, lo, hi, out, H, G, D, scale, dv=None, window=0, slopes=None, gate=None,
+                      gate_ld=0):
+    """Rows ``lo .. hi`` of a step against the paged cache: keys of ``D`` columns whose first ``dv`` are the value, an
+    optional window (0: none), distance penalty and output gate.  Any size, 32-bit or bf16."""
+    dims = (ctypes.c_int * 8)(hi - lo, H, G, D, dv or D, window, cache.shape[1], rows.tables.shape[1])
+    ptrs = (ctypes.c_void_p * 9)(*[t.data_ptr() if t is not None else None for t in
+                                   (q, cache, rows.tables, rows.row_seq[lo:hi], rows.pos[lo:hi], rows.slots[lo:hi], slopes,
+                                    gate, out)])
     LAUNCHES["window_attention"] += 1
-    _lib.check(_lib.kernels().gk_window_attn(
-        int(q.dtype == torch.float32), _lib.ptr(q), q_ld, _lib.ptr(cache), _lib.ptr(rows.tables),
-        _lib.ptr(rows.row_seq[lo:hi]), _lib.ptr(rows.pos[lo:hi]), _lib.ptr(rows.slots[lo:hi]), _lib.ptr(slopes),
-        _lib.ptr(out), dims, float(scale), _lib.stream_ptr()), "window_attn")
+    _lib.check(_lib.kernels().gk_window_attn(int(q.dtype == torch.float32), ptrs, q_ld, gate_ld, dims, float(scale),
+                                             _lib.stream_ptr()), "window_attn")
 
 
 def window_attention(proj, q_off: int, k_off: int, heads: int, kv_heads: int, dim: int, rows: StepRows, cache, slopes,
@@ -81,7 +85,7 @@ def window_attention(proj, q_off: int, k_off: int, heads: int, kv_heads: int, di
     tiled = bf16 and D in (64, 128)
     if not tiled:
         append_keys(proj, k_off, G * D, rows.slots, cache)
-        _general(proj[:, q_off:], proj.stride(0), cache, rows, 0, T, slopes, out, H, G, D, window, scale)
+        general_attention(proj[:, q_off:], proj.stride(0), cache, rows, 0, T, out, H, G, D, scale, None, window, slopes)
         return out
     if P:
         append_keys(proj[:P], k_off, G * D, rows.slots[:P], cache)
@@ -94,7 +98,7 @@ def window_attention(proj, q_off: int, k_off: int, heads: int, kv_heads: int, di
                                              _lib.ptr(out), dims, float(scale), _lib.ptr(_lib.err_flag(proj.device)),
                                              _lib.stream_ptr()), "window_prefill")
         else:
-            _general(proj[:, q_off:], proj.stride(0), cache, rows, 0, P, slopes, out, H, G, D, window, scale)
+            general_attention(proj[:, q_off:], proj.stride(0), cache, rows, 0, P, out, H, G, D, scale, None, window, slopes)
     if T > P:
         B = T - P
         ptab = rows.tables[rows.n_portions:]

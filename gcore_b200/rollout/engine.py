@@ -170,9 +170,10 @@ class _Sched:
 
 
 def _count_launches() -> int:
-    from ..ops import attention, gemm, matrix_memory, optim, rl, sandwich, vocab, window_attention
-    return sum(sum(m.LAUNCHES.values()) for m in (attention, fused, gemm, matrix_memory, optim, rl, sandwich, vocab,
-                                                  window_attention))
+    from ..ops import (attention, depth, gemm, latent_attention, matrix_memory, moe, optim, rl, sandwich, vocab,
+                       window_attention)
+    return sum(sum(m.LAUNCHES.values()) for m in (attention, depth, fused, gemm, latent_attention, matrix_memory, moe, optim,
+                                                  rl, sandwich, vocab, window_attention))
 
 
 class LayerWeights:
@@ -215,7 +216,7 @@ class RolloutWeights:
         model = getattr(model, "language_model", model)  # vision-language wrapper: the decoder is what serves
         if isinstance(model, PlanDecoder):
             w.plan = cls._serving_module(model, clone)
-            w.embed, w.final_ln, w.head = w.plan.embed.detach(), w.plan.final_gain.detach(), w.plan.head.detach()
+            w.embed, w.final_ln, w.head = (t.detach() for t in (w.plan.embed, w.plan.final_gain, w.plan.output_weight))
             return w
         w.embed = f(model.embedding.word_embeddings.weight)
         w.final_ln = f(model.decoder.final_layernorm.weight)
@@ -349,8 +350,7 @@ class InferEngine:
     # ------------------------------------------------------------------ memory
     def _kv_bytes_per_block(self):
         if self.plan is not None:
-            es = self.w.embed.element_size()
-            return sum(math.prod(self.plan.layers[r.layer].cache_shape()) for r in self.cfg.layer_plan.runs) * self.bs * es
+            return self.plan.cache_bytes_per_token() * self.bs
         if self.mla_dim:
             return len(self.w.layers) * self.bs * self.mla_dim * 2
         return 2 * len(self.w.layers) * self.bs * self.hk * self.D * 2
@@ -364,20 +364,19 @@ class InferEngine:
                 if self.device.type == "cuda":
                     free, total = torch.cuda.mem_get_info(self.device)
                     if self.plan is not None:
-                        free -= self.max_running * sum(self.plan.layers[r.layer].state_bytes()
-                                                       for r in self.cfg.layer_plan.runs)
+                        free -= self.max_running * self.plan.state_bytes_per_slot()
                     budget = int(free * self.gpu_memory_utilization)
-                    n = max(min(need, budget // self._kv_bytes_per_block()), self.max_blocks + 1)
+                    # a purely recurrent plan caches nothing: its blocks cost no memory
+                    n = max(min(need, budget // max(1, self._kv_bytes_per_block())), self.max_blocks + 1)
                 else:
                     n = need
             self.num_blocks = n
             dt = self.w.embed.dtype
             if self.plan is not None:
-                # per layer run: one cached row serves as key and value, and one recurrent state per request slot
-                per_run = [self.plan.layers[r.layer] for r in self.cfg.layer_plan.runs]
-                self.k_cache = [torch.zeros(n, self.bs, *ly.cache_shape(), dtype=dt, device=self.device) for ly in per_run]
+                # per layer run: a paged cache whose rows are key and value, a recurrent state per request slot, or both
+                self.k_cache = self.plan.new_caches(n, self.bs, self.device)
                 self.v_cache = []
-                self.memory = [ly.new_state(self.max_running, self.device) for ly in per_run]
+                self.memory = self.plan.new_states(self.max_running, self.device)
             elif self.mla_dim:
                 # latent cache: one row of (kv_lora + rope) values per token, shared by all heads; block ``n`` is a
                 # sink for the rows of inactive batch slots
@@ -885,18 +884,21 @@ class InferEngine:
         pos = torch.arange(T, dtype=torch.int32) - (cu[:-1] - first_t)[row_seq.long()]
         slots = bt[row_seq.long(), (pos // self.bs).long()] * self.bs + pos % self.bs
         ctx = (first_t + 1)[n_port:]
+        cu_ctx = torch.zeros(n_port + 1, dtype=torch.int32)
+        cu_ctx[1:] = (first_t + lens_t)[:n_port].cumsum(0)
         parts = [torch.tensor([t for e in order for t in entries[e][2]], dtype=torch.int32), pos, slots.to(torch.int32),
-                 torch.tensor(self.sched.states(rids), dtype=torch.int32), first_t, cu[:n_port + 1], ctx, row_seq,
-                 bt.reshape(-1)]
+                 torch.tensor(self.sched.states(rids), dtype=torch.int32), first_t, cu[:n_port + 1], cu_ctx, ctx,
+                 row_seq, bt.reshape(-1)]
         packed = torch.cat(parts)
         if self.device.type == "cuda":
             packed = packed.pin_memory()
         io_counters.add_h2d(io_counters.tensor_bytes(packed))
-        tok, pos, slots, states, first_d, cu_d, ctx, row_seq, tables = packed.to(self.device, non_blocking=True).split(
+        tok, pos, slots, states, first_d, cu_d, ctx_d, ctx, row_seq, tables = packed.to(self.device, non_blocking=True).split(
             [p.numel() for p in parts])
         rows = StepRows(tokens=tok.long(), pos=pos, slots=slots, tables=tables.view(n, self.max_blocks), states=states,
                         first_pos=first_d, cu=cu_d, ctx=ctx, row_seq=row_seq, n_portions=n_port, portion_rows=port_rows,
-                        max_portion=max(lens[:n_port], default=0), max_ctx=max((f + 1 for f in first[n_port:]), default=1))
+                        max_portion=max(lens[:n_port], default=0), max_ctx=max((f + 1 for f in first[n_port:]), default=1), cu_ctx=ctx_d, ctx_rows=int(cu_ctx[-1]),
+                        max_first=max(first[:n_port], default=0))
         base = [0] * n
         for k, e in enumerate(order):
             base[e] = int(cu[k])
@@ -1159,12 +1161,14 @@ class InferEngine:
                     src = torch.tensor([a for a, _ in copies], device=dev)
                     dst = torch.tensor([b for _, b in copies], device=dev)
                     for c in self.k_cache + self.v_cache:
-                        c[dst] = c[src]
+                        if c is not None:
+                            c[dst] = c[src]
                 if self.plan is not None and len(owners) > len(pre):
                     pairs = [(r.rid, c.rid) for r in pre for c in children.get(r.rid, [])]
                     s_src, s_dst = (torch.tensor(self.sched.states([p[k] for p in pairs]), device=dev) for k in (0, 1))
                     for state in self.memory:
-                        state.copy_slots(s_src, s_dst)
+                        if state is not None:
+                            state.copy_slots(s_src, s_dst)
                 for c in owners:
                     place(c, *first[c.rid])
             if self.ep_group is not None:

@@ -14,7 +14,7 @@ import torch
 
 from ..models.config import ModelConfig, from_hf_config
 from ..models.gpt import GPTModel
-from ..models.plan_decoder import PlanDecoder
+from ..models.plan_decoder import build_decoder
 from ..ops import _lib, attention, fused, sandwich
 from ..ops import matrix_memory as mm
 from ..ops import window_attention as wa
@@ -52,7 +52,7 @@ def build(kind, s, positions, requests, block=64):
     dev = torch.device("cuda")
     if kind == "nafitar":
         cfg = from_hf_config(nafitar_conf(s, positions))
-        model = PlanDecoder(cfg, dev).randomize()
+        model = build_decoder(cfg, dev).randomize()
     else:
         cfg = ModelConfig(arch="llama", num_layers=s["layers"], hidden_size=s["width"], num_attention_heads=s["heads"],
                           num_kv_heads=s["kv"], head_dim=s["dim"], ffn_hidden_size=s["ff"], vocab_size=VOCAB,

@@ -5,7 +5,7 @@ from dataclasses import replace
 import torch
 
 from gcore_b200.models.config import from_hf_config
-from gcore_b200.models.plan_decoder import PlanDecoder
+from gcore_b200.models.plan_decoder import build_decoder
 from gcore_b200.rollout.engine import InferEngine, RolloutWeights
 
 
@@ -36,7 +36,7 @@ def round_conf(window=70, loop=(0, 1, 2), positions=1024):
 
 def make_engine(c, W, dtype="float32", device="cpu", **kw):
     cfg = replace(from_hf_config(c), dtype=dtype)
-    model = PlanDecoder(cfg, device).load_tensors(W)
+    model = build_decoder(cfg, device).load_tensors(W)
     kw = {**dict(max_running_requests=4, max_model_len=min(c["max_positions"], 512), kv_block_size=16,
                  use_cuda_graph=device != "cpu"), **kw}
     return InferEngine(cfg, RolloutWeights.from_model(model), device=torch.device(device), **kw)

@@ -7,7 +7,7 @@ import pytest
 import torch
 
 from gcore_b200.models.config import MODEL_ARCH, from_hf_config
-from gcore_b200.models.plan_decoder import PlanDecoder
+from gcore_b200.models.plan_decoder import build_decoder
 from gcore_b200.rollout.engine import RolloutWeights, SamplingParams
 from tests import nafitar_util as nu
 from tests.oracle import nafitar as oracle
@@ -48,8 +48,8 @@ def test_checkpoint_tensors_must_fit_exactly():
     for bad in ({k: v for k, v in W.items() if k != "l1.mix.right.i.b"}, {**W, "l1.norm2": W["l0.norm2"]},
                 {**W, "l0.mix.left.o": W["l0.mix.left.o"][:, :-1]}):
         with pytest.raises((KeyError, ValueError)):
-            PlanDecoder(cfg).load_tensors(bad)
-    m = PlanDecoder(cfg).load_tensors(W)
+            build_decoder(cfg).load_tensors(bad)
+    m = build_decoder(cfg).load_tensors(W)
     ly = m.layers[0]   # padded heads: real rows in place, zero rows between them
     q = ly.in_proj[ly.off["q"]:ly.off["k"]].view(6, ly.att_dim, -1)
     assert torch.equal(q[:, :20, :44].reshape(120, 44), W["l0.mix.left.q"]) and not q[:, 20:].any() and not q[..., 44:].any()
@@ -57,7 +57,7 @@ def test_checkpoint_tensors_must_fit_exactly():
 
 def test_serving_copy_owns_its_weights():
     c = nu.uneven_conf(positions=32)
-    m = PlanDecoder(from_hf_config(c)).load_tensors(oracle.random_weights(c))
+    m = build_decoder(from_hf_config(c)).load_tensors(oracle.random_weights(c))
     shared, own = RolloutWeights.from_model(m), RolloutWeights.from_model(m, clone=True)
     assert shared.plan is m and own.plan is not m
     assert all(a.data_ptr() != b.data_ptr() and torch.equal(a, b) for a, b in zip(shared.tensors(), own.tensors()))
@@ -85,11 +85,11 @@ def test_new_weights_replace_the_old_ones():
     c = nu.uneven_conf(positions=64)
     Wa, Wb = oracle.random_weights(c, seed=1), oracle.random_weights(c, seed=2)
     eng = nu.make_engine(c, Wa, max_model_len=64)
-    other = PlanDecoder(eng.cfg).load_tensors(Wb)
+    other = build_decoder(eng.cfg).load_tensors(Wb)
     seq = nu.tokens(20, 75, 1)
     eng.update_weights(RolloutWeights.from_model(other))
     nu.assert_close(nu.run_alone(eng, seq, [20]), oracle.forward(Wb, c, seq))
-    eng.load_weights_from(PlanDecoder(eng.cfg).load_tensors(Wa))
+    eng.load_weights_from(build_decoder(eng.cfg).load_tensors(Wa))
     nu.assert_close(nu.run_alone(eng, seq, [20]), oracle.forward(Wa, c, seq))
 
 
