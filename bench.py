@@ -272,7 +272,8 @@ def main():
                     "model's optimizer state shares the GPU with the activations")
     ap.add_argument("--serve", nargs="*", default=None, metavar="SIZE",
                     help="instead of the recipe: prefill and decode throughput of layer-plan decoders beside the closest "
-                    "dense model, kernel by kernel (sizes: see gcore_b200/tools/serve_bench.py; default all); one JSON line")
+                    "uniform model, kernel by kernel (sizes: see gcore_b200/tools/serve_bench.py; default all); one JSON line")
+    ap.add_argument("--serve-design", default="nafitar", choices=("nafitar", "kedesun"), help="design that --serve measures")
     args = ap.parse_args()
     if args.serve is not None:
         return serve_bench(args)
@@ -455,7 +456,7 @@ def serve_bench(args):
     clocks = ClockSampler(0, period_s=0.2)
     clocks.start()
     clocks.mark()
-    out = sb.run(args.serve or None)
+    out = sb.run(args.serve or None, design=args.serve_design)
     out["clocks"] = clocks.stop()
     print(json.dumps({"metric": "serve_prefill_decode_tokens_per_s", **out}))
     return 0

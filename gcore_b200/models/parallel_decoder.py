@@ -42,7 +42,7 @@ class LatentAttentionMixer(nn.Module):
                                       magnitude=spec.rot.magnitude(), eps=eps)
         self.out_columns = spec.heads * vdim
         self.gain = _buf(torch.zeros(spec.kv_rank, dtype=torch.float32, device=device))
-        self.freq = _buf(torch.tensor(spec.rot.frequencies(), dtype=torch.float32, device=device))
+        self.turns = _buf(la.rotation_turns(spec.rot.frequencies()).to(device))
         self.up_kv = _buf(torch.zeros(spec.heads * (dim + vdim), rank, dtype=dtype, device=device))
 
     def cache_shape(self):
@@ -71,7 +71,7 @@ class LatentAttentionMixer(nn.Module):
         put(out.view(out.shape[0], H, ly.vdim), take(p + "o", W, H * s.vdim).view(W, H, s.vdim))
 
     def forward(self, proj, rows, cache, state, out):
-        la.latent_attention(proj, self.layout, self.gain, self.freq, self.up_kv, rows, cache, out)
+        la.latent_attention(proj, self.layout, self.gain, self.turns, self.up_kv, rows, cache, out)
 
 
 class RetentionMixer(nn.Module):
@@ -240,7 +240,7 @@ class ParallelDecoder(PlanDecoder):
         g = torch.Generator(device=self.embed.device).manual_seed(seed)
         for name, p in self.named_parameters():
             leaf = name.rsplit(".", 1)[-1]
-            if leaf in ("freq", "decay"):
+            if leaf in ("turns", "decay"):
                 continue
             if leaf == "avg":
                 p.fill_(0.3 / p.numel())

@@ -4,7 +4,8 @@
 //   * latent_prep_kernel    a packed projection row -> its cache row (norm of the latent in 32-bit, rotation), the queries'
 //                           rotated parts in place, and a copy of the cache row in the portion's contiguous context;
 //   * latent_gather_kernel  cache rows of the tokens in front of a portion -> the portion's contiguous context.
-// The rotation pairs dimension 2i with 2i + 1; angle and rotation are 32-bit.
+// The rotation pairs dimension 2i with 2i + 1, all in 32-bit.  A pair's speed is given in turns per position as two floats
+// (value and remainder), so the fraction of a turn is as exact at position 10^6 as at position 1.
 #include "host_utils.h"
 #include "row_ops.cuh"
 #include <type_traits>
@@ -27,7 +28,7 @@ struct LatentPrepParams {
   int q_rot;
   int d_off;               // latent columns, then the shared key part at d_off + CV
   const float* gain;       // [C]
-  const float* freq;       // [rot / 2]
+  const float2* turns;     // [rot / 2] turns per position: value, remainder
   const int* pos;
   const int* slots;        // cache slot of every row; negative: not stored
   T* cache;                // rows of CV + DR
@@ -50,8 +51,11 @@ __global__ void __launch_bounds__(LP_THREADS) latent_prep_kernel(const LatentPre
   T* pr = p.proj + row * p.ld;
   const int pos = p.pos[row], slot = p.slots[row];
   for (int i = tid; i < half; i += LP_THREADS) {
+    const float2 f = p.turns[i];
+    const float x = static_cast<float>(pos), t = x * f.x;
+    const float frac = (t - rintf(t)) + fmaf(x, f.y, fmaf(x, f.x, -t));
     float s, c;
-    sincosf(static_cast<float>(pos) * p.freq[i], &s, &c);
+    sincospif(2.f * frac, &s, &c);
     s_cos[i] = c * p.magnitude;
     s_sin[i] = s * p.magnitude;
   }
@@ -108,7 +112,7 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const uint4* __restr
 
 using namespace gk;
 
-// ptrs: {proj, gain, freq, pos, slots, cache, context, row_seq, cu_ctx}; context null: single tokens only
+// ptrs: {proj, gain, turns, pos, slots, cache, context, row_seq, cu_ctx}; context null: single tokens only
 // dims: {rows, context_rows, q_off, q_hs, q_rot, d_off, H, C, CV, rot, DR}
 GK_EXPORT int gk_latent_prep(int is_fp32, void* const* ptrs, long long ld, const int* dims, float eps, float magnitude,
                              void* stream) {
@@ -121,7 +125,7 @@ GK_EXPORT int gk_latent_prep(int is_fp32, void* const* ptrs, long long ld, const
     p.proj = static_cast<T*>(ptrs[0]);
     p.ld = ld;
     p.gain = static_cast<const float*>(ptrs[1]);
-    p.freq = static_cast<const float*>(ptrs[2]);
+    p.turns = static_cast<const float2*>(ptrs[2]);
     p.pos = static_cast<const int*>(ptrs[3]);
     p.slots = static_cast<const int*>(ptrs[4]);
     p.cache = static_cast<T*>(ptrs[5]);

@@ -5,6 +5,7 @@ folded into query and output.  CPU tensors run the plain PyTorch definition."""
 from __future__ import annotations
 
 import ctypes
+import math
 from dataclasses import dataclass
 from typing import Dict
 
@@ -58,16 +59,22 @@ class LatentLayout:
         return self.row_rank + self.row_rot
 
 
+def rotation_turns(frequencies) -> torch.Tensor:
+    """[pairs, 2] 32-bit: turns per position of every rotated pair as value and remainder."""
+    t = torch.tensor(frequencies, dtype=torch.float64) / (2 * math.pi)
+    return torch.stack([t.float(), (t - t.float().double()).float()], -1)
+
+
 def _rotate(x, cos, sin):
     u, v = x[..., 0::2], x[..., 1::2]
     return torch.stack([u * cos - v * sin, v * cos + u * sin], -1).flatten(-2)
 
 
-def _ref(proj, ly: LatentLayout, gain, freq, up_kv, rows: StepRows, cache, out):
+def _ref(proj, ly: LatentLayout, gain, turns, up_kv, rows: StepRows, cache, out):
     T, H, bs = proj.shape[0], ly.heads, cache.shape[1]
     p = proj.float()
-    a = rows.pos.float()[:, None] * freq
-    cos, sin = torch.cos(a) * ly.magnitude, torch.sin(a) * ly.magnitude
+    a = 2 * math.pi * rows.pos.double()[:, None] * turns.double().sum(-1)
+    cos, sin = (torch.cos(a) * ly.magnitude).float(), (torch.sin(a) * ly.magnitude).float()
     c = p[:, ly.down:ly.down + ly.rank]
     row = torch.zeros(T, ly.row)
     row[:, :ly.rank] = c * torch.rsqrt(c.pow(2).mean(-1, keepdim=True) + ly.eps) * gain
@@ -92,9 +99,9 @@ def _ref(proj, ly: LatentLayout, gain, freq, up_kv, rows: StepRows, cache, out):
     return out
 
 
-def _prep(proj, ly: LatentLayout, gain, freq, rows: StepRows, cache, context):
+def _prep(proj, ly: LatentLayout, gain, turns, rows: StepRows, cache, context):
     ptrs = (ctypes.c_void_p * 9)(*[t.data_ptr() if t is not None else None for t in
-                                   (proj, gain, freq, rows.pos, rows.slots, cache, context, rows.row_seq, rows.cu_ctx)])
+                                   (proj, gain, turns, rows.pos, rows.slots, cache, context, rows.row_seq, rows.cu_ctx)])
     dims = (ctypes.c_int * 11)(proj.shape[0], rows.portion_rows if context is not None else 0, ly.q, ly.dim + ly.row_rot,
                                ly.dim, ly.down, ly.heads, ly.rank, ly.row_rank, ly.rot, ly.row_rot)
     LAUNCHES["latent_attention"] += 1
@@ -173,19 +180,19 @@ def _absorbed(proj, ly: LatentLayout, up_kv, rows: StepRows, lo: int, hi: int, c
     _bmm(o_lat, uv.transpose(1, 2), out[lo:hi].view(T, H, ly.vdim).transpose(0, 1))
 
 
-def latent_attention(proj, ly: LatentLayout, gain, freq, up_kv, rows: StepRows, cache, out):
+def latent_attention(proj, ly: LatentLayout, gain, turns, up_kv, rows: StepRows, cache, out):
     """Appends every row's ``[latent | rotated key part]`` to ``cache`` [blocks, block_size, 1, row] and writes the gated
     attention output [T, heads * vdim] to ``out`` (any row stride).  The queries' rotated parts in ``proj`` are rotated in
-    place.  ``up_kv`` [heads * (dim + vdim), row_rank]: key rows of all heads, then value rows; ``gain`` [rank] and ``freq``
-    [rot / 2] are 32-bit."""
+    place.  ``up_kv`` [heads * (dim + vdim), row_rank]: key rows of all heads, then value rows; ``gain`` [rank] is
+    32-bit, ``turns`` comes from ``rotation_turns``."""
     cache = cache.view(cache.shape[0], cache.shape[1], ly.row)
     if not proj.is_cuda:
-        return _ref(proj, ly, gain, freq, up_kv, rows, cache, out)
+        return _ref(proj, ly, gain, turns, up_kv, rows, cache, out)
     T, P = proj.shape[0], rows.portion_rows
     tiled = P > 0 and proj.dtype == torch.bfloat16 and bool(
         _lib.kernels().gk_latent_prefill_supported(ly.dim, up8(ly.rot), ly.vdim))
     context = torch.empty(rows.ctx_rows, ly.row, dtype=proj.dtype, device=proj.device) if tiled else None
-    _prep(proj, ly, gain, freq, rows, cache, context)
+    _prep(proj, ly, gain, turns, rows, cache, context)
     if tiled:
         _portions(proj, ly, up_kv, rows, cache, context, out)
     elif P:

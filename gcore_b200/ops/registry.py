@@ -44,7 +44,8 @@ def resolve(name: str, impl: Optional[str] = None) -> Callable:
 
 
 def _populate():
-    from . import attention, fused, gemm, matrix_memory, optim, quant, rl, sandwich, vocab, window_attention
+    from . import (attention, depth, fused, gemm, latent_attention, matrix_memory, moe, optim, quant, rl, sandwich, vocab,
+                   window_attention)
     for mod, names in ((gemm, ("gemm", "grouped_gemm", "grouped_wgrad", "linear")),
                        (fused, ("rmsnorm", "rope", "swiglu")),
                        (attention, ("flash_attn_varlen", "flash_attn_qkvpacked", "paged_decode", "kv_append_rope")),
@@ -52,7 +53,9 @@ def _populate():
                        (optim, ("adam_step", "sumsq", "axpy_cast")),
                        (quant, ("quant_act_1x128", "quant_weight_128x128", "quant_fp4_1x32", "gemm_fp8_blockscaled")),
                        (sandwich, ("embed_rows", "add_sublayer", "norm_rows")),
-                       (window_attention, ("window_attention",)), (matrix_memory, ("matrix_memory",)),
+                       (window_attention, ("window_attention",)), (matrix_memory, ("matrix_memory", "retention")),
+                       (latent_attention, ("latent_attention",)), (depth, ("add_layer",)),
+                       (moe, ("activate", "choose", "expert_rows", "routed_experts")),
                        (rl, ("fused_grpo_loss", "gae"))):
         for n in names:
             fn = getattr(mod, n, None)

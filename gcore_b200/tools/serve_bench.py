@@ -1,9 +1,10 @@
 """Serving throughput of layer-plan decoders beside the closest uniform model at equal size (``bench.py --serve``).
 
-For a few real-model layer sizes (random weights) it times, on the device, a prefill step and a captured decode step of a
-Nafitar engine and of a dense grouped-query decoder with the same width, heads, window, feed-forward and layer count, and
-then every kernel the design added beside the like kernel of that model: time, the time its bytes or FLOPs would take at
-the measured peaks, and the ratio of the two.  Inputs of every timed launch rotate over buffers larger than L2."""
+For a few real-model layer sizes (random weights) it times, on the device, a prefill step and a captured decode step of an
+engine of the design and of the closest uniform model - for Nafitar a dense grouped-query decoder with the same width,
+heads, window, feed-forward and layer count, for Kedesun a latent-attention decoder with experts (``serve_bench_kedesun.py``)
+- and then every kernel the design added beside the like kernel of that model: time, the time its bytes or FLOPs would take
+at the measured peaks, and the ratio of the two.  Inputs of every timed launch rotate over buffers larger than L2."""
 from __future__ import annotations
 
 import json
@@ -48,15 +49,22 @@ def nafitar_conf(s, positions):
                 vocab=VOCAB, width=s["width"])
 
 
+def dense_config(s):
+    return ModelConfig(arch="llama", num_layers=s["layers"], hidden_size=s["width"], num_attention_heads=s["heads"],
+                       num_kv_heads=s["kv"], head_dim=s["dim"], ffn_hidden_size=s["ff"], vocab_size=VOCAB, qkv_bias=True,
+                       sliding_window=s["window"])
+
+
 def build(kind, s, positions, requests, block=64):
+    """Engine of a layer-plan design (``nafitar``, ``kedesun``) or of the uniform model it is compared with (``dense``,
+    ``latent``)."""
+    from . import serve_bench_kedesun as sk
     dev = torch.device("cuda")
-    if kind == "nafitar":
-        cfg = from_hf_config(nafitar_conf(s, positions))
+    if kind in ("nafitar", "kedesun"):
+        cfg = from_hf_config(nafitar_conf(s, positions) if kind == "nafitar" else sk.conf(s))
         model = build_decoder(cfg, dev).randomize()
     else:
-        cfg = ModelConfig(arch="llama", num_layers=s["layers"], hidden_size=s["width"], num_attention_heads=s["heads"],
-                          num_kv_heads=s["kv"], head_dim=s["dim"], ffn_hidden_size=s["ff"], vocab_size=VOCAB,
-                          qkv_bias=True, sliding_window=s["window"])
+        cfg = dense_config(s) if kind == "dense" else sk.latent_config(s)
         model = GPTModel(cfg, recompute="none", device=dev)
     eng = InferEngine(cfg, RolloutWeights.from_model(model), max_running_requests=requests, max_model_len=positions,
                       kv_block_size=block, max_prefill_tokens=1 << 20, device=dev)
@@ -171,7 +179,7 @@ def _rows(prompts, length, ctx, B, bs, dev):
     return StepRows(tokens=torch.zeros(T, dtype=torch.int64, device=dev), pos=pos, slots=slots, tables=tab,
                     states=torch.arange(n, dtype=torch.int32, device=dev), first_pos=first, cu=cu, ctx=ctxs, row_seq=seq,
                     n_portions=prompts, portion_rows=prompts * length, max_portion=length if prompts else 0,
-                    max_ctx=ctx + 1), n * nb
+                    max_ctx=ctx + 1, cu_ctx=cu, ctx_rows=prompts * length), n * nb
 
 
 def kernel_table(s, prompts, length, B, ctx, bs=64):
@@ -255,31 +263,42 @@ def kernel_table(s, prompts, length, B, ctx, bs=64):
     return table
 
 
-def run(sizes=None, iters=10):
+def _families():
+    from . import serve_bench_kedesun as sk
+    active = lambda eng, s, n: n - 2 * VOCAB * s["width"]
+    return {"nafitar": dict(like="dense", sizes=SIZES, active=active, table=kernel_table,
+                            decode_bytes=lambda kind, s, eng, B, ctx: decode_bytes(kind, s, eng, B, ctx)),
+            "kedesun": dict(like="latent", sizes=sk.SIZES, active=sk.active_weights, table=sk.kernel_table,
+                            decode_bytes=sk.decode_bytes)}
+
+
+def run(sizes=None, iters=10, design="nafitar"):
     hbm, flops, which = peaks()
-    out = {"peaks": which, "gpu": torch.cuda.get_device_name(0), "dtype": "bf16", "data": "synthetic", "sizes": {}}
+    fam = _families()[design]
+    out = {"design": design, "peaks": which, "gpu": torch.cuda.get_device_name(0), "dtype": "bf16", "data": "synthetic",
+           "sizes": {}}
     prompts, length, ctx = 4, 4096, 4096
-    for name in sizes or SIZES:
-        s = SIZES[name]
+    for name in sizes or fam["sizes"]:
+        s = fam["sizes"][name]
         rec = {"layer": s, "prefill": {}, "decode": {}}
-        for kind in ("nafitar", "dense"):
+        for kind in (design, fam["like"]):
             eng = build(kind, s, ctx + 256, 64)
             n_params = sum(t.numel() for t in eng.w.tensors())
             ms = prefill_step(eng, prompts, length, max(3, iters // 2))
             T = prompts * length
             rec["prefill"][kind] = {"ms": round(ms, 3), "tokens_per_s": round(T / ms * 1e3),
-                                    "gemm_roofline_fraction": round(2.0 * T * (n_params - 2 * VOCAB * s["width"]) / flops
+                                    "gemm_roofline_fraction": round(2.0 * T * fam["active"](eng, s, n_params) / flops
                                                                     / (ms * 1e-3), 3)}
             for B in (8, 64):
                 ms = decode_step(eng, B, ctx, iters * 3)
                 rec["decode"][f"{kind}_b{B}"] = {"ms": round(ms, 4), "tokens_per_s": round(B / ms * 1e3),
-                                                 "hbm_roofline_fraction": round(decode_bytes(kind, s, eng, B, ctx) / hbm
-                                                                                / (ms * 1e-3), 3)}
+                                                 "hbm_roofline_fraction": round(fam["decode_bytes"](kind, s, eng, B, ctx)
+                                                                                / hbm / (ms * 1e-3), 3)}
             del eng
             torch.cuda.empty_cache()
         rec["kernels"] = []
         for B in (8, 64):
-            for phase, k, t, i, lk, lt, li in kernel_table(s, prompts, length, B, ctx):
+            for phase, k, t, i, lk, lt, li in fam["table"](s, prompts, length, B, ctx):
                 if phase == "prefill" and B != 8:
                     continue
                 r = {"phase": phase if phase == "prefill" else f"{phase} b{B}", "kernel": k, "us": round(t, 2),

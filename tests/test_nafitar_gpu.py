@@ -8,39 +8,12 @@ import torch
 from gcore_b200.ops import matrix_memory as mm
 from gcore_b200.ops import sandwich
 from gcore_b200.ops import window_attention as wa
-from gcore_b200.ops.rows import StepRows
 from gcore_b200.rollout.engine import SamplingParams
 from tests import nafitar_util as nu
 from tests.oracle import nafitar as oracle
 
 pytestmark = pytest.mark.gpu
 DT = {"float32": torch.float32, "bfloat16": torch.bfloat16}
-
-
-def make_rows(segments, block_size, n_blocks, n_slots, seed=0, device="cuda"):
-    """StepRows of ``segments`` = [(first position, length)] on shuffled cache blocks and state slots; portions (length
-    > 1) must come first."""
-    g = torch.Generator().manual_seed(seed)
-    perm = torch.randperm(n_blocks, generator=g).tolist()
-    mb = max((f + l + block_size - 1) // block_size for f, l in segments)
-    tab = torch.zeros(len(segments), mb, dtype=torch.int32)
-    for i, (f, l) in enumerate(segments):
-        for b in range((f + l + block_size - 1) // block_size):
-            tab[i, b] = perm.pop()
-    lens = [l for _, l in segments]
-    n_port = sum(l > 1 for l in lens)
-    assert all(l > 1 for l in lens[:n_port])
-    seq = torch.repeat_interleave(torch.arange(len(segments), dtype=torch.int32), torch.tensor(lens))
-    pos = torch.cat([torch.arange(f, f + l, dtype=torch.int32) for f, l in segments])
-    slots = tab[seq.long(), (pos // block_size).long()] * block_size + pos % block_size
-    cu = torch.tensor([sum(lens[:i]) for i in range(n_port + 1)], dtype=torch.int32)
-    states = torch.randperm(n_slots, generator=g)[:len(segments)].to(torch.int32)
-    first = torch.tensor([f for f, _ in segments], dtype=torch.int32)
-    d = lambda t: t.to(device)
-    return StepRows(tokens=torch.zeros(pos.numel(), dtype=torch.int64, device=device), pos=d(pos), slots=d(slots.int()),
-                    tables=d(tab), states=d(states), first_pos=d(first), cu=d(cu), ctx=d((first + 1)[n_port:].contiguous()),
-                    row_seq=d(seq), n_portions=n_port, portion_rows=int(cu[-1]), max_portion=max(lens[:n_port], default=0),
-                    max_ctx=max((f + 1 for f, l in segments if l == 1), default=1))
 
 
 # ---------------------------------------------------------------------------------------------------- attention alone
@@ -52,7 +25,7 @@ def test_window_attention_alone(H, G, D, window, bs, dtype):
     torch.manual_seed(1)
     segs = [(0, 150), (333, 70), (63, 2), (127, 65), (5, 2), (500, 1), (0, 1), (64, 1), (window + 3, 1), (255, 1)]
     total = [f + l for f, l in segs]
-    rows = make_rows(segs, bs, sum((t + bs - 1) // bs for t in total) + 5, 16)
+    rows = nu.make_rows(segs, bs, sum((t + bs - 1) // bs for t in total) + 5, 16)
     dt = DT[dtype]
     ld, q_off, k_off = H * D + G * D + 24, 8, 8 + H * D
     keys = [torch.randn(t, G, D).to(dt).double() for t in total]
@@ -98,7 +71,7 @@ def test_decode_splits_of_a_long_window_agree():
     """One request whose window is cut into many splits = the same with one split."""
     torch.manual_seed(2)
     H, G, D, window, bs = 8, 1, 128, 4000, 64
-    rows = make_rows([(5000, 1)], bs, 90, 2)
+    rows = nu.make_rows([(5000, 1)], bs, 90, 2)
     cache = torch.randn(91, bs, G, D, device="cuda").bfloat16()
     proj = torch.randn(1, (H + G) * D, device="cuda").bfloat16()
     sl = torch.tensor(oracle.slopes(H), device="cuda")
@@ -120,7 +93,7 @@ def test_matrix_memory_alone(heads, dim, vdim, width, dtype, finish, monkeypatch
     torch.manual_seed(3)
     dt = DT[dtype]
     segs = [(0, 300), (70, 130), (0, 2), (40, 7), (128, 128), (0, 1), (9, 1), (200, 1)]
-    rows = make_rows(segs, 16, 200, 12)
+    rows = nu.make_rows(segs, 16, 200, 12)
     ofs = [0, heads * dim, 2 * heads * dim, 2 * heads * dim + heads * vdim]
     ld = ofs[3] + heads * vdim
     m = dict(heads=heads, dim=dim, vdim=vdim, gate_cap=7.0)
