@@ -132,8 +132,8 @@ class RetentionSpec:
     def __post_init__(self):
         if min(self.heads, self.dim, self.vdim) < 1 or len(self.decay) != self.heads:
             raise ValueError("retention needs positive sizes and one decay per head")
-        if not all(0 < d <= 1 for d in self.decay):
-            raise ValueError("retention decays must lie in (0, 1]")
+        if not all(0 <= d <= 1 for d in self.decay):
+            raise ValueError("retention decays must lie in [0, 1]")
 
 
 @dataclass(frozen=True)

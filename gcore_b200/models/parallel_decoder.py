@@ -152,10 +152,10 @@ class ExpertFeedForward(nn.Module):
 
     def forward(self, h, proj, out, counts):
         s = self.spec
-        logits = linear_forward(h, self.router, out_dtype=torch.float32)
+        logits, choice = moe.route_tokens(h, self.router, s.experts, s.top, self.correction, counts)
         if self.shared:
             moe.activate(moe.RELU2, proj, self.shared, 0, out, row_logit=logits[:, s.experts])
-        return moe.routed_experts(h, logits, s.top, self.correction, self.up, self.down, counts)
+        return moe.routed_experts(h, choice, self.up, self.down, counts)
 
 
 class ParallelLayer(nn.Module):

@@ -230,6 +230,7 @@ def _declare_kernels(lib: ctypes.CDLL):
     d("gk_expert_rows", [P, P, P, P, P, P, P, I, I, I, I, P])
     d("gk_grouped_gemm_f32", [P, P, P, P, I, I, I, I, P])
     d("gk_router_dispatch", [P, L, P, P, P, P, P, L, I, I, I, I, F, P])
+    d("gk_router_fused", [I, P, P, P, I, I, P, P, P, P, P, L, I, I, I, I, F, P])
     d("gk_latent_prep", [I, P, L, P, F, F, P])
     d("gk_latent_gather", [P, P, P, P, P, I, I, I, I, I, P])
     d("gk_latent_prefill", [P, P, P, F, P])

@@ -317,33 +317,52 @@ __global__ void __launch_bounds__(THREADS, 2) mla_paged_decode_kernel(
   }
 }
 
-// Merges the live KV splits of one (request, head): scratch rows are [CV values | running max | running sum].
-__global__ void mla_decode_combine_kernel(const float* __restrict__ scratch, const int* __restrict__ ctx_len,
-                                          __nv_bfloat16* __restrict__ out, long long os_b, long long os_h, int H,
-                                          int CV, int nsplit_total, int split_tokens,
-                                          const __nv_bfloat16* __restrict__ gate, long long gate_ld) {
+// Merges the live KV splits of one (request, head): scratch rows are [CV values | running max | running sum].  One column
+// pair per thread; the splits' weights are computed once per CTA.
+constexpr int COMBINE_THREADS = 256;
+__global__ void __launch_bounds__(COMBINE_THREADS) mla_decode_combine_kernel(
+    const float* __restrict__ scratch, const int* __restrict__ ctx_len, __nv_bfloat16* __restrict__ out, long long os_b,
+    long long os_h, int H, int CV, int nsplit_total, int split_tokens, const __nv_bfloat16* __restrict__ gate,
+    long long gate_ld) {
+  __shared__ float s_w[COMBINE_THREADS];
+  __shared__ float s_red[COMBINE_THREADS / 32];
   pdl_launch_dependents();
   pdl_wait();
-  const int b = blockIdx.x, h = blockIdx.y;
+  const int b = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
   const float* base = scratch + (static_cast<long long>(b) * H + h) * nsplit_total * (CV + 2);
   int nsplit = (ctx_len[b] + split_tokens - 1) / split_tokens;
   if (nsplit < 1) nsplit = 1;
-  if (nsplit > nsplit_total) nsplit = nsplit_total;
-  float m = -FLT_MAX;
-  for (int s = 0; s < nsplit; ++s) m = fmaxf(m, base[s * (CV + 2) + CV]);
-  float l = 0.f;
-  for (int s = 0; s < nsplit; ++s) {
-    const float ms = base[s * (CV + 2) + CV];
-    l += base[s * (CV + 2) + CV + 1] * (ms == -FLT_MAX ? 0.f : __expf(ms - m));
-  }
+  if (nsplit > nsplit_total) nsplit = nsplit_total;       // at most COMBINE_THREADS (plan)
+  const float ms = tid < nsplit ? base[static_cast<long long>(tid) * (CV + 2) + CV] : -FLT_MAX;
+  const float ls = tid < nsplit ? base[static_cast<long long>(tid) * (CV + 2) + CV + 1] : 0.f;
+  float m = ms;
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffff, m, o));
+  if ((tid & 31) == 0) s_red[tid >> 5] = m;
+  __syncthreads();
+#pragma unroll
+  for (int w = 0; w < COMBINE_THREADS / 32; ++w) m = fmaxf(m, s_red[w]);
+  const float wt = ms == -FLT_MAX ? 0.f : __expf(ms - m);
+  s_w[tid] = wt;
+  float l = ls * wt;
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffff, l, o);
+  __syncthreads();
+  if ((tid & 31) == 0) s_red[tid >> 5] = l;
+  __syncthreads();
+  l = 0.f;
+#pragma unroll
+  for (int w = 0; w < COMBINE_THREADS / 32; ++w) l += s_red[w];
   const float inv = l > 0.f ? gate_of(gate, gate_ld, b, h) / l : 0.f;
-  for (int d = threadIdx.x; d < CV; d += blockDim.x) {
-    float acc = 0.f;
+  for (int d = tid * 2; d < CV; d += COMBINE_THREADS * 2) {
+    float2 acc = make_float2(0.f, 0.f);
+#pragma unroll 8
     for (int s = 0; s < nsplit; ++s) {
-      const float ms = base[s * (CV + 2) + CV];
-      acc += base[s * (CV + 2) + d] * (ms == -FLT_MAX ? 0.f : __expf(ms - m));
+      const float2 v = *reinterpret_cast<const float2*>(base + static_cast<long long>(s) * (CV + 2) + d);
+      acc.x = fmaf(v.x, s_w[s], acc.x);
+      acc.y = fmaf(v.y, s_w[s], acc.y);
     }
-    out[b * os_b + h * os_h + d] = __float2bfloat16(acc * inv);
+    *reinterpret_cast<__nv_bfloat162*>(out + b * os_b + h * os_h + d) = __floats2bfloat162_rn(acc.x * inv, acc.y * inv);
   }
 }
 
@@ -355,6 +374,7 @@ static void plan(int B, int H, int max_ctx, int* nsplit, int* split_tokens) {
   if (ns < 1) ns = 1;
   int want = target_ctas() / (groups > 0 ? groups : 1);
   if (want < 1) want = 1;
+  if (want > COMBINE_THREADS) want = COMBINE_THREADS;
   if (want < ns) ns = want;
   int st = ((max_ctx + ns - 1) / ns + TILE - 1) / TILE * TILE;
   if (st < MIN_SPLIT) st = MIN_SPLIT;
@@ -419,7 +439,7 @@ static int decode(const void* q_lat, long long qs_b, long long qs_h, const void*
 #undef GK_MLA_LAUNCH
 #undef GK_MLA_ARGS
   if (nsplit > 1) {
-    launch_k(mla_decode_combine_kernel, dim3(B, H), dim3(128), 0, st, static_cast<const float*>(scratch), ctx_len,
+    launch_k(mla_decode_combine_kernel, dim3(B, H), dim3(COMBINE_THREADS), 0, st, static_cast<const float*>(scratch), ctx_len,
              reinterpret_cast<__nv_bfloat16*>(out), os_b, os_h, H, CV, nsplit, split_tokens, gate, gate_ld);
   }
   return launch_status();

@@ -27,33 +27,47 @@ struct ActParams {
   int F;                    // columns, a multiple of 4
 };
 
+// 32-bit rows take the exact exponential and quotient, bf16 rows the fast ones (their error is far below the rounding).
+__device__ __forceinline__ float act_sigmoid(float z, float) { return 1.f / (1.f + expf(-z)); }
+__device__ __forceinline__ float act_sigmoid(float z, __nv_bfloat16) { return __fdividef(1.f, 1.f + __expf(-z)); }
+
+template <typename T, int ACT>
+__device__ __forceinline__ float4 act4(const T* gate, const T* up, float w) {
+  float4 u = ld4(up);
+  if (ACT == ACT_SILU_GATE) {
+    const float4 g = ld4(gate);
+    u.x *= g.x * act_sigmoid(g.x, T()); u.y *= g.y * act_sigmoid(g.y, T());
+    u.z *= g.z * act_sigmoid(g.z, T()); u.w *= g.w * act_sigmoid(g.w, T());
+  } else {
+    u.x = fmaxf(u.x, 0.f); u.y = fmaxf(u.y, 0.f); u.z = fmaxf(u.z, 0.f); u.w = fmaxf(u.w, 0.f);
+    u.x *= u.x; u.y *= u.y; u.z *= u.z; u.w *= u.w;
+  }
+  u.x *= w; u.y *= w; u.z *= w; u.w *= w;
+  return u;
+}
+
+// grid (column groups of 4 * blockDim.x, row groups): a thread keeps its columns and walks rows, four at a time so that
+// their loads overlap.
 template <typename T, int ACT>
 __global__ void __launch_bounds__(256) ffn_act_kernel(const ActParams<T> p) {
   pdl_launch_dependents();
   pdl_wait();
-  const int fv = p.F >> 2;
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
+  if (c >= p.F) return;
   long long rows = p.rows;
   if (p.n_rows_dev && *p.n_rows_dev < rows) rows = *p.n_rows_dev;
-  const long long n = rows * fv;
-  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < n;
-       i += static_cast<long long>(gridDim.x) * blockDim.x) {
-    const long long row = i / fv;
-    const int c = static_cast<int>(i - row * fv) * 4;
-    const T* s = p.src + row * p.src_ld + c;
-    float4 u = ld4(s + p.up_off);
-    if (ACT == ACT_SILU_GATE) {
-      const float4 g = ld4(s);
-      u.x *= g.x / (1.f + expf(-g.x)); u.y *= g.y / (1.f + expf(-g.y));
-      u.z *= g.z / (1.f + expf(-g.z)); u.w *= g.w / (1.f + expf(-g.w));
-    } else {
-      u.x = fmaxf(u.x, 0.f); u.y = fmaxf(u.y, 0.f); u.z = fmaxf(u.z, 0.f); u.w = fmaxf(u.w, 0.f);
-      u.x *= u.x; u.y *= u.y; u.z *= u.z; u.w *= u.w;
+  for (long long r0 = static_cast<long long>(blockIdx.y) * 4; r0 < rows; r0 += static_cast<long long>(gridDim.y) * 4) {
+    float4 u[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const long long row = r0 + i < rows ? r0 + i : rows - 1;
+      const float w = p.row_logit ? 1.f / (1.f + expf(-p.row_logit[row * p.logit_ld])) : 1.f;
+      const T* s = p.src + row * p.src_ld + c;
+      u[i] = act4<T, ACT>(s, s + p.up_off, w);
     }
-    if (p.row_logit) {
-      const float w = 1.f / (1.f + expf(-p.row_logit[row * p.logit_ld]));
-      u.x *= w; u.y *= w; u.z *= w; u.w *= w;
-    }
-    st4(p.dst + row * p.dst_ld + c, u);
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+      if (r0 + i < rows) st4(p.dst + (r0 + i) * p.dst_ld + c, u[i]);
   }
 }
 
@@ -139,12 +153,15 @@ __global__ void __launch_bounds__(256) grouped_f32_kernel(const float* __restric
 
 template <typename T>
 int launch_act(int act, const ActParams<T>& p, cudaStream_t st) {
-  const long long n = p.rows * (p.F >> 2);
-  long long blocks = (n + 255) / 256;
-  if (blocks > sm_count() * 16) blocks = sm_count() * 16;
-  const dim3 grid(static_cast<unsigned>(blocks));
-  if (act == ACT_SILU_GATE) launch_k(ffn_act_kernel<T, ACT_SILU_GATE>, grid, dim3(256), 0, st, p);
-  else if (act == ACT_RELU2) launch_k(ffn_act_kernel<T, ACT_RELU2>, grid, dim3(256), 0, st, p);
+  const int cols = p.F >> 2;
+  const int threads = cols >= 256 ? 256 : (cols + 31) / 32 * 32;
+  const unsigned gx = static_cast<unsigned>((cols + threads - 1) / threads);
+  long long gy = (p.rows + 3) / 4;
+  const long long most = (sm_count() * 16 + gx - 1) / gx;
+  if (gy > most) gy = most;
+  const dim3 grid(gx, static_cast<unsigned>(gy)), block(threads);
+  if (act == ACT_SILU_GATE) launch_k(ffn_act_kernel<T, ACT_SILU_GATE>, grid, block, 0, st, p);
+  else if (act == ACT_RELU2) launch_k(ffn_act_kernel<T, ACT_RELU2>, grid, block, 0, st, p);
   else return -3;
   return launch_status();
 }

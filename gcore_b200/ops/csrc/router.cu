@@ -6,8 +6,10 @@
 // chain topk / scatter / masked_fill / topk / gather / sum / div of the PyTorch formulation (the semantics of the
 // reference's routers: softmax top-k with renormalisation for the Qwen MoE families, sigmoid + bias + node-limited
 // groups for the DeepSeek families, gpatch_v4/models/deepseek_v4/modeling_deepseek_v4.py:1120-1219).
-// Ties go to the lower expert index.
+// Ties go to the lower expert index.  For few tokens (decode steps) router_fused_kernel computes the logits in the same
+// launch, one CTA per token.
 #include "host_utils.h"
+#include "row_ops.cuh"
 #include <cfloat>
 #include <stdint.h>
 
@@ -40,14 +42,9 @@ __device__ __forceinline__ void warp_argmax(float& v, int& i) {
   }
 }
 
+// One warp routes token t from its logits in `row`.
 template <int VPT>
-__global__ void __launch_bounds__(256) router_fwd_kernel(RouterParams p) {
-  const long long t = (blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x) >> 5;
-  const int lane = threadIdx.x & 31;
-  gk::pdl_launch_dependents();
-  gk::pdl_wait();
-  if (t >= p.T) return;
-  const float* row = p.logits + t * p.ld;
+__device__ __forceinline__ void route_token(const RouterParams& p, long long t, int lane, const float* row) {
   float sc[VPT], sel[VPT];
   // ---- scores (lanes past the last expert hold none)
   if (p.sigmoid) {
@@ -173,6 +170,60 @@ __global__ void __launch_bounds__(256) router_fwd_kernel(RouterParams p) {
     out_w[lane] = wv / denom * p.scale;
     if (p.counts) p.place[t * p.K + lane] = atomicAdd(p.counts + iv, 1);
   }
+}
+
+template <int VPT>
+__global__ void __launch_bounds__(256) router_fwd_kernel(RouterParams p) {
+  const long long t = (blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x) >> 5;
+  gk::pdl_launch_dependents();
+  gk::pdl_wait();
+  if (t >= p.T) return;
+  route_token<VPT>(p, t, threadIdx.x & 31, p.logits + t * p.ld);
+}
+
+constexpr int RF_WARPS = 16;
+constexpr int RF_MAX_ROWS = 516;
+
+// logits[t, r] = h[t] . w[r] for the `n_rows` rows of w (the experts, then rows the router only projects), then the
+// choice among the first E.  H is a multiple of 8.
+template <typename T, int VPT>
+__global__ void __launch_bounds__(RF_WARPS * 32) router_fused_kernel(RouterParams p, const T* __restrict__ h,
+                                                                     const T* __restrict__ w, float* __restrict__ logits,
+                                                                     int H, int n_rows) {
+  extern __shared__ float rf_h[];
+  __shared__ float s_logit[RF_MAX_ROWS];
+  gk::pdl_launch_dependents();
+  gk::pdl_wait();
+  const long long t = blockIdx.x;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  for (int d = tid * 4; d < H; d += RF_WARPS * 128) gk::st4(rf_h + d, gk::ld4(h + t * H + d));
+  __syncthreads();
+  for (int r0 = warp * 4; r0 < n_rows; r0 += RF_WARPS * 4) {      // four rows at a time: their loads overlap
+    float a[4] = {0.f, 0.f, 0.f, 0.f};
+    const T* wr[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) wr[i] = w + static_cast<long long>(r0 + i < n_rows ? r0 + i : n_rows - 1) * H;
+#pragma unroll 2
+    for (int d = lane * 4; d < H; d += 128) {
+      const float4 x = gk::ld4(rf_h + d);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float4 y = gk::ld4(wr[i] + d);
+        a[i] = fmaf(x.x, y.x, fmaf(x.y, y.y, fmaf(x.z, y.z, fmaf(x.w, y.w, a[i]))));
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) a[i] += __shfl_xor_sync(0xffffffffu, a[i], o);
+      if (lane == 0 && r0 + i < n_rows) {
+        s_logit[r0 + i] = a[i];
+        logits[t * n_rows + r0 + i] = a[i];
+      }
+    }
+  }
+  __syncthreads();
+  if (warp == 0) route_token<VPT>(p, t, lane, s_logit);
 }
 
 struct RouterBwdParams {
@@ -304,6 +355,32 @@ GK_EXPORT int gk_router_dispatch(const float* logits, long long ld, const float*
   p.topk_group = 1; p.sigmoid = sigmoid; p.norm = norm; p.scale = scale;
   p.ld = ld; p.counts = counts; p.place = place;
   return router_launch(p, reinterpret_cast<cudaStream_t>(stream));
+}
+
+// The same from the tokens themselves, h [T, H] and w [n_rows, H] (n_rows >= E; H % 8 == 0, at most 11264): also writes the
+// logits [T, n_rows].
+GK_EXPORT int gk_router_fused(int is_fp32, const void* h, const void* w, float* logits, int H, int n_rows, const float* bias,
+                              long long* idx, float* weight, int* counts, int* place, long long T, int E, int K, int sigmoid,
+                              int norm, float scale, void* stream) {
+  if (T <= 0) return 0;
+  if (n_rows < E || n_rows > RF_MAX_ROWS || H % 8 || H > 11264 || !counts || !place || E < 1 || K < 1 || K > MAX_K || K > E)
+    return -1;
+  RouterParams p;
+  p.logits = logits; p.bias = bias; p.replay = nullptr; p.idx = idx; p.w = weight; p.T = T; p.E = E; p.K = K; p.G = 1;
+  p.topk_group = 1; p.sigmoid = sigmoid; p.norm = norm; p.scale = scale;
+  p.ld = n_rows; p.counts = counts; p.place = place;
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  return dispatch_vpt(E, p, [&](auto v) {
+    constexpr int VPT = decltype(v)::value;
+    const dim3 grid(static_cast<unsigned>(T)), block(RF_WARPS * 32);
+    if (is_fp32)
+      gk::launch_k(router_fused_kernel<float, VPT>, grid, block, H * sizeof(float), st, p, static_cast<const float*>(h),
+                   static_cast<const float*>(w), logits, H, n_rows);
+    else
+      gk::launch_k(router_fused_kernel<__nv_bfloat16, VPT>, grid, block, H * sizeof(float), st, p,
+                   static_cast<const __nv_bfloat16*>(h), static_cast<const __nv_bfloat16*>(w), logits, H, n_rows);
+    return gk::launch_status();
+  });
 }
 
 GK_EXPORT int gk_router_bwd(const float* logits, const long long* idx, const float* dw, float* dlogits, long long T,

@@ -8,7 +8,7 @@ import ctypes
 import torch
 
 from . import _lib
-from .gemm import grouped_gemm
+from .gemm import grouped_gemm, linear_forward
 from .router import route_ref
 
 LAUNCHES = {"moe": 0}
@@ -35,7 +35,7 @@ def activate(kind: int, src, cols: int, up_off: int, dst, row_logit=None, n_rows
     return dst
 
 
-def choose(logits, experts: int, top: int, correction, counts, place=None):
+def choose(logits, experts: int, top: int, correction, counts):
     """Softmax scores of ``logits[:, :experts]`` (32-bit), the ``top`` experts by score + ``correction``, their scores
     normalised.  Returns ``(expert [T, top] int64, weight [T, top], place [T, top] int32)`` and adds to ``counts`` [experts]
     int32 how many tokens chose each; ``place`` numbers the tokens of one expert."""
@@ -47,15 +47,37 @@ def choose(logits, experts: int, top: int, correction, counts, place=None):
             place[i] = counts[e]
             counts[e] += 1
         return idx, w, place.view(T, top)
-    dev = logits.device
-    idx = torch.empty(T, top, dtype=torch.int64, device=dev)
-    w = torch.empty(T, top, dtype=torch.float32, device=dev)
-    place = torch.empty(T, top, dtype=torch.int32, device=dev)
+    idx, w, place = _choice_buffers(T, top, logits.device)
     LAUNCHES["moe"] += 1
     _lib.check(_lib.kernels().gk_router_dispatch(
         _lib.ptr(logits), logits.stride(0), _lib.ptr(correction), _lib.ptr(idx), _lib.ptr(w), _lib.ptr(counts),
         _lib.ptr(place), T, experts, top, 0, 1, 1.0, _lib.stream_ptr()), "router_dispatch")
     return idx, w, place
+
+
+def _choice_buffers(T, top, device):
+    return (torch.empty(T, top, dtype=torch.int64, device=device), torch.empty(T, top, dtype=torch.float32, device=device),
+            torch.empty(T, top, dtype=torch.int32, device=device))
+
+
+FUSED_TOKENS, FUSED_WIDTH = 128, 11264      # up to here a CTA per token computes the logits itself
+
+
+def route_tokens(h, router, experts: int, top: int, correction, counts):
+    """``choose`` on the logits ``h @ router^T``; ``router`` [experts + extra, H] may hold rows that are only projected.
+    Returns ``(logits [T, rows], choice)``."""
+    T, n = h.shape[0], router.shape[0]
+    if not h.is_cuda or T > FUSED_TOKENS or h.shape[1] > FUSED_WIDTH:
+        logits = linear_forward(h, router, out_dtype=torch.float32)
+        return logits, choose(logits, experts, top, correction, counts)
+    logits = torch.empty(T, n, dtype=torch.float32, device=h.device)
+    idx, w, place = _choice_buffers(T, top, h.device)
+    LAUNCHES["moe"] += 1
+    _lib.check(_lib.kernels().gk_router_fused(
+        int(h.dtype == torch.float32), _lib.ptr(h), _lib.ptr(router), _lib.ptr(logits), h.shape[1], n, _lib.ptr(correction),
+        _lib.ptr(idx), _lib.ptr(w), _lib.ptr(counts), _lib.ptr(place), T, experts, top, 0, 1, 1.0, _lib.stream_ptr()),
+        "router_fused")
+    return logits, (idx, w, place)
 
 
 def expert_rows_bound(tokens: int, top: int, experts: int) -> int:
@@ -98,10 +120,10 @@ def grouped(x, w, offsets):
     return grouped_gemm(x, w, offsets, out_dtype=x.dtype)
 
 
-def routed_experts(h, logits, top: int, correction, up, down, counts):
-    """Every token through its ``top`` experts ``down(relu(up h)^2)``: returns ``(rows, dest, weight)``, the experts' outputs
-    in expert order and where a token finds its own.  ``counts``: [experts] int32, zero."""
-    idx, w, place = choose(logits, up.shape[0], top, correction, counts)
+def routed_experts(h, choice, up, down, counts):
+    """Every token through its chosen experts ``down(relu(up h)^2)``: returns ``(rows, dest, weight)``, the experts' outputs
+    in expert order and where a token finds its own."""
+    idx, w, place = choice
     x, dest, offsets = expert_rows(h, counts, idx, place)
     a = grouped(x, up, offsets)
     activate(RELU2, a, a.shape[1], 0, a, n_rows=offsets[-1:])

@@ -7,10 +7,12 @@ import math
 import torch
 
 from ..models.config import ModelConfig
+from ..models.moe import build_dispatch_plan, padded_rows_bound
 from ..ops import attention, depth, fused, moe
 from ..ops import latent_attention as la
 from ..ops import matrix_memory as mm
-from ..ops.gemm import grouped_gemm, linear_forward
+from ..ops.gemm import grouped_gemm
+from ..ops.router import route
 
 # width, attention heads and head sizes (unrotated, rotated, value), latent size, retention heads and sizes, dense and
 # expert feed-forwards, layers (every fourth layer is latent attention; feed-forwards alternate between dense and experts)
@@ -54,33 +56,29 @@ def latent_config(s):
                        moe_ffn_hidden_size=ff, moe_shared_expert_ffn=ff, first_k_dense=0, moe_layer_freq=2)
 
 
-def _expert_weights(s):
-    """(all routed experts, one of them) of the design's expert layers; the compared model's hold about the same."""
-    one = 2 * s["eff"] * s["width"]
-    return s["experts"] * one, one
-
-
 def active_weights(eng, s, n):
-    from .serve_bench import VOCAB
-    every, one = _expert_weights(s)
-    emb = VOCAB * s["width"] * (1 if eng.plan is not None else 2)
-    return n - emb - (s["layers"] // 2) * (every - s["top"] * one)
+    """Weights a token is multiplied with, without the vocabulary matrices."""
+    cfg = eng.cfg
+    if eng.plan is None:
+        return cfg.active_parameters() - 2 * cfg.vocab_size * cfg.hidden_size
+    return cfg.num_parameters(include_embedding=False) - _idle_experts(s, s["top"])
+
+
+def _idle_experts(s, used):
+    """Weights of the routed experts beyond ``used`` per expert layer (about the same in the compared model)."""
+    return (s["layers"] // 2) * (s["experts"] - used) * 2 * s["eff"] * s["width"]
 
 
 def decode_bytes(kind, s, eng, B, ctx):
     """HBM bytes one decode step has to move: weights once (of the experts, those that B tokens choose at random), cached
     latents, recurrent state in and out."""
-    from .serve_bench import VOCAB
-    w = sum(t.numel() * t.element_size() for t in eng.w.tensors())
-    if eng.plan is None:
-        w -= VOCAB * s["width"] * 2               # of the two vocabulary matrices one is read
-    every, one = _expert_weights(s)
+    cfg = eng.cfg
     hit = s["experts"] * (1 - (1 - s["top"] / s["experts"]) ** B)
-    w -= (s["layers"] // 2) * 2 * (every - hit * one)
+    w = cfg.num_parameters(include_embedding=False) + cfg.vocab_size * cfg.hidden_size - _idle_experts(s, hit)
     n_lat = s["layers"] // 4 if kind == "kedesun" else s["layers"]
     cache = n_lat * B * (ctx + 1) * (s["rank"] + s["rot"]) * 2
     state = (s["layers"] - n_lat) * 2 * 4 * B * s["rh"] * s["rk"] * s["rv"]
-    return w + cache + state
+    return 2 * w + cache + state
 
 
 def kernel_table(s, prompts, length, B, ctx, bs=64):
@@ -173,32 +171,23 @@ def kernel_table(s, prompts, length, B, ctx, bs=64):
         like = graph_us([lambda a=a: fused.swiglu(a) for a in srcs])
         table.append((phase, "ffn_act (silu gate)", t, ideal(n * ff * 6), "swiglu", like, ideal(n * ff * 6)))
         del srcs, dst
-        logits, corr = torch.randn(n, E + 1, **f32), torch.zeros(E, **f32)
-        counts = torch.zeros(E, dtype=torch.int32, device=dev)
+        corr, counts = torch.zeros(E, **f32), torch.zeros(E, dtype=torch.int32, device=dev)
         router = torch.randn(E + 1, width, **bf)
-        t = graph_us([lambda y=y: linear_forward(y, router, out_dtype=torch.float32) for y in ys])
         rw = router.float()[:E].contiguous()
-        like = graph_us([lambda y=y: torch.nn.functional.linear(y.float(), rw) for y in ys])
-        table.append((phase, "router logits", t, ideal(n * width * 2 + E * width * 2), "router logits (fp32 copy)", like,
-                      ideal(n * width * 2 + E * width * 4)))
 
         def pick(y):
             counts.zero_()
-            idx, _, place = moe.choose(logits, E, K, corr, counts)
+            _, (idx, _, place) = moe.route_tokens(y, router, E, K, corr, counts)
             return moe.expert_rows(y, counts, idx, place)
 
-        from ..models.moe import build_dispatch_plan, padded_rows_bound
-        from ..ops.router import route
-        lg = logits[:, :E].contiguous()
-
         def like_pick(y):
-            idx, _ = route(lg, None, None, K)
+            idx, _ = route(torch.nn.functional.linear(y.float(), rw), None, None, K)
             dst_, _ = build_dispatch_plan(idx.reshape(-1), E)
             xp = torch.zeros(padded_rows_bound(n * K, E), width, **bf)
             return xp.index_copy(0, dst_, y[torch.arange(n, device=dev).repeat_interleave(K)])
         t, like = graph_us([lambda y=y: pick(y) for y in ys]), graph_us([lambda y=y: like_pick(y) for y in ys])
-        table.append((phase, "choice + expert rows", t, ideal(n * width * 2 * (1 + K)), "route + dispatch", like,
-                      ideal(n * width * 2 * (1 + K))))
+        i = ideal(n * width * 2 * (2 + K) + E * width * 2)
+        table.append((phase, "logits + choice + expert rows", t, i, "logits + route + dispatch", like, i))
         xs, _, offs = pick(ys[0])
         n_w = max(2, math.ceil(3e8 / (E * eff * width * 2)))
         ups = [torch.randn(E, eff, width, **bf) for _ in range(n_w)]

@@ -157,7 +157,7 @@ def test_retention_alone(heads, dim, vdim, true, dtype, finish, monkeypatch):
     segs = [(0, 300), (70, 130), (0, 2), (40, 7), (128, 128), (3, 129), (0, 1), (9, 1), (200, 1)]
     rows = ku.make_rows(segs, 16, 240, 12)
     ofs = [0, heads * dim, 2 * heads * dim, 2 * heads * dim + heads * vdim]
-    decay = [[0.97], [0.6, 1.0], [0.004, 0.9, 0.9995], [1e-30, 0.5, 0.999, 1.0]][heads - 1]
+    decay = [[0.97], [0.6, 1.0], [0.004, 0.9, 0.9995], [0.0, 0.5, 0.999, 1.0]][heads - 1]
     state = mm.MemoryState.allocate(12, heads, dim, vdim, "cuda", gated=False)
     state.S.fill_(99.0)                                  # what earlier requests left
     proj, wants, states = [], [], []
@@ -241,6 +241,26 @@ def test_choice_of_experts_alone(E, K):
 
 
 @DTYPES
+@pytest.mark.parametrize("T,E,K,width", [(1, 1, 1, 8), (8, 12, 2, 200), (128, 33, 5, 1000), (3, 512, 8, 4096), (40, 64, 4, 11264),
+                                         (129, 9, 2, 64)])
+def test_routing_from_the_tokens(T, E, K, width, dtype):
+    """One launch for few tokens, product and choice for many: the same logits and choice."""
+    torch.manual_seed(8)
+    h, router = torch.randn(T, width).to(DT[dtype]), (torch.randn(E + 1, width) * width ** -0.5 * 2).to(DT[dtype])
+    corr, counts = torch.randn(E) * 0.01, torch.zeros(E, dtype=torch.int32, device="cuda")
+    logits, (idx, w, place) = moe.route_tokens(h.cuda(), router.cuda(), E, K, corr.cuda(), counts)
+    want = h.double() @ router.double().T
+    assert (logits.double().cpu() - want).abs().max() < 2e-5 and int(counts.sum()) == T * K
+    got = logits.double().cpu()
+    for t in range(T):
+        ref = dict(oracle.choose_experts(got[t, :E], corr.double(), K))
+        assert set(idx[t].tolist()) == set(ref)
+        assert all(abs(x - ref[e]) < 1e-5 for e, x in zip(idx[t].tolist(), w[t].tolist()))
+    flat = idx * 1000 + place
+    assert flat.unique().numel() == T * K and (place < counts[idx]).all()
+
+
+@DTYPES
 @pytest.mark.parametrize("T,E,K,F,width", [(1, 5, 2, 24, 48), (8, 64, 4, 128, 256), (300, 12, 3, 72, 200), (130, 7, 1, 136, 64),
                                            (40, 200, 6, 16, 32)])
 def test_routed_experts_alone(T, E, K, F, width, dtype):
@@ -252,7 +272,8 @@ def test_routed_experts_alone(T, E, K, F, width, dtype):
     corr[0], corr[-1] = 9.0, -9.0
     up, down = (torch.randn(E, F, width) * width ** -0.5).to(dt), (torch.randn(E, width, F) * F ** -0.5).to(dt)
     counts = torch.zeros(E, dtype=torch.int32, device="cuda")
-    rows, dest, w = moe.routed_experts(h.cuda(), logits.cuda(), K, corr.cuda(), up.cuda(), down.cuda(), counts)
+    choice = moe.choose(logits.cuda(), E, K, corr.cuda(), counts)
+    rows, dest, w = moe.routed_experts(h.cuda(), choice, up.cuda(), down.cuda(), counts)
     got = (rows[dest.long()].double() * w[:, :, None].double()).sum(1).cpu()
     assert int(counts[0]) == T and int(counts[-1]) == 0
     for t in range(T):
