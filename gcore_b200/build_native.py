@@ -33,8 +33,8 @@ NVCC_FLAGS = [
     "--expt-relaxed-constexpr",
 ]
 # sources of models that promise 32-bit arithmetic where they say so: compiled without the approximate math functions
-EXACT_MATH = {"depth_average", "latent_attention", "matrix_memory", "matrix_memory_chunk", "moe_serve", "router",
-              "sandwich_norm", "window_attention", "window_prefill"}
+EXACT_MATH = {"depth_average", "diff_attention", "diff_prefill", "latent_attention", "matrix_memory", "matrix_memory_chunk",
+              "moe_serve", "router", "sandwich_norm", "stream_mix", "window_attention", "window_prefill"}
 # sources one served architecture needs: ``ensure_kernels`` builds only these when the full library is not there
 KERNEL_SETS = {
     "nafitar": ("comm", "elementwise", "gemm_skinny", "gemm_tcgen05", "gemm_wide", "matrix_memory", "matrix_memory_chunk",
@@ -42,6 +42,9 @@ KERNEL_SETS = {
     "kedesun": ("attention_fwd", "comm", "depth_average", "elementwise", "gemm_skinny", "gemm_tcgen05", "gemm_wide",
                 "latent_attention", "matrix_memory", "matrix_memory_chunk", "mla_decode", "moe_serve", "router",
                 "sample_filtered", "sandwich_norm", "vocab", "window_attention"),
+    "lobutar": ("attention_fwd", "comm", "diff_attention", "diff_prefill", "elementwise", "gemm_skinny", "gemm_tcgen05",
+                "gemm_wide", "latent_attention", "mla_decode", "moe_serve", "router", "sample_filtered", "sandwich_norm",
+                "stream_mix", "vocab", "window_attention"),
 }
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-Wall", "-pthread"]
 

@@ -6,8 +6,8 @@ from __future__ import annotations
 from dataclasses import dataclass, field, fields
 from typing import Tuple, Any, Dict, List, Optional
 
-from .layer_plan import (DenseSpec, ExpertsSpec, LatentAttentionSpec, LayerPlan, ParallelLayerSpec, kedesun_plan,
-                         nafitar_plan)
+from .layer_plan import (DenseSpec, DifferentialAttentionSpec, ExpertsSpec, LatentAttentionSpec, LayerPlan,
+                         ParallelLayerSpec, StreamLayerSpec, kedesun_plan, lobutar_plan, nafitar_plan)
 
 
 @dataclass
@@ -138,32 +138,44 @@ class ModelConfig:
 
     def _plan_parameters(self, include_embedding: bool) -> int:
         h, total = self.hidden_size, self.hidden_size * (1 + self.layer_plan.loop_times)
+        S = self.layer_plan.streams
         for i, sp in enumerate(self.layer_plan.layers):
-            if isinstance(sp, ParallelLayerSpec):
-                total += self._parallel_layer_parameters(sp, i)
+            if isinstance(sp, (ParallelLayerSpec, StreamLayerSpec)):
+                total += self._mixer_parameters(sp.mixer) + self._ffn_parameters(sp.ffn)
+                if isinstance(sp, ParallelLayerSpec):
+                    total += h + i + 2                                              # norm, depth average
+                else:
+                    total += (h + S * (S + 2)) * (1 if sp.ffn is None else 2)       # norms, hyper-connections
                 continue
             a, m = sp.attention, sp.memory
             total += (2 * a.heads + a.kv_heads) * a.dim * h + (a.heads + a.kv_heads) * a.dim
             total += m.heads * (2 * m.dim + 3 * m.vdim + 2) * h + m.heads * (m.vdim + 2)
             total += (4 if not sp.ffn else 6) * h + 3 * sp.ffn * h
         if include_embedding:
-            total += self.vocab_size * h if self.tie_word_embeddings else \
-                (2 * self.vocab_size + self.max_position_embeddings) * h
+            positions = 0 if S else self.max_position_embeddings
+            total += self.vocab_size * h if self.tie_word_embeddings else (2 * self.vocab_size + positions) * h
         return total
 
-    def _parallel_layer_parameters(self, sp: ParallelLayerSpec, index: int) -> int:
-        h, m, f = self.hidden_size, sp.mixer, sp.ffn
-        n = h + index + 2                       # norm, depth average
+    def _mixer_parameters(self, m) -> int:
+        h = self.hidden_size
         if isinstance(m, LatentAttentionSpec):
-            n += m.heads * (m.dim + m.rot_dim + m.vdim + 1) * h + (m.kv_rank + m.rot_dim) * h
-            n += m.kv_rank * (1 + m.heads * (m.dim + m.vdim))
-        else:
-            n += m.heads * (2 * m.dim + 3 * m.vdim) * h
+            gates = m.heads * (m.vdim if m.gate == "element" else 1)
+            return (m.heads * (m.dim + m.rot_dim + m.vdim) + gates + m.kv_rank + m.rot_dim) * h \
+                + m.kv_rank * (1 + m.heads * (m.dim + m.vdim)) + (m.heads if m.sink else 0)
+        if isinstance(m, DifferentialAttentionSpec):
+            qkv = (m.heads + m.kv_heads) * 2 * m.dim + m.kv_heads * m.vdim
+            return (qkv + m.heads + m.heads * m.vdim) * h + qkv + h + 4 * m.dim
+        return m.heads * (2 * m.dim + 3 * m.vdim) * h
+
+    def _ffn_parameters(self, f) -> int:
+        h = self.hidden_size
         if isinstance(f, DenseSpec):
-            n += 3 * f.ff * h
-        elif isinstance(f, ExpertsSpec):
-            n += f.experts * (2 * f.ff * h + h + 1) + ((2 * f.shared_ff + 1) * h if f.shared_ff else 0)
-        return n
+            return 3 * f.ff * h
+        if isinstance(f, ExpertsSpec):
+            mats = 3 if f.act == "silu_gate" else 2
+            shared = (mats * f.shared_ff + (1 if f.shared_gate else 0)) * h if f.shared_ff else 0
+            return f.experts * (mats * f.ff * h + h + 1) + shared
+        return 0
 
     def active_parameters(self) -> int:
         if not self.is_moe:
@@ -182,7 +194,7 @@ class ModelConfig:
 
 MODEL_ARCH = ("llama", "llama4", "qwen2", "qwen2_5_vl", "qwen3", "qwen3_moe", "qwen3_vl", "qwen3_vl_moe", "qwen2_moe",
               "qwen2_vl", "deepseek_v3", "mistral", "gemma3_text", "seed_oss", "gpt_oss", "nafitar",
-              "kedesun")
+              "kedesun", "lobutar")
 
 PRESETS: Dict[str, Dict[str, Any]] = {
     # tiny Llama-style decoder
@@ -244,8 +256,19 @@ def from_kedesun_config(conf: Dict[str, Any], dtype: str = "bfloat16") -> ModelC
                        max_position_embeddings=ROTARY_POSITIONS, dtype=dtype, layer_plan=plan)
 
 
+def from_lobutar_config(conf: Dict[str, Any], dtype: str = "bfloat16") -> ModelConfig:
+    """Maps a Lobutar ``config.json`` (``architecture``, ``layers``, ``streams``, ``norm``, ``vocab``, ``width``)."""
+    plan = lobutar_plan(conf)
+    m = plan.layers[0].mixer
+    ffn = next((sp.ffn for sp in plan.layers if sp.ffn is not None), None)
+    return ModelConfig(arch="lobutar", num_layers=len(plan.runs), hidden_size=conf["width"], num_attention_heads=m.heads,
+                       num_kv_heads=getattr(m, "kv_heads", m.heads), head_dim=m.dim, ffn_hidden_size=ffn.ff if ffn else 0,
+                       vocab_size=conf["vocab"], rms_norm_eps=float(conf["norm"]["eps"]),
+                       max_position_embeddings=ROTARY_POSITIONS, dtype=dtype, layer_plan=plan)
+
+
 # architectures whose config.json names them in ``architecture``: reader of that file
-ARCH_READERS = {"nafitar": from_nafitar_config, "kedesun": from_kedesun_config}
+ARCH_READERS = {"nafitar": from_nafitar_config, "kedesun": from_kedesun_config, "lobutar": from_lobutar_config}
 
 
 def from_hf_config(hf: Dict[str, Any]) -> ModelConfig:

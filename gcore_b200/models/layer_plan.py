@@ -5,12 +5,13 @@ layers one by one - which mixers a layer runs, the size of each, its feed-forwar
 shared weights.  Every run of a layer (a looped layer counts once per pass) owns its cache and state, so the serving engine
 sizes both from ``LayerPlan.runs``.
 
-Two kinds of layer are described: ``LayerSpec`` (two mixers side by side, then a feed-forward, norms before and after each)
-and ``ParallelLayerSpec`` (one mixer and a feed-forward that read the same normed input)."""
+Three kinds of layer are described: ``LayerSpec`` (two mixers side by side, then a feed-forward, norms before and after
+each), ``ParallelLayerSpec`` (one mixer and a feed-forward that read the same normed input) and ``StreamLayerSpec`` (a mixer,
+then a feed-forward, each reading a mixture of several residual streams and writing to all of them)."""
 from __future__ import annotations
 
 import math
-from dataclasses import dataclass
+from dataclasses import dataclass, replace
 from typing import Any, Dict, List, Optional, Tuple, Union
 
 
@@ -104,8 +105,9 @@ class RotarySpec:
 @dataclass(frozen=True)
 class LatentAttentionSpec:
     """Causal softmax attention over a cached latent: per token one normed vector of ``kv_rank`` that every head expands to
-    its own key (``dim``) and value (``vdim``), and one rotated key part of ``rot_dim`` that all heads share; the output of
-    a head is scaled by a sigmoid gate."""
+    its own key (``dim``) and value (``vdim``), and one rotated key part of ``rot_dim`` that all heads share.  ``window``:
+    position i sees j with ``0 <= i - j < window`` (0: every j <= i); ``sink``: a learned logit per head joins the softmax
+    denominator; ``gate``: the output is scaled by sigmoids, one per "head" or one per "element"."""
     heads: int
     dim: int
     rot_dim: int
@@ -113,12 +115,38 @@ class LatentAttentionSpec:
     kv_rank: int
     scale: float
     rot: RotarySpec
+    window: int = 0
+    sink: bool = False
+    gate: str = "head"
 
     def __post_init__(self):
-        if min(self.heads, self.dim, self.vdim, self.kv_rank) < 1:
+        if min(self.heads, self.dim, self.vdim, self.kv_rank) < 1 or self.window < 0:
             raise ValueError("latent-attention sizes must be positive")
+        if self.gate not in ("head", "element"):
+            raise ValueError(f"unknown output gate {self.gate!r}")
         if self.rot.dims != self.rot_dim:
             raise ValueError("the rotation must cover the rotated key part")
+
+
+@dataclass(frozen=True)
+class DifferentialAttentionSpec:
+    """Grouped-query causal attention whose heads subtract two softmax maps over the same values: per head two queries and
+    per key/value head two keys of ``dim``, the first ``rot.dims`` of them rotated; the difference ``a1 - lambda * a2`` is
+    normed over the head's ``vdim`` values, scaled by ``1 - diff`` and by a sigmoid gate of the head.  lambda is learned
+    (four vectors of ``dim``) around ``diff``.  The projections have biases."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    diff: float
+    rot: RotarySpec
+
+    def __post_init__(self):
+        if self.heads < 1 or self.kv_heads < 1 or self.heads % self.kv_heads:
+            raise ValueError("query heads must be a positive multiple of the key/value heads")
+        if min(self.dim, self.vdim) < 1 or self.rot.dims > self.dim:
+            raise ValueError("attention sizes must be positive and hold the rotated dimensions")
 
 
 @dataclass(frozen=True)
@@ -144,22 +172,46 @@ class DenseSpec:
 
 @dataclass(frozen=True)
 class ExpertsSpec:
-    """Mixture of small feed-forwards ``down(relu(up h)^2)``: softmax scores, chosen with a correction that the weights do
-    not carry, and a shared expert (``shared_ff`` = 0: none) behind a sigmoid gate of one number per token."""
+    """Mixture of small feed-forwards, ``down(relu(up h)^2)`` ("relu2") or ``down(silu(gate h) * up h)`` ("silu_gate").  The
+    ``top`` experts are chosen by score + correction; the weights carry the scores alone, normalised or not, times
+    ``scale``.  Scores are a softmax or sigmoids of the router's logits.  With ``groups`` > 1 only experts of the ``keep``
+    groups of neighbours with the largest sum of two best choice scores take part.  A shared expert (``shared_ff`` = 0:
+    none) runs for every token, behind a sigmoid gate of one number per token if ``shared_gate``."""
     experts: int
     top: int
     ff: int
     shared_ff: int = 0
+    act: str = "relu2"
+    score: str = "softmax"
+    normalize: bool = True
+    scale: float = 1.0
+    groups: int = 1
+    keep: int = 1
+    shared_gate: bool = True
 
     def __post_init__(self):
         if not 1 <= self.top <= self.experts or self.ff < 1 or self.shared_ff < 0:
             raise ValueError("experts need positive sizes and at most as many choices as experts")
+        if self.act not in ("relu2", "silu_gate") or self.score not in ("softmax", "sigmoid"):
+            raise ValueError(f"unknown expert activation {self.act!r} or score {self.score!r}")
+        if self.groups < 1 or self.experts % self.groups or not 1 <= self.keep <= self.groups:
+            raise ValueError("expert groups must be equal and some of them kept")
+        if self.top > self.experts // self.groups * self.keep:
+            raise ValueError("the kept groups hold fewer experts than are chosen")
 
 
 @dataclass(frozen=True)
 class ParallelLayerSpec:
     """One layer whose mixer and feed-forward (None: none) read the same normed input."""
     mixer: Union[LatentAttentionSpec, RetentionSpec]
+    ffn: Union[DenseSpec, ExpertsSpec, None] = None
+
+
+@dataclass(frozen=True)
+class StreamLayerSpec:
+    """One layer of a decoder with several residual streams (hyper-connections): a mixer, then a feed-forward (None: none),
+    each behind its own norm."""
+    mixer: Union[LatentAttentionSpec, DifferentialAttentionSpec]
     ffn: Union[DenseSpec, ExpertsSpec, None] = None
 
 
@@ -174,21 +226,41 @@ class LayerRun:
 
 @dataclass(frozen=True)
 class LayerPlan:
-    layers: Tuple[Union[LayerSpec, ParallelLayerSpec], ...]
+    """``layers``: the layers that own weights.  They run in order, with a looped range, or, with ``order``, as it lists them
+    (a layer may run any number of times).  ``names``: the layers' numbers in the checkpoint when they are not 0, 1, ..."""
+    layers: Tuple[Union[LayerSpec, ParallelLayerSpec, StreamLayerSpec], ...]
     loop_start: int = 0
     loop_stop: int = 0
     loop_times: int = 0          # 0: no loop
+    order: Tuple[int, ...] = ()
+    names: Tuple[int, ...] = ()
+    streams: int = 0             # residual streams of a decoder with hyper-connections
 
     def __post_init__(self):
         if not self.layers:
             raise ValueError("a layer plan needs at least one layer")
         if self.loop_times < 0 or (self.loop_times and not 0 <= self.loop_start < self.loop_stop <= len(self.layers)):
             raise ValueError("the looped layers must be a non-empty range of the layer list")
+        if self.order and (self.loop_times or not all(0 <= i < len(self.layers) for i in self.order)):
+            raise ValueError("the order of a plan's runs names layers of the plan and goes without a loop")
+        if self.names and len(self.names) != len(self.layers):
+            raise ValueError("a plan's layer names must cover its layers")
+
+    def name(self, i: int) -> int:
+        """Number of layer i in the checkpoint."""
+        return self.names[i] if self.names else i
+
+    def windows(self) -> List[int]:
+        """Distinct attention windows of the latent mixers (0: unlimited)."""
+        mixers = [getattr(sp, "mixer", None) for sp in self.layers]
+        return sorted({m.window for m in mixers if isinstance(m, LatentAttentionSpec)})
 
     @property
     def runs(self) -> List[LayerRun]:
         order: List[Tuple[int, Optional[int]]] = []
-        if self.loop_times:
+        if self.order:
+            order = [(i, None) for i in self.order]
+        elif self.loop_times:
             order += [(i, None) for i in range(self.loop_start)]
             for t in range(self.loop_times):
                 order += [(i, t if i == self.loop_start else None) for i in range(self.loop_start, self.loop_stop)]
@@ -258,6 +330,61 @@ def _feed_forward(m: Optional[Dict[str, Any]], where: str):
     router, shared = _need(m, "router", where), m.get("shared")
     return ExpertsSpec(experts=_need(router, "experts", where), top=_need(router, "top", where),
                        ff=_need(_need(m, "expert", where), "ff", where), shared_ff=shared["ff"] if shared else 0)
+
+
+def _differential_attention(m: Dict[str, Any], where: str) -> DifferentialAttentionSpec:
+    return DifferentialAttentionSpec(rot=_rotation(_need(m, "rot", where), where + ".rot"),
+                                     **{k: float(_need(m, k, where)) for k in ("scale", "diff")},
+                                     **{k: _need(m, k, where) for k in ("heads", "kv_heads", "dim", "vdim")})
+
+
+def _window_latent_attention(m: Dict[str, Any], where: str) -> LatentAttentionSpec:
+    window = _need(_need(m, "mask", where), "size", where + ".mask")
+    if window < 1:
+        raise ValueError(f"{where}.mask: the window must be positive")
+    return replace(_latent_attention(m, where), window=window, sink=True, gate="element")
+
+
+STREAM_MIXER_READERS = {"attention": _differential_attention, "latent_attention": _window_latent_attention}
+
+
+def _grouped_experts(m: Optional[Dict[str, Any]], where: str):
+    """Feed-forward of a stream layer: experts are gated, with sigmoid scores that are not normalised."""
+    spec = _feed_forward(m, where)
+    if not isinstance(spec, ExpertsSpec):
+        return spec
+    router = m["router"]
+    groups = router.get("groups") or {"count": 1, "keep": 1}
+    return replace(spec, act="silu_gate", score="sigmoid", normalize=False, scale=float(router.get("scale", 1.0)),
+                   groups=_need(groups, "count", where + ".router.groups"),
+                   keep=_need(groups, "keep", where + ".router.groups"), shared_gate=False)
+
+
+def lobutar_plan(conf: Dict[str, Any]) -> LayerPlan:
+    """Layer plan of a Lobutar ``config.json``.  Entries with ``weights_of`` run another entry's layer once more."""
+    entries = _need(conf, "layers", "config")
+    owner = []
+    for i, entry in enumerate(entries):
+        j, seen = i, set()
+        while entries[j].get("weights_of") is not None:
+            seen.add(j)
+            j = entries[j]["weights_of"]
+            if not 0 <= j < len(entries) or j in seen:
+                raise ValueError(f"layers[{i}]: 'weights_of' names no layer with weights")
+        owner.append(j)
+    names = [i for i, j in enumerate(owner) if i == j]
+    layers = []
+    for i in names:
+        where, entry = f"layers[{i}]", entries[i]
+        reader = STREAM_MIXER_READERS.get(entry.get("type"))
+        if reader is None:
+            raise ValueError(f"{where}: unknown mixer type {entry.get('type')!r}")
+        layers.append(StreamLayerSpec(reader(_need(entry, "mixer", where), where + ".mixer"),
+                                      _grouped_experts(entry.get("mlp"), where + ".mlp")))
+    streams = _need(conf, "streams", "config")
+    if streams < 1:
+        raise ValueError("a decoder needs at least one residual stream")
+    return LayerPlan(tuple(layers), order=tuple(names.index(j) for j in owner), names=tuple(names), streams=streams)
 
 
 def kedesun_plan(conf: Dict[str, Any]) -> LayerPlan:

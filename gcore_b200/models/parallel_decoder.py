@@ -3,10 +3,7 @@ input and hand on a weighted average over depth (Kedesun).
 
 Because both sublayers read the same input and are summed, a layer has two projections only: one into
 ``[mixer columns | feed-forward columns]`` and one out of ``[mixer output | feed-forward activation]``, whose product is the
-sum of the two.  Routed experts are added to it, still in expert order, by the residual step.
-
-Every block of columns is a multiple of 8 wide and heads are padded with zero rows to the sizes the kernels store; zero
-padding changes no score, state or output, and means are taken over the true sizes."""
+sum of the two.  Routed experts are added to it, still in expert order, by the residual step."""
 from __future__ import annotations
 
 import math
@@ -14,64 +11,12 @@ import math
 import torch
 import torch.nn as nn
 
-from ..ops import depth, latent_attention as la, matrix_memory as mm, moe, sandwich
+from ..ops import depth, matrix_memory as mm, sandwich
 from ..ops.gemm import linear_forward
 from .config import ModelConfig
-from .layer_plan import DenseSpec, ExpertsSpec, LatentAttentionSpec, ParallelLayerSpec, RetentionSpec
-from .plan_decoder import CheckpointTensors, PlanDecoder, _buf, _up, put, put_heads
-
-
-def _columns(*sizes):
-    """Offsets of consecutive blocks and their total."""
-    at, n = [], 0
-    for s in sizes:
-        at.append(n)
-        n += s
-    return at, n
-
-
-class LatentAttentionMixer(nn.Module):
-    def __init__(self, spec: LatentAttentionSpec, width: int, eps: float, dtype, device):
-        super().__init__()
-        self.spec, self.width = spec, width
-        rank, rot = la.cached_row(spec.kv_rank, spec.rot_dim)
-        dim, vdim = _up(spec.dim, 8), _up(spec.vdim, 8)
-        (q, down, gate), self.columns = _columns(spec.heads * (dim + rot), rank + rot, _up(spec.heads, 8))
-        self.layout = la.LatentLayout(q=q, down=down, gate=gate, heads=spec.heads, dim=dim, vdim=vdim, rank=spec.kv_rank,
-                                      row_rank=rank, rot=spec.rot_dim, row_rot=rot, scale=spec.scale,
-                                      magnitude=spec.rot.magnitude(), eps=eps)
-        self.out_columns = spec.heads * vdim
-        self.gain = _buf(torch.zeros(spec.kv_rank, dtype=torch.float32, device=device))
-        self.turns = _buf(la.rotation_turns(spec.rot.frequencies()).to(device))
-        self.up_kv = _buf(torch.zeros(spec.heads * (dim + vdim), rank, dtype=dtype, device=device))
-
-    def cache_shape(self):
-        return 1, self.layout.row
-
-    def new_state(self, slots, device):
-        return None
-
-    def state_bytes(self):
-        return 0
-
-    def load(self, take, p: str, rows, out):
-        s, ly, W = self.spec, self.layout, self.width
-        H, d, r, C = s.heads, s.dim, s.rot_dim, s.kv_rank
-        q = take(p + "q", H * (d + r), W).view(H, d + r, W)
-        dst = rows[ly.q:ly.q + H * (ly.dim + ly.row_rot)].view(H, ly.dim + ly.row_rot, -1)
-        put(dst, q[:, :d])
-        put(dst[:, ly.dim:], q[:, d:])
-        down = take(p + "dkv", C + r, W)
-        put(rows[ly.down:], down[:C])
-        put(rows[ly.down + ly.row_rank:], down[C:])
-        put(rows[ly.gate:], take(p + "g", H, W))
-        put(self.gain, take(p + "dkv.norm", C).float())
-        put_heads(self.up_kv[:H * ly.dim], take(p + "uk", H * d, C), H, d, ly.dim)
-        put_heads(self.up_kv[H * ly.dim:], take(p + "uv", H * s.vdim, C), H, s.vdim, ly.vdim)
-        put(out.view(out.shape[0], H, ly.vdim), take(p + "o", W, H * s.vdim).view(W, H, s.vdim))
-
-    def forward(self, proj, rows, cache, state, out):
-        la.latent_attention(proj, self.layout, self.gain, self.turns, self.up_kv, rows, cache, out)
+from .layer_plan import ExpertsSpec, LatentAttentionSpec, ParallelLayerSpec, RetentionSpec
+from .plan_decoder import CheckpointTensors, PlanDecoder, _buf, put, put_heads
+from .plan_modules import DenseFeedForward, ExpertFeedForward, LatentAttentionMixer, blocks
 
 
 class RetentionMixer(nn.Module):
@@ -80,7 +25,7 @@ class RetentionMixer(nn.Module):
         self.spec, self.width, self.eps = spec, width, eps
         self.dim, self.vdim = mm.padded_key_dim(spec.dim), mm.padded_value_dim(spec.vdim)
         H = spec.heads
-        self.at, self.columns = _columns(H * self.dim, H * self.dim, H * self.vdim, H * self.vdim)
+        self.at, self.columns = blocks(H * self.dim, H * self.dim, H * self.vdim, H * self.vdim)
         self.out_columns = H * self.vdim
         self.decay = _buf(torch.tensor(spec.decay, dtype=torch.float32, device=device))
 
@@ -102,60 +47,6 @@ class RetentionMixer(nn.Module):
     def forward(self, proj, rows, cache, state, out):
         s = self.spec
         mm.retention(proj, *self.at, self.decay, s.dim ** -0.5, s.heads, self.dim, self.vdim, s.vdim, rows, state, self.eps, out)
-
-
-class DenseFeedForward(nn.Module):
-    def __init__(self, spec: DenseSpec, width: int, width_pad: int, dtype, device):
-        super().__init__()
-        self.spec, self.width, self.ff = spec, width, _up(spec.ff, 8)
-        self.columns, self.out_columns = 2 * self.ff, self.ff
-
-    def load(self, take, p: str, rows, out):
-        f, W = self.spec.ff, self.width
-        put(rows, take(p + "gate", f, W))
-        put(rows[self.ff:], take(p + "up", f, W))
-        put(out, take(p + "down", W, f))
-
-    def forward(self, h, proj, out, counts):
-        moe.activate(moe.SILU_GATE, proj, self.ff, self.ff, out)
-        return None
-
-
-class ExpertFeedForward(nn.Module):
-    """The shared expert is part of the layer's two projections; routed experts run on the grouped GEMM."""
-
-    def __init__(self, spec: ExpertsSpec, width: int, width_pad: int, dtype, device):
-        super().__init__()
-        if spec.experts > moe.MAX_EXPERTS or spec.top > moe.MAX_TOP:
-            raise ValueError(f"at most {moe.MAX_EXPERTS} experts and {moe.MAX_TOP} choices are supported")
-        self.spec, self.width = spec, width
-        self.ff, self.shared = _up(spec.ff, 8), _up(spec.shared_ff, 8)
-        self.columns = self.out_columns = self.shared
-        act = dict(dtype=dtype, device=device)
-        E = spec.experts
-        self.router = _buf(torch.zeros(E + (1 if self.shared else 0), width_pad, **act))   # + the shared expert's gate
-        self.correction = _buf(torch.zeros(E, dtype=torch.float32, device=device))
-        self.up = _buf(torch.zeros(E, self.ff, width_pad, **act))
-        self.down = _buf(torch.zeros(E, width_pad, self.ff, **act))
-
-    def load(self, take, p: str, rows, out):
-        s, W = self.spec, self.width
-        put(self.router, take(p + "router", s.experts, W))
-        put(self.correction, take(p + "correction", s.experts).float())
-        for e in range(s.experts):
-            put(self.up[e], take(f"{p}e{e}.up", s.ff, W))
-            put(self.down[e], take(f"{p}e{e}.down", W, s.ff))
-        if self.shared:
-            put(rows, take(p + "shared.up", s.shared_ff, W))
-            put(out, take(p + "shared.down", W, s.shared_ff))
-            put(self.router[s.experts:], take(p + "shared.sg", 1, W))
-
-    def forward(self, h, proj, out, counts):
-        s = self.spec
-        logits, choice = moe.route_tokens(h, self.router, s.experts, s.top, self.correction, counts)
-        if self.shared:
-            moe.activate(moe.RELU2, proj, self.shared, 0, out, row_logit=logits[:, s.experts])
-        return moe.routed_experts(h, choice, self.up, self.down, counts)
 
 
 class ParallelLayer(nn.Module):

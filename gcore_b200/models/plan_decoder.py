@@ -25,7 +25,7 @@ from ..ops import sandwich
 from ..ops import window_attention as wa
 from ..ops.gemm import linear_forward
 from .config import ModelConfig
-from .layer_plan import LayerSpec, ParallelLayerSpec
+from .layer_plan import LayerSpec, ParallelLayerSpec, StreamLayerSpec
 
 
 def _up(n: int, m: int) -> int:
@@ -59,6 +59,11 @@ class CheckpointTensors:
         if tuple(t.shape) != shape:
             raise ValueError(f"'{name}' has shape {tuple(t.shape)}, the configuration says {shape}")
         return t
+
+    def drop(self, *names: str):
+        """Tensors the configuration has no use for, if they are there."""
+        for n in names:
+            self.left.pop(n, None)
 
     def done(self):
         if self.left:
@@ -164,7 +169,7 @@ class PlanDecoder(nn.Module):
 
     # ---- what the engine allocates for every layer run
     def new_caches(self, blocks: int, block_size: int, device) -> list:
-        """Paged cache of every run: one row per token serves as key and value; None for runs without one."""
+        """Paged cache of every run, one row (of any shape) per token; None for runs without one."""
         shapes = [self.layers[r.layer].cache_shape() for r in self.cfg.layer_plan.runs]
         return [torch.zeros(blocks, block_size, *s, dtype=self.dtype, device=device) if s else None for s in shapes]
 
@@ -281,5 +286,6 @@ class SandwichDecoder(PlanDecoder):
 def build_decoder(cfg: ModelConfig, device=None) -> PlanDecoder:
     """The serving module of a layer-plan configuration."""
     from .parallel_decoder import ParallelDecoder
-    cls = ParallelDecoder if isinstance(cfg.layer_plan.layers[0], ParallelLayerSpec) else SandwichDecoder
-    return cls(cfg, device)
+    from .stream_decoder import StreamDecoder
+    cls = {ParallelLayerSpec: ParallelDecoder, StreamLayerSpec: StreamDecoder, LayerSpec: SandwichDecoder}
+    return cls[type(cfg.layer_plan.layers[0])](cfg, device)

@@ -210,14 +210,14 @@ def _declare_kernels(lib: ctypes.CDLL):
     d("gk_paged_decode_append", [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, F, I, I, I, F, P])
     d("gk_paged_set_target_ctas", [I], None)
     d("gk_mla_paged_decode", [P, L, L, P, L, L, P, P, P, P, L, L, P, I, I, I, I, I, I, I, F, P])
-    d("gk_mla_paged_decode_gated", [P, L, L, P, L, L, P, P, P, P, L, L, P, I, I, I, I, I, I, I, F, P, L, P])
+    d("gk_mla_paged_decode_gated", [P, L, L, P, L, L, P, P, P, P, L, L, P, I, I, I, I, I, I, I, F, P, L, I, P, P])
     d("gk_mla_decode_scratch", [I, I, I, I, ctypes.POINTER(L)], None)
     d("gk_mla_decode_supported", [I, I])
     d("gk_mla_set_target_ctas", [I], None)
     d("gk_sandwich_norm", [I, I, P, P, F, P])
     d("gk_swiglu_f32", [P, P, L, I, P])
     d("gk_append_keys", [P, L, L, I, P, P, I, P])
-    d("gk_window_attn", [I, P, L, L, P, F, P])
+    d("gk_window_attn", [I, I, P, P, P, F, P])
     d("gk_shared_kv_decode", [P, L, P, P, P, P, P, P, P, P, F, P])
     d("gk_shared_kv_decode_scratch", [I, I, I, I], L)
     d("gk_shared_decode_set_target_ctas", [I], None)
@@ -229,10 +229,20 @@ def _declare_kernels(lib: ctypes.CDLL):
     d("gk_ffn_act", [I, I, P, P, P, P])
     d("gk_expert_rows", [P, P, P, P, P, P, P, I, I, I, I, P])
     d("gk_grouped_gemm_f32", [P, P, P, P, I, I, I, I, P])
-    d("gk_router_dispatch", [P, L, P, P, P, P, P, L, I, I, I, I, F, P])
-    d("gk_router_fused", [I, P, P, P, I, I, P, P, P, P, P, L, I, I, I, I, F, P])
+    d("gk_router_dispatch", [P, L, P, P, P, P, P, L, I, I, I, I, F, I, I, P])
+    d("gk_router_fused", [I, P, P, P, I, I, P, P, P, P, P, L, I, I, I, I, F, I, I, P])
     d("gk_latent_prep", [I, P, L, P, F, F, P])
-    d("gk_latent_gather", [P, P, P, P, P, I, I, I, I, I, P])
+    d("gk_latent_gather", [P, P, P, P, P, P, I, I, I, I, I, P])
+    d("gk_gate_columns", [I, P, L, P, L, I, I, P])
+    d("gk_stream_mix", [I, P, P, F, P])
+    d("gk_rotate_append", [I, P, L, P, F, P])
+    d("gk_diff_prefill", [P, P, P, P, P])
+    d("gk_diff_prefill_supported", [I, I])
+    d("gk_diff_decode", [P, P, P, P, P])
+    d("gk_diff_decode_supported", [I, I])
+    d("gk_diff_decode_scratch", [I, I, I, I, I], L)
+    d("gk_diff_set_target_ctas", [I], None)
+    d("gk_diff_combine", [I, I, P, L, L, P, P, P])
     d("gk_latent_prefill", [P, P, P, F, P])
     d("gk_latent_prefill_supported", [I, I, I])
     d("gk_attn_fwd", [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, I, P, P])

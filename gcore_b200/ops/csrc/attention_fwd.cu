@@ -18,7 +18,7 @@
 // LAT instances serve latent attention over prompt portions: the last 64-wide chunk of queries and keys is a rotated part
 // that comes from matrices of its own (the key's is shared by all heads), heads narrower than the tile are zero-filled by
 // the loads, probabilities enter P V as two bf16 terms (rounded value and remainder, 16 significant bits), and the output
-// is scaled by a sigmoid gate per (token, head).
+// is scaled by a sigmoid gate per (token, head) or per output element.
 #include "ptx.cuh"
 #include "host_utils.h"
 #include <float.h>
@@ -41,8 +41,9 @@ struct FaParams {
   int causal, window;
   float scale;
   int* err;
-  const __nv_bfloat16* gate;   // LAT: [Tq, Hq] logits, gate_ld apart, or null
+  const __nv_bfloat16* gate;   // LAT: rows of logits, gate_ld apart, or null
   long long gate_ld;
+  int gate_cols;               // LAT: gate logits per head: 1 or dv
   int dv;                      // LAT: value columns in use (a multiple of 8)
 };
 
@@ -337,7 +338,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
       if (p.sinks) l += exp2f(p.sinks[h] * 1.4426950408889634f - m_use);
       float inv = l > 0.f ? 1.f / l : 0.f;
       const bool valid = qi < lq;
-      if (LAT && p.gate && valid)
+      if (LAT && p.gate && valid && p.gate_cols == 1)
         inv /= 1.f + exp2f(-1.4426950408889634f * __bfloat162float(p.gate[static_cast<long long>(q_beg + qi) * p.gate_ld + h]));
       __nv_bfloat16* orow = p.out + static_cast<long long>(q_beg + qi) * p.o_stride_t + static_cast<long long>(h) * (LAT ? p.dv : DV);
 #pragma unroll
@@ -354,11 +355,24 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__
 #pragma unroll
           for (int j = 0; j < 4; ++j) {
             if (LAT && c * 32 + j * 8 >= p.dv) break;
+            float v[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) v[e] = __uint_as_float(r[8 * j + e]) * inv;
+            if (LAT && p.gate && p.gate_cols != 1) {
+              const uint4 g = *reinterpret_cast<const uint4*>(p.gate + static_cast<long long>(q_beg + qi) * p.gate_ld +
+                                                              static_cast<long long>(h) * p.gate_cols + c * 32 + j * 8);
+              const uint32_t gw[4] = {g.x, g.y, g.z, g.w};
+#pragma unroll
+              for (int e = 0; e < 8; ++e) {
+                const float z = bf16_bits_to_float(static_cast<uint16_t>(e & 1 ? gw[e >> 1] >> 16 : gw[e >> 1] & 0xffff));
+                v[e] = __fdividef(v[e], 1.f + exp2f(-1.4426950408889634f * z));
+              }
+            }
             uint4 w;
-            w.x = pack_bf16x2(__uint_as_float(r[8 * j + 0]) * inv, __uint_as_float(r[8 * j + 1]) * inv);
-            w.y = pack_bf16x2(__uint_as_float(r[8 * j + 2]) * inv, __uint_as_float(r[8 * j + 3]) * inv);
-            w.z = pack_bf16x2(__uint_as_float(r[8 * j + 4]) * inv, __uint_as_float(r[8 * j + 5]) * inv);
-            w.w = pack_bf16x2(__uint_as_float(r[8 * j + 6]) * inv, __uint_as_float(r[8 * j + 7]) * inv);
+            w.x = pack_bf16x2(v[0], v[1]);
+            w.y = pack_bf16x2(v[2], v[3]);
+            w.z = pack_bf16x2(v[4], v[5]);
+            w.w = pack_bf16x2(v[6], v[7]);
             *reinterpret_cast<uint4*>(orow + c * 32 + j * 8) = w;
           }
         }
@@ -424,7 +438,7 @@ GK_EXPORT int gk_attn_fwd(const void* q, const void* k, const void* v, void* out
   p.lse = lse; p.tq_total = Tq;
   p.Hq = Hq; p.Hk = Hk; p.causal = causal; p.window = window; p.scale = scale;
   p.err = reinterpret_cast<int*>(se[1]);
-  p.gate = nullptr; p.gate_ld = 0; p.dv = Dv;
+  p.gate = nullptr; p.gate_ld = 0; p.gate_cols = 1; p.dv = Dv;
   dim3 grid((max_q + FA_BM - 1) / FA_BM, Hq, B);
   cudaStream_t st = reinterpret_cast<cudaStream_t>(se[0]);
   if (D == 192) return launch_fa<192, 128>(tq, tk, tv, tq, tk, p, grid, st);
@@ -438,16 +452,19 @@ GK_EXPORT int gk_latent_prefill_supported(int dim, int rot, int vdim) {
 }
 
 // Latent attention over prompt portions whose context lies expanded and contiguous: query i of portion b sees the keys
-// 0 .. lk - lq + i of its context.  q [Tq rows, q_ld]: head h has `dim` unrotated columns at q_off + h * q_hs and `rot`
+// 0 .. lk - lq + i of its context, or the last `window` of them (0: all); sinks [H] (or null) join the denominators.  q [Tq rows, q_ld]: head h has `dim` unrotated columns at q_off + h * q_hs and `rot`
 // rotated ones behind them; kv [Tk rows, kv_ld]: head h has its `dim` key columns at h * dim and `vdim` value columns at
-// H * dim + h * vdim; kr [Tk rows, kr_ld]: the rotated key part of all heads; gate [Tq rows, gate_ld]: one logit per head.
+// H * dim + h * vdim; kr [Tk rows, kr_ld]: the rotated key part of all heads; gate [Tq rows, gate_ld]: gate_cols logits per
+// head, 1 or vdim.
 // All widths, offsets and strides are multiples of 8 elements.
-// ptrs: {q, kv, kr, gate, out, cu_q, cu_k, err};  lds: {q_ld, kv_ld, kr_ld, gate_ld, out_ld}
-// dims: {portions, Tq, Tk, H, dim, rot, vdim, q_hs, max_q}
+// ptrs: {q, kv, kr, gate, out, cu_q, cu_k, err, sinks};  lds: {q_ld, kv_ld, kr_ld, gate_ld, out_ld}
+// dims: {portions, Tq, Tk, H, dim, rot, vdim, q_hs, max_q, window, gate_cols}
 GK_EXPORT int gk_latent_prefill(void* const* ptrs, const long long* lds, const int* dims, float scale, void* stream) {
   const int B = dims[0], Tq = dims[1], Tk = dims[2], H = dims[3], dim = dims[4], rot = dims[5], vdim = dims[6];
   if (!gk_latent_prefill_supported(dim, rot, vdim)) return -1;
   if (dim % 8 || rot % 8 || vdim % 8 || dims[7] % 8 || lds[0] % 8 || lds[1] % 8 || lds[2] % 8 || lds[4] % 8) return -2;
+  if (dims[9] < 0 || (dims[10] != 1 && (dims[10] != vdim || lds[3] % 8 || (reinterpret_cast<uintptr_t>(ptrs[3]) & 15))))
+    return -2;
   if (B == 0 || Tq == 0) return 0;
   const __nv_bfloat16 *q = static_cast<const __nv_bfloat16*>(ptrs[0]), *kv = static_cast<const __nv_bfloat16*>(ptrs[1]),
                       *kr = static_cast<const __nv_bfloat16*>(ptrs[2]);
@@ -461,13 +478,14 @@ GK_EXPORT int gk_latent_prefill(void* const* ptrs, const long long* lds, const i
   if (make_tmap_3d(&tv, kv + static_cast<long long>(H) * dim, 2, Tk, H, vdim, lds[1], vdim, FA_BN, 1, 64, true)) return -6;
   if (make_tmap_3d(&tkr, kr, 2, Tk, 1, rot, lds[2], rot, FA_BN, 1, 64, true)) return -7;
   FaParams p;
-  p.cu_q = static_cast<const int*>(ptrs[5]); p.cu_k = static_cast<const int*>(ptrs[6]); p.sinks = nullptr;
+  p.cu_q = static_cast<const int*>(ptrs[5]); p.cu_k = static_cast<const int*>(ptrs[6]);
+  p.sinks = static_cast<const float*>(ptrs[8]);
   p.out = static_cast<__nv_bfloat16*>(ptrs[4]);
   p.o_stride_t = lds[4];
   p.lse = nullptr; p.tq_total = Tq;
-  p.Hq = H; p.Hk = H; p.causal = 1; p.window = 0; p.scale = scale;
+  p.Hq = H; p.Hk = H; p.causal = 1; p.window = dims[9]; p.scale = scale;
   p.err = static_cast<int*>(ptrs[7]);
-  p.gate = static_cast<const __nv_bfloat16*>(ptrs[3]); p.gate_ld = lds[3]; p.dv = vdim;
+  p.gate = static_cast<const __nv_bfloat16*>(ptrs[3]); p.gate_ld = lds[3]; p.gate_cols = dims[10]; p.dv = vdim;
   const dim3 grid((dims[8] + FA_BM - 1) / FA_BM, H, B);
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   if (dim <= 64)

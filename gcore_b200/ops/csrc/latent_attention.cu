@@ -3,10 +3,12 @@
 // at its position], both padded with zeros; it serves every head.
 //   * latent_prep_kernel    a packed projection row -> its cache row (norm of the latent in 32-bit, rotation), the queries'
 //                           rotated parts in place, and a copy of the cache row in the portion's contiguous context;
-//   * latent_gather_kernel  cache rows of the tokens in front of a portion -> the portion's contiguous context.
-// The rotation pairs dimension 2i with 2i + 1, all in 32-bit.  A pair's speed is given in turns per position as two floats
-// (value and remainder), so the fraction of a turn is as exact at position 10^6 as at position 1.
+//   * latent_gather_kernel  cache rows of the tokens in front of a portion -> the portion's contiguous context;
+//   * gate_columns_kernel   attention output times the sigmoid of a gate per element.
+// A portion's context starts at position 0 or, under a window, at the first position its first row sees.  The rotation pairs
+// dimension 2i with 2i + 1 (rotary.cuh).
 #include "host_utils.h"
+#include "rotary.cuh"
 #include "row_ops.cuh"
 #include <type_traits>
 
@@ -35,6 +37,7 @@ struct LatentPrepParams {
   T* context;              // [context rows, CV + DR] or null
   const int* row_seq;      // with context: portion of every row
   const int* cu_ctx;       //   first context row of every portion
+  const int* ctx_start;    //   position of that row, or null: 0
   int rows, context_rows;  //   rows that belong to portions (they come first)
   int H, C, CV, rot, DR;
   float eps, magnitude;
@@ -51,11 +54,8 @@ __global__ void __launch_bounds__(LP_THREADS) latent_prep_kernel(const LatentPre
   T* pr = p.proj + row * p.ld;
   const int pos = p.pos[row], slot = p.slots[row];
   for (int i = tid; i < half; i += LP_THREADS) {
-    const float2 f = p.turns[i];
-    const float x = static_cast<float>(pos), t = x * f.x;
-    const float frac = (t - rintf(t)) + fmaf(x, f.y, fmaf(x, f.x, -t));
     float s, c;
-    sincospif(2.f * frac, &s, &c);
+    rotation_at(pos, p.turns[i], &s, &c);
     s_cos[i] = c * p.magnitude;
     s_sin[i] = s * p.magnitude;
   }
@@ -67,8 +67,11 @@ __global__ void __launch_bounds__(LP_THREADS) latent_prep_kernel(const LatentPre
   const float r = 1.f / sqrtf(block_sum2(ss, 0.f, red).x / p.C + p.eps);      // also orders the angles for all threads
   const int width = p.CV + p.DR;
   T* dst = slot >= 0 ? p.cache + static_cast<long long>(slot) * width : nullptr;
-  T* ctx = p.context && row < p.context_rows
-               ? p.context + (static_cast<long long>(p.cu_ctx[p.row_seq[row]]) + pos) * width : nullptr;
+  T* ctx = nullptr;
+  if (p.context && row < p.context_rows) {
+    const int b = p.row_seq[row];
+    ctx = p.context + (static_cast<long long>(p.cu_ctx[b]) + pos - (p.ctx_start ? p.ctx_start[b] : 0)) * width;
+  }
   for (int c = tid; c < width; c += LP_THREADS) {
     float v = 0.f;
     if (c < p.C) {
@@ -94,17 +97,36 @@ __global__ void __launch_bounds__(LP_THREADS) latent_prep_kernel(const LatentPre
 __global__ void __launch_bounds__(256) latent_gather_kernel(const uint4* __restrict__ cache, const int* __restrict__ tables,
                                                             int max_blocks, int block_size,
                                                             const int* __restrict__ first_pos,
-                                                            const int* __restrict__ cu_ctx, uint4* __restrict__ context,
-                                                            int vec) {
+                                                            const int* __restrict__ cu_ctx,
+                                                            const int* __restrict__ ctx_start,
+                                                            uint4* __restrict__ context, int vec) {
   pdl_launch_dependents();
   pdl_wait();
-  const int b = blockIdx.y, n = first_pos[b], lane = threadIdx.x & 31;
+  const int b = blockIdx.y, start = ctx_start ? ctx_start[b] : 0, n = first_pos[b] - start, lane = threadIdx.x & 31;
   const int* table = tables + static_cast<long long>(b) * max_blocks;
   uint4* out = context + static_cast<long long>(cu_ctx[b]) * vec;
   for (int j = blockIdx.x * 8 + (threadIdx.x >> 5); j < n; j += gridDim.x * 8) {
-    const uint4* src = cache + (static_cast<long long>(table[j / block_size]) * block_size + j % block_size) * vec;
+    const int at = start + j;
+    const uint4* src = cache + (static_cast<long long>(table[at / block_size]) * block_size + at % block_size) * vec;
     uint4* dst = out + static_cast<long long>(j) * vec;
     for (int c = lane; c < vec; c += 32) dst[c] = src[c];
+  }
+}
+
+// x[r, c] *= sigmoid(gate[r, c]), four columns per thread
+template <typename T>
+__global__ void __launch_bounds__(256) gate_columns_kernel(T* __restrict__ x, long long x_ld, const T* __restrict__ gate,
+                                                           long long gate_ld, int rows, int vec) {
+  pdl_launch_dependents();
+  pdl_wait();
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < static_cast<long long>(rows) * vec;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const long long r = i / vec;
+    const int c = static_cast<int>(i - r * vec) * 4;
+    float4 v = ld4(x + r * x_ld + c);
+    const float4 g = ld4(gate + r * gate_ld + c);
+    v.x /= 1.f + expf(-g.x); v.y /= 1.f + expf(-g.y); v.z /= 1.f + expf(-g.z); v.w /= 1.f + expf(-g.w);
+    st4(x + r * x_ld + c, v);
   }
 }
 
@@ -112,7 +134,8 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const uint4* __restr
 
 using namespace gk;
 
-// ptrs: {proj, gain, turns, pos, slots, cache, context, row_seq, cu_ctx}; context null: single tokens only
+// ptrs: {proj, gain, turns, pos, slots, cache, context, row_seq, cu_ctx, ctx_start}; context null: single tokens only;
+// ctx_start null: contexts start at position 0
 // dims: {rows, context_rows, q_off, q_hs, q_rot, d_off, H, C, CV, rot, DR}
 GK_EXPORT int gk_latent_prep(int is_fp32, void* const* ptrs, long long ld, const int* dims, float eps, float magnitude,
                              void* stream) {
@@ -132,6 +155,7 @@ GK_EXPORT int gk_latent_prep(int is_fp32, void* const* ptrs, long long ld, const
     p.context = static_cast<T*>(ptrs[6]);
     p.row_seq = static_cast<const int*>(ptrs[7]);
     p.cu_ctx = static_cast<const int*>(ptrs[8]);
+    p.ctx_start = static_cast<const int*>(ptrs[9]);
     p.rows = dims[0]; p.context_rows = dims[1]; p.q_off = dims[2]; p.q_hs = dims[3]; p.q_rot = dims[4]; p.d_off = dims[5];
     p.H = dims[6]; p.C = dims[7]; p.CV = dims[8]; p.rot = dims[9]; p.DR = dims[10];
     p.eps = eps; p.magnitude = magnitude;
@@ -141,15 +165,35 @@ GK_EXPORT int gk_latent_prep(int is_fp32, void* const* ptrs, long long ld, const
   return is_fp32 ? fill(static_cast<float*>(nullptr)) : fill(static_cast<__nv_bfloat16*>(nullptr));
 }
 
-// Rows 0 .. first_pos[b] - 1 of every portion's request from the paged cache to its context.
-GK_EXPORT int gk_latent_gather(const void* cache, const int* tables, const int* first_pos, const int* cu_ctx, void* context,
-                               int portions, int max_blocks, int block_size, int row_bytes, int max_first, void* stream) {
+// Rows ctx_start[b] (null: 0) .. first_pos[b] - 1 of every portion's request from the paged cache to its context; max_rows
+// bounds their number.
+GK_EXPORT int gk_latent_gather(const void* cache, const int* tables, const int* first_pos, const int* cu_ctx,
+                               const int* ctx_start, void* context, int portions, int max_blocks, int block_size,
+                               int row_bytes, int max_rows, void* stream) {
   if (row_bytes % 16) return -1;
-  if (portions == 0 || max_first == 0) return 0;
-  int blocks = (max_first + 7) / 8;
+  if (portions == 0 || max_rows == 0) return 0;
+  int blocks = (max_rows + 7) / 8;
   if (blocks > sm_count() * 4) blocks = sm_count() * 4;
   launch_k(latent_gather_kernel, dim3(blocks, portions), dim3(256), 0, reinterpret_cast<cudaStream_t>(stream),
-           static_cast<const uint4*>(cache), tables, max_blocks, block_size, first_pos, cu_ctx, static_cast<uint4*>(context),
-           row_bytes / 16);
+           static_cast<const uint4*>(cache), tables, max_blocks, block_size, first_pos, cu_ctx, ctx_start,
+           static_cast<uint4*>(context), row_bytes / 16);
+  return launch_status();
+}
+
+// Columns, strides: multiples of 4 elements, rows 8- (bf16) or 16-byte (32-bit) aligned.
+GK_EXPORT int gk_gate_columns(int is_fp32, void* x, long long x_ld, const void* gate, long long gate_ld, int rows, int cols,
+                              void* stream) {
+  if (cols % 4 || x_ld % 4 || gate_ld % 4) return -1;
+  if (rows == 0 || cols == 0) return 0;
+  long long blocks = (static_cast<long long>(rows) * (cols / 4) + 255) / 256;
+  if (blocks > sm_count() * 8) blocks = sm_count() * 8;
+  const dim3 grid(static_cast<unsigned>(blocks)), block(256);
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  if (is_fp32)
+    launch_k(gate_columns_kernel<float>, grid, block, 0, st, static_cast<float*>(x), x_ld, static_cast<const float*>(gate),
+             gate_ld, rows, cols / 4);
+  else
+    launch_k(gate_columns_kernel<__nv_bfloat16>, grid, block, 0, st, static_cast<__nv_bfloat16*>(x), x_ld,
+             static_cast<const __nv_bfloat16*>(gate), gate_ld, rows, cols / 4);
   return launch_status();
 }

@@ -14,7 +14,8 @@
 //     (Evaluating each exponential once and passing P through shared memory costs a third barrier per tile and
 //     measured 5 % slower: the kernel is bound by issue latency at two warps per scheduler, not by the exponentials.)
 // SPLIT instances keep the probabilities at 16 significant bits (two bf16 terms, rounded value and remainder), and any
-// instance can scale the output by a sigmoid gate per (request, head).
+// instance can scale the output by a sigmoid gate per (request, head), look at the last `window` positions only, and take a
+// learned logit per head (a sink) into the softmax denominator.
 // Stands in for the latent decode kernels the reference reaches through its serving engines and its own
 // gpatch_v4/models/deepseek_v4/kernel/flash_mla_wrapper.py:56-160.
 #include "host_utils.h"
@@ -86,6 +87,12 @@ __device__ __forceinline__ float gate_of(const __nv_bfloat16* gate, long long ga
   return gate ? 1.f / (1.f + __expf(-__bfloat162float(gate[b * gate_ld + h]))) : 1.f;
 }
 
+__device__ __forceinline__ int window_start(int len, int window) { return window > 0 && len > window ? len - window : 0; }
+// a head's softmax denominator with its sink's share; m: the maximum `l` is relative to
+__device__ __forceinline__ float with_sink(const float* sinks, int h, float l, float m) {
+  return sinks ? l + __expf(sinks[h] - m) : l;
+}
+
 // q_lat [B, H, CV] and q_rope [B, H, DR] and out [B, H, CV] are addressed through (batch, head) strides in elements,
 // so the batched projections around the kernel can keep their head-major layout.
 template <int CV, int DR, bool SPLIT>
@@ -94,7 +101,7 @@ __global__ void __launch_bounds__(THREADS, 2) mla_paged_decode_kernel(
     long long rs_b, long long rs_h, const __nv_bfloat16* __restrict__ cache, const int* __restrict__ block_table,
     int max_blocks, const int* __restrict__ ctx_len, __nv_bfloat16* __restrict__ out, long long os_b, long long os_h,
     float* __restrict__ scratch, int H, int block_size, float scale, int nsplit, int split_tokens,
-    const __nv_bfloat16* __restrict__ gate, long long gate_ld) {
+    const __nv_bfloat16* __restrict__ gate, long long gate_ld, int window, const float* __restrict__ sinks) {
   using G = Geo<CV, DR>;
   extern __shared__ __align__(128) uint8_t mla_smem[];
   uint8_t* sq = mla_smem;
@@ -105,7 +112,7 @@ __global__ void __launch_bounds__(THREADS, 2) mla_paged_decode_kernel(
   pdl_wait();
   const int b = blockIdx.x, hg = blockIdx.y, split = blockIdx.z;
   const int len = ctx_len[b];
-  const int s0 = split * split_tokens;
+  const int s0 = window_start(len, window) + split * split_tokens;
   if (split > 0 && s0 >= len) return;   // the combine kernel reads the live splits only
   int s1 = s0 + split_tokens;
   if (s1 > len) s1 = len;
@@ -299,7 +306,8 @@ __global__ void __launch_bounds__(THREADS, 2) mla_paged_decode_kernel(
     if (head >= H) continue;
     const int col0 = warp * G::COLS_PER_WARP + cq;
     if (nsplit == 1) {
-      const float inv = l_run[h] > 0.f ? gate_of(gate, gate_ld, b, head) / l_run[h] : 0.f;
+      const float l = with_sink(sinks, head, l_run[h], m_run[h]);
+      const float inv = l > 0.f ? gate_of(gate, gate_ld, b, head) / l : 0.f;
       __nv_bfloat16* dst = out + b * os_b + head * os_h + col0;
 #pragma unroll
       for (int j = 0; j < G::NT; ++j) {
@@ -323,14 +331,15 @@ constexpr int COMBINE_THREADS = 256;
 __global__ void __launch_bounds__(COMBINE_THREADS) mla_decode_combine_kernel(
     const float* __restrict__ scratch, const int* __restrict__ ctx_len, __nv_bfloat16* __restrict__ out, long long os_b,
     long long os_h, int H, int CV, int nsplit_total, int split_tokens, const __nv_bfloat16* __restrict__ gate,
-    long long gate_ld) {
+    long long gate_ld, int window, const float* __restrict__ sinks) {
   __shared__ float s_w[COMBINE_THREADS];
   __shared__ float s_red[COMBINE_THREADS / 32];
   pdl_launch_dependents();
   pdl_wait();
   const int b = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
   const float* base = scratch + (static_cast<long long>(b) * H + h) * nsplit_total * (CV + 2);
-  int nsplit = (ctx_len[b] + split_tokens - 1) / split_tokens;
+  const int len = ctx_len[b];
+  int nsplit = (len - window_start(len, window) + split_tokens - 1) / split_tokens;
   if (nsplit < 1) nsplit = 1;
   if (nsplit > nsplit_total) nsplit = nsplit_total;       // at most COMBINE_THREADS (plan)
   const float ms = tid < nsplit ? base[static_cast<long long>(tid) * (CV + 2) + CV] : -FLT_MAX;
@@ -353,6 +362,7 @@ __global__ void __launch_bounds__(COMBINE_THREADS) mla_decode_combine_kernel(
   l = 0.f;
 #pragma unroll
   for (int w = 0; w < COMBINE_THREADS / 32; ++w) l += s_red[w];
+  l = with_sink(sinks, h, l, m);
   const float inv = l > 0.f ? gate_of(gate, gate_ld, b, h) / l : 0.f;
   for (int d = tid * 2; d < CV; d += COMBINE_THREADS * 2) {
     float2 acc = make_float2(0.f, 0.f);
@@ -388,7 +398,8 @@ template <int CV, int DR, bool SPLIT>
 static int launch(const void* q_lat, long long qs_b, long long qs_h, const void* q_rope, long long rs_b,
                   long long rs_h, const void* cache, const int* block_table, int max_blocks, const int* ctx_len,
                   void* out, long long os_b, long long os_h, float* scratch, int B, int H, int block_size, float scale,
-                  int nsplit, int split_tokens, const __nv_bfloat16* gate, long long gate_ld, cudaStream_t st) {
+                  int nsplit, int split_tokens, const __nv_bfloat16* gate, long long gate_ld, int window,
+                  const float* sinks, cudaStream_t st) {
   using G = Geo<CV, DR>;
   static bool configured = false;
   if (!configured) {
@@ -399,7 +410,7 @@ static int launch(const void* q_lat, long long qs_b, long long qs_h, const void*
            reinterpret_cast<const __nv_bfloat16*>(q_lat), qs_b, qs_h, reinterpret_cast<const __nv_bfloat16*>(q_rope),
            rs_b, rs_h, reinterpret_cast<const __nv_bfloat16*>(cache), block_table, max_blocks, ctx_len,
            reinterpret_cast<__nv_bfloat16*>(out), os_b, os_h, scratch, H, block_size, scale, nsplit, split_tokens, gate,
-           gate_ld);
+           gate_ld, window, sinks);
   return 0;
 }
 
@@ -423,15 +434,16 @@ GK_EXPORT void gk_mla_decode_scratch(int B, int H, int CV, int max_ctx, long lon
 static int decode(const void* q_lat, long long qs_b, long long qs_h, const void* q_rope, long long rs_b, long long rs_h,
                   const void* cache, const int* block_table, const int* ctx_len, void* out, long long os_b, long long os_h,
                   float* scratch, int B, int H, int CV, int DR, int block_size, int max_blocks, int max_ctx, float scale,
-                  bool split, const __nv_bfloat16* gate, long long gate_ld, cudaStream_t st) {
+                  bool split, const __nv_bfloat16* gate, long long gate_ld, int window, const float* sinks,
+                  cudaStream_t st) {
   if (!gk_mla_decode_supported(CV, DR)) return -1;
   if ((qs_b | qs_h | rs_b | rs_h) % 8 || (os_b | os_h) % 2) return -3;
   if (B == 0 || H == 0) return 0;
   int nsplit, split_tokens;
-  plan(B, H, max_ctx, &nsplit, &split_tokens);
+  plan(B, H, window > 0 && window < max_ctx ? window : max_ctx, &nsplit, &split_tokens);
   if (nsplit > 1 && !scratch) return -2;
 #define GK_MLA_ARGS q_lat, qs_b, qs_h, q_rope, rs_b, rs_h, cache, block_table, max_blocks, ctx_len, out, os_b, os_h, \
-                    scratch, B, H, block_size, scale, nsplit, split_tokens, gate, gate_ld, st
+                    scratch, B, H, block_size, scale, nsplit, split_tokens, gate, gate_ld, window, sinks, st
 #define GK_MLA_LAUNCH(cv, dr) (split ? launch<cv, dr, true>(GK_MLA_ARGS) : launch<cv, dr, false>(GK_MLA_ARGS))
   if (CV == 512) GK_MLA_LAUNCH(512, 64);
   else if (CV == 256) GK_MLA_LAUNCH(256, 64);
@@ -440,7 +452,8 @@ static int decode(const void* q_lat, long long qs_b, long long qs_h, const void*
 #undef GK_MLA_ARGS
   if (nsplit > 1) {
     launch_k(mla_decode_combine_kernel, dim3(B, H), dim3(COMBINE_THREADS), 0, st, static_cast<const float*>(scratch), ctx_len,
-             reinterpret_cast<__nv_bfloat16*>(out), os_b, os_h, H, CV, nsplit, split_tokens, gate, gate_ld);
+             reinterpret_cast<__nv_bfloat16*>(out), os_b, os_h, H, CV, nsplit, split_tokens, gate, gate_ld,
+             window, sinks);
   }
   return launch_status();
 }
@@ -452,16 +465,18 @@ GK_EXPORT int gk_mla_paged_decode(const void* q_lat, long long qs_b, long long q
                                   int B, int H, int CV, int DR, int block_size, int max_blocks, int max_ctx,
                                   float scale, void* stream) {
   return decode(q_lat, qs_b, qs_h, q_rope, rs_b, rs_h, cache, block_table, ctx_len, out, os_b, os_h, scratch, B, H, CV, DR,
-                block_size, max_blocks, max_ctx, scale, false, nullptr, 0, reinterpret_cast<cudaStream_t>(stream));
+                block_size, max_blocks, max_ctx, scale, false, nullptr, 0, 0, nullptr, reinterpret_cast<cudaStream_t>(stream));
 }
 
-// The same with 32-bit-like probabilities (two bf16 terms) and a gate: logits [B, gate_ld], one per head, or null.
+// The same with 32-bit-like probabilities (two bf16 terms), a gate (logits [B, gate_ld], one per head, or null), a window
+// (0: none; the scratch may then be sized for max_ctx = window) and sinks [H] (or null).
 GK_EXPORT int gk_mla_paged_decode_gated(const void* q_lat, long long qs_b, long long qs_h, const void* q_rope,
                                         long long rs_b, long long rs_h, const void* cache, const int* block_table,
                                         const int* ctx_len, void* out, long long os_b, long long os_h, float* scratch,
                                         int B, int H, int CV, int DR, int block_size, int max_blocks, int max_ctx,
-                                        float scale, const void* gate, long long gate_ld, void* stream) {
+                                        float scale, const void* gate, long long gate_ld, int window,
+                                        const float* sinks, void* stream) {
   return decode(q_lat, qs_b, qs_h, q_rope, rs_b, rs_h, cache, block_table, ctx_len, out, os_b, os_h, scratch, B, H, CV, DR,
                 block_size, max_blocks, max_ctx, scale, true, static_cast<const __nv_bfloat16*>(gate), gate_ld,
-                reinterpret_cast<cudaStream_t>(stream));
+                window, sinks, reinterpret_cast<cudaStream_t>(stream));
 }

@@ -16,7 +16,7 @@
 namespace gkr {
 
 constexpr int MAX_K = 16;
-constexpr int MAX_G = 8;
+constexpr int MAX_G = 32;   // a lane per group
 
 struct RouterParams {
   const float* logits;      // [T, E]
@@ -88,12 +88,10 @@ __device__ __forceinline__ void route_token(const RouterParams& p, long long t, 
     for (int i = 0; i < VPT; ++i)
       sel[i] = lane + 32 * i < p.E ? sc[i] + (p.bias ? p.bias[lane + 32 * i] : 0.f) : -FLT_MAX;
     if (p.G > 1) {
-      // group score = sum of the two best selection scores inside the group
+      // group score = sum of the two best selection scores inside the group (of the only one in a group of one)
       const int gs = p.E / p.G;
-      float gscore[MAX_G];
-#pragma unroll
-      for (int g = 0; g < MAX_G; ++g) {
-        if (g >= p.G) break;
+      float mine = -FLT_MAX;               // lane g: score of group g
+      for (int g = 0; g < p.G; ++g) {
         float a = -FLT_MAX, b = -FLT_MAX;  // a >= b
 #pragma unroll
         for (int i = 0; i < VPT; ++i) {
@@ -109,20 +107,18 @@ __device__ __forceinline__ void route_token(const RouterParams& p, long long t, 
           const float nb = fmaxf(fminf(a, oa), fmaxf(b, ob));
           a = na; b = nb;
         }
-        gscore[g] = a + b;
+        if (lane == g) mine = gs > 1 ? a + b : a;
       }
+      int rank = 0;
+      for (int g = 0; g < p.G; ++g) {
+        const float other = __shfl_sync(0xffffffffu, mine, g);
+        rank += (other > mine || (other == mine && g < lane)) ? 1 : 0;
+      }
+      const unsigned kept = __ballot_sync(0xffffffffu, lane < p.G && rank < p.topk_group);
 #pragma unroll
-      for (int g = 0; g < MAX_G; ++g) {
-        if (g >= p.G) break;
-        int rank = 0;
-#pragma unroll
-        for (int h = 0; h < MAX_G; ++h)
-          if (h < p.G) rank += (gscore[h] > gscore[g] || (gscore[h] == gscore[g] && h < g)) ? 1 : 0;
-        if (rank >= p.topk_group) {
-#pragma unroll
-          for (int i = 0; i < VPT; ++i)
-            if ((lane + 32 * i) / gs == g) sel[i] = -FLT_MAX;
-        }
+      for (int i = 0; i < VPT; ++i) {
+        const int g = (lane + 32 * i) / gs;
+        if (g >= p.G || !((kept >> g) & 1u)) sel[i] = -FLT_MAX;
       }
     }
 #pragma unroll
@@ -321,10 +317,13 @@ int dispatch_vpt(int E, const P& p, F launch) {
 
 using namespace gkr;
 
+static bool router_valid(const RouterParams& p) {
+  return p.E >= 1 && p.K >= 1 && p.K <= MAX_K && p.K <= p.E && p.G >= 1 && p.G <= MAX_G && p.E % p.G == 0 &&
+         (p.G == 1 || (p.topk_group >= 1 && p.topk_group <= p.G));
+}
+
 static int router_launch(const RouterParams& p, cudaStream_t st) {
-  if (p.E < 1 || p.K < 1 || p.K > MAX_K || p.K > p.E || p.G < 1 || p.G > MAX_G || p.E % p.G ||
-      (p.G > 1 && (p.topk_group < 1 || p.topk_group > p.G)))
-    return -1;
+  if (!router_valid(p)) return -1;
   const unsigned blocks = static_cast<unsigned>((p.T + 7) / 8);
   return dispatch_vpt(p.E, p, [&](auto v) {
     gk::launch_k(router_fwd_kernel<decltype(v)::value>, dim3(blocks), dim3(256), 0, st, p);
@@ -332,7 +331,7 @@ static int router_launch(const RouterParams& p, cudaStream_t st) {
   });
 }
 
-// E <= 512; K <= 16; G <= 8 and E % G == 0.  Returns -2 for an expert count without a kernel.
+// E <= 512; K <= 16; G <= 32 and E % G == 0.  Returns -2 for an expert count without a kernel.
 GK_EXPORT int gk_router_fwd(const float* logits, const float* bias, const long long* replay, long long* idx, float* w,
                             long long T, int E, int K, int G, int topk_group, int sigmoid, int norm, float scale,
                             void* stream) {
@@ -347,12 +346,13 @@ GK_EXPORT int gk_router_fwd(const float* logits, const float* bias, const long l
 // Routing of served models: logits rows `ld` floats apart, and the dispatch bookkeeping in the same launch (counts [E],
 // cleared by the caller, and every choice's place [T, K] among its expert's tokens; the places' order is not fixed).
 GK_EXPORT int gk_router_dispatch(const float* logits, long long ld, const float* bias, long long* idx, float* w, int* counts,
-                                 int* place, long long T, int E, int K, int sigmoid, int norm, float scale, void* stream) {
+                                 int* place, long long T, int E, int K, int sigmoid, int norm, float scale, int G,
+                                 int topk_group, void* stream) {
   if (T <= 0) return 0;
   if (ld < E || !counts || !place) return -1;
   RouterParams p;
-  p.logits = logits; p.bias = bias; p.replay = nullptr; p.idx = idx; p.w = w; p.T = T; p.E = E; p.K = K; p.G = 1;
-  p.topk_group = 1; p.sigmoid = sigmoid; p.norm = norm; p.scale = scale;
+  p.logits = logits; p.bias = bias; p.replay = nullptr; p.idx = idx; p.w = w; p.T = T; p.E = E; p.K = K; p.G = G;
+  p.topk_group = topk_group; p.sigmoid = sigmoid; p.norm = norm; p.scale = scale;
   p.ld = ld; p.counts = counts; p.place = place;
   return router_launch(p, reinterpret_cast<cudaStream_t>(stream));
 }
@@ -361,14 +361,14 @@ GK_EXPORT int gk_router_dispatch(const float* logits, long long ld, const float*
 // logits [T, n_rows].
 GK_EXPORT int gk_router_fused(int is_fp32, const void* h, const void* w, float* logits, int H, int n_rows, const float* bias,
                               long long* idx, float* weight, int* counts, int* place, long long T, int E, int K, int sigmoid,
-                              int norm, float scale, void* stream) {
+                              int norm, float scale, int G, int topk_group, void* stream) {
   if (T <= 0) return 0;
-  if (n_rows < E || n_rows > RF_MAX_ROWS || H % 8 || H > 11264 || !counts || !place || E < 1 || K < 1 || K > MAX_K || K > E)
-    return -1;
+  if (n_rows < E || n_rows > RF_MAX_ROWS || H % 8 || H > 11264 || !counts || !place) return -1;
   RouterParams p;
-  p.logits = logits; p.bias = bias; p.replay = nullptr; p.idx = idx; p.w = weight; p.T = T; p.E = E; p.K = K; p.G = 1;
-  p.topk_group = 1; p.sigmoid = sigmoid; p.norm = norm; p.scale = scale;
+  p.logits = logits; p.bias = bias; p.replay = nullptr; p.idx = idx; p.w = weight; p.T = T; p.E = E; p.K = K; p.G = G;
+  p.topk_group = topk_group; p.sigmoid = sigmoid; p.norm = norm; p.scale = scale;
   p.ld = n_rows; p.counts = counts; p.place = place;
+  if (!router_valid(p)) return -1;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   return dispatch_vpt(E, p, [&](auto v) {
     constexpr int VPT = decltype(v)::value;

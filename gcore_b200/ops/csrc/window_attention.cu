@@ -3,8 +3,9 @@
 //   * append_keys_kernel      copies the new keys of a packed projection into their cache slots;
 //   * window_attn_kernel      any row (prompt portion or decoded token), any head size, 32-bit or bf16 storage, one warp
 //                             per (row, head): the true 32-bit path and the sizes the tensor-core kernels do not cover.
-//                             The value may be the first columns of the key row only, and window, penalty and an output
-//                             gate are optional, so absorbed latent attention runs on it too;
+//                             Keys and values may lie anywhere in a cached row and several keys may share a value, and
+//                             window, penalty, sink and output gate are optional, so absorbed latent attention and
+//                             differential attention run on it too;
 //   * shared_kv_decode_kernel one new token per request, bf16, head sizes 64 and 128: mma.sync tiles with the query heads
 //                             of a group as rows (a group is far below the 64-row minimum of a tcgen05 instruction), KV
 //                             splits, append of the new key fused in.
@@ -14,6 +15,7 @@
 #include "host_utils.h"
 #include <cuda_bf16.h>
 #include <float.h>
+#include <type_traits>
 
 namespace gk {
 
@@ -41,72 +43,91 @@ __global__ void append_keys_kernel(const uint4* __restrict__ proj, long long ld_
 constexpr int WA_WARPS = 8;
 constexpr int WA_MAX_D = 1024;
 
-// One warp per (row, query head).  slots[row] < 0 marks an inactive row (zero output).  D: key columns, DV <= D: value
-// columns (DV <= 32 * NR); window 0: unlimited; slopes, gate (one logit per row and head, rows gate_ld apart): or null.
-template <typename T, int NR>
-__global__ void __launch_bounds__(WA_WARPS * 32) window_attn_kernel(
-    const T* __restrict__ q, long long q_ld, const T* __restrict__ cache, const int* __restrict__ tables, int max_blocks,
-    int block_size, const int* __restrict__ row_seq, const int* __restrict__ pos, const int* __restrict__ slots,
-    const float* __restrict__ slopes, const T* __restrict__ gate, long long gate_ld, T* __restrict__ out, int rows, int H,
-    int G, int D, int DV, int window, float scale) {
+template <typename T, typename O>
+struct WindowAttnParams {
+  const T* q;               // head h of a row at h * D
+  long long q_ld;
+  const T* cache;           // rows of `cache_row` elements: key kh at kh * D, value g at v_off + g * v_stride
+  long long cache_row;
+  int v_off, v_stride;
+  const int *tables, *row_seq, *pos, *slots;   // slots[row] < 0 marks an inactive row (zero output)
+  int max_blocks, block_size;
+  const float* slopes;      // [H] or null
+  const float* sinks;       // [H] or null: a logit that joins the softmax denominator
+  const T* gate;            // one logit per row and head, rows gate_ld apart, or null
+  long long gate_ld;
+  O* out;                   // [rows, H, DV]
+  int rows, H, G, maps;     // H query heads over G values, `maps` keys per value: head h takes key (g, h % maps)
+  int D, DV, window;        // window 0: unlimited
+  float scale;
+};
+
+// One warp per (row, query head); DV <= 32 * NR.
+template <typename T, typename O, int NR>
+__global__ void __launch_bounds__(WA_WARPS * 32) window_attn_kernel(const WindowAttnParams<T, O> p) {
   extern __shared__ float wa_q[];
   pdl_launch_dependents();
   pdl_wait();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, D = p.D, DV = p.DV;
   const long long item = static_cast<long long>(blockIdx.x) * WA_WARPS + warp;
-  if (item >= static_cast<long long>(rows) * H) return;
-  const int row = static_cast<int>(item / H), h = static_cast<int>(item - static_cast<long long>(row) * H);
-  T* orow = out + (static_cast<long long>(row) * H + h) * DV;
+  if (item >= static_cast<long long>(p.rows) * p.H) return;
+  const int row = static_cast<int>(item / p.H), h = static_cast<int>(item - static_cast<long long>(row) * p.H);
+  O* orow = p.out + (static_cast<long long>(row) * p.H + h) * DV;
   float acc[NR];
 #pragma unroll
   for (int r = 0; r < NR; ++r) acc[r] = 0.f;
   float m = -FLT_MAX, l = 0.f;
-  if (slots[row] >= 0) {
+  if (p.slots[row] >= 0) {
+    if (p.sinks) {
+      m = p.sinks[h];
+      l = lane == 0 ? 1.f : 0.f;
+    }
     float* sq = wa_q + warp * D;
-    const T* qr = q + row * q_ld + static_cast<long long>(h) * D;
+    const T* qr = p.q + row * p.q_ld + static_cast<long long>(h) * D;
     for (int d = lane; d < D; d += 32) sq[d] = wa_f(qr[d]);
     __syncwarp();
-    const int g = h / (H / G), i = pos[row];
-    const int* table = tables + static_cast<long long>(row_seq[row]) * max_blocks;
-    const float slope = slopes ? slopes[h] : 0.f;
-    int j0 = window > 0 ? i - window + 1 : 0;
+    const int g = h / (p.H / p.G), i = p.pos[row];
+    const long long k_off = static_cast<long long>(g * p.maps + h % p.maps) * D;
+    const long long v_off = p.v_off + static_cast<long long>(g) * p.v_stride;
+    const int* table = p.tables + static_cast<long long>(p.row_seq[row]) * p.max_blocks;
+    const float slope = p.slopes ? p.slopes[h] : 0.f;
+    int j0 = p.window > 0 ? i - p.window + 1 : 0;
     if (j0 < 0) j0 = 0;
     for (int base = j0; base <= i; base += 32) {
       const int j = base + lane;
       const int nt = i + 1 - base < 32 ? i + 1 - base : 32;
       float s = -FLT_MAX;
-      long long koff = 0;
+      long long at = 0;
       if (j <= i) {
-        const long long slot = static_cast<long long>(table[j / block_size]) * block_size + j % block_size;
-        koff = (slot * G + g) * D;
-        const T* kr = cache + koff;
+        at = (static_cast<long long>(table[j / p.block_size]) * p.block_size + j % p.block_size) * p.cache_row;
+        const T* kr = p.cache + at + k_off;
         float a = 0.f;
         for (int d = 0; d < D; ++d) a = fmaf(sq[d], wa_f(kr[d]), a);
-        s = a * scale - slope * static_cast<float>(i - j);
+        s = a * p.scale - slope * static_cast<float>(i - j);
       }
       float mx = s;
 #pragma unroll
       for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffff, mx, o));
       const float mn = fmaxf(m, mx);
       const float c = expf(m - mn);            // 0 on the first tile (m = -FLT_MAX)
-      const float p = j <= i ? expf(s - mn) : 0.f;
+      const float e = j <= i ? expf(s - mn) : 0.f;
       m = mn;
-      l = l * c + p;
+      l = l * c + e;
 #pragma unroll
       for (int r = 0; r < NR; ++r) acc[r] *= c;
       for (int t = 0; t < nt; ++t) {
-        const float pt = __shfl_sync(0xffffffff, p, t);
-        const T* kr = cache + __shfl_sync(0xffffffff, koff, t);
+        const float pt = __shfl_sync(0xffffffff, e, t);
+        const T* vr = p.cache + __shfl_sync(0xffffffff, at, t) + v_off;
 #pragma unroll
         for (int r = 0; r < NR; ++r)
-          if (r * 32 + lane < DV) acc[r] = fmaf(pt, wa_f(kr[r * 32 + lane]), acc[r]);
+          if (r * 32 + lane < DV) acc[r] = fmaf(pt, wa_f(vr[r * 32 + lane]), acc[r]);
       }
     }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffff, l, o);
   }
   float inv = l > 0.f ? 1.f / l : 0.f;
-  if (gate) inv /= 1.f + expf(-wa_f(gate[row * gate_ld + h]));
+  if (p.gate) inv /= 1.f + expf(-wa_f(p.gate[row * p.gate_ld + h]));
 #pragma unroll
   for (int r = 0; r < NR; ++r)
     if (r * 32 + lane < DV) wa_st(orow + r * 32 + lane, acc[r] * inv);
@@ -387,33 +408,15 @@ __global__ void shared_kv_combine_kernel(const float* __restrict__ scratch, cons
   out[(static_cast<long long>(b) * H + h) * D + d] = __float2bfloat16(l > 0.f ? acc / l : 0.f);
 }
 
-struct WindowAttnArgs {
-  const void* q;
-  long long q_ld;
-  const void* cache;
-  const int *tables, *row_seq, *pos, *slots;
-  const float* slopes;
-  const void* gate;
-  long long gate_ld;
-  void* out;
-  int rows, H, G, D, DV, window, block_size, max_blocks;
-  float scale;
-};
-
-template <typename T, int NR>
-int launch_window_attn(const WindowAttnArgs& a, cudaStream_t st) {
-  const long long items = static_cast<long long>(a.rows) * a.H;
-  launch_k(window_attn_kernel<T, NR>, dim3(static_cast<unsigned>((items + WA_WARPS - 1) / WA_WARPS)), dim3(WA_WARPS * 32),
-           WA_WARPS * a.D * sizeof(float), st, static_cast<const T*>(a.q), a.q_ld, static_cast<const T*>(a.cache), a.tables,
-           a.max_blocks, a.block_size, a.row_seq, a.pos, a.slots, a.slopes, static_cast<const T*>(a.gate), a.gate_ld,
-           static_cast<T*>(a.out), a.rows, a.H, a.G, a.D, a.DV, a.window, a.scale);
+template <typename T, typename O>
+int launch_window_attn(const WindowAttnParams<T, O>& p, cudaStream_t st) {
+  const long long items = static_cast<long long>(p.rows) * p.H;
+  const dim3 grid(static_cast<unsigned>((items + WA_WARPS - 1) / WA_WARPS)), block(WA_WARPS * 32);
+  const size_t smem = WA_WARPS * p.D * sizeof(float);
+  if (p.DV <= 128) launch_k(window_attn_kernel<T, O, 4>, grid, block, smem, st, p);
+  else if (p.DV <= 512) launch_k(window_attn_kernel<T, O, 16>, grid, block, smem, st, p);
+  else launch_k(window_attn_kernel<T, O, 32>, grid, block, smem, st, p);
   return launch_status();
-}
-
-inline int window_attn(bool f32, const WindowAttnArgs& a, cudaStream_t st) {
-  if (a.DV <= 128) return f32 ? launch_window_attn<float, 4>(a, st) : launch_window_attn<__nv_bfloat16, 4>(a, st);
-  if (a.DV <= 512) return f32 ? launch_window_attn<float, 16>(a, st) : launch_window_attn<__nv_bfloat16, 16>(a, st);
-  return f32 ? launch_window_attn<float, 32>(a, st) : launch_window_attn<__nv_bfloat16, 32>(a, st);
 }
 
 // Splits the window so that the grid about fills the GPU once, never finer than 128 tokens.
@@ -479,21 +482,36 @@ GK_EXPORT int gk_append_keys(const void* proj, long long ld_bytes, long long off
   return launch_status();
 }
 
-// ptrs: {q, cache, tables, row_seq, pos, slots, slopes, gate, out}; slopes, gate: or null
-// dims: {rows, H, G, D, DV, window, block_size, max_blocks}; window 0: unlimited
-GK_EXPORT int gk_window_attn(int is_fp32, void* const* ptrs, long long q_ld, long long gate_ld, const int* dims, float scale,
+// ptrs: {q, cache, tables, row_seq, pos, slots, slopes, gate, out, sinks}; slopes, gate, sinks: or null
+// lds: {q_ld, gate_ld, cache_row};  window 0: unlimited;  out_fp32: 32-bit output of bf16 rows
+// dims: {rows, H, G, maps, D, DV, v_off, v_stride, window, block_size, max_blocks}
+GK_EXPORT int gk_window_attn(int is_fp32, int out_fp32, void* const* ptrs, const long long* lds, const int* dims, float scale,
                              void* stream) {
-  WindowAttnArgs a;
-  a.q = ptrs[0]; a.q_ld = q_ld; a.cache = ptrs[1];
-  a.tables = static_cast<const int*>(ptrs[2]); a.row_seq = static_cast<const int*>(ptrs[3]);
-  a.pos = static_cast<const int*>(ptrs[4]); a.slots = static_cast<const int*>(ptrs[5]);
-  a.slopes = static_cast<const float*>(ptrs[6]);
-  a.gate = ptrs[7]; a.gate_ld = gate_ld; a.out = ptrs[8];
-  a.rows = dims[0]; a.H = dims[1]; a.G = dims[2]; a.D = dims[3]; a.DV = dims[4]; a.window = dims[5];
-  a.block_size = dims[6]; a.max_blocks = dims[7]; a.scale = scale;
-  if (a.G < 1 || a.H % a.G || a.D > WA_MAX_D || a.DV < 1 || a.DV > a.D || a.window < 0) return -1;
-  if (a.rows == 0) return 0;
-  return window_attn(is_fp32 != 0, a, reinterpret_cast<cudaStream_t>(stream));
+  const int H = dims[1], G = dims[2], maps = dims[3], D = dims[4], DV = dims[5];
+  if (G < 1 || H % G || maps < 1 || (H / G) % maps || D < 1 || D > WA_MAX_D || DV < 1 || DV > WA_MAX_D || dims[8] < 0)
+    return -1;
+  if (static_cast<long long>(G) * maps * D > lds[2] || dims[6] + static_cast<long long>(G - 1) * dims[7] + DV > lds[2])
+    return -1;
+  if (dims[0] == 0) return 0;
+  auto fill = [&](auto* tag, auto* otag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    using O = std::remove_pointer_t<decltype(otag)>;
+    WindowAttnParams<T, O> p;
+    p.q = static_cast<const T*>(ptrs[0]); p.q_ld = lds[0];
+    p.cache = static_cast<const T*>(ptrs[1]); p.cache_row = lds[2];
+    p.v_off = dims[6]; p.v_stride = dims[7];
+    p.tables = static_cast<const int*>(ptrs[2]); p.row_seq = static_cast<const int*>(ptrs[3]);
+    p.pos = static_cast<const int*>(ptrs[4]); p.slots = static_cast<const int*>(ptrs[5]);
+    p.max_blocks = dims[10]; p.block_size = dims[9];
+    p.slopes = static_cast<const float*>(ptrs[6]); p.sinks = static_cast<const float*>(ptrs[9]);
+    p.gate = static_cast<const T*>(ptrs[7]); p.gate_ld = lds[1];
+    p.out = static_cast<O*>(ptrs[8]);
+    p.rows = dims[0]; p.H = H; p.G = G; p.maps = maps; p.D = D; p.DV = DV; p.window = dims[8]; p.scale = scale;
+    return launch_window_attn(p, reinterpret_cast<cudaStream_t>(stream));
+  };
+  float* f = nullptr;
+  __nv_bfloat16* h = nullptr;
+  return is_fp32 ? fill(f, f) : out_fp32 ? fill(h, f) : fill(h, h);
 }
 
 GK_EXPORT void gk_shared_decode_set_target_ctas(int n) { shared_decode_target_ctas() = n > 0 ? n : 444; }

@@ -1,6 +1,6 @@
 """Latent attention over the rows of a serving step: a paged cache with one row ``[normed latent | rotated key part]`` per
 token, shared by all heads (``csrc/latent_attention.cu``, ``csrc/attention_fwd.cu``, ``csrc/mla_decode.cu``).  Prompt portions
-expand their whole context to per-head keys and values; single tokens work on the latent itself, with the up-projections
+expand the context they see to per-head keys and values; single tokens work on the latent itself, with the up-projections
 folded into query and output.  CPU tensors run the plain PyTorch definition."""
 from __future__ import annotations
 
@@ -53,6 +53,8 @@ class LatentLayout:
     scale: float
     magnitude: float
     eps: float
+    window: int = 0      # positions a token sees, itself included; 0: all before it
+    gate_cols: int = 1   # gate logits per head: one, or one per (padded) value column
 
     @property
     def row(self):
@@ -70,7 +72,7 @@ def _rotate(x, cos, sin):
     return torch.stack([u * cos - v * sin, v * cos + u * sin], -1).flatten(-2)
 
 
-def _ref(proj, ly: LatentLayout, gain, turns, up_kv, rows: StepRows, cache, out):
+def _ref(proj, ly: LatentLayout, gain, turns, up_kv, rows: StepRows, cache, out, sinks=None):
     T, H, bs = proj.shape[0], ly.heads, cache.shape[1]
     p = proj.float()
     a = 2 * math.pi * rows.pos.double()[:, None] * turns.double().sum(-1)
@@ -85,23 +87,27 @@ def _ref(proj, ly: LatentLayout, gain, turns, up_kv, rows: StepRows, cache, out)
     q = p[:, ly.q:ly.q + H * (ly.dim + ly.row_rot)].view(T, H, -1)
     qr = _rotate(q[..., ly.dim:ly.dim + ly.rot], cos[:, None], sin[:, None])
     uk, uv = up_kv[:H * ly.dim].float().view(H, ly.dim, -1), up_kv[H * ly.dim:].float().view(H, ly.vdim, -1)
-    g = torch.sigmoid(p[:, ly.gate:ly.gate + H])
+    g = torch.sigmoid(p[:, ly.gate:ly.gate + H * ly.gate_cols].view(T, H, -1))
     for t in range(T):
         if rows.slots[t] < 0:
             out[t] = 0
             continue
-        j = torch.arange(int(rows.pos[t]) + 1)
+        i = int(rows.pos[t])
+        j = torch.arange(max(0, i - ly.window + 1) if ly.window else 0, i + 1)
         ctx = flat[rows.tables[rows.row_seq[t], j // bs].long() * bs + j % bs].float()
         lat, rot = ctx[:, :ly.row_rank], ctx[:, ly.row_rank:ly.row_rank + ly.rot]
         s = (torch.einsum("hd,hdc,nc->hn", q[t, :, :ly.dim], uk, lat) + qr[t] @ rot.T) * ly.scale
-        o = torch.einsum("hn,nc,hvc->hv", torch.softmax(s, -1), lat, uv) * g[t][:, None]
+        w = torch.softmax(s if sinks is None else torch.cat([s, sinks[:, None]], 1), -1)[:, :len(j)]
+        o = torch.einsum("hn,nc,hvc->hv", w, lat, uv) * g[t]
         out[t] = o.reshape(-1).to(out.dtype)
     return out
 
 
 def _prep(proj, ly: LatentLayout, gain, turns, rows: StepRows, cache, context):
-    ptrs = (ctypes.c_void_p * 9)(*[t.data_ptr() if t is not None else None for t in
-                                   (proj, gain, turns, rows.pos, rows.slots, cache, context, rows.row_seq, rows.cu_ctx)])
+    ctx = rows.contexts[ly.window] if context is not None else None
+    ptrs = (ctypes.c_void_p * 10)(*[t.data_ptr() if t is not None else None for t in
+                                    (proj, gain, turns, rows.pos, rows.slots, cache, context, rows.row_seq,
+                                     ctx.cu if ctx else None, ctx.start if ctx else None)])
     dims = (ctypes.c_int * 11)(proj.shape[0], rows.portion_rows if context is not None else 0, ly.q, ly.dim + ly.row_rot,
                                ly.dim, ly.down, ly.heads, ly.rank, ly.row_rank, ly.rot, ly.row_rot)
     LAUNCHES["latent_attention"] += 1
@@ -109,21 +115,21 @@ def _prep(proj, ly: LatentLayout, gain, turns, rows: StepRows, cache, context):
                                              float(ly.magnitude), _lib.stream_ptr()), "latent_prep")
 
 
-def _portions(proj, ly: LatentLayout, up_kv, rows: StepRows, cache, context, out):
+def _portions(proj, ly: LatentLayout, up_kv, rows: StepRows, cache, context, out, sinks):
     """Prompt portions: the rest of the context from the cache, expansion, tcgen05 attention."""
-    lib, n = _lib.kernels(), rows.n_portions
-    if rows.max_first:
+    lib, n, ctx = _lib.kernels(), rows.n_portions, rows.contexts[ly.window]
+    if ctx.max_before:
         LAUNCHES["latent_attention"] += 1
-        _lib.check(lib.gk_latent_gather(_lib.ptr(cache), _lib.ptr(rows.tables), _lib.ptr(rows.first_pos),
-                                        _lib.ptr(rows.cu_ctx), _lib.ptr(context), n, rows.tables.shape[1], cache.shape[1],
-                                        ly.row * context.element_size(), rows.max_first, _lib.stream_ptr()), "latent_gather")
+        _lib.check(lib.gk_latent_gather(_lib.ptr(cache), _lib.ptr(rows.tables), _lib.ptr(rows.first_pos), _lib.ptr(ctx.cu),
+                                        _lib.ptr(ctx.start), _lib.ptr(context), n, rows.tables.shape[1], cache.shape[1],
+                                        ly.row * context.element_size(), ctx.max_before, _lib.stream_ptr()), "latent_gather")
     kv = linear_forward(context[:, :ly.row_rank], up_kv)
     q, kr, gate = proj[:, ly.q:], context[:, ly.row_rank:], proj[:, ly.gate:]
-    ptrs = (ctypes.c_void_p * 8)(*[t.data_ptr() for t in (q, kv, kr, gate, out, rows.cu, rows.cu_ctx,
-                                                          _lib.err_flag(proj.device))])
+    ptrs = (ctypes.c_void_p * 9)(*[t.data_ptr() if t is not None else None for t in
+                                   (q, kv, kr, gate, out, rows.cu, ctx.cu, _lib.err_flag(proj.device), sinks)])
     lds = (ctypes.c_longlong * 5)(proj.stride(0), kv.stride(0), context.stride(0), proj.stride(0), out.stride(0))
-    dims = (ctypes.c_int * 9)(n, rows.portion_rows, rows.ctx_rows, ly.heads, ly.dim, up8(ly.rot), ly.vdim,
-                              ly.dim + ly.row_rot, rows.max_portion)
+    dims = (ctypes.c_int * 11)(n, rows.portion_rows, ctx.rows, ly.heads, ly.dim, up8(ly.rot), ly.vdim,
+                               ly.dim + ly.row_rot, rows.max_portion, ly.window, ly.gate_cols)
     LAUNCHES["latent_attention"] += 1
     _lib.check(lib.gk_latent_prefill(ptrs, lds, dims, float(ly.scale), _lib.stream_ptr()), "latent_prefill")
 
@@ -149,7 +155,7 @@ def _decode_scratch(device, floats: int):
     return buf
 
 
-def _absorbed(proj, ly: LatentLayout, up_kv, rows: StepRows, lo: int, hi: int, cache, out):
+def _absorbed(proj, ly: LatentLayout, up_kv, rows: StepRows, lo: int, hi: int, cache, out, sinks):
     """Rows ``lo .. hi`` on the latent itself: query times key up-projection, attention over the cached rows, value
     up-projection.  Single tokens in bf16 take the decode kernel, everything else the general one."""
     T, H = hi - lo, ly.heads
@@ -158,45 +164,53 @@ def _absorbed(proj, ly: LatentLayout, up_kv, rows: StepRows, lo: int, hi: int, c
     uk, uv = up_kv[:H * ly.dim].view(H, ly.dim, -1), up_kv[H * ly.dim:].view(H, ly.vdim, -1)
     kw = dict(dtype=proj.dtype, device=proj.device)
     lib = _lib.kernels()
+    gate = p[:, ly.gate:]
+    head_gate = gate if ly.gate_cols == 1 else None     # the attention kernels apply one per head themselves
     if lo == rows.portion_rows and proj.dtype == torch.bfloat16 and lib.gk_mla_decode_supported(ly.row_rank, ly.row_rot):
         q_lat = _bmm(q[..., :ly.dim].transpose(0, 1), uk, torch.empty(H, T, ly.row_rank, **kw))
         o_lat = torch.empty_like(q_lat)
         need = ctypes.c_longlong()
-        lib.gk_mla_decode_scratch(T, H, ly.row_rank, rows.max_ctx, ctypes.byref(need))
-        scratch, gate, tab = _decode_scratch(proj.device, max(need.value, 1)), p[:, ly.gate:], rows.tables[rows.n_portions:]
+        span = min(ly.window, rows.max_ctx) if ly.window else rows.max_ctx
+        lib.gk_mla_decode_scratch(T, H, ly.row_rank, span, ctypes.byref(need))
+        scratch, tab = _decode_scratch(proj.device, max(need.value, 1)), rows.tables[rows.n_portions:]
         LAUNCHES["latent_attention"] += 1
         _lib.check(lib.gk_mla_paged_decode_gated(
             _lib.ptr(q_lat), q_lat.stride(1), q_lat.stride(0), _lib.ptr(q[..., ly.dim:]), q.stride(0), q.stride(1),
             _lib.ptr(cache), _lib.ptr(tab), _lib.ptr(rows.ctx), _lib.ptr(o_lat), o_lat.stride(1), o_lat.stride(0),
             _lib.ptr(scratch), T, H, ly.row_rank, ly.row_rot, cache.shape[1], rows.tables.shape[1], rows.max_ctx,
-            float(ly.scale), _lib.ptr(gate), p.stride(0), _lib.stream_ptr()), "mla_paged_decode_gated")
+            float(ly.scale), _lib.ptr(head_gate), p.stride(0), ly.window, _lib.ptr(sinks), _lib.stream_ptr()),
+            "mla_paged_decode_gated")
     else:
         q_abs, o = torch.empty(T, H, ly.row, **kw), torch.empty(T, H, ly.row_rank, **kw)
         q_abs[..., ly.row_rank:].copy_(q[..., ly.dim:])
         _bmm(q[..., :ly.dim].transpose(0, 1), uk, q_abs[..., :ly.row_rank].transpose(0, 1))
         general_attention(q_abs, H * ly.row, cache, rows, lo, hi, o, H, 1, ly.row, ly.scale, ly.row_rank,
-                          gate=p[:, ly.gate:], gate_ld=p.stride(0))
+                          ly.window, gate=head_gate, gate_ld=p.stride(0), sinks=sinks)
         o_lat = o.transpose(0, 1)
     _bmm(o_lat, uv.transpose(1, 2), out[lo:hi].view(T, H, ly.vdim).transpose(0, 1))
+    if head_gate is None:
+        LAUNCHES["latent_attention"] += 1
+        _lib.check(lib.gk_gate_columns(int(proj.dtype == torch.float32), _lib.ptr(out[lo:hi]), out.stride(0), _lib.ptr(gate),
+                                       p.stride(0), T, H * ly.vdim, _lib.stream_ptr()), "gate_columns")
 
 
-def latent_attention(proj, ly: LatentLayout, gain, turns, up_kv, rows: StepRows, cache, out):
+def latent_attention(proj, ly: LatentLayout, gain, turns, up_kv, rows: StepRows, cache, out, sinks=None):
     """Appends every row's ``[latent | rotated key part]`` to ``cache`` [blocks, block_size, 1, row] and writes the gated
     attention output [T, heads * vdim] to ``out`` (any row stride).  The queries' rotated parts in ``proj`` are rotated in
     place.  ``up_kv`` [heads * (dim + vdim), row_rank]: key rows of all heads, then value rows; ``gain`` [rank] is
-    32-bit, ``turns`` comes from ``rotation_turns``."""
+    32-bit, ``turns`` comes from ``rotation_turns``; ``sinks`` [heads] 32-bit join the softmax denominators."""
     cache = cache.view(cache.shape[0], cache.shape[1], ly.row)
     if not proj.is_cuda:
-        return _ref(proj, ly, gain, turns, up_kv, rows, cache, out)
+        return _ref(proj, ly, gain, turns, up_kv, rows, cache, out, sinks)
     T, P = proj.shape[0], rows.portion_rows
     tiled = P > 0 and proj.dtype == torch.bfloat16 and bool(
         _lib.kernels().gk_latent_prefill_supported(ly.dim, up8(ly.rot), ly.vdim))
-    context = torch.empty(rows.ctx_rows, ly.row, dtype=proj.dtype, device=proj.device) if tiled else None
+    context = torch.empty(rows.contexts[ly.window].rows, ly.row, dtype=proj.dtype, device=proj.device) if tiled else None
     _prep(proj, ly, gain, turns, rows, cache, context)
     if tiled:
-        _portions(proj, ly, up_kv, rows, cache, context, out)
+        _portions(proj, ly, up_kv, rows, cache, context, out, sinks)
     elif P:
-        _absorbed(proj, ly, up_kv, rows, 0, P, cache, out)
+        _absorbed(proj, ly, up_kv, rows, 0, P, cache, out, sinks)
     if T > P:
-        _absorbed(proj, ly, up_kv, rows, P, T, cache, out)
+        _absorbed(proj, ly, up_kv, rows, P, T, cache, out, sinks)
     return out

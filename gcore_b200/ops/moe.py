@@ -13,7 +13,7 @@ from .router import route_ref
 
 LAUNCHES = {"moe": 0}
 SEG = 128               # expert segments are padded to the grouped GEMM's tile height
-MAX_EXPERTS, MAX_TOP = 512, 16
+MAX_EXPERTS, MAX_TOP, MAX_GROUPS = 512, 16, 32
 SILU_GATE, RELU2 = 0, 1
 
 
@@ -35,13 +35,14 @@ def activate(kind: int, src, cols: int, up_off: int, dst, row_logit=None, n_rows
     return dst
 
 
-def choose(logits, experts: int, top: int, correction, counts):
-    """Softmax scores of ``logits[:, :experts]`` (32-bit), the ``top`` experts by score + ``correction``, their scores
-    normalised.  Returns ``(expert [T, top] int64, weight [T, top], place [T, top] int32)`` and adds to ``counts`` [experts]
-    int32 how many tokens chose each; ``place`` numbers the tokens of one expert."""
+def choose(logits, experts: int, top: int, correction, counts, sigmoid=False, norm=True, scale=1.0, groups=1, keep=1):
+    """Scores of ``logits[:, :experts]`` (32-bit; a softmax or sigmoids), the ``top`` experts by score + ``correction``
+    among the best ``keep`` of ``groups`` groups of neighbours, their scores (normalised with ``norm``) times ``scale``.
+    Returns ``(expert [T, top] int64, weight [T, top], place [T, top] int32)`` and adds to ``counts`` [experts] int32 how
+    many tokens chose each; ``place`` numbers the tokens of one expert."""
     T = logits.shape[0]
     if not logits.is_cuda:
-        idx, w = route_ref(logits[:, :experts], correction, None, top, 1, 1, False, True, 1.0)
+        idx, w = route_ref(logits[:, :experts], correction, None, top, groups, keep, sigmoid, norm, scale)
         place, flat = torch.zeros(T * top, dtype=torch.int32), idx.reshape(-1).tolist()
         for i, e in enumerate(flat):
             place[i] = counts[e]
@@ -51,7 +52,7 @@ def choose(logits, experts: int, top: int, correction, counts):
     LAUNCHES["moe"] += 1
     _lib.check(_lib.kernels().gk_router_dispatch(
         _lib.ptr(logits), logits.stride(0), _lib.ptr(correction), _lib.ptr(idx), _lib.ptr(w), _lib.ptr(counts),
-        _lib.ptr(place), T, experts, top, 0, 1, 1.0, _lib.stream_ptr()), "router_dispatch")
+        _lib.ptr(place), T, experts, top, int(sigmoid), int(norm), float(scale), groups, keep, _lib.stream_ptr()), "router_dispatch")
     return idx, w, place
 
 
@@ -63,20 +64,20 @@ def _choice_buffers(T, top, device):
 FUSED_TOKENS, FUSED_WIDTH = 128, 11264      # up to here a CTA per token computes the logits itself
 
 
-def route_tokens(h, router, experts: int, top: int, correction, counts):
+def route_tokens(h, router, experts: int, top: int, correction, counts, sigmoid=False, norm=True, scale=1.0, groups=1, keep=1):
     """``choose`` on the logits ``h @ router^T``; ``router`` [experts + extra, H] may hold rows that are only projected.
     Returns ``(logits [T, rows], choice)``."""
     T, n = h.shape[0], router.shape[0]
     if not h.is_cuda or T > FUSED_TOKENS or h.shape[1] > FUSED_WIDTH:
         logits = linear_forward(h, router, out_dtype=torch.float32)
-        return logits, choose(logits, experts, top, correction, counts)
+        return logits, choose(logits, experts, top, correction, counts, sigmoid, norm, scale, groups, keep)
     logits = torch.empty(T, n, dtype=torch.float32, device=h.device)
     idx, w, place = _choice_buffers(T, top, h.device)
     LAUNCHES["moe"] += 1
     _lib.check(_lib.kernels().gk_router_fused(
         int(h.dtype == torch.float32), _lib.ptr(h), _lib.ptr(router), _lib.ptr(logits), h.shape[1], n, _lib.ptr(correction),
-        _lib.ptr(idx), _lib.ptr(w), _lib.ptr(counts), _lib.ptr(place), T, experts, top, 0, 1, 1.0, _lib.stream_ptr()),
-        "router_fused")
+        _lib.ptr(idx), _lib.ptr(w), _lib.ptr(counts), _lib.ptr(place), T, experts, top, int(sigmoid), int(norm), float(scale),
+        groups, keep, _lib.stream_ptr()), "router_fused")
     return logits, (idx, w, place)
 
 
@@ -120,11 +121,14 @@ def grouped(x, w, offsets):
     return grouped_gemm(x, w, offsets, out_dtype=x.dtype)
 
 
-def routed_experts(h, choice, up, down, counts):
-    """Every token through its chosen experts ``down(relu(up h)^2)``: returns ``(rows, dest, weight)``, the experts' outputs
-    in expert order and where a token finds its own."""
+def routed_experts(h, choice, up, down, counts, act: int = RELU2):
+    """Every token through its chosen experts, ``down(relu(up h)^2)`` (RELU2) or ``down(silu(gate h) * up h)`` (SILU_GATE:
+    ``up`` holds the gate rows, then the up rows): returns ``(rows, dest, weight)``, the experts' outputs in expert order and
+    where a token finds its own."""
     idx, w, place = choice
     x, dest, offsets = expert_rows(h, counts, idx, place)
     a = grouped(x, up, offsets)
-    activate(RELU2, a, a.shape[1], 0, a, n_rows=offsets[-1:])
-    return grouped(a, down, offsets), dest, w
+    F = down.shape[2]
+    b = a if act == RELU2 else torch.empty(a.shape[0], F, dtype=a.dtype, device=a.device)
+    activate(act, a, F, F if act == SILU_GATE else 0, b, n_rows=offsets[-1:])
+    return grouped(b, down, offsets), dest, w

@@ -23,7 +23,7 @@ def route_ref(logits, bias, replay, K, n_group, topk_group, sigmoid, norm, scale
     else:
         sel = scores + bias if bias is not None else scores
         if n_group > 1:
-            grp = sel.view(-1, n_group, E // n_group).topk(2, dim=-1).values.sum(-1)
+            grp = sel.view(-1, n_group, E // n_group).topk(min(2, E // n_group), dim=-1).values.sum(-1)
             gidx = grp.topk(topk_group, dim=-1).indices
             gmask = torch.zeros_like(grp).scatter_(1, gidx, 1.0)
             sel = sel.masked_fill(gmask[:, :, None].expand(-1, n_group, E // n_group).reshape(-1, E) == 0,

@@ -60,16 +60,20 @@ def append_keys(proj, k_off, n, slots, cache):
 
 
 def general_attention(q, q_ld, cache, rows: StepRows, lo, hi, out, H, G, D, scale, dv=None, window=0, slopes=None, gate=None,
-                      gate_ld=0):
-    """Rows ``lo .. hi`` of a step against the paged cache: keys of ``D`` columns whose first ``dv`` are the value, an
-    optional window (0: none), distance penalty and output gate.  Any size, 32-bit or bf16."""
-    dims = (ctypes.c_int * 8)(hi - lo, H, G, D, dv or D, window, cache.shape[1], rows.tables.shape[1])
-    ptrs = (ctypes.c_void_p * 9)(*[t.data_ptr() if t is not None else None for t in
-                                   (q, cache, rows.tables, rows.row_seq[lo:hi], rows.pos[lo:hi], rows.slots[lo:hi], slopes,
-                                    gate, out)])
+                      gate_ld=0, sinks=None, maps=1, v_off=0, v_stride=None):
+    """Rows ``lo .. hi`` of a step against the paged cache, whose rows hold G * ``maps`` keys of ``D`` columns and, at
+    ``v_off``, G values of ``dv`` columns ``v_stride`` apart (default: a value is the first columns of its key).  Optional
+    window (0: none), distance penalty, sink logits and output gate.  Any size, 32-bit or bf16; ``out`` may be 32-bit."""
+    row = cache.stride(1)
+    dims = (ctypes.c_int * 11)(hi - lo, H, G, maps, D, dv or D, v_off, D if v_stride is None else v_stride, window,
+                               cache.shape[1], rows.tables.shape[1])
+    ptrs = (ctypes.c_void_p * 10)(*[t.data_ptr() if t is not None else None for t in
+                                    (q, cache, rows.tables, rows.row_seq[lo:hi], rows.pos[lo:hi], rows.slots[lo:hi], slopes,
+                                     gate, out, sinks)])
+    lds = (ctypes.c_longlong * 3)(q_ld, gate_ld, row)
     LAUNCHES["window_attention"] += 1
-    _lib.check(_lib.kernels().gk_window_attn(int(q.dtype == torch.float32), ptrs, q_ld, gate_ld, dims, float(scale),
-                                             _lib.stream_ptr()), "window_attn")
+    _lib.check(_lib.kernels().gk_window_attn(int(q.dtype == torch.float32), int(out.dtype == torch.float32), ptrs, lds, dims,
+                                             float(scale), _lib.stream_ptr()), "window_attn")
 
 
 def window_attention(proj, q_off: int, k_off: int, heads: int, kv_heads: int, dim: int, rows: StepRows, cache, slopes,

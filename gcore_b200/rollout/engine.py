@@ -35,7 +35,7 @@ from ..models.plan_decoder import PlanDecoder
 from ..ops import _lib, fused
 from ..ops.attention import flash_attn_varlen, kv_append_rope, mla_paged_decode, paged_decode_append
 from ..ops.gemm import linear_forward
-from ..ops.rows import StepRows
+from ..ops.rows import PortionContexts, StepRows, portion_contexts
 from ..ops.vocab import apply_top_k_top_p, sample, sample_filtered
 from ..utils import io_counters
 
@@ -170,10 +170,11 @@ class _Sched:
 
 
 def _count_launches() -> int:
-    from ..ops import (attention, depth, gemm, latent_attention, matrix_memory, moe, optim, rl, sandwich, vocab,
-                       window_attention)
-    return sum(sum(m.LAUNCHES.values()) for m in (attention, depth, fused, gemm, latent_attention, matrix_memory, moe, optim,
-                                                  rl, sandwich, vocab, window_attention))
+    from ..ops import (attention, depth, diff_attention, gemm, latent_attention, matrix_memory, moe, optim, rl, sandwich,
+                       streams, vocab, window_attention)
+    return sum(sum(m.LAUNCHES.values()) for m in (attention, depth, diff_attention, fused, gemm, latent_attention,
+                                                  matrix_memory, moe, optim, rl, sandwich, streams, vocab,
+                                                  window_attention))
 
 
 class LayerWeights:
@@ -884,21 +885,23 @@ class InferEngine:
         pos = torch.arange(T, dtype=torch.int32) - (cu[:-1] - first_t)[row_seq.long()]
         slots = bt[row_seq.long(), (pos // self.bs).long()] * self.bs + pos % self.bs
         ctx = (first_t + 1)[n_port:]
-        cu_ctx = torch.zeros(n_port + 1, dtype=torch.int32)
-        cu_ctx[1:] = (first_t + lens_t)[:n_port].cumsum(0)
+        windows = self.cfg.layer_plan.windows()
+        ctxs = [portion_contexts(first[:n_port], lens[:n_port], w) for w in windows]
         parts = [torch.tensor([t for e in order for t in entries[e][2]], dtype=torch.int32), pos, slots.to(torch.int32),
-                 torch.tensor(self.sched.states(rids), dtype=torch.int32), first_t, cu[:n_port + 1], cu_ctx, ctx,
-                 row_seq, bt.reshape(-1)]
+                 torch.tensor(self.sched.states(rids), dtype=torch.int32), first_t, cu[:n_port + 1], ctx,
+                 row_seq, bt.reshape(-1)] + [t for start, off, _, _ in ctxs for t in (start, off)]
         packed = torch.cat(parts)
         if self.device.type == "cuda":
             packed = packed.pin_memory()
         io_counters.add_h2d(io_counters.tensor_bytes(packed))
-        tok, pos, slots, states, first_d, cu_d, ctx_d, ctx, row_seq, tables = packed.to(self.device, non_blocking=True).split(
+        tok, pos, slots, states, first_d, cu_d, ctx, row_seq, tables, *rest = packed.to(self.device, non_blocking=True).split(
             [p.numel() for p in parts])
+        contexts = {w: PortionContexts(cu=rest[2 * k + 1], start=rest[2 * k] if w else None, rows=ctxs[k][2],
+                                       max_before=ctxs[k][3]) for k, w in enumerate(windows)}
         rows = StepRows(tokens=tok.long(), pos=pos, slots=slots, tables=tables.view(n, self.max_blocks), states=states,
                         first_pos=first_d, cu=cu_d, ctx=ctx, row_seq=row_seq, n_portions=n_port, portion_rows=port_rows,
-                        max_portion=max(lens[:n_port], default=0), max_ctx=max((f + 1 for f in first[n_port:]), default=1), cu_ctx=ctx_d, ctx_rows=int(cu_ctx[-1]),
-                        max_first=max(first[:n_port], default=0))
+                        max_portion=max(lens[:n_port], default=0), max_ctx=max((f + 1 for f in first[n_port:]), default=1),
+                        contexts=contexts)
         base = [0] * n
         for k, e in enumerate(order):
             base[e] = int(cu[k])

@@ -19,7 +19,7 @@ from ..models.plan_decoder import build_decoder
 from ..ops import _lib, attention, fused, sandwich
 from ..ops import matrix_memory as mm
 from ..ops import window_attention as wa
-from ..ops.rows import StepRows
+from ..ops.rows import PortionContexts, StepRows
 from ..rollout.engine import InferEngine, RolloutWeights, SamplingParams
 
 SIZES = {
@@ -159,7 +159,7 @@ def graph_us(fns, replays=20):
     return event_ms(g.replay, replays) * 1e3 / len(fns)
 
 
-def _rows(prompts, length, ctx, B, bs, dev):
+def _rows(prompts, length, ctx, B, bs, dev, windows=(0,)):
     """Rows of ``prompts`` whole prompts, or (``prompts`` = 0) of B single tokens at context ``ctx``."""
     if prompts:
         n, T = prompts, prompts * length
@@ -174,12 +174,13 @@ def _rows(prompts, length, ctx, B, bs, dev):
         pos = torch.full((n,), ctx, dtype=torch.int32, device=dev)
         seq = torch.arange(n, dtype=torch.int32, device=dev)
         first, cu, ctxs = pos, None, pos + 1
+    contexts = {w: PortionContexts(cu=cu, start=first if w else None, rows=prompts * length, max_before=0) for w in windows}
     tab = torch.arange(n * nb, dtype=torch.int32, device=dev).view(n, nb)
     slots = (tab[seq.long(), (pos // bs).long()] * bs + pos % bs).int()
     return StepRows(tokens=torch.zeros(T, dtype=torch.int64, device=dev), pos=pos, slots=slots, tables=tab,
                     states=torch.arange(n, dtype=torch.int32, device=dev), first_pos=first, cu=cu, ctx=ctxs, row_seq=seq,
                     n_portions=prompts, portion_rows=prompts * length, max_portion=length if prompts else 0,
-                    max_ctx=ctx + 1, cu_ctx=cu, ctx_rows=prompts * length), n * nb
+                    max_ctx=ctx + 1, contexts=contexts), n * nb
 
 
 def kernel_table(s, prompts, length, B, ctx, bs=64):

@@ -1,0 +1,57 @@
+"""Small Lobutar configurations for the tests."""
+from tests.plan_util import assert_close, make_engine, make_rows, rms_error, run_alone, run_mixed, tokens  # noqa: F401
+
+
+def rotation(dims, base):
+    return dict(dims=dims, base=base)
+
+
+def attention(heads, kv_heads, dim, vdim, rot, scale, diff, mlp, base=400.0):
+    return dict(type="attention", mlp=mlp, mixer=dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, scale=scale, diff=diff,
+                                                      rot=rotation(rot, base)))
+
+
+def latent(heads, dim, rot_dim, vdim, kv_rank, window, scale, mlp, base=600.0):
+    return dict(type="latent_attention", mlp=mlp, mixer=dict(
+        heads=heads, dim=dim, rot_dim=rot_dim, vdim=vdim, kv_rank=kv_rank, scale=scale, mask=dict(size=window),
+        rot=rotation(rot_dim, base)))
+
+
+def again(layers, j):
+    """A layer that runs layer j's weights once more."""
+    return dict(type=layers[j]["type"], mixer=layers[j]["mixer"], mlp=layers[j]["mlp"], weights_of=j)
+
+
+def dense(ff):
+    return dict(kind="dense", ff=ff)
+
+
+def experts(n, top, ff, shared, groups=1, keep=1, scale=1.0):
+    return dict(kind="moe", expert=dict(ff=ff), shared=dict(ff=shared) if shared else None,
+                router=dict(experts=n, top=top, scale=scale, groups=dict(count=groups, keep=keep)))
+
+
+def conf(layers, width, vocab, streams=2, eps=1e-5):
+    return dict(architecture="Lobutar", layers=layers, norm=dict(eps=eps), streams=streams, vocab=vocab, width=width)
+
+
+def uneven_conf():
+    """Layers that share no size, odd widths everywhere, every kind of feed-forward behind every mixer and none, a layer that
+    comes back twice with others between."""
+    ly = [attention(6, 2, 20, 12, 6, 0.3, 0.2, experts(6, 2, 20, 28, groups=3, keep=2, scale=2.5)),
+          latent(3, 20, 6, 12, 36, 9, 0.3, dense(36)),
+          attention(3, 3, 10, 30, 10, 0.25, 0.55, None, base=90.0),
+          latent(2, 10, 14, 30, 50, 1, 0.2, experts(5, 3, 12, 0), base=50.0)]
+    ly.append(again(ly, 0))
+    ly += [attention(1, 1, 12, 4, 2, 0.4, 0.0, dense(52)), latent(5, 8, 4, 8, 24, 70, 0.4, None), again(ly, 0)]
+    ly.append(again(ly, 6))
+    return conf(ly, width=44, vocab=75, streams=3)
+
+
+def round_conf():
+    """Sizes the tensor-core kernels take without padding."""
+    ly = [attention(8, 2, 64, 128, 64, 0.11, 0.4, dense(384)),
+          latent(8, 64, 32, 64, 128, 48, 0.11, experts(16, 4, 128, 128, groups=4, keep=2, scale=1.7)),
+          attention(4, 4, 128, 64, 32, 0.08, 0.7, experts(12, 3, 64, 256, groups=2, keep=1, scale=0.8), base=9000.0)]
+    ly += [again(ly, 1), latent(4, 128, 64, 128, 256, 100, 0.08, dense(256), base=9000.0), again(ly, 2)]
+    return conf(ly, width=256, vocab=320, streams=2)

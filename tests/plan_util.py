@@ -6,13 +6,13 @@ import torch
 
 from gcore_b200.models.config import from_hf_config
 from gcore_b200.models.plan_decoder import build_decoder
-from gcore_b200.ops.rows import StepRows
+from gcore_b200.ops.rows import PortionContexts, StepRows, portion_contexts
 from gcore_b200.rollout.engine import InferEngine, RolloutWeights
 
 
-def make_rows(segments, block_size, n_blocks, n_slots, seed=0, device="cuda"):
+def make_rows(segments, block_size, n_blocks, n_slots, seed=0, device="cuda", windows=(0,)):
     """StepRows of ``segments`` = [(first position, length)] on shuffled cache blocks and state slots; portions (length
-    > 1) must come first."""
+    > 1) must come first.  ``windows``: the attention windows whose contexts the rows carry."""
     g = torch.Generator().manual_seed(seed)
     perm = torch.randperm(n_blocks, generator=g).tolist()
     mb = max((f + l + block_size - 1) // block_size for f, l in segments)
@@ -29,13 +29,15 @@ def make_rows(segments, block_size, n_blocks, n_slots, seed=0, device="cuda"):
     cu = torch.tensor([sum(lens[:i]) for i in range(n_port + 1)], dtype=torch.int32)
     states = torch.randperm(n_slots, generator=g)[:len(segments)].to(torch.int32)
     first = torch.tensor([f for f, _ in segments], dtype=torch.int32)
-    ends = torch.tensor([0] + [f + l for f, l in segments[:n_port]])
     d = lambda t: t.to(device)
+    contexts = {}
+    for w in windows:
+        start, off, n, before = portion_contexts([f for f, _ in segments[:n_port]], lens[:n_port], w)
+        contexts[w] = PortionContexts(cu=d(off), start=d(start) if w else None, rows=n, max_before=before)
     return StepRows(tokens=torch.zeros(pos.numel(), dtype=torch.int64, device=device), pos=d(pos), slots=d(slots.int()),
                     tables=d(tab), states=d(states), first_pos=d(first), cu=d(cu), ctx=d((first + 1)[n_port:].contiguous()),
                     row_seq=d(seq), n_portions=n_port, portion_rows=int(cu[-1]), max_portion=max(lens[:n_port], default=0),
-                    max_ctx=max((f + 1 for f, l in segments if l == 1), default=1), cu_ctx=d(ends.cumsum(0).int()),
-                    ctx_rows=int(ends.sum()), max_first=max((f for f, l in segments if l > 1), default=0))
+                    max_ctx=max((f + 1 for f, l in segments if l == 1), default=1), contexts=contexts)
 
 
 def make_engine(c, W, dtype="float32", device="cpu", **kw):
