@@ -141,6 +141,8 @@ class ExpertFeedForward(nn.Module):
         super().__init__()
         if spec.experts > moe.MAX_EXPERTS or spec.top > moe.MAX_TOP:
             raise ValueError(f"at most {moe.MAX_EXPERTS} experts and {moe.MAX_TOP} choices are supported")
+        if spec.groups > moe.MAX_GROUPS:
+            raise ValueError(f"at most {moe.MAX_GROUPS} expert groups are supported")
         self.spec, self.width = spec, width
         self.ff, self.shared = _up(spec.ff, 8), _up(spec.shared_ff, 8)
         self.act = moe.SILU_GATE if spec.act == "silu_gate" else moe.RELU2

@@ -2,8 +2,8 @@
 
 For a few real-model layer sizes (random weights) it times, on the device, a prefill step and a captured decode step of an
 engine of the design and of the closest uniform model - for Nafitar a dense grouped-query decoder with the same width,
-heads, window, feed-forward and layer count, for Kedesun a latent-attention decoder with experts (``serve_bench_kedesun.py``)
-- and then every kernel the design added beside the like kernel of that model: time, the time its bytes or FLOPs would take
+heads, window, feed-forward and layer count, for Kedesun and Lobutar a latent-attention decoder with experts
+(``serve_bench_kedesun.py``, ``serve_bench_lobutar.py``) - and then every kernel the design added beside the like kernel of that model: time, the time its bytes or FLOPs would take
 at the measured peaks, and the ratio of the two.  Inputs of every timed launch rotate over buffers larger than L2."""
 from __future__ import annotations
 
@@ -56,15 +56,16 @@ def dense_config(s):
 
 
 def build(kind, s, positions, requests, block=64):
-    """Engine of a layer-plan design (``nafitar``, ``kedesun``) or of the uniform model it is compared with (``dense``,
-    ``latent``)."""
-    from . import serve_bench_kedesun as sk
+    """Engine of a layer-plan design (``nafitar``, ``kedesun``, ``lobutar``) or of the uniform model it is compared with
+    (``dense``, ``latent``: Kedesun's, ``grouped``: Lobutar's)."""
+    from . import serve_bench_kedesun as sk, serve_bench_lobutar as sl
     dev = torch.device("cuda")
-    if kind in ("nafitar", "kedesun"):
-        cfg = from_hf_config(nafitar_conf(s, positions) if kind == "nafitar" else sk.conf(s))
+    plans = {"nafitar": lambda: nafitar_conf(s, positions), "kedesun": lambda: sk.conf(s), "lobutar": lambda: sl.conf(s)}
+    if kind in plans:
+        cfg = from_hf_config(plans[kind]())
         model = build_decoder(cfg, dev).randomize()
     else:
-        cfg = dense_config(s) if kind == "dense" else sk.latent_config(s)
+        cfg = {"dense": dense_config, "latent": sk.latent_config, "grouped": sl.latent_config}[kind](s)
         model = GPTModel(cfg, recompute="none", device=dev)
     eng = InferEngine(cfg, RolloutWeights.from_model(model), max_running_requests=requests, max_model_len=positions,
                       kv_block_size=block, max_prefill_tokens=1 << 20, device=dev)
@@ -265,12 +266,14 @@ def kernel_table(s, prompts, length, B, ctx, bs=64):
 
 
 def _families():
-    from . import serve_bench_kedesun as sk
+    from . import serve_bench_kedesun as sk, serve_bench_lobutar as sl
     active = lambda eng, s, n: n - 2 * VOCAB * s["width"]
     return {"nafitar": dict(like="dense", sizes=SIZES, active=active, table=kernel_table,
                             decode_bytes=lambda kind, s, eng, B, ctx: decode_bytes(kind, s, eng, B, ctx)),
             "kedesun": dict(like="latent", sizes=sk.SIZES, active=sk.active_weights, table=sk.kernel_table,
-                            decode_bytes=sk.decode_bytes)}
+                            decode_bytes=sk.decode_bytes),
+            "lobutar": dict(like="grouped", sizes=sl.SIZES, active=sl.active_weights, table=sl.kernel_table,
+                            decode_bytes=sl.decode_bytes)}
 
 
 def run(sizes=None, iters=10, design="nafitar"):

@@ -114,7 +114,7 @@ def kernel_table(s, prompts, length, B, ctx, bs=64):
     up, la_linear = mix.up_kv, la.linear_forward
     la.linear_forward = lambda *a: kv            # the attention kernel alone
     try:
-        t = graph_us([lambda p=p: la._portions(p, ly, up, rows, cache, context, out) for p in projs])
+        t = graph_us([lambda p=p: la._portions(p, ly, up, rows, cache, context, out, None) for p in projs])
     finally:
         la.linear_forward = la_linear
     fl = 2.0 * pairs * H * (dim + rot + vdim)
@@ -215,7 +215,7 @@ def kernel_table(s, prompts, length, B, ctx, bs=64):
     o_lat = torch.empty_like(q_lat)
     bmm, la._bmm = la._bmm, lambda a, b, out: out      # the attention kernel alone
     try:
-        t = graph_us([lambda c=c: la._absorbed(proj, ly, mix.up_kv, rows, 0, B, c, out) for c in caches])
+        t = graph_us([lambda c=c: la._absorbed(proj, ly, mix.up_kv, rows, 0, B, c, out, None) for c in caches])
     finally:
         la._bmm = bmm
     like = graph_us([lambda c=c: attention.mla_paged_decode(q_lat.transpose(0, 1), q_rope, c, rows.tables, rows.ctx, ctx + 1,

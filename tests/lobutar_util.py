@@ -1,5 +1,9 @@
 """Small Lobutar configurations for the tests."""
-from tests.plan_util import assert_close, make_engine, make_rows, rms_error, run_alone, run_mixed, tokens  # noqa: F401
+import torch
+
+from tests import plan_util
+from tests.oracle import lobutar as oracle
+from tests.plan_util import make_engine, make_rows, rms_error, run_alone, run_mixed, tokens  # noqa: F401
 
 
 def rotation(dims, base):
@@ -55,3 +59,42 @@ def round_conf():
           attention(4, 4, 128, 64, 32, 0.08, 0.7, experts(12, 3, 64, 256, groups=2, keep=1, scale=0.8), base=9000.0)]
     ly += [again(ly, 1), latent(4, 128, 64, 128, 256, 100, 0.08, dense(256), base=9000.0), again(ly, 2)]
     return conf(ly, width=256, vocab=320, streams=2)
+
+
+def decisive(W, c, level=4.0):
+    """The same weights with expert choices that bf16 rounding cannot turn: the residual's first column carries the token's
+    parity untouched through every layer, the routers read mainly that, and the corrections are well apart."""
+    W = dict(W)
+    W["embed"] = W["embed"].clone()
+    W["embed"][:, 0] = torch.tensor([level, -level]).repeat(c["vocab"])[:c["vocab"]]
+    for k, v in W.items():
+        end = k.rsplit(".", 1)[-1]
+        if end == "down" or k.endswith((".mix.o", ".mix.o.b")):
+            W[k] = v.clone()
+            W[k][0] = 0
+        elif end in ("norm1", "norm2"):
+            W[k] = v.clone()
+            W[k][0] = 1
+        elif end in ("in", "mix") and ".hc" in k:       # the streams' parities add up and keep their size
+            W[k] = (v.abs().float() / v.abs().float().sum(0)).to(v.dtype)
+        elif end == "router":
+            E = v.shape[0]
+            W[k] = v * 0.1
+            W[k][:, 0] = torch.tensor([1.0, -1.0, 1.0, 1.0, -1.0, -1.0, -1.0]).repeat(E)[:E]
+        elif end == "correction":
+            E = v.shape[0]
+            W[k] = (torch.arange(E) * 5 % 17 * 0.3 / 17 + torch.arange(E) * 0.7 / E).to(v.dtype)
+    return W
+
+
+def weights(c, seed, dtype="float32"):
+    """Random weights, for bf16 with expert choices that rounding cannot turn."""
+    W = oracle.random_weights(c, seed=seed)
+    return decisive(W, c) if dtype == "bfloat16" else W
+
+
+def assert_close(got, want, dtype="float32", what=None):
+    if dtype == "float32":
+        return plan_util.assert_close(got, want, dtype, what)
+    e = rms_error(got, want)
+    assert e.max() < 0.1 and e.quantile(0.9) < 0.03, (what, float(e.max()), float(e.quantile(0.9)), int(e.argmax()))

@@ -239,7 +239,7 @@ def test_window_sink_and_gate_alone(H, dim, rot, vdim, rank, bs, window, dtype):
             w = torch.stack([oracle.softmax_with_sink(sc[h], sink[h].double()) for h in range(H)])
             want = torch.einsum("hn,nhv->hv", w, v[j]) * torch.sigmoid(gate[r])
             err = (got[at + r, :, :vdim] - want).abs().max() / want.abs().max().clamp_min(0.5)
-            assert err < (5e-5 if dtype == "float32" else 3e-2), (f, l, r, float(err))
+            assert err < (5e-5 if dtype == "float32" else 5e-2), (f, l, r, float(err))
         stored = flat[where(s, torch.arange(f, f + l))].double().cpu()
         assert (stored[:, :rank] - lat[f:]).abs().max() < (1e-5 if dtype == "float32" else 4e-2)
 
@@ -354,7 +354,7 @@ def test_gated_experts_from_the_tokens(T, dtype):
 @pytest.mark.parametrize("which", ["uneven", "round"])
 def test_portions_and_decoding_match_whole_sequences(which, dtype):
     c = lu.uneven_conf() if which == "uneven" else lu.round_conf()
-    W = oracle.random_weights(c, seed=5)
+    W = lu.weights(c, 5, dtype)
     eng = lu.make_engine(c, W, dtype, "cuda")
     for n, seed in ((1, 1), (2, 2), (150, 3), (260, 4)):
         seq = lu.tokens(n, c["vocab"], seed)
@@ -370,7 +370,7 @@ def test_portions_and_decoding_match_whole_sequences(which, dtype):
 @pytest.mark.parametrize("block", [8, 64])
 def test_mixed_batches_on_reused_pages_and_slots(dtype, block):
     c = lu.round_conf()
-    W = oracle.random_weights(c, seed=6)
+    W = lu.weights(c, 6, dtype)
     eng = lu.make_engine(c, W, dtype, "cuda", kv_block_size=block, num_kv_blocks=4 * 256 // block, max_model_len=256)
     seqs = [lu.tokens(n, c["vocab"], 20 + n) for n in (200, 31, 64, 1, 129, 65, 90, 17, 240)]
     for s, got in zip(seqs, lu.run_mixed(eng, seqs, [1, 1, 2, 3, 16, 63, 64, 65, 100], seed=7)):
@@ -381,7 +381,7 @@ def test_mixed_batches_on_reused_pages_and_slots(dtype, block):
 def test_the_batch_does_not_matter():
     """bf16 logits of one request alone and in a batch of others differ by rounding only."""
     c = lu.round_conf()
-    W = oracle.random_weights(c, seed=12)
+    W = lu.weights(c, 12, "bfloat16")
     eng = lu.make_engine(c, W, "bfloat16", "cuda", max_model_len=256)
     seqs = [lu.tokens(n, c["vocab"], 70 + n) for n in (120, 77, 33, 5)]
     for s, got in zip(seqs, lu.run_mixed(eng, seqs, [1, 2, 30, 64], seed=8)):
@@ -391,7 +391,7 @@ def test_the_batch_does_not_matter():
 def test_true_32_bit_whatever_the_matrix_mode():
     """The 32-bit engine stays exact when the process allows TF32."""
     c = lu.round_conf()
-    W = oracle.random_weights(c, seed=8)
+    W = lu.weights(c, 8)
     eng = lu.make_engine(c, W, "float32", "cuda")
     seq = lu.tokens(70, c["vocab"], 9)
     torch.backends.cuda.matmul.allow_tf32 = True
@@ -407,7 +407,7 @@ def test_greedy_generation_through_the_scheduler(dtype):
     """generate(): captured decode graphs, more requests than slots, prompts longer than a prefill step, samples that
     share a prompt - every token is the plain implementation's choice (or ties with it within rounding)."""
     c = lu.uneven_conf() if dtype == "float32" else lu.round_conf()
-    W = oracle.random_weights(c, seed=10)
+    W = lu.weights(c, 10, dtype)
     eng = lu.make_engine(c, W, dtype, "cuda", max_prefill_tokens=50, sync_interval=3, max_model_len=256)
     prompts = [lu.tokens(n, c["vocab"], 40 + n) for n in (1, 5, 33, 120, 64)]
     reqs = eng.generate(prompts, SamplingParams(max_new_tokens=40, greedy=True), n=2)
@@ -428,7 +428,7 @@ def test_greedy_generation_through_the_scheduler(dtype):
 def test_long_decoding_past_the_window():
     ly = [lu.attention(4, 2, 32, 64, 16, 0.17, 0.5, lu.dense(64)), lu.latent(4, 32, 8, 32, 64, 50, 0.15, lu.dense(64))]
     c = lu.conf(ly + [lu.again(ly, 1), lu.again(ly, 0)], 64, 128)
-    W = oracle.random_weights(c, seed=11)
+    W = lu.weights(c, 11, "bfloat16")
     eng = lu.make_engine(c, W, "bfloat16", "cuda", max_model_len=1024)
     seq = lu.tokens(400, c["vocab"], 12)
     lu.assert_close(lu.run_alone(eng, seq, [20] + [1] * 380), oracle.forward(W, c, seq), "bfloat16")
@@ -436,7 +436,7 @@ def test_long_decoding_past_the_window():
 
 def _checkpoint(path, c, seed):
     from safetensors.torch import save_file
-    W = oracle.random_weights(c, seed=seed)
+    W = lu.weights(c, seed, "bfloat16")
     save_file({k: v.contiguous() for k, v in W.items()}, str(path / "model.safetensors"))
     (path / "config.json").write_text(json.dumps(c))
     return W
@@ -479,3 +479,16 @@ def test_trace_replay_through_the_executable_entry(tmp_path):
         got = torch.from_numpy(np.fromfile(tmp_path / f"{n}.f32", "<f4").reshape(-1, c["vocab"]).copy())
         lu.assert_close(got, want)
     assert eng.get_load()["free_blocks"] == eng.num_blocks
+
+
+def test_serving_benchmark_runs_on_a_small_size():
+    from gcore_b200.tools import serve_bench as sb
+    from gcore_b200.tools import serve_bench_lobutar as sl
+    s = dict(width=256, heads=4, kv=2, dim=32, vdim=96, lh=4, ldim=128, lrot=64, lv=128, rank=512, window=70, ff=512, experts=32,
+             top=2, eff=192, groups=4, keep=2, streams=2, layers=4)
+    for kind in ("lobutar", "grouped"):
+        eng = sb.build(kind, s, 512, 4)
+        assert sb.prefill_step(eng, 2, 130, 2) > 0 and sb.decode_step(eng, 4, 200, 2) > 0
+        assert sl.decode_bytes(kind, s, eng, 4, 200) > 0
+    table = sl.kernel_table(s, 2, 130, 4, 200)
+    assert {r[0] for r in table} == {"prefill", "decode"} and all(r[2] > 0 for r in table)
