@@ -5,15 +5,18 @@
 // One CTA = 128 query rows of one head of one portion, both maps.  The portion's keys and those that earlier steps cached are
 // read through the block table, tile by tile (64 keys, on 64-key boundaries of the sequence), by TMA; heads narrower than the
 // tile are zero-filled by the loads.  A value tile serves both maps.  The probabilities feed the tensor core as two bf16 terms
-// (rounded value, remainder), i.e. with 16 significant bits.  With M = 128 every TMEM lane is one query row.
+// (rounded value, remainder), i.e. with 16 significant bits; they replace the scores in tensor memory (64 32-bit columns of S
+// become 32 + 32 columns of packed pairs) and are the A operand of P V from there, so neither they nor their loads touch
+// shared memory.  With M = 128 every TMEM lane is one query row.
 //
 //   warps 0-3, 4-7  softmax / O-correction of map 1, map 2 (thread t of a warpgroup <-> query row t <-> TMEM lane t); at the
 //                   end both warpgroups read both accumulators, each for half of the columns, so the difference, its norm and
 //                   the gate never leave the SM
 //   warp 8          TMA producer (both queries once, then [key 1, key 2 | value] tiles into a ring)
-//   warp 9          MMA issuer: both S_{j+1} are issued before P_j V_j, so score products overlap the softmax
+//   warp 9          MMA issuer: both S_{j+1} are issued before P_j V_j, so score products overlap the softmax; they go to the
+//                   buffer of P_{j-1} once its product is done
 //
-// TMEM columns (all 512, one CTA per SM): S of map m, buffer b at [64 (2m + b), +64); O of map m at [256 + m DV, +DV).
+// TMEM columns (all 512, one CTA per SM): S and P of map m, buffer b at [64 (2m + b), +64); O of map m at [256 + m DV, +DV).
 // Values wider than 128 columns take one CTA per 128 of them, which stores the difference for a finishing kernel.
 #include "ptx.cuh"
 #include "host_utils.h"
@@ -46,13 +49,12 @@ __device__ __forceinline__ void df_sync_softmax() { asm volatile("bar.sync 1, 25
 template <int DQ, int DV>
 struct DfGeo {
   static constexpr int NCH = DQ / 64, NCHV = DV / 64;
-  static constexpr int STAGES = DQ == 64 ? 3 : 2;
+  static constexpr int STAGES = DQ == 64 ? 4 : 3;
   static constexpr int Q_BYTES = 2 * DF_BM * DQ * 2;
   static constexpr int K_BYTES = 2 * NCH * DF_CHUNK;
   static constexpr int V_BYTES = NCHV * DF_CHUNK;
   static constexpr int STAGE = K_BYTES + V_BYTES;
-  static constexpr int P_BYTES = DF_BM * DF_BN * 2;        // one term of one map
-  static constexpr int BARS = Q_BYTES + STAGES * STAGE + 4 * P_BYTES;
+  static constexpr int BARS = Q_BYTES + STAGES * STAGE;
   static constexpr int SMEM = BARS + 256 + 2048;
   static_assert(SMEM <= 232448, "shared memory of one CTA");
 };
@@ -66,15 +68,13 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* sQ = smem_raw;                                 // map, chunk
   uint8_t* sKV = sQ + Geo::Q_BYTES;                       // stage: key map, chunk | value chunk
-  uint8_t* sP = sKV + STAGES * Geo::STAGE;                // map, term
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem_raw + Geo::BARS);
   uint64_t* q_full = bars;                                // 1
   uint64_t* k_full = q_full + 1;                          // STAGES
   uint64_t* v_full = k_full + STAGES;                     // STAGES
   uint64_t* kv_empty = v_full + STAGES;                   // STAGES
   uint64_t* s_full = kv_empty + STAGES;                   // map, buffer
-  uint64_t* s_empty = s_full + 4;                         // map, buffer (128 arrivals)
-  uint64_t* p_full = s_empty + 4;                         // map (128 arrivals)
+  uint64_t* p_full = s_full + 4;                          // map (128 arrivals)
   uint64_t* pv_done = p_full + 2;                         // map
   uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(pv_done + 2);
   float* s_inv = reinterpret_cast<float*>(smem_raw + Geo::BARS + 256);   // map, row
@@ -103,10 +103,7 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       mbar_init(&v_full[i], 1);
       mbar_init(&kv_empty[i], 1);
     }
-    for (int i = 0; i < 4; ++i) {
-      mbar_init(&s_full[i], 1);
-      mbar_init(&s_empty[i], 128);
-    }
+    for (int i = 0; i < 4; ++i) mbar_init(&s_full[i], 1);
     for (int i = 0; i < 2; ++i) {
       mbar_init(&p_full[i], 128);
       mbar_init(&pv_done[i], 1);
@@ -173,7 +170,7 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       if (!mbar_wait(&k_full[s], (it / STAGES) & 1, p.err, ERR_WAIT_FULL)) return false;
 #pragma unroll
       for (int m = 0; m < 2; ++m) {
-        if (it >= 2 && !mbar_wait(&s_empty[2 * m + sb], ((it - 2) >> 1) & 1, p.err, ERR_WAIT_TMEM_EMPTY)) return false;
+        if (it >= 2 && !mbar_wait(&pv_done[m], it & 1, p.err, ERR_WAIT_TMEM_EMPTY)) return false;   // P of it - 2
         tc_fence_after();
         if (lane == 0) {
           const uint32_t qa = smem_u32(sQ + m * NCH * DF_BM * 128), ka = smem_u32(sKV + s * Geo::STAGE + m * NCH * DF_CHUNK);
@@ -205,12 +202,11 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
           const uint32_t va = smem_u32(sKV + s * Geo::STAGE + Geo::K_BYTES);
 #pragma unroll
           for (int term = 0; term < 2; ++term) {
-            const uint32_t pa = smem_u32(sP + (2 * m + term) * Geo::P_BYTES);
+            const uint32_t pa = tmem_base + (2 * m + (it & 1)) * DF_BN + term * 32;
 #pragma unroll
             for (int k4 = 0; k4 < DF_BN / 16; ++k4)
-              umma_f16(tmem_o + m * DV, make_smem_desc_sw128(pa + k4 * 32, 16, 1024),
-                       make_smem_desc_sw128(va + k4 * 2048, DF_CHUNK, 1024), idesc_o,
-                       (it > 0 || term > 0 || k4 > 0) ? 1u : 0u);
+              umma_f16_ts(tmem_o + m * DV, pa + k4 * 8, make_smem_desc_sw128(va + k4 * 2048, DF_CHUNK, 1024), idesc_o,
+                          (it > 0 || term > 0 || k4 > 0) ? 1u : 0u);
           }
           if (m == 1) umma_commit(&kv_empty[s]);
           umma_commit(&pv_done[m]);
@@ -242,20 +238,18 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
 #pragma unroll
         for (int j = 0; j < 32; ++j) sv[c * 32 + j] = __uint_as_float(r[j]);
       }
-      tc_fence_before();
-      mbar_arrive(&s_empty[sb]);
       const int kbase = it * DF_BN;
-      float mx = -FLT_MAX;
-      if (kbase + DF_BN - 1 <= pi) {
+      if (kbase + DF_BN - 1 > pi) {
 #pragma unroll
-        for (int j = 0; j < DF_BN; ++j) mx = fmaxf(mx, sv[j]);
-      } else {
-#pragma unroll
-        for (int j = 0; j < DF_BN; ++j) {
-          sv[j] = kbase + j <= pi ? sv[j] : -FLT_MAX;
-          mx = fmaxf(mx, sv[j]);
-        }
+        for (int j = 0; j < DF_BN; ++j) sv[j] = kbase + j <= pi ? sv[j] : -FLT_MAX;
       }
+      // with two warps on a scheduler the length of a dependent chain counts: eight maxima and four sums at a time
+      float mx8[8];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) mx8[j] = sv[j];
+#pragma unroll
+      for (int j = 8; j < DF_BN; ++j) mx8[j & 7] = fmaxf(mx8[j & 7], sv[j]);
+      float mx = fmaxf(fmaxf(fmaxf(mx8[0], mx8[1]), fmaxf(mx8[2], mx8[3])), fmaxf(fmaxf(mx8[4], mx8[5]), fmaxf(mx8[6], mx8[7])));
       if (mx != -FLT_MAX) mx *= sl2;       // log2 domain (the scale is positive)
       // the running maximum moves only when the tile exceeds it by more than 2^8, so the accumulator in tensor memory
       // is rescaled on few tiles; the probabilities then reach at most 256
@@ -264,52 +258,45 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       const float m_new = grow ? m_cand : m;
       const float m_use = m_new == -FLT_MAX ? 0.f : m_new;
       const float corr = grow ? ex2(m - m_use) : 1.f;
-      float ps = 0.f;
+      float ps[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
       for (int j = 0; j < DF_BN; ++j) {
-        const float e = ex2(fmaf(sv[j], sl2, -m_use));   // masked scores underflow to exactly 0
-        sv[j] = e;
-        ps += e;
+        sv[j] = ex2(fmaf(sv[j], sl2, -m_use));           // masked scores underflow to exactly 0
+        ps[j & 3] += sv[j];
       }
-      l = l * corr + ps;
+      l = l * corr + ((ps[0] + ps[1]) + (ps[2] + ps[3]));
       m = m_new;
-      if (it > 0) {
+      if (it > 0 && __any_sync(0xffffffff, grow)) {
         ok = mbar_wait(&pv_done[map], (it - 1) & 1, p.err, ERR_WAIT_MISC);
         if (!ok) break;
         tc_fence_after();
-        if (__any_sync(0xffffffff, grow)) {
 #pragma unroll
-          for (int c = 0; c < DV / 32; ++c) {
-            uint32_t r[32];
-            tmem_ld32(my_o + c * 32, r);
-            tmem_ld_wait();
+        for (int c = 0; c < DV / 32; ++c) {
+          uint32_t r[32];
+          tmem_ld32(my_o + c * 32, r);
+          tmem_ld_wait();
 #pragma unroll
-            for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(__uint_as_float(r[j]) * corr);
-            tmem_st32(my_o + c * 32, r);
-          }
-          tmem_st_wait();
+          for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(__uint_as_float(r[j]) * corr);
+          tmem_st32(my_o + c * 32, r);
         }
       }
-      // P -> shared, K-major with the 128-byte swizzle: 16-byte unit u of row r sits at unit u ^ (r & 7)
-      uint8_t* rowp = sP + 2 * map * Geo::P_BYTES + row * 128;
+      // P over S: a column holds the keys 2j and 2j + 1; rounded values first, remainders behind
+      uint32_t w[32];
 #pragma unroll
-      for (int u = 0; u < 8; ++u) {
-        uint32_t w[4], v[4];
+      for (int j = 0; j < 32; ++j) w[j] = pack_bf16x2(sv[2 * j], sv[2 * j + 1]);
+      tmem_st32(tmem_base + lane_addr + sb * DF_BN, w);
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const float a = sv[u * 8 + 2 * e], c = sv[u * 8 + 2 * e + 1];
-          w[e] = pack_bf16x2(a, c);
-          v[e] = pack_bf16x2(a - bf16_bits_to_float(static_cast<uint16_t>(w[e] & 0xffff)),
-                             c - bf16_bits_to_float(static_cast<uint16_t>(w[e] >> 16)));
-        }
-        const int o = (u ^ (row & 7)) << 4;
-        *reinterpret_cast<uint4*>(rowp + o) = make_uint4(w[0], w[1], w[2], w[3]);
-        *reinterpret_cast<uint4*>(rowp + Geo::P_BYTES + o) = make_uint4(v[0], v[1], v[2], v[3]);
-      }
-      fence_proxy_async();
+      for (int j = 0; j < 32; ++j)
+        w[j] = pack_bf16x2(sv[2 * j] - bf16_bits_to_float(static_cast<uint16_t>(w[j] & 0xffff)),
+                           sv[2 * j + 1] - bf16_bits_to_float(static_cast<uint16_t>(w[j] >> 16)));
+      tmem_st32(tmem_base + lane_addr + sb * DF_BN + 32, w);
+      tmem_st_wait();
       tc_fence_before();
       mbar_arrive(&p_full[map]);
     }
+    // S of the last tile waited for the product two tiles back only: wait for the last two in turn, a parity does not tell
+    // phases two apart
+    if (ok && ntiles > 1) ok = mbar_wait(&pv_done[map], ntiles & 1, p.err, ERR_WAIT_MISC);
     if (ok) ok = mbar_wait(&pv_done[map], (ntiles - 1) & 1, p.err, ERR_WAIT_MISC);
     // both accumulators are complete behind this barrier (every thread of both warpgroups arrives, whatever its waits did)
     s_inv[map * 128 + row] = l > 0.f ? 1.f / l : 0.f;
