@@ -74,9 +74,9 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   uint64_t* v_full = k_full + STAGES;                     // STAGES
   uint64_t* kv_empty = v_full + STAGES;                   // STAGES
   uint64_t* s_full = kv_empty + STAGES;                   // map, buffer
-  uint64_t* p_full = s_full + 4;                          // map (128 arrivals)
-  uint64_t* pv_done = p_full + 2;                         // map
-  uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(pv_done + 2);
+  uint64_t* p_full = s_full + 4;                          // map, buffer (128 arrivals): a map may be a tile ahead of the other
+  uint64_t* pv_done = p_full + 4;                         // map, buffer
+  uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(pv_done + 4);
   float* s_inv = reinterpret_cast<float*>(smem_raw + Geo::BARS + 256);   // map, row
   float* s_ss = s_inv + 256;
 
@@ -103,8 +103,8 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       mbar_init(&v_full[i], 1);
       mbar_init(&kv_empty[i], 1);
     }
-    for (int i = 0; i < 4; ++i) mbar_init(&s_full[i], 1);
-    for (int i = 0; i < 2; ++i) {
+    for (int i = 0; i < 4; ++i) {
+      mbar_init(&s_full[i], 1);
       mbar_init(&p_full[i], 128);
       mbar_init(&pv_done[i], 1);
     }
@@ -170,7 +170,7 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       if (!mbar_wait(&k_full[s], (it / STAGES) & 1, p.err, ERR_WAIT_FULL)) return false;
 #pragma unroll
       for (int m = 0; m < 2; ++m) {
-        if (it >= 2 && !mbar_wait(&pv_done[m], it & 1, p.err, ERR_WAIT_TMEM_EMPTY)) return false;   // P of it - 2
+        if (it >= 2 && !mbar_wait(&pv_done[2 * m + sb], ((it - 2) >> 1) & 1, p.err, ERR_WAIT_TMEM_EMPTY)) return false;   // P of it - 2
         tc_fence_after();
         if (lane == 0) {
           const uint32_t qa = smem_u32(sQ + m * NCH * DF_BM * 128), ka = smem_u32(sKV + s * Geo::STAGE + m * NCH * DF_CHUNK);
@@ -195,7 +195,7 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       ok = mbar_wait(&v_full[s], (it / STAGES) & 1, p.err, ERR_WAIT_FULL);
 #pragma unroll
       for (int m = 0; m < 2; ++m) {
-        if (ok) ok = mbar_wait(&p_full[m], it & 1, p.err, ERR_WAIT_MISC);
+        if (ok) ok = mbar_wait(&p_full[2 * m + (it & 1)], (it >> 1) & 1, p.err, ERR_WAIT_MISC);
         if (!ok) break;
         tc_fence_after();
         if (lane == 0) {
@@ -209,7 +209,7 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
                           (it > 0 || term > 0 || k4 > 0) ? 1u : 0u);
           }
           if (m == 1) umma_commit(&kv_empty[s]);
-          umma_commit(&pv_done[m]);
+          umma_commit(&pv_done[2 * m + (it & 1)]);
         }
         __syncwarp();
       }
@@ -267,7 +267,7 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       l = l * corr + ((ps[0] + ps[1]) + (ps[2] + ps[3]));
       m = m_new;
       if (it > 0 && __any_sync(0xffffffff, grow)) {
-        ok = mbar_wait(&pv_done[map], (it - 1) & 1, p.err, ERR_WAIT_MISC);
+        ok = mbar_wait(&pv_done[sb ^ 1], ((it - 1) >> 1) & 1, p.err, ERR_WAIT_MISC);
         if (!ok) break;
         tc_fence_after();
 #pragma unroll
@@ -292,12 +292,10 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       tmem_st32(tmem_base + lane_addr + sb * DF_BN + 32, w);
       tmem_st_wait();
       tc_fence_before();
-      mbar_arrive(&p_full[map]);
+      mbar_arrive(&p_full[sb]);
     }
-    // S of the last tile waited for the product two tiles back only: wait for the last two in turn, a parity does not tell
-    // phases two apart
-    if (ok && ntiles > 1) ok = mbar_wait(&pv_done[map], ntiles & 1, p.err, ERR_WAIT_MISC);
-    if (ok) ok = mbar_wait(&pv_done[map], (ntiles - 1) & 1, p.err, ERR_WAIT_MISC);
+    // a buffer's barrier is at most one phase ahead or behind here: its product before this one was done when S was issued
+    if (ok) ok = mbar_wait(&pv_done[2 * map + ((ntiles - 1) & 1)], ((ntiles - 1) >> 1) & 1, p.err, ERR_WAIT_MISC);
     // both accumulators are complete behind this barrier (every thread of both warpgroups arrives, whatever its waits did)
     s_inv[map * 128 + row] = l > 0.f ? 1.f / l : 0.f;
     tc_fence_before();
