@@ -44,6 +44,33 @@ struct DfParams {
   int* err;
 };
 
+// Two 32-bit numbers in a register pair: one instruction works on both.
+__device__ __forceinline__ uint64_t pair2(float lo, float hi) {
+  uint64_t v;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(v) : "f"(lo), "f"(hi));
+  return v;
+}
+__device__ __forceinline__ float2 unpair2(uint64_t v) {
+  float2 r;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+  return r;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ uint64_t add2(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+__device__ __forceinline__ float max3(float a, float b, float c) {
+  float d;
+  asm("max.f32 %0, %1, %2, %3;" : "=f"(d) : "f"(a), "f"(b), "f"(c));
+  return d;
+}
+
 __device__ __forceinline__ void df_sync_softmax() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
 
 template <int DQ, int DV>
@@ -74,7 +101,7 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   uint64_t* v_full = k_full + STAGES;                     // STAGES
   uint64_t* kv_empty = v_full + STAGES;                   // STAGES
   uint64_t* s_full = kv_empty + STAGES;                   // map, buffer
-  uint64_t* p_full = s_full + 4;                          // map, buffer (128 arrivals): a map may be a tile ahead of the other
+  uint64_t* p_full = s_full + 4;                          // map, buffer (an arrival per warp): a map may be a tile ahead of the other
   uint64_t* pv_done = p_full + 4;                         // map, buffer
   uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(pv_done + 4);
   float* s_inv = reinterpret_cast<float*>(smem_raw + Geo::BARS + 256);   // map, row
@@ -105,7 +132,7 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     }
     for (int i = 0; i < 4; ++i) {
       mbar_init(&s_full[i], 1);
-      mbar_init(&p_full[i], 128);
+      mbar_init(&p_full[i], 4);
       mbar_init(&pv_done[i], 1);
     }
     fence_barrier_init();
@@ -164,6 +191,10 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     // ------------------------------------------------------------------ MMA issuer
     constexpr uint32_t idesc_s = make_idesc(DF_BM, DF_BN, 1, 1, 0, 0);
     constexpr uint32_t idesc_o = make_idesc(DF_BM, DV, 1, 1, 0, 1);
+    // descriptors of the first operands; the others are a distance away (the address is their lowest field, in 16-byte units)
+    const uint64_t q_desc = make_smem_desc_sw128(smem_u32(sQ), 16, 1024), kv_desc = make_smem_desc_sw128(smem_u32(sKV), 16, 1024);
+    const uint64_t v_desc = make_smem_desc_sw128(smem_u32(sKV + Geo::K_BYTES), DF_CHUNK, 1024);
+    const bool leader = elect_one();
     bool ok = mbar_wait(q_full, 0, p.err, ERR_WAIT_FULL);
     auto issue_s = [&](int it) -> bool {
       const int s = it % STAGES, sb = it & 1;
@@ -172,13 +203,13 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       for (int m = 0; m < 2; ++m) {
         if (it >= 2 && !mbar_wait(&pv_done[2 * m + sb], ((it - 2) >> 1) & 1, p.err, ERR_WAIT_TMEM_EMPTY)) return false;   // P of it - 2
         tc_fence_after();
-        if (lane == 0) {
-          const uint32_t qa = smem_u32(sQ + m * NCH * DF_BM * 128), ka = smem_u32(sKV + s * Geo::STAGE + m * NCH * DF_CHUNK);
+        const uint64_t qd = q_desc + (m * NCH * DF_BM * 128 >> 4);
+        const uint64_t kd = kv_desc + (s * Geo::STAGE + m * NCH * DF_CHUNK >> 4);
+        if (leader) {
 #pragma unroll
           for (int k4 = 0; k4 < DQ / 16; ++k4)
-            umma_f16(tmem_base + (2 * m + sb) * DF_BN,
-                     make_smem_desc_sw128(qa + (k4 >> 2) * DF_BM * 128 + (k4 & 3) * 32, 16, 1024),
-                     make_smem_desc_sw128(ka + (k4 >> 2) * DF_CHUNK + (k4 & 3) * 32, 16, 1024), idesc_s, k4 > 0 ? 1u : 0u);
+            umma_f16(tmem_base + (2 * m + sb) * DF_BN, qd + ((k4 >> 2) * DF_BM * 128 + (k4 & 3) * 32 >> 4),
+                     kd + ((k4 >> 2) * DF_CHUNK + (k4 & 3) * 32 >> 4), idesc_s, k4 > 0 ? 1u : 0u);
           umma_commit(&s_full[2 * m + sb]);
         }
         __syncwarp();
@@ -198,14 +229,14 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         if (ok) ok = mbar_wait(&p_full[2 * m + (it & 1)], (it >> 1) & 1, p.err, ERR_WAIT_MISC);
         if (!ok) break;
         tc_fence_after();
-        if (lane == 0) {
-          const uint32_t va = smem_u32(sKV + s * Geo::STAGE + Geo::K_BYTES);
+        const uint64_t vd = v_desc + (s * Geo::STAGE >> 4);
+        const uint32_t pa = tmem_base + (2 * m + (it & 1)) * DF_BN;
+        if (leader) {
 #pragma unroll
           for (int term = 0; term < 2; ++term) {
-            const uint32_t pa = tmem_base + (2 * m + (it & 1)) * DF_BN + term * 32;
 #pragma unroll
             for (int k4 = 0; k4 < DF_BN / 16; ++k4)
-              umma_f16_ts(tmem_o + m * DV, pa + k4 * 8, make_smem_desc_sw128(va + k4 * 2048, DF_CHUNK, 1024), idesc_o,
+              umma_f16_ts(tmem_o + m * DV, pa + term * 32 + k4 * 8, vd + (k4 * 2048 >> 4), idesc_o,
                           (it > 0 || term > 0 || k4 > 0) ? 1u : 0u);
           }
           if (m == 1) umma_commit(&kv_empty[s]);
@@ -230,26 +261,29 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       if (!ok) break;
       tc_fence_after();
       float sv[DF_BN];
-#pragma unroll
-      for (int c = 0; c < DF_BN / 32; ++c) {
-        uint32_t r[32];
-        tmem_ld32(tmem_base + lane_addr + sb * DF_BN + c * 32, r);
+      {
+        uint32_t r0[32], r1[32];         // both loads in flight
+        tmem_ld32(tmem_base + lane_addr + sb * DF_BN, r0);
+        tmem_ld32(tmem_base + lane_addr + sb * DF_BN + 32, r1);
         tmem_ld_wait();
 #pragma unroll
-        for (int j = 0; j < 32; ++j) sv[c * 32 + j] = __uint_as_float(r[j]);
+        for (int j = 0; j < 32; ++j) {
+          sv[j] = __uint_as_float(r0[j]);
+          sv[32 + j] = __uint_as_float(r1[j]);
+        }
       }
       const int kbase = it * DF_BN;
       if (kbase + DF_BN - 1 > pi) {
 #pragma unroll
         for (int j = 0; j < DF_BN; ++j) sv[j] = kbase + j <= pi ? sv[j] : -FLT_MAX;
       }
-      // with two warps on a scheduler the length of a dependent chain counts: eight maxima and four sums at a time
-      float mx8[8];
+      // four maxima at a time (chains are short), three operands an instruction
+      float mx4[4];
 #pragma unroll
-      for (int j = 0; j < 8; ++j) mx8[j] = sv[j];
+      for (int j = 0; j < 4; ++j) mx4[j] = max3(sv[3 * j], sv[3 * j + 1], sv[3 * j + 2]);
 #pragma unroll
-      for (int j = 8; j < DF_BN; ++j) mx8[j & 7] = fmaxf(mx8[j & 7], sv[j]);
-      float mx = fmaxf(fmaxf(fmaxf(mx8[0], mx8[1]), fmaxf(mx8[2], mx8[3])), fmaxf(fmaxf(mx8[4], mx8[5]), fmaxf(mx8[6], mx8[7])));
+      for (int j = 12; j < DF_BN; j += 2) mx4[(j >> 1) & 3] = max3(mx4[(j >> 1) & 3], sv[j], sv[j + 1]);
+      float mx = fmaxf(max3(mx4[0], mx4[1], mx4[2]), mx4[3]);
       if (mx != -FLT_MAX) mx *= sl2;       // log2 domain (the scale is positive)
       // the running maximum moves only when the tile exceeds it by more than 2^8, so the accumulator in tensor memory
       // is rescaled on few tiles; the probabilities then reach at most 256
@@ -258,13 +292,17 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       const float m_new = grow ? m_cand : m;
       const float m_use = m_new == -FLT_MAX ? 0.f : m_new;
       const float corr = grow ? ex2(m - m_use) : 1.f;
-      float ps[4] = {0.f, 0.f, 0.f, 0.f};
+      const uint64_t sl2x2 = pair2(sl2, sl2), m2 = pair2(-m_use, -m_use), minus1 = pair2(-1.f, -1.f);
+      uint64_t ps[4] = {0, 0, 0, 0};
 #pragma unroll
-      for (int j = 0; j < DF_BN; ++j) {
-        sv[j] = ex2(fmaf(sv[j], sl2, -m_use));           // masked scores underflow to exactly 0
-        ps[j & 3] += sv[j];
+      for (int j = 0; j < DF_BN / 2; ++j) {
+        const float2 x = unpair2(fma2(pair2(sv[2 * j], sv[2 * j + 1]), sl2x2, m2));
+        sv[2 * j] = ex2(x.x);                            // masked scores underflow to exactly 0
+        sv[2 * j + 1] = ex2(x.y);
+        ps[j & 3] = add2(ps[j & 3], pair2(sv[2 * j], sv[2 * j + 1]));
       }
-      l = l * corr + ((ps[0] + ps[1]) + (ps[2] + ps[3]));
+      const float2 sum = unpair2(add2(add2(ps[0], ps[1]), add2(ps[2], ps[3])));
+      l = l * corr + (sum.x + sum.y);
       m = m_new;
       if (it > 0 && __any_sync(0xffffffff, grow)) {
         ok = mbar_wait(&pv_done[sb ^ 1], ((it - 1) >> 1) & 1, p.err, ERR_WAIT_MISC);
@@ -286,13 +324,16 @@ diff_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       for (int j = 0; j < 32; ++j) w[j] = pack_bf16x2(sv[2 * j], sv[2 * j + 1]);
       tmem_st32(tmem_base + lane_addr + sb * DF_BN, w);
 #pragma unroll
-      for (int j = 0; j < 32; ++j)
-        w[j] = pack_bf16x2(sv[2 * j] - bf16_bits_to_float(static_cast<uint16_t>(w[j] & 0xffff)),
-                           sv[2 * j + 1] - bf16_bits_to_float(static_cast<uint16_t>(w[j] >> 16)));
+      for (int j = 0; j < 32; ++j) {
+        const float2 r = unpair2(fma2(pair2(__uint_as_float(w[j] << 16), __uint_as_float(w[j] & 0xffff0000u)), minus1,
+                                      pair2(sv[2 * j], sv[2 * j + 1])));
+        w[j] = pack_bf16x2(r.x, r.y);
+      }
       tmem_st32(tmem_base + lane_addr + sb * DF_BN + 32, w);
       tmem_st_wait();
       tc_fence_before();
-      mbar_arrive(&p_full[sb]);
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&p_full[sb]);
     }
     // a buffer's barrier is at most one phase ahead or behind here: its product before this one was done when S was issued
     if (ok) ok = mbar_wait(&pv_done[2 * map + ((ntiles - 1) & 1)], ((ntiles - 1) >> 1) & 1, p.err, ERR_WAIT_MISC);
