@@ -33,8 +33,9 @@ NVCC_FLAGS = [
     "--expt-relaxed-constexpr",
 ]
 # sources of models that promise 32-bit arithmetic where they say so: compiled without the approximate math functions
-EXACT_MATH = {"depth_average", "diff_attention", "diff_prefill", "latent_attention", "matrix_memory", "matrix_memory_chunk",
-              "moe_serve", "router", "sandwich_norm", "stream_mix", "window_attention", "window_prefill"}
+EXACT_MATH = {"conv_norm", "depth_average", "diff_attention", "diff_prefill", "latent_attention", "matrix_memory",
+              "matrix_memory_chunk", "moe_serve", "router", "sandwich_norm", "scored_attention", "scored_prefill", "stream_mix",
+              "window_attention", "window_prefill"}
 # sources one served architecture needs: ``ensure_kernels`` builds only these when the full library is not there
 KERNEL_SETS = {
     "nafitar": ("comm", "elementwise", "gemm_skinny", "gemm_tcgen05", "gemm_wide", "matrix_memory", "matrix_memory_chunk",
@@ -45,6 +46,9 @@ KERNEL_SETS = {
     "lobutar": ("attention_fwd", "comm", "diff_attention", "diff_prefill", "elementwise", "gemm_skinny", "gemm_tcgen05",
                 "gemm_wide", "latent_attention", "mla_decode", "moe_serve", "router", "sample_filtered", "sandwich_norm",
                 "stream_mix", "vocab", "window_attention"),
+    "rezulorn": ("comm", "conv_norm", "elementwise", "gemm_skinny", "gemm_tcgen05", "gemm_wide", "matrix_memory",
+                 "matrix_memory_chunk", "moe_serve", "sample_filtered", "scored_attention", "scored_prefill", "vocab",
+                 "window_attention"),
 }
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-Wall", "-pthread"]
 

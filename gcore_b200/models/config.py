@@ -7,7 +7,8 @@ from dataclasses import dataclass, field, fields
 from typing import Tuple, Any, Dict, List, Optional
 
 from .layer_plan import (DenseSpec, DifferentialAttentionSpec, ExpertsSpec, LatentAttentionSpec, LayerPlan,
-                         ParallelLayerSpec, StreamLayerSpec, kedesun_plan, lobutar_plan, nafitar_plan)
+                         ParallelLayerSpec, StreamLayerSpec, kedesun_plan, lobutar_plan, nafitar_plan,
+                         rezulorn_plan)
 
 
 @dataclass
@@ -194,7 +195,7 @@ class ModelConfig:
 
 MODEL_ARCH = ("llama", "llama4", "qwen2", "qwen2_5_vl", "qwen3", "qwen3_moe", "qwen3_vl", "qwen3_vl_moe", "qwen2_moe",
               "qwen2_vl", "deepseek_v3", "mistral", "gemma3_text", "seed_oss", "gpt_oss", "nafitar",
-              "kedesun", "lobutar")
+              "kedesun", "lobutar", "rezulorn")
 
 PRESETS: Dict[str, Dict[str, Any]] = {
     # tiny Llama-style decoder
@@ -267,8 +268,21 @@ def from_lobutar_config(conf: Dict[str, Any], dtype: str = "bfloat16") -> ModelC
                        max_position_embeddings=ROTARY_POSITIONS, dtype=dtype, layer_plan=plan)
 
 
+def from_rezulorn_config(conf: Dict[str, Any], dtype: str = "bfloat16") -> ModelConfig:
+    """Maps a Rezulorn ``config.json`` (``architecture``, ``canon``, ``layers``, ``logit_scale``, ``norm``, ``residual_mult``,
+    ``vocab``, ``width``)."""
+    plan = rezulorn_plan(conf)
+    m = plan.layers[0].mixers[0]
+    ffn = next((sp.ffn for sp in plan.layers if sp.ffn is not None), None)
+    return ModelConfig(arch="rezulorn", num_layers=len(plan.layers), hidden_size=conf["width"], num_attention_heads=m.heads,
+                       num_kv_heads=getattr(m, "kv_heads", m.heads), head_dim=m.dim, ffn_hidden_size=ffn.ff if ffn else 0,
+                       vocab_size=conf["vocab"], rms_norm_eps=float(conf["norm"]["eps"]),
+                       max_position_embeddings=ROTARY_POSITIONS, dtype=dtype, layer_plan=plan)
+
+
 # architectures whose config.json names them in ``architecture``: reader of that file
-ARCH_READERS = {"nafitar": from_nafitar_config, "kedesun": from_kedesun_config, "lobutar": from_lobutar_config}
+ARCH_READERS = {"nafitar": from_nafitar_config, "kedesun": from_kedesun_config, "lobutar": from_lobutar_config,
+                "rezulorn": from_rezulorn_config}
 
 
 def from_hf_config(hf: Dict[str, Any]) -> ModelConfig:

@@ -5,9 +5,10 @@ layers one by one - which mixers a layer runs, the size of each, its feed-forwar
 shared weights.  Every run of a layer (a looped layer counts once per pass) owns its cache and state, so the serving engine
 sizes both from ``LayerPlan.runs``.
 
-Three kinds of layer are described: ``LayerSpec`` (two mixers side by side, then a feed-forward, norms before and after
-each), ``ParallelLayerSpec`` (one mixer and a feed-forward that read the same normed input) and ``StreamLayerSpec`` (a mixer,
-then a feed-forward, each reading a mixture of several residual streams and writing to all of them)."""
+Four kinds of layer are described: ``LayerSpec`` (two mixers side by side, then a feed-forward, norms before and after
+each), ``ParallelLayerSpec`` (one mixer and a feed-forward that read the same normed input), ``StreamLayerSpec`` (a mixer,
+then a feed-forward, each reading a mixture of several residual streams and writing to all of them) and ``ConvLayerSpec`` (one
+mixer or a weighted sum of several, then a feed-forward, each behind a norm and a short convolution over time)."""
 from __future__ import annotations
 
 import math
@@ -75,18 +76,28 @@ class YarnSpec:
 
 @dataclass(frozen=True)
 class RotarySpec:
-    """Rotation of ``dims`` dimensions, neighbours paired (2i with 2i + 1), angle = position * base^(-2i/dims)."""
+    """Rotation of ``dims`` dimensions, angle = position * base^(-2i/dims) / ``slow``.  Pair i is two neighbours (2i with
+    2i + 1) or, with ``halves``, dimension i and dimension i + dims/2."""
     dims: int
     base: float
     scaling: Optional[YarnSpec] = None
+    slow: float = 1.0
+    halves: bool = False
 
     def __post_init__(self):
-        if self.dims < 2 or self.dims % 2 or self.base <= 1:
-            raise ValueError("a rotation needs an even number of dimensions and a base above 1")
+        if self.dims < 2 or self.dims % 2 or self.base <= 1 or self.slow <= 0:
+            raise ValueError("a rotation needs an even number of dimensions, a base above 1 and a positive scaling")
+
+    def neighbours(self, dim: int) -> List[int]:
+        """Order of a head's ``dim`` dimensions in which pair i is 2i with 2i + 1.  Applied to queries and keys alike it
+        changes neither their products nor their norms."""
+        n = self.dims
+        turned = [i // 2 + (i % 2) * (n // 2) for i in range(n)] if self.halves else list(range(n))
+        return turned + list(range(n, dim))
 
     def frequencies(self) -> List[float]:
         n, sc = self.dims, self.scaling
-        freq = [self.base ** (-2.0 * i / n) for i in range(n // 2)]
+        freq = [self.base ** (-2.0 * i / n) / self.slow for i in range(n // 2)]
         if sc is None:
             return freq
 
@@ -150,24 +161,70 @@ class DifferentialAttentionSpec:
 
 
 @dataclass(frozen=True)
+class ScoredAttentionSpec:
+    """Grouped-query attention with a bias on every score.  Queries and keys may be rotated (``rot``) and then divided by
+    their root mean square (``unit``).  ``weights``: "softmax" of the scores, or "sigmoid" of each, not normalised over the
+    keys.  ``distance``: two learned numbers per head take ``r1 * ln(1 + r2 * (i - j))`` off a score; ``head_bias``: a learned
+    number per head is added to it.  ``window`` (0: none): position i sees j with ``0 <= i - j < window``, and the first
+    ``keep`` positions."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    weights: str = "softmax"
+    rot: Optional[RotarySpec] = None
+    unit: bool = False
+    distance: bool = False
+    head_bias: bool = False
+    window: int = 0
+    keep: int = 0
+
+    def __post_init__(self):
+        if self.heads < 1 or self.kv_heads < 1 or self.heads % self.kv_heads:
+            raise ValueError("query heads must be a positive multiple of the key/value heads")
+        if min(self.dim, self.vdim) < 1 or (self.rot is not None and self.rot.dims > self.dim):
+            raise ValueError("attention sizes must be positive and hold the rotated dimensions")
+        if min(self.window, self.keep) < 0:
+            raise ValueError("a window and its kept positions must not be negative")
+        if self.weights not in ("softmax", "sigmoid"):
+            raise ValueError(f"unknown attention weights {self.weights!r}")
+
+
+@dataclass(frozen=True)
 class RetentionSpec:
-    """Linear attention with one fixed decay per head: a ``dim x vdim`` state per head in 32-bit."""
+    """Linear attention with one fixed decay per head: a ``dim x vdim`` state per head in 32-bit.  Queries and keys may be
+    rotated (``rot``); ``act``: "silu" on queries, keys and values, or "".  The output is normed per "head" or over all heads
+    together ("joint", with a gain), and gated by a "silu" or "sigmoid"; ``scale``: factor of a query-key product."""
     heads: int
     dim: int
     vdim: int
     decay: Tuple[float, ...]
+    scale: Optional[float] = None        # default: dim^-1/2
+    rot: Optional[RotarySpec] = None
+    act: str = ""
+    norm: str = "head"
+    gate: str = "silu"
 
     def __post_init__(self):
         if min(self.heads, self.dim, self.vdim) < 1 or len(self.decay) != self.heads:
             raise ValueError("retention needs positive sizes and one decay per head")
         if not all(0 <= d <= 1 for d in self.decay):
             raise ValueError("retention decays must lie in [0, 1]")
+        if self.act not in ("", "silu") or (self.norm, self.gate) not in (("head", "silu"), ("joint", "sigmoid")):
+            raise ValueError(f"unknown retention activation {self.act!r}, norm {self.norm!r} or gate {self.gate!r}")
+        if self.rot is not None and (self.rot.dims > self.dim or self.act):
+            raise ValueError("rotated dimensions must lie in the head, and go without an activation")
+
+    def product_scale(self) -> float:
+        return self.dim ** -0.5 if self.scale is None else self.scale
 
 
 @dataclass(frozen=True)
 class DenseSpec:
-    """Gated feed-forward: ``down(silu(gate h) * up h)``."""
+    """Feed-forward: ``down(silu(gate h) * up h)`` ("silu_gate") or ``down(relu(up h)^2)`` ("relu2")."""
     ff: int
+    act: str = "silu_gate"
 
 
 @dataclass(frozen=True)
@@ -216,6 +273,19 @@ class StreamLayerSpec:
 
 
 @dataclass(frozen=True)
+class ConvLayerSpec:
+    """One layer: the sum of ``mixers`` times their ``scales``, then a feed-forward (None: none), each behind a norm and a short
+    causal convolution over time."""
+    mixers: Tuple[Union[ScoredAttentionSpec, RetentionSpec], ...]
+    scales: Tuple[float, ...]
+    ffn: Optional[DenseSpec] = None
+
+    def __post_init__(self):
+        if not self.mixers or len(self.mixers) != len(self.scales):
+            raise ValueError("a layer needs a mixer, and one scale per mixer")
+
+
+@dataclass(frozen=True)
 class LayerRun:
     """One execution of a layer: ``index`` numbers the runs (= the cache / state set), ``layer`` names the weights.
     ``opens_pass`` is the pass number when this run is the first of a pass of the loop, else None."""
@@ -228,13 +298,16 @@ class LayerRun:
 class LayerPlan:
     """``layers``: the layers that own weights.  They run in order, with a looped range, or, with ``order``, as it lists them
     (a layer may run any number of times).  ``names``: the layers' numbers in the checkpoint when they are not 0, 1, ..."""
-    layers: Tuple[Union[LayerSpec, ParallelLayerSpec, StreamLayerSpec], ...]
+    layers: Tuple[Union[LayerSpec, ParallelLayerSpec, StreamLayerSpec, ConvLayerSpec], ...]
     loop_start: int = 0
     loop_stop: int = 0
     loop_times: int = 0          # 0: no loop
     order: Tuple[int, ...] = ()
     names: Tuple[int, ...] = ()
     streams: int = 0             # residual streams of a decoder with hyper-connections
+    taps: int = 0                # taps of the convolution in front of every sublayer
+    residual_mult: float = 1.0   # factor of what a sublayer adds to the residual
+    logit_scale: float = 1.0
 
     def __post_init__(self):
         if not self.layers:
@@ -385,6 +458,58 @@ def lobutar_plan(conf: Dict[str, Any]) -> LayerPlan:
     if streams < 1:
         raise ValueError("a decoder needs at least one residual stream")
     return LayerPlan(tuple(layers), order=tuple(names.index(j) for j in owner), names=tuple(names), streams=streams)
+
+
+def _halves_rotation(d: Dict[str, Any], where: str) -> RotarySpec:
+    sc = d.get("scaling")
+    return RotarySpec(dims=_need(d, "dims", where), base=float(_need(d, "base", where)), halves=True,
+                      slow=float(_need(sc, "factor", where + ".scaling")) if sc else 1.0)
+
+
+def _distance_attention(m: Dict[str, Any], where: str) -> ScoredAttentionSpec:
+    mask = _need(m, "mask", where)
+    if _need(mask, "size", where + ".mask") < 1:
+        raise ValueError(f"{where}.mask: the window must be positive")
+    return ScoredAttentionSpec(distance=True, window=mask["size"], keep=_need(mask, "keep_first", where + ".mask"),
+                               scale=float(_need(m, "scale", where)),
+                               **{k: _need(m, k, where) for k in ("heads", "kv_heads", "dim", "vdim")})
+
+
+def _sigmoid_attention(m: Dict[str, Any], where: str) -> ScoredAttentionSpec:
+    return ScoredAttentionSpec(weights="sigmoid", unit=True, head_bias=True, scale=float(_need(m, "scale", where)),
+                               rot=_halves_rotation(_need(m, "rot", where), where + ".rot"),
+                               **{k: _need(m, k, where) for k in ("heads", "kv_heads", "dim", "vdim")})
+
+
+def _conv_mixers(kind: str, m: Dict[str, Any], where: str):
+    """Mixers of a layer of ``kind`` and their scales."""
+    if kind == "attention":
+        return (_distance_attention(m, where),), (1.0,)
+    if kind == "lightning":
+        return (replace(_retention(m, where), scale=1.0, act="silu", norm="joint", gate="sigmoid"),), (1.0,)
+    if kind != "parallel":
+        raise ValueError(f"{where}: unknown mixer type {kind!r}")
+    left, right = _need(m, "left", where), _need(m, "right", where)
+    turned = replace(_retention(right, where + ".right"),
+                     rot=_halves_rotation(_need(right, "rot", where + ".right"), where + ".right.rot"))
+    return (_sigmoid_attention(left, where + ".left"), turned), tuple(float(_need(m, k, where))
+                                                                      for k in ("left_scale", "right_scale"))
+
+
+def rezulorn_plan(conf: Dict[str, Any]) -> LayerPlan:
+    """Layer plan of a Rezulorn ``config.json``."""
+    layers = []
+    for i, entry in enumerate(_need(conf, "layers", "config")):
+        where = f"layers[{i}]"
+        ffn = _feed_forward(entry.get("mlp"), where + ".mlp")
+        if ffn is not None and not isinstance(ffn, DenseSpec):
+            raise ValueError(f"{where}.mlp: unknown feed-forward kind {entry['mlp'].get('kind')!r}")
+        layers.append(ConvLayerSpec(*_conv_mixers(entry.get("type"), _need(entry, "mixer", where), where + ".mixer"),
+                                    replace(ffn, act="relu2") if ffn is not None else None))
+    taps = _need(_need(conf, "canon", "config"), "taps", "canon")
+    if taps < 1:
+        raise ValueError("the input convolution needs at least one tap")
+    return LayerPlan(tuple(layers), taps=taps, **{k: float(_need(conf, k, "config")) for k in ("residual_mult", "logit_scale")})
 
 
 def kedesun_plan(conf: Dict[str, Any]) -> LayerPlan:

@@ -11,42 +11,12 @@ import math
 import torch
 import torch.nn as nn
 
-from ..ops import depth, matrix_memory as mm, sandwich
+from ..ops import depth, sandwich
 from ..ops.gemm import linear_forward
 from .config import ModelConfig
-from .layer_plan import ExpertsSpec, LatentAttentionSpec, ParallelLayerSpec, RetentionSpec
-from .plan_decoder import CheckpointTensors, PlanDecoder, _buf, put, put_heads
-from .plan_modules import DenseFeedForward, ExpertFeedForward, LatentAttentionMixer, blocks
-
-
-class RetentionMixer(nn.Module):
-    def __init__(self, spec: RetentionSpec, width: int, eps: float, dtype, device):
-        super().__init__()
-        self.spec, self.width, self.eps = spec, width, eps
-        self.dim, self.vdim = mm.padded_key_dim(spec.dim), mm.padded_value_dim(spec.vdim)
-        H = spec.heads
-        self.at, self.columns = blocks(H * self.dim, H * self.dim, H * self.vdim, H * self.vdim)
-        self.out_columns = H * self.vdim
-        self.decay = _buf(torch.tensor(spec.decay, dtype=torch.float32, device=device))
-
-    def cache_shape(self):
-        return None
-
-    def new_state(self, slots, device):
-        return mm.MemoryState.allocate(slots, self.spec.heads, self.dim, self.vdim, device, gated=False)
-
-    def state_bytes(self):
-        return mm.MemoryState.bytes_per_slot(self.spec.heads, self.dim, self.vdim, gated=False)
-
-    def load(self, take, p: str, rows, out):
-        s, W, H = self.spec, self.width, self.spec.heads
-        for at, nm, dim, pad in zip(self.at, "qkvg", (s.dim, s.dim, s.vdim, s.vdim), (self.dim, self.dim, self.vdim, self.vdim)):
-            put_heads(rows[at:at + H * pad], take(p + nm, H * dim, W), H, dim, pad)
-        put(out.view(out.shape[0], H, self.vdim), take(p + "o", W, H * s.vdim).view(W, H, s.vdim))
-
-    def forward(self, proj, rows, cache, state, out):
-        s = self.spec
-        mm.retention(proj, *self.at, self.decay, s.dim ** -0.5, s.heads, self.dim, self.vdim, s.vdim, rows, state, self.eps, out)
+from .layer_plan import ExpertsSpec, LatentAttentionSpec, ParallelLayerSpec
+from .plan_decoder import CheckpointTensors, PlanDecoder, _buf, put
+from .plan_modules import DenseFeedForward, ExpertFeedForward, LatentAttentionMixer, RetentionMixer
 
 
 class ParallelLayer(nn.Module):

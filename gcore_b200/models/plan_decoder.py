@@ -25,7 +25,7 @@ from ..ops import sandwich
 from ..ops import window_attention as wa
 from ..ops.gemm import linear_forward
 from .config import ModelConfig
-from .layer_plan import LayerSpec, ParallelLayerSpec, StreamLayerSpec
+from .layer_plan import ConvLayerSpec, LayerSpec, ParallelLayerSpec, StreamLayerSpec
 
 
 def _up(n: int, m: int) -> int:
@@ -285,7 +285,9 @@ class SandwichDecoder(PlanDecoder):
 
 def build_decoder(cfg: ModelConfig, device=None) -> PlanDecoder:
     """The serving module of a layer-plan configuration."""
+    from .conv_decoder import ConvDecoder
     from .parallel_decoder import ParallelDecoder
     from .stream_decoder import StreamDecoder
-    cls = {ParallelLayerSpec: ParallelDecoder, StreamLayerSpec: StreamDecoder, LayerSpec: SandwichDecoder}
+    cls = {ParallelLayerSpec: ParallelDecoder, StreamLayerSpec: StreamDecoder, LayerSpec: SandwichDecoder,
+           ConvLayerSpec: ConvDecoder}
     return cls[type(cfg.layer_plan.layers[0])](cfg, device)

@@ -11,8 +11,9 @@ import math
 import torch
 import torch.nn as nn
 
-from ..ops import diff_attention as da, latent_attention as la, moe
-from .layer_plan import DenseSpec, DifferentialAttentionSpec, ExpertsSpec, LatentAttentionSpec
+from ..ops import diff_attention as da, latent_attention as la, matrix_memory as mm, moe, scored_attention as sa
+from .layer_plan import (DenseSpec, DifferentialAttentionSpec, ExpertsSpec, LatentAttentionSpec, RetentionSpec,
+                         ScoredAttentionSpec)
 from .plan_decoder import _buf, _up, put, put_heads
 
 
@@ -117,20 +118,113 @@ class DifferentialAttentionMixer(nn.Module):
         da.differential_attention(proj, self.layout, self.turns, self.lam, rows, cache, out)
 
 
+def _head_order(rot, dim: int):
+    """Dimensions of a head in the order the kernels rotate (neighbours paired), or None if that is their own order."""
+    return rot.neighbours(dim) if rot is not None and rot.halves else None
+
+
+def _take_heads(take, name: str, heads: int, dim: int, width: int, order=None):
+    t = take(name, heads * dim, width)
+    return t if order is None else t.view(heads, dim, width)[:, order].reshape(heads * dim, width)
+
+
+class ScoredAttentionMixer(nn.Module):
+    def __init__(self, spec: ScoredAttentionSpec, width: int, eps: float, dtype, device, out_scale: float = 1.0):
+        super().__init__()
+        self.spec, self.width, self.out_scale = spec, width, out_scale
+        H, G, dim, vdim = spec.heads, spec.kv_heads, _up(spec.dim, 8), _up(spec.vdim, 8)
+        (q, k, v), self.columns = blocks(H * dim, G * dim, G * vdim)
+        self.layout = sa.ScoredLayout(q=q, k=k, v=v, heads=H, kv_heads=G, dim=dim, true_dim=spec.dim, vdim=vdim, scale=spec.scale,
+                                      eps=eps, unit=spec.unit, sigmoid=spec.weights == "sigmoid", window=spec.window,
+                                      keep=spec.keep if spec.window else 0)
+        self.out_columns = H * vdim
+        f32 = dict(dtype=torch.float32, device=device)
+        self.turns = _buf(la.rotation_turns(spec.rot.frequencies()).to(device)) if spec.rot is not None else None
+        self.r1, self.r2 = (_buf(torch.zeros(H, **f32)) if spec.distance else None for _ in range(2))
+        self.head_bias = _buf(torch.zeros(H, **f32)) if spec.head_bias else None
+
+    def cache_shape(self):
+        return (self.layout.row,)
+
+    def new_state(self, slots, device):
+        return None
+
+    def state_bytes(self):
+        return 0
+
+    def load(self, take, p: str, rows, out):
+        s, ly, W = self.spec, self.layout, self.width
+        order = _head_order(s.rot, s.dim)
+        for at, nm, n, dim, pad, o in ((ly.q, "q", s.heads, s.dim, ly.dim, order), (ly.k, "k", s.kv_heads, s.dim, ly.dim, order),
+                                       (ly.v, "v", s.kv_heads, s.vdim, ly.vdim, None)):
+            put_heads(rows[at:at + n * pad], _take_heads(take, p + nm, n, dim, W, o), n, dim, pad)
+        for nm, dst in (("r1", self.r1), ("r2", self.r2), ("pb", self.head_bias)):
+            if dst is not None:
+                put(dst, take(p + nm, s.heads).float())
+        put(out.view(out.shape[0], s.heads, ly.vdim), take(p + "o", W, s.heads * s.vdim).view(W, s.heads, s.vdim))
+
+    def forward(self, proj, rows, cache, state, out):
+        sa.scored_attention(proj, self.layout, rows, cache, out, self.turns, (self.r1, self.r2) if self.spec.distance else None,
+                            self.head_bias, self.out_scale)
+
+
+class RetentionMixer(nn.Module):
+    def __init__(self, spec: RetentionSpec, width: int, eps: float, dtype, device, out_scale: float = 1.0):
+        super().__init__()
+        self.spec, self.width, self.eps, self.out_scale = spec, width, eps, out_scale
+        self.dim, self.vdim = mm.padded_key_dim(spec.dim), mm.padded_value_dim(spec.vdim)
+        H = spec.heads
+        self.at, self.columns = blocks(H * self.dim, H * self.dim, H * self.vdim, H * self.vdim)
+        self.out_columns = H * self.vdim
+        f32 = dict(dtype=torch.float32, device=device)
+        self.decay = _buf(torch.tensor(spec.decay, **f32))
+        self.turns = _buf(la.rotation_turns(spec.rot.frequencies()).to(device)) if spec.rot is not None else None
+        self.gain = _buf(torch.zeros(H * self.vdim, **f32)) if spec.norm == "joint" else None
+
+    def cache_shape(self):
+        return None
+
+    def new_state(self, slots, device):
+        return mm.MemoryState.allocate(slots, self.spec.heads, self.dim, self.vdim, device, gated=False)
+
+    def state_bytes(self):
+        return mm.MemoryState.bytes_per_slot(self.spec.heads, self.dim, self.vdim, gated=False)
+
+    def load(self, take, p: str, rows, out):
+        s, W, H = self.spec, self.width, self.spec.heads
+        order = _head_order(s.rot, s.dim)
+        for at, nm, dim, pad, o in zip(self.at, "qkvg", (s.dim, s.dim, s.vdim, s.vdim),
+                                       (self.dim, self.dim, self.vdim, self.vdim), (order, order, None, None)):
+            put_heads(rows[at:at + H * pad], _take_heads(take, p + nm, H, dim, W, o), H, dim, pad)
+        if self.gain is not None:
+            put_heads(self.gain, take(p + "norm", H * s.vdim).float(), H, s.vdim, self.vdim)
+        put(out.view(out.shape[0], H, self.vdim), take(p + "o", W, H * s.vdim).view(W, H, s.vdim))
+
+    def forward(self, proj, rows, cache, state, out):
+        s = self.spec
+        mm.retention(proj, *self.at, self.decay, s.product_scale(), s.heads, self.dim, self.vdim, s.vdim, rows, state, self.eps,
+                     out, self.turns, s.act == "silu", self.gain, self.out_scale)
+
+
 class DenseFeedForward(nn.Module):
     def __init__(self, spec: DenseSpec, width: int, width_pad: int, dtype, device):
         super().__init__()
         self.spec, self.width, self.ff = spec, width, _up(spec.ff, 8)
-        self.columns, self.out_columns = 2 * self.ff, self.ff
+        self.gated = spec.act == "silu_gate"
+        self.columns, self.out_columns = (2 if self.gated else 1) * self.ff, self.ff
 
     def load(self, take, p: str, rows, out):
         f, W = self.spec.ff, self.width
-        put(rows, take(p + "gate", f, W))
-        put(rows[self.ff:], take(p + "up", f, W))
+        if self.gated:
+            put(rows, take(p + "gate", f, W))
+        put(rows[self.columns - self.ff:], take(p + "up", f, W))
         put(out, take(p + "down", W, f))
 
     def forward(self, h, proj, out, counts):
-        moe.activate(moe.SILU_GATE, proj, self.ff, self.ff, out)
+        if self.gated:
+            moe.activate(moe.SILU_GATE, proj, self.ff, self.ff, out)
+        else:
+            moe.activate(moe.RELU2, proj, self.ff, 0, out)
         return None
 
 

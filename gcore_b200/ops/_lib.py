@@ -217,14 +217,14 @@ def _declare_kernels(lib: ctypes.CDLL):
     d("gk_sandwich_norm", [I, I, P, P, F, P])
     d("gk_swiglu_f32", [P, P, L, I, P])
     d("gk_append_keys", [P, L, L, I, P, P, I, P])
-    d("gk_window_attn", [I, I, P, P, P, F, P])
+    d("gk_window_attn", [I, I, P, P, P, P, P])
     d("gk_shared_kv_decode", [P, L, P, P, P, P, P, P, P, P, F, P])
     d("gk_shared_kv_decode_scratch", [I, I, I, I], L)
     d("gk_shared_decode_set_target_ctas", [I], None)
     d("gk_window_prefill", [P, L, P, P, P, P, P, P, P, F, P, P])
-    d("gk_matrix_memory_scan", [I, P, L, L, P, F, F, F, P])
+    d("gk_matrix_memory_scan", [I, P, L, L, P, P, P])
     d("gk_matrix_memory_chunk", [P, L, P, F, F, P])
-    d("gk_memory_output", [I, P, P, L, P, P, L, P, F, P])
+    d("gk_memory_output", [I, P, P, L, P, P, L, P, F, F, P])
     d("gk_depth_average", [I, P, L, P, F, P])
     d("gk_ffn_act", [I, I, P, P, P, P])
     d("gk_expert_rows", [P, P, P, P, P, P, P, I, I, I, I, P])
@@ -243,6 +243,16 @@ def _declare_kernels(lib: ctypes.CDLL):
     d("gk_diff_decode_scratch", [I, I, I, I, I], L)
     d("gk_diff_set_target_ctas", [I], None)
     d("gk_diff_combine", [I, I, P, L, L, P, P, P])
+    d("gk_conv_norm", [I, P, P, P, P])
+    d("gk_head_prep", [I, P, L, P, F, P])
+    d("gk_silu_columns", [I, P, L, I, I, I, P])
+    d("gk_scored_prefill", [P, P, P, P, P])
+    d("gk_scored_prefill_supported", [I, I])
+    d("gk_scored_decode", [P, P, P, P, P])
+    d("gk_scored_decode_supported", [I, I])
+    d("gk_scored_decode_scratch", [I, I, I, I, I, I, I], L)
+    d("gk_scored_set_target_ctas", [I], None)
+    d("gk_memory_output_joint", [I, P, P, L, P, P, L, P, P, P])
     d("gk_latent_prefill", [P, P, P, F, P])
     d("gk_latent_prefill_supported", [I, I, I])
     d("gk_attn_fwd", [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, I, P, P])

@@ -9,12 +9,16 @@
 // bf16 prompt portions run the chunkwise kernel in matrix_memory_chunk.cu.
 //
 // Retention is the same recurrence with constant gates and without normaliser and maximum: S_t = decay S + k v^T, output
-// S^T q, normed per head without a gain and gated by a silu.  The RET instances of the kernels compute it.
+// S^T q, normed per head without a gain and gated by a silu, or normed over all heads together with a gain and gated by a
+// sigmoid (memory_output_joint_kernel).  The RET instances of the kernels compute it.  The scan can rotate queries and keys, or
+// apply a silu to queries, keys and values, as it reads them (in 32-bit).
 //
 // State layout per layer run: S [slots, heads, dim, vdim], n [slots, heads, slices, dim], m [slots, heads, slices]: a head's
 // value columns are cut into slices of 64 that different CTAs own, and each keeps its own copy of n and m, so no CTA
 // reads what another one writes.
 #include "host_utils.h"
+#include "rotary.cuh"
+#include "row_ops.cuh"
 #include <cuda_bf16.h>
 #include <type_traits>
 
@@ -22,6 +26,7 @@ namespace gk {
 
 constexpr int MM_SLICE = 64;
 constexpr int MM_THREADS = 256;
+constexpr int MM_MAX_ROT = 512;
 
 __device__ __forceinline__ float mm_f(float v) { return v; }
 __device__ __forceinline__ float mm_f(__nv_bfloat16 v) { return __bfloat162float(v); }
@@ -66,8 +71,10 @@ struct ScanParams {
   int g_off, vdim_true;    // FINISH
   float eps;               // FINISH
   const float* decay;      // RET: [heads]; gates, n and m are absent
+  const float2* turns;     // RET: [rot / 2] turns per position (value, remainder): leading dimensions rotated, neighbours paired
+  int rot, act;            // RET: act: silu on queries, keys and values
   int width, heads, dim, vdim, slices;
-  float cap, q_scale;
+  float cap, q_scale, out_scale;
 };
 
 __device__ __forceinline__ void mm_cluster_arrive() { asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory"); }
@@ -82,6 +89,7 @@ __device__ __forceinline__ void mm_st1(float* p, float v) { *p = v; }
 __device__ __forceinline__ void mm_st1(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
 
 __device__ __forceinline__ float mm_gate(float g, bool silu) { return (silu ? g : 1.f) / (1.f + expf(-g)); }
+__device__ __forceinline__ float mm_silu(float g) { return g / (1.f + expf(-g)); }
 
 // grid (heads * slices, segments).  Thread (warp w, lane): rows rg, rg + 16, ... with rg = 2 w + lane / 16; columns
 // 4 * (lane % 16) .. + 3 of the slice.  R = rows per thread.
@@ -92,6 +100,7 @@ __global__ void __launch_bounds__(MM_THREADS, R <= 8 ? 3 : R <= 16 ? 2 : 1) matr
   __shared__ float gred[2][8];
   __shared__ float peer_ss[8];      // FINISH: sum of squares of every slice of the head
   __shared__ float warp_ss[2];
+  __shared__ float s_cos[RET ? 8 * R : 1], s_sin[RET ? 8 * R : 1];   // rot / 2 of them
   pdl_launch_dependents();
   pdl_wait();
   const int head = blockIdx.x / p.slices, slice = blockIdx.x % p.slices, seg = blockIdx.y;
@@ -145,12 +154,29 @@ __global__ void __launch_bounds__(MM_THREADS, R <= 8 ? 3 : R <= 16 ? 2 : 1) matr
   for (int row = r_beg, it = 0; row < r_end; ++row, ++it) {
     const int buf = it & 1;
     const T* pr = p.proj + row * p.ld;
+    const T *qr = pr + p.q_off + static_cast<long long>(head) * p.dim, *kr = pr + p.k_off + static_cast<long long>(head) * p.dim;
+    if (RET && p.rot) {
+      __syncthreads();       // the row before has read its angles
+      for (int i = tid; i < p.rot >> 1; i += MM_THREADS) rotation_at(p.first_pos[seg] + it, p.turns[i], &s_sin[i], &s_cos[i]);
+      __syncthreads();
+    }
     for (int d = tid; d < 16 * R; d += MM_THREADS) {
-      sq[buf][d] = d < p.dim ? mm_f(pr[p.q_off + static_cast<long long>(head) * p.dim + d]) * p.q_scale : 0.f;
-      sk[buf][d] = d < p.dim ? mm_f(pr[p.k_off + static_cast<long long>(head) * p.dim + d]) : 0.f;
+      float q = d < p.dim ? mm_f(qr[d]) : 0.f, k = d < p.dim ? mm_f(kr[d]) : 0.f;
+      if (RET && d < p.rot) {
+        const float c = s_cos[d >> 1], s = d & 1 ? s_sin[d >> 1] : -s_sin[d >> 1];
+        q = q * c + mm_f(qr[d ^ 1]) * s;
+        k = k * c + mm_f(kr[d ^ 1]) * s;
+      }
+      if (RET && p.act) {
+        q = mm_silu(q);
+        k = mm_silu(k);
+      }
+      sq[buf][d] = q * p.q_scale;
+      sk[buf][d] = k;
     }
     float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
     if (live) v = mm_ld4(pr + p.v_off + static_cast<long long>(head) * p.vdim + col);
+    if (RET && p.act) v = make_float4(mm_silu(v.x), mm_silu(v.y), mm_silu(v.z), mm_silu(v.w));
     float gi = 0.f, gf = 0.f;
     if (RET) {
     } else if (p.gates) {
@@ -245,7 +271,8 @@ __global__ void __launch_bounds__(MM_THREADS, R <= 8 ? 3 : R <= 16 ? 2 : 1) matr
         float ss = 0.f;
         for (int x = 0; x < p.slices; ++x) ss += peer_ss[x];
         const float r = 1.f / sqrtf(ss / p.vdim_true + p.eps);
-        mm_st1(p.y + row * p.y_ld + static_cast<long long>(head) * p.vdim + oc, o * r * gain * mm_gate(gate, RET));
+        mm_st1(p.y + row * p.y_ld + static_cast<long long>(head) * p.vdim + oc,
+               o * r * gain * mm_gate(gate, RET) * p.out_scale);
       }
     }
   }
@@ -258,7 +285,7 @@ template <typename T>
 __global__ void __launch_bounds__(256) memory_output_kernel(const float* __restrict__ o, const T* __restrict__ proj,
                                                             long long ld, int g_off, const float* __restrict__ gain,
                                                             T* __restrict__ y, long long y_ld, int rows, int heads, int vdim,
-                                                            int vdim_true, float eps) {
+                                                            int vdim_true, float eps, float out_scale) {
   pdl_launch_dependents();
   pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -274,7 +301,7 @@ __global__ void __launch_bounds__(256) memory_output_kernel(const float* __restr
   }
 #pragma unroll
   for (int s = 16; s > 0; s >>= 1) ss += __shfl_xor_sync(0xffffffff, ss, s);
-  const float r = 1.f / sqrtf(ss / vdim_true + eps);
+  const float r = out_scale / sqrtf(ss / vdim_true + eps);
   for (int c = lane * 4; c < vdim; c += 128) {
     const float4 v = *reinterpret_cast<const float4*>(src + c);
     const float4 g = mm_ld4(proj + row * ld + g_off + static_cast<long long>(head) * vdim + c);
@@ -282,6 +309,42 @@ __global__ void __launch_bounds__(256) memory_output_kernel(const float* __restr
     mm_st4(y + row * y_ld + static_cast<long long>(head) * vdim + c, v.x * r * w.x / (1.f + expf(-g.x)),
            v.y * r * w.y / (1.f + expf(-g.y)), v.z * r * w.z / (1.f + expf(-g.z)), v.w * r * w.w / (1.f + expf(-g.w)));
   }
+}
+
+// y = o / rms(o over all heads) * gain * sigmoid(g) * out_scale.  One CTA per row; cols = heads * vdim, of which cols_true are in
+// use (the others are zero).
+template <typename T>
+__global__ void __launch_bounds__(256) memory_output_joint_kernel(const float* __restrict__ o, const T* __restrict__ proj,
+                                                                  long long ld, int g_off, const float* __restrict__ gain,
+                                                                  T* __restrict__ y, long long y_ld, int cols, int cols_true,
+                                                                  float eps, float out_scale) {
+  __shared__ float red[64];
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long row = blockIdx.x;
+  const float* src = o + row * cols;
+  constexpr int KEEP = 4;              // groups a thread holds between the two passes; the rest are read again
+  float4 v[KEEP];
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k) {
+    const int c = (threadIdx.x + k * 256) * 4;
+    v[k] = c < cols ? ld4(src + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    ss += sq4(v[k]);
+  }
+  for (int c = (threadIdx.x + KEEP * 256) * 4; c < cols; c += 1024) ss += sq4(ld4(src + c));
+  const float r = out_scale / sqrtf(block_sum2(ss, 0.f, red).x / cols_true + eps);
+  auto put = [&](int c, const float4& a) {
+    const float4 g = mm_ld4(proj + row * ld + g_off + c), w = ld4(gain + c);
+    mm_st4(y + row * y_ld + c, a.x * r * w.x / (1.f + expf(-g.x)), a.y * r * w.y / (1.f + expf(-g.y)),
+           a.z * r * w.z / (1.f + expf(-g.z)), a.w * r * w.w / (1.f + expf(-g.w)));
+  };
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k) {
+    const int c = (threadIdx.x + k * 256) * 4;
+    if (c < cols) put(c, v[k]);
+  }
+  for (int c = (threadIdx.x + KEEP * 256) * 4; c < cols; c += 1024) put(c, ld4(src + c));
 }
 
 template <typename T, int R, bool RET>
@@ -325,16 +388,20 @@ int launch_scan(const ScanParams<T>& p, int segments, cudaStream_t st) {
 
 using namespace gk;
 
-// ptrs: {proj, h, gate_w, gates, gate_b, cu, first_pos, slots, S, n, m, out, y, gain, decay}; y (finished output, one row
-// per segment, at most 512 value columns, rows y_ld apart) replaces out; decay (retention) replaces h to gate_b, n, m, gain.
-// dims: {segments, q_off, k_off, v_off, width, heads, dim, vdim, g_off, vdim_true}
-GK_EXPORT int gk_matrix_memory_scan(int is_fp32, void* const* ptrs, long long ld, long long y_ld, const int* dims, float cap,
-                                    float q_scale, float eps, void* stream) {
+// ptrs: {proj, h, gate_w, gates, gate_b, cu, first_pos, slots, S, n, m, out, y, gain, decay, turns}; y (finished output, one
+// row per segment, at most 512 value columns, rows y_ld apart) replaces out; decay (retention) replaces h to gate_b, n, m, gain;
+// turns: retention with rot.  dims: {segments, q_off, k_off, v_off, width, heads, dim, vdim, g_off, vdim_true, rot, act}
+// floats: {cap, q_scale, eps, out_scale}
+GK_EXPORT int gk_matrix_memory_scan(int is_fp32, void* const* ptrs, long long ld, long long y_ld, const int* dims,
+                                    const float* floats, void* stream) {
   if (dims[0] == 0) return 0;
   const bool ret = ptrs[14] != nullptr;
   if (dims[7] % 4 || ld % 4 || dims[3] % 4 || (!ret && !ptrs[3] && dims[4] % 4)) return -1;
   if (ptrs[12] && (ptrs[5] || dims[7] > 8 * MM_SLICE || (!ret && !ptrs[13]))) return -3;
   if (!ret && (!ptrs[4] || !ptrs[9] || !ptrs[10])) return -4;
+  if (dims[10] < 0 || dims[10] % 2 || dims[10] > dims[6] || dims[10] > MM_MAX_ROT || (dims[10] && !ptrs[15]) ||
+      (!ret && (dims[10] || dims[11])) || (dims[10] && dims[11]))
+    return -5;
   auto fill = [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
     ScanParams<T> p;
@@ -354,11 +421,12 @@ GK_EXPORT int gk_matrix_memory_scan(int is_fp32, void* const* ptrs, long long ld
     p.y = static_cast<T*>(ptrs[12]);
     p.gain = static_cast<const float*>(ptrs[13]);
     p.decay = static_cast<const float*>(ptrs[14]);
-    p.g_off = dims[8]; p.vdim_true = dims[9]; p.eps = eps; p.y_ld = y_ld;
+    p.g_off = dims[8]; p.vdim_true = dims[9]; p.eps = floats[2]; p.y_ld = y_ld;
+    p.turns = static_cast<const float2*>(ptrs[15]); p.rot = dims[10]; p.act = dims[11];
     p.q_off = dims[1]; p.k_off = dims[2]; p.v_off = dims[3];
     p.width = dims[4]; p.heads = dims[5]; p.dim = dims[6]; p.vdim = dims[7];
     p.slices = (p.vdim + MM_SLICE - 1) / MM_SLICE;
-    p.cap = cap; p.q_scale = q_scale;
+    p.cap = floats[0]; p.q_scale = floats[1]; p.out_scale = floats[3];
     cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
     return ret ? launch_scan<T, true>(p, dims[0], st) : launch_scan<T, false>(p, dims[0], st);
   };
@@ -367,7 +435,7 @@ GK_EXPORT int gk_matrix_memory_scan(int is_fp32, void* const* ptrs, long long ld
 
 // gain null: no gain, silu in place of the sigmoid.  dims: {rows, heads, vdim, vdim_true, g_off}
 GK_EXPORT int gk_memory_output(int is_fp32, const float* o, const void* proj, long long ld, const float* gain, void* y,
-                               long long y_ld, const int* dims, float eps, void* stream) {
+                               long long y_ld, const int* dims, float eps, float out_scale, void* stream) {
   const long long items = static_cast<long long>(dims[0]) * dims[1];
   if (items == 0) return 0;
   if (dims[2] % 4 || ld % 4 || y_ld % 4 || dims[4] % 4) return -1;
@@ -375,9 +443,24 @@ GK_EXPORT int gk_memory_output(int is_fp32, const float* o, const void* proj, lo
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   if (is_fp32)
     launch_k(memory_output_kernel<float>, grid, dim3(256), 0, st, o, static_cast<const float*>(proj), ld, dims[4], gain,
-             static_cast<float*>(y), y_ld, dims[0], dims[1], dims[2], dims[3], eps);
+             static_cast<float*>(y), y_ld, dims[0], dims[1], dims[2], dims[3], eps, out_scale);
   else
     launch_k(memory_output_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, o, static_cast<const __nv_bfloat16*>(proj), ld,
-             dims[4], gain, static_cast<__nv_bfloat16*>(y), y_ld, dims[0], dims[1], dims[2], dims[3], eps);
+             dims[4], gain, static_cast<__nv_bfloat16*>(y), y_ld, dims[0], dims[1], dims[2], dims[3], eps, out_scale);
   return launch_status();
+}
+
+// All heads normed together.  dims: {rows, cols, cols_true, g_off};  floats: {eps, out_scale}
+GK_EXPORT int gk_memory_output_joint(int is_fp32, const float* o, const void* proj, long long ld, const float* gain, void* y,
+                                     long long y_ld, const int* dims, const float* floats, void* stream) {
+  if (dims[0] == 0) return 0;
+  if (dims[1] < 4 || dims[1] % 4 || dims[2] < 1 || dims[2] > dims[1] || ld % 4 || y_ld % 4 || dims[3] % 4 || !gain) return -1;
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  auto go = [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    launch_k(memory_output_joint_kernel<T>, dim3(dims[0]), dim3(256), 0, st, o, static_cast<const T*>(proj), ld, dims[3], gain,
+             static_cast<T*>(y), y_ld, dims[1], dims[2], floats[0], floats[1]);
+    return launch_status();
+  };
+  return is_fp32 ? go(static_cast<float*>(nullptr)) : go(static_cast<__nv_bfloat16*>(nullptr));
 }

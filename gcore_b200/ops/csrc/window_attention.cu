@@ -3,9 +3,10 @@
 //   * append_keys_kernel      copies the new keys of a packed projection into their cache slots;
 //   * window_attn_kernel      any row (prompt portion or decoded token), any head size, 32-bit or bf16 storage, one warp
 //                             per (row, head): the true 32-bit path and the sizes the tensor-core kernels do not cover.
-//                             Keys and values may lie anywhere in a cached row and several keys may share a value, and
-//                             window, penalty, sink and output gate are optional, so absorbed latent attention and
-//                             differential attention run on it too;
+//                             Keys and values may lie anywhere in a cached row and several keys may share a value;
+//                             window, kept first positions, penalties, sink and output gate are optional and sigmoids may
+//                             take the softmax's place, so absorbed latent attention, differential attention and attention
+//                             with scored distances or sigmoid weights run on it too;
 //   * shared_kv_decode_kernel one new token per request, bf16, head sizes 64 and 128: mma.sync tiles with the query heads
 //                             of a group as rows (a group is far below the 64-row minimum of a tcgen05 instruction), KV
 //                             splits, append of the new key fused in.
@@ -56,10 +57,14 @@ struct WindowAttnParams {
   const float* sinks;       // [H] or null: a logit that joins the softmax denominator
   const T* gate;            // one logit per row and head, rows gate_ld apart, or null
   long long gate_ld;
-  O* out;                   // [rows, H, DV]
+  const float *r1, *r2;     // [H] or null: r1 ln(1 + r2 distance) is taken off a score
+  const float* head_bias;   // [H] or null: added to a score
+  O* out;                   // head h of a row at h * DV, rows out_ld apart
+  long long out_ld;
   int rows, H, G, maps;     // H query heads over G values, `maps` keys per value: head h takes key (g, h % maps)
-  int D, DV, window;        // window 0: unlimited
-  float scale;
+  int D, DV, window, keep;  // window 0: unlimited; the first `keep` positions are seen whatever the window
+  int sigmoid;              // weights are sigmoids of the scores, not normalised
+  float scale, out_scale;
 };
 
 // One warp per (row, query head); DV <= 32 * NR.
@@ -72,7 +77,7 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attn_kernel(const Window
   const long long item = static_cast<long long>(blockIdx.x) * WA_WARPS + warp;
   if (item >= static_cast<long long>(p.rows) * p.H) return;
   const int row = static_cast<int>(item / p.H), h = static_cast<int>(item - static_cast<long long>(row) * p.H);
-  O* orow = p.out + (static_cast<long long>(row) * p.H + h) * DV;
+  O* orow = p.out + row * p.out_ld + static_cast<long long>(h) * DV;
   float acc[NR];
 #pragma unroll
   for (int r = 0; r < NR; ++r) acc[r] = 0.f;
@@ -90,31 +95,39 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attn_kernel(const Window
     const long long k_off = static_cast<long long>(g * p.maps + h % p.maps) * D;
     const long long v_off = p.v_off + static_cast<long long>(g) * p.v_stride;
     const int* table = p.tables + static_cast<long long>(p.row_seq[row]) * p.max_blocks;
-    const float slope = p.slopes ? p.slopes[h] : 0.f;
+    const float slope = p.slopes ? p.slopes[h] : 0.f, bias = p.head_bias ? p.head_bias[h] : 0.f;
+    const float r1 = p.r1 ? p.r1[h] : 0.f, r2 = p.r1 ? p.r2[h] : 0.f;
     int j0 = p.window > 0 ? i - p.window + 1 : 0;
     if (j0 < 0) j0 = 0;
-    for (int base = j0; base <= i; base += 32) {
-      const int j = base + lane;
-      const int nt = i + 1 - base < 32 ? i + 1 - base : 32;
+    const int kept = p.keep < j0 ? p.keep : j0, count = kept + i + 1 - j0;   // places: kept positions, then the window
+    for (int base = 0; base < count; base += 32) {
+      const int place = base + lane, j = place < kept ? place : j0 + place - kept;
+      const int nt = count - base < 32 ? count - base : 32;
       float s = -FLT_MAX;
       long long at = 0;
-      if (j <= i) {
+      if (place < count) {
         at = (static_cast<long long>(table[j / p.block_size]) * p.block_size + j % p.block_size) * p.cache_row;
         const T* kr = p.cache + at + k_off;
         float a = 0.f;
         for (int d = 0; d < D; ++d) a = fmaf(sq[d], wa_f(kr[d]), a);
-        s = a * p.scale - slope * static_cast<float>(i - j);
+        s = a * p.scale - slope * static_cast<float>(i - j) + bias;
+        if (p.r1) s -= r1 * log1pf(r2 * static_cast<float>(i - j));
       }
       float mx = s;
 #pragma unroll
       for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffff, mx, o));
       const float mn = fmaxf(m, mx);
-      const float c = expf(m - mn);            // 0 on the first tile (m = -FLT_MAX)
-      const float e = j <= i ? expf(s - mn) : 0.f;
-      m = mn;
-      l = l * c + e;
+      float e;
+      if (p.sigmoid) {
+        e = place < count ? 1.f / (1.f + expf(-s)) : 0.f;
+      } else {
+        const float c = expf(m - mn);            // 0 on the first tile (m = -FLT_MAX)
+        e = place < count ? expf(s - mn) : 0.f;
+        m = mn;
+        l = l * c + e;
 #pragma unroll
-      for (int r = 0; r < NR; ++r) acc[r] *= c;
+        for (int r = 0; r < NR; ++r) acc[r] *= c;
+      }
       for (int t = 0; t < nt; ++t) {
         const float pt = __shfl_sync(0xffffffff, e, t);
         const T* vr = p.cache + __shfl_sync(0xffffffff, at, t) + v_off;
@@ -126,7 +139,7 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attn_kernel(const Window
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffff, l, o);
   }
-  float inv = l > 0.f ? 1.f / l : 0.f;
+  float inv = p.sigmoid ? p.out_scale : l > 0.f ? p.out_scale / l : 0.f;
   if (p.gate) inv /= 1.f + expf(-wa_f(p.gate[row * p.gate_ld + h]));
 #pragma unroll
   for (int r = 0; r < NR; ++r)
@@ -482,13 +495,16 @@ GK_EXPORT int gk_append_keys(const void* proj, long long ld_bytes, long long off
   return launch_status();
 }
 
-// ptrs: {q, cache, tables, row_seq, pos, slots, slopes, gate, out, sinks}; slopes, gate, sinks: or null
-// lds: {q_ld, gate_ld, cache_row};  window 0: unlimited;  out_fp32: 32-bit output of bf16 rows
-// dims: {rows, H, G, maps, D, DV, v_off, v_stride, window, block_size, max_blocks}
-GK_EXPORT int gk_window_attn(int is_fp32, int out_fp32, void* const* ptrs, const long long* lds, const int* dims, float scale,
-                             void* stream) {
+// ptrs: {q, cache, tables, row_seq, pos, slots, slopes, gate, out, sinks, r1, r2, head_bias}; slopes, gate and all behind out:
+// or null;  lds: {q_ld, gate_ld, cache_row, out_ld};  window 0: unlimited;  out_fp32: 32-bit output of bf16 rows
+// dims: {rows, H, G, maps, D, DV, v_off, v_stride, window, block_size, max_blocks, keep, sigmoid};  floats: {scale, out_scale}
+GK_EXPORT int gk_window_attn(int is_fp32, int out_fp32, void* const* ptrs, const long long* lds, const int* dims,
+                             const float* floats, void* stream) {
   const int H = dims[1], G = dims[2], maps = dims[3], D = dims[4], DV = dims[5];
   if (G < 1 || H % G || maps < 1 || (H / G) % maps || D < 1 || D > WA_MAX_D || DV < 1 || DV > WA_MAX_D || dims[8] < 0)
+    return -1;
+  if (dims[11] < 0 || lds[3] < static_cast<long long>(H) * DV || (ptrs[10] != nullptr) != (ptrs[11] != nullptr) ||
+      (dims[12] && ptrs[9]))
     return -1;
   if (static_cast<long long>(G) * maps * D > lds[2] || dims[6] + static_cast<long long>(G - 1) * dims[7] + DV > lds[2])
     return -1;
@@ -506,7 +522,10 @@ GK_EXPORT int gk_window_attn(int is_fp32, int out_fp32, void* const* ptrs, const
     p.slopes = static_cast<const float*>(ptrs[6]); p.sinks = static_cast<const float*>(ptrs[9]);
     p.gate = static_cast<const T*>(ptrs[7]); p.gate_ld = lds[1];
     p.out = static_cast<O*>(ptrs[8]);
-    p.rows = dims[0]; p.H = H; p.G = G; p.maps = maps; p.D = D; p.DV = DV; p.window = dims[8]; p.scale = scale;
+    p.rows = dims[0]; p.H = H; p.G = G; p.maps = maps; p.D = D; p.DV = DV; p.window = dims[8];
+    p.r1 = static_cast<const float*>(ptrs[10]); p.r2 = static_cast<const float*>(ptrs[11]);
+    p.head_bias = static_cast<const float*>(ptrs[12]); p.out_ld = lds[3];
+    p.keep = dims[11]; p.sigmoid = dims[12]; p.scale = floats[0]; p.out_scale = floats[1];
     return launch_window_attn(p, reinterpret_cast<cudaStream_t>(stream));
   };
   float* f = nullptr;

@@ -1,5 +1,6 @@
 """Recurrent matrix memories over the rows of a serving step (``csrc/matrix_memory.cu``, ``csrc/matrix_memory_chunk.cu``): the
-gated memory of an mLSTM, and retention, whose decay is fixed per head.  CPU tensors run the plain PyTorch definition."""
+gated memory of an mLSTM, and retention, whose decay is fixed per head (with a norm per head and a silu gate, or a joint norm and
+a sigmoid gate, and with rotated or activated inputs).  CPU tensors run the plain PyTorch definition."""
 from __future__ import annotations
 
 import ctypes
@@ -10,6 +11,7 @@ import torch
 
 from . import _lib
 from .gemm import linear_forward
+from .head_prep import head_prep, rotate_heads, silu_columns
 from .rows import StepRows
 
 LAUNCHES = {"matrix_memory": 0}
@@ -82,16 +84,19 @@ def _ref(proj, offs, gates, gate_b, cap, q_scale, heads, dim, vdim, rows: StepRo
 
 
 def _scan(proj, offs, h, gate_w, gates, gate_b, cap, q_scale, heads, dim, vdim, cu, first_pos, slots, st, out=None,
-          finish=None, decay=None):
-    """Token by token.  ``finish`` = (y, gain, g_off, vdim_true, eps): the normed, gated output in place of ``out``."""
-    y, gain, g_off, vdim_true, eps = finish if finish is not None else (None, None, 0, vdim, 0.0)
-    ptrs = (ctypes.c_void_p * 15)(*[t.data_ptr() if t is not None else None for t in
+          finish=None, decay=None, turns=None, act=False):
+    """Token by token.  ``finish`` = (y, gain, g_off, vdim_true, eps, out_scale): the normed, gated output in place of ``out``.
+    ``turns`` / ``act``: queries and keys are rotated, or queries, keys and values pass a silu, as they are read."""
+    y, gain, g_off, vdim_true, eps, out_scale = finish if finish is not None else (None, None, 0, vdim, 0.0, 1.0)
+    ptrs = (ctypes.c_void_p * 16)(*[t.data_ptr() if t is not None else None for t in
                                     (proj, h, gate_w, gates, gate_b, cu, first_pos, slots, st.S, st.n, st.m, out, y, gain,
-                                     decay)])
-    dims = (ctypes.c_int * 10)(slots.numel(), *offs, h.shape[1] if h is not None else 0, heads, dim, vdim, g_off, vdim_true)
+                                     decay, turns)])
+    dims = (ctypes.c_int * 12)(slots.numel(), *offs, h.shape[1] if h is not None else 0, heads, dim, vdim, g_off, vdim_true,
+                               2 * turns.shape[0] if turns is not None else 0, int(act))
     LAUNCHES["matrix_memory"] += 1
     _lib.check(_lib.kernels().gk_matrix_memory_scan(int(proj.dtype == torch.float32), ptrs, proj.stride(0),
-                                                    y.stride(0) if y is not None else 0, dims, float(cap), float(q_scale), float(eps), _lib.stream_ptr()),
+                                                    y.stride(0) if y is not None else 0, dims,
+                                                    (ctypes.c_float * 4)(cap, q_scale, eps, out_scale), _lib.stream_ptr()),
                "matrix_memory_scan")
 
 
@@ -108,17 +113,29 @@ def _chunk(proj, offs, gates, gate_b, cap, q_scale, heads, dim, vdim, rows: Step
                                                      _lib.stream_ptr()), "matrix_memory_chunk")
 
 
-def _output(o, proj, g_off, gain, vdim_true, eps, y=None):
+def _output(o, proj, g_off, gain, vdim_true, eps, y=None, joint=False, out_scale=1.0):
+    """Head outputs ``o`` [T, heads, vdim] normed (per head, or ``joint``) and gated: by a sigmoid with a gain, by a silu
+    without."""
     T, heads, vdim = o.shape
     if not o.is_cuda:
-        n = (o * torch.rsqrt(o.pow(2).sum(-1, keepdim=True) / vdim_true + eps)).reshape(T, -1)
+        if joint:
+            n = o.reshape(T, -1)
+            n = n * torch.rsqrt(n.pow(2).sum(-1, keepdim=True) / (heads * vdim_true) + eps) * gain * out_scale
+            return (n * torch.sigmoid(proj[:, g_off:g_off + heads * vdim].float())).to(proj.dtype)
+        n = (o * torch.rsqrt(o.pow(2).sum(-1, keepdim=True) / vdim_true + eps) * out_scale).reshape(T, -1)
         z = proj[:, g_off:g_off + heads * vdim].float()
         return (n * gain * torch.sigmoid(z) if gain is not None else n * torch.nn.functional.silu(z)).to(proj.dtype)
-    dims = (ctypes.c_int * 5)(T, heads, vdim, vdim_true, g_off)
     LAUNCHES["matrix_memory"] += 1
+    if joint:
+        dims = (ctypes.c_int * 4)(T, heads * vdim, heads * vdim_true, g_off)
+        _lib.check(_lib.kernels().gk_memory_output_joint(
+            int(proj.dtype == torch.float32), _lib.ptr(o), _lib.ptr(proj), proj.stride(0), _lib.ptr(gain), _lib.ptr(y),
+            y.stride(0), dims, (ctypes.c_float * 2)(eps, out_scale), _lib.stream_ptr()), "memory_output_joint")
+        return y
+    dims = (ctypes.c_int * 5)(T, heads, vdim, vdim_true, g_off)
     _lib.check(_lib.kernels().gk_memory_output(int(proj.dtype == torch.float32), _lib.ptr(o), _lib.ptr(proj),
                                                proj.stride(0), _lib.ptr(gain), _lib.ptr(y), y.stride(0), dims,
-                                               float(eps), _lib.stream_ptr()), "memory_output")
+                                               float(eps), float(out_scale), _lib.stream_ptr()), "memory_output")
     return y
 
 
@@ -148,7 +165,7 @@ def matrix_memory(proj, q_off: int, k_off: int, v_off: int, g_off: int, h, gate_
         single = (proj[P:], offs, h[P:], gate_w, None, *common, None, rows.first_pos[n:], rows.states[n:], state)
         slices = (vdim + SLICE - 1) // SLICE
         if slices <= FINISH_SLICES and slices * heads * (T - P) <= FINISH_CTAS:
-            _scan(*single, finish=(y[P:], gain, g_off, vdim_true, eps))
+            _scan(*single, finish=(y[P:], gain, g_off, vdim_true, eps, 1.0))
         else:
             o = torch.empty(T - P, heads, vdim, dtype=torch.float32, device=proj.device)
             _scan(*single, o)
@@ -156,50 +173,66 @@ def matrix_memory(proj, q_off: int, k_off: int, v_off: int, g_off: int, h, gate_
     return y
 
 
-def _retention_ref(proj, offs, decay, q_scale, heads, dim, vdim, rows: StepRows, st: MemoryState):
+def _retention_ref(proj, offs, decay, q_scale, heads, dim, vdim, rows: StepRows, st: MemoryState, turns, act):
     q_off, k_off, v_off = offs
     T = proj.shape[0]
+    p = proj.float()
+    q, k, v = (p[:, o:o + heads * d].view(T, heads, d) for o, d in ((q_off, dim), (k_off, dim), (v_off, vdim)))
+    if turns is not None:
+        q, k = (rotate_heads(x, turns, rows.pos) for x in (q, k))
+    if act:
+        q, k, v = (torch.nn.functional.silu(x) for x in (q, k, v))
     out = torch.zeros(T, heads, vdim)
     for t in range(T):
         slot = int(rows.states[rows.row_seq[t]])
         if slot < 0:
             continue
         S = torch.zeros_like(st.S[slot]) if int(rows.pos[t]) == 0 else st.S[slot]
-        q = proj[t, q_off:q_off + heads * dim].view(heads, dim).float() * q_scale
-        k = proj[t, k_off:k_off + heads * dim].view(heads, dim).float()
-        v = proj[t, v_off:v_off + heads * vdim].view(heads, vdim).float()
-        st.S[slot] = decay[:, None, None] * S + k[:, :, None] * v[:, None, :]
-        out[t] = torch.einsum("hdv,hd->hv", st.S[slot], q)
+        st.S[slot] = decay[:, None, None] * S + k[t][:, :, None] * v[t][:, None, :]
+        out[t] = torch.einsum("hdv,hd->hv", st.S[slot], q[t]) * q_scale
     return out
 
 
 def retention(proj, q_off: int, k_off: int, v_off: int, g_off: int, decay, q_scale: float, heads: int, dim: int, vdim: int,
-              vdim_true: int, rows: StepRows, state: MemoryState, eps: float, y):
+              vdim_true: int, rows: StepRows, state: MemoryState, eps: float, y, turns=None, act: bool = False, gain=None,
+              out_scale: float = 1.0):
     """Retention over the rows of a step: ``S <- decay_h S + k v^T``, head output ``S^T q * q_scale`` divided by its root
-    mean square (over ``vdim_true`` columns) and multiplied by ``silu(g)``, written to ``y`` [T, heads * vdim] (any row
-    stride).  ``decay``: [heads] 32-bit."""
+    mean square (over ``vdim_true`` columns) and multiplied by ``silu(g)``; with ``gain`` [heads * vdim], all heads' outputs
+    divided by their common root mean square and multiplied by ``gain * sigmoid(g)``.  Times ``out_scale``, written to ``y``
+    [T, heads * vdim] (any row stride).  ``decay``: [heads] 32-bit.  Queries and keys are rotated with ``turns`` (neighbours
+    paired), or queries, keys and values pass a silu with ``act``; both may happen in place."""
     T, P, n = proj.shape[0], rows.portion_rows, rows.n_portions
     offs = (q_off, k_off, v_off)
+    joint = gain is not None
     if not proj.is_cuda:
-        o = _retention_ref(proj, offs, decay, q_scale, heads, dim, vdim, rows, state)
-        y.copy_(_output(o, proj, g_off, None, vdim_true, eps))
+        o = _retention_ref(proj, offs, decay, q_scale, heads, dim, vdim, rows, state, turns, act)
+        y.copy_(_output(o, proj, g_off, gain, vdim_true, eps, joint=joint, out_scale=out_scale))
         return y
     common = (None, None, 0.0, q_scale, heads, dim, vdim)
     f32 = dict(dtype=torch.float32, device=proj.device)
     if P:
         o = torch.empty(P, heads, vdim, **f32)
+        if turns is not None:
+            head_prep(proj, rows, 0, P, q_off, heads, k_off, heads, dim, turns=turns)
+        if act:
+            sizes = (heads * dim, heads * dim, heads * vdim)
+            if offs == (q_off, q_off + sizes[0], q_off + sizes[0] + sizes[1]):
+                silu_columns(proj[:P], q_off, sum(sizes))
+            else:
+                for at, size in zip(offs, sizes):
+                    silu_columns(proj[:P], at, size)
         if proj.dtype == torch.bfloat16 and dim <= CHUNK_MAX_KEY_DIM and rows.max_portion > SCAN_MAX_TOKENS:
             _chunk(proj, offs, *common, rows, state, o, decay)
         else:
             _scan(proj, offs, None, None, *common, rows.cu, rows.first_pos, rows.states[:n], state, o, decay=decay)
-        _output(o, proj, g_off, None, vdim_true, eps, y[:P])
+        _output(o, proj, g_off, gain, vdim_true, eps, y[:P], joint, out_scale)
     if T > P:
         single = (proj[P:], offs, None, None, *common, None, rows.first_pos[n:], rows.states[n:], state)
         slices = (vdim + SLICE - 1) // SLICE
-        if slices <= FINISH_SLICES and slices * heads * (T - P) <= FINISH_CTAS:
-            _scan(*single, finish=(y[P:], None, g_off, vdim_true, eps), decay=decay)
+        if not joint and slices <= FINISH_SLICES and slices * heads * (T - P) <= FINISH_CTAS:
+            _scan(*single, finish=(y[P:], None, g_off, vdim_true, eps, out_scale), decay=decay, turns=turns, act=act)
         else:
             o = torch.empty(T - P, heads, vdim, **f32)
-            _scan(*single, o, decay=decay)
-            _output(o, proj[P:], g_off, None, vdim_true, eps, y[P:])
+            _scan(*single, o, decay=decay, turns=turns, act=act)
+            _output(o, proj[P:], g_off, gain, vdim_true, eps, y[P:], joint, out_scale)
     return y

@@ -60,20 +60,24 @@ def append_keys(proj, k_off, n, slots, cache):
 
 
 def general_attention(q, q_ld, cache, rows: StepRows, lo, hi, out, H, G, D, scale, dv=None, window=0, slopes=None, gate=None,
-                      gate_ld=0, sinks=None, maps=1, v_off=0, v_stride=None):
+                      gate_ld=0, sinks=None, maps=1, v_off=0, v_stride=None, keep=0, distance=None, head_bias=None,
+                      sigmoid=False, out_scale=1.0):
     """Rows ``lo .. hi`` of a step against the paged cache, whose rows hold G * ``maps`` keys of ``D`` columns and, at
     ``v_off``, G values of ``dv`` columns ``v_stride`` apart (default: a value is the first columns of its key).  Optional
-    window (0: none), distance penalty, sink logits and output gate.  Any size, 32-bit or bf16; ``out`` may be 32-bit."""
+    window (0: none) beside the first ``keep`` positions, penalties (``slopes`` times the distance; ``distance`` = (r1, r2):
+    r1 ln(1 + r2 distance)), bias per head, sink logits and output gate; ``sigmoid``: sigmoids of the scores in place of the
+    softmax.  Any size, 32-bit or bf16; ``out`` [rows, H * dv] or [rows, H, ...] (any row stride) may be 32-bit."""
     row = cache.stride(1)
-    dims = (ctypes.c_int * 11)(hi - lo, H, G, maps, D, dv or D, v_off, D if v_stride is None else v_stride, window,
-                               cache.shape[1], rows.tables.shape[1])
-    ptrs = (ctypes.c_void_p * 10)(*[t.data_ptr() if t is not None else None for t in
+    dims = (ctypes.c_int * 13)(hi - lo, H, G, maps, D, dv or D, v_off, D if v_stride is None else v_stride, window,
+                               cache.shape[1], rows.tables.shape[1], keep, int(sigmoid))
+    r1, r2 = distance if distance is not None else (None, None)
+    ptrs = (ctypes.c_void_p * 13)(*[t.data_ptr() if t is not None else None for t in
                                     (q, cache, rows.tables, rows.row_seq[lo:hi], rows.pos[lo:hi], rows.slots[lo:hi], slopes,
-                                     gate, out, sinks)])
-    lds = (ctypes.c_longlong * 3)(q_ld, gate_ld, row)
+                                     gate, out, sinks, r1, r2, head_bias)])
+    lds = (ctypes.c_longlong * 4)(q_ld, gate_ld, row, H * (dv or D) if out.dim() > 2 else out.stride(0))
     LAUNCHES["window_attention"] += 1
     _lib.check(_lib.kernels().gk_window_attn(int(q.dtype == torch.float32), int(out.dtype == torch.float32), ptrs, lds, dims,
-                                             float(scale), _lib.stream_ptr()), "window_attn")
+                                             (ctypes.c_float * 2)(scale, out_scale), _lib.stream_ptr()), "window_attn")
 
 
 def window_attention(proj, q_off: int, k_off: int, heads: int, kv_heads: int, dim: int, rows: StepRows, cache, slopes,

@@ -170,11 +170,11 @@ class _Sched:
 
 
 def _count_launches() -> int:
-    from ..ops import (attention, depth, diff_attention, gemm, latent_attention, matrix_memory, moe, optim, rl, sandwich,
-                       streams, vocab, window_attention)
-    return sum(sum(m.LAUNCHES.values()) for m in (attention, depth, diff_attention, fused, gemm, latent_attention,
-                                                  matrix_memory, moe, optim, rl, sandwich, streams, vocab,
-                                                  window_attention))
+    from ..ops import (attention, conv_norm, depth, diff_attention, gemm, head_prep, latent_attention, matrix_memory, moe, optim,
+                       rl, sandwich, scored_attention, streams, vocab, window_attention)
+    return sum(sum(m.LAUNCHES.values()) for m in (attention, conv_norm, depth, diff_attention, fused, gemm, head_prep,
+                                                  latent_attention, matrix_memory, moe, optim, rl, sandwich,
+                                                  scored_attention, streams, vocab, window_attention))
 
 
 class LayerWeights:
