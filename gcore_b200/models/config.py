@@ -6,9 +6,9 @@ from __future__ import annotations
 from dataclasses import dataclass, field, fields
 from typing import Tuple, Any, Dict, List, Optional
 
-from .layer_plan import (DenseSpec, DifferentialAttentionSpec, ExpertsSpec, LatentAttentionSpec, LayerPlan,
-                         ParallelLayerSpec, StreamLayerSpec, kedesun_plan, lobutar_plan, nafitar_plan,
-                         rezulorn_plan)
+from .layer_plan import (ConvLayerSpec, DenseSpec, DifferentialAttentionSpec, ExpertsSpec, LatentAttentionSpec, LayerPlan,
+                         LayerSpec, ParallelLayerSpec, ScoredAttentionSpec, StreamLayerSpec, kedesun_plan, lobutar_plan,
+                         nafitar_plan, rezulorn_plan)
 
 
 @dataclass
@@ -148,12 +148,16 @@ class ModelConfig:
                 else:
                     total += (h + S * (S + 2)) * (1 if sp.ffn is None else 2)       # norms, hyper-connections
                 continue
+            if isinstance(sp, ConvLayerSpec):
+                total += sum(self._mixer_parameters(m) for m in sp.mixers) + self._ffn_parameters(sp.ffn)
+                total += (1 if sp.ffn is None else 2) * (1 + self.layer_plan.taps) * h          # norms, convolutions
+                continue
             a, m = sp.attention, sp.memory
             total += (2 * a.heads + a.kv_heads) * a.dim * h + (a.heads + a.kv_heads) * a.dim
             total += m.heads * (2 * m.dim + 3 * m.vdim + 2) * h + m.heads * (m.vdim + 2)
             total += (4 if not sp.ffn else 6) * h + 3 * sp.ffn * h
         if include_embedding:
-            positions = 0 if S else self.max_position_embeddings
+            positions = self.max_position_embeddings if isinstance(self.layer_plan.layers[0], LayerSpec) else 0
             total += self.vocab_size * h if self.tie_word_embeddings else (2 * self.vocab_size + positions) * h
         return total
 
@@ -166,12 +170,14 @@ class ModelConfig:
         if isinstance(m, DifferentialAttentionSpec):
             qkv = (m.heads + m.kv_heads) * 2 * m.dim + m.kv_heads * m.vdim
             return (qkv + m.heads + m.heads * m.vdim) * h + qkv + h + 4 * m.dim
-        return m.heads * (2 * m.dim + 3 * m.vdim) * h
+        if isinstance(m, ScoredAttentionSpec):
+            return (m.heads + m.kv_heads) * (m.dim + m.vdim) * h + (2 * m.distance + m.head_bias) * m.heads
+        return m.heads * (2 * m.dim + 3 * m.vdim) * h + (m.heads * m.vdim if m.norm == "joint" else 0)
 
     def _ffn_parameters(self, f) -> int:
         h = self.hidden_size
         if isinstance(f, DenseSpec):
-            return 3 * f.ff * h
+            return (3 if f.act == "silu_gate" else 2) * f.ff * h
         if isinstance(f, ExpertsSpec):
             mats = 3 if f.act == "silu_gate" else 2
             shared = (mats * f.shared_ff + (1 if f.shared_gate else 0)) * h if f.shared_ff else 0

@@ -176,13 +176,13 @@ class ConvDecoder(PlanDecoder):
         return self
 
     def final_rows(self, x, rows=None):
-        return cn.norm_rows(x, self.final_gain, self.norm, self.embed.dtype, rows)
+        return cn.conv_norm_rows(x, self.final_gain, self.norm, self.embed.dtype, rows)
 
     def forward(self, rows, caches, states, final=True, record=None):
         runs, mult, spec = self.cfg.layer_plan.runs, self.cfg.layer_plan.residual_mult, self.norm
         subs = [(s, states[r.index].rings[k]) for r in runs for k, s in enumerate(self.layers[r.layer].sublayers())]
         first, ring = subs[0]
-        x, h = cn.embed_rows(rows, self.embed, first.gain, first.taps, ring, spec)
+        x, h = cn.conv_embed_rows(rows, self.embed, first.gain, first.taps, ring, spec)
         at = 0
 
         def join(y):
@@ -191,9 +191,9 @@ class ConvDecoder(PlanDecoder):
             at += 1
             if at < len(subs):
                 sub, ring = subs[at]
-                x, h = cn.add_sublayer(x, y, mult, spec, sub.gain, rows, sub.taps, ring)
+                x, h = cn.conv_add_sublayer(x, y, mult, spec, sub.gain, rows, sub.taps, ring)
             else:
-                x, h = cn.add_sublayer(x, y, mult, spec, self.final_gain if final else None, keep=not final or record is not None)
+                x, h = cn.conv_add_sublayer(x, y, mult, spec, self.final_gain if final else None, keep=not final or record is not None)
 
         for r in runs:
             layer = self.layers[r.layer]

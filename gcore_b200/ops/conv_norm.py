@@ -74,7 +74,7 @@ def _launch(rows: Optional[StepRows], n_rows: int, H: int, spec: NormSpec, mult:
     _lib.check(_lib.kernels().gk_conv_norm(int(fp32), ptrs, dims, floats, _lib.stream_ptr()), "conv_norm")
 
 
-def embed_rows(rows: StepRows, embed, gain, taps, ring, spec: NormSpec):
+def conv_embed_rows(rows: StepRows, embed, gain, taps, ring, spec: NormSpec):
     """``x = embed[token]``; returns ``(x, h)`` with ``h`` the convolved norm of ``x``, the input of the first sublayer."""
     T, H = rows.tokens.numel(), embed.shape[1]
     if not embed.is_cuda:
@@ -87,7 +87,7 @@ def embed_rows(rows: StepRows, embed, gain, taps, ring, spec: NormSpec):
     return x, h
 
 
-def add_sublayer(x, y, mult: float, spec: NormSpec, gain=None, rows: Optional[StepRows] = None, taps=None, ring=None,
+def conv_add_sublayer(x, y, mult: float, spec: NormSpec, gain=None, rows: Optional[StepRows] = None, taps=None, ring=None,
                  keep: bool = True):
     """``x + mult * y`` and, with ``gain``, its norm in ``y``'s dtype, convolved when ``taps`` are given.  Returns
     ``(x_new, h)``; ``x`` stays as it is (a row of ``h`` reads its neighbours), and without ``keep`` ``x_new`` is None."""
@@ -104,7 +104,7 @@ def add_sublayer(x, y, mult: float, spec: NormSpec, gain=None, rows: Optional[St
     return new, h
 
 
-def norm_rows(x, gain, spec: NormSpec, dtype, pick=None):
+def conv_norm_rows(x, gain, spec: NormSpec, dtype, pick=None):
     """``norm(x[pick]) * gain`` of the 32-bit residual, in ``dtype``."""
     if not x.is_cuda:
         return norm(x if pick is None else x[pick], gain, spec).to(dtype)

@@ -44,8 +44,8 @@ def resolve(name: str, impl: Optional[str] = None) -> Callable:
 
 
 def _populate():
-    from . import (attention, depth, diff_attention, fused, gemm, latent_attention, matrix_memory, moe, optim, quant, rl,
-                   sandwich, streams, vocab, window_attention)
+    from . import (attention, conv_norm, depth, diff_attention, fused, gemm, head_prep, latent_attention, matrix_memory, moe,
+                   optim, quant, rl, sandwich, scored_attention, streams, vocab, window_attention)
     for mod, names in ((gemm, ("gemm", "grouped_gemm", "grouped_wgrad", "linear")),
                        (fused, ("rmsnorm", "rope", "swiglu")),
                        (attention, ("flash_attn_varlen", "flash_attn_qkvpacked", "paged_decode", "kv_append_rope")),
@@ -56,6 +56,8 @@ def _populate():
                        (window_attention, ("window_attention",)), (matrix_memory, ("matrix_memory", "retention")),
                        (latent_attention, ("latent_attention",)), (depth, ("add_layer",)),
                        (diff_attention, ("differential_attention",)), (streams, ("connect",)),
+                       (conv_norm, ("conv_embed_rows", "conv_add_sublayer", "conv_norm_rows")),
+                       (head_prep, ("head_prep", "silu_columns")), (scored_attention, ("scored_attention",)),
                        (moe, ("activate", "choose", "expert_rows", "routed_experts")),
                        (rl, ("fused_grpo_loss", "gae"))):
         for n in names:
