@@ -273,7 +273,8 @@ def main():
     ap.add_argument("--serve", nargs="*", default=None, metavar="SIZE",
                     help="instead of the recipe: prefill and decode throughput of layer-plan decoders beside the closest "
                     "uniform model, kernel by kernel (sizes: see gcore_b200/tools/serve_bench.py; default all); one JSON line")
-    ap.add_argument("--serve-design", default="nafitar", choices=("nafitar", "kedesun", "lobutar"), help="design that --serve measures")
+    ap.add_argument("--serve-design", default="nafitar", choices=("nafitar", "kedesun", "lobutar", "rezulorn"),
+                    help="design that --serve measures")
     args = ap.parse_args()
     if args.serve is not None:
         return serve_bench(args)

@@ -15,7 +15,7 @@ from . import _lib
 from .rows import StepRows
 
 LAUNCHES = {"conv_norm": 0}
-MAX_TAPS, MAX_WIDTH = 16, 8192
+MAX_TAPS, MAX_WIDTH = 16, 16384
 STORED_TAPS = (2, 3, 4, 8, 16)      # taps the kernel is built for; others are padded with zero taps in front
 
 

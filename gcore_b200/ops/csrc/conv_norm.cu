@@ -3,11 +3,13 @@
 //     x_t <- x_t + mult * y_t;   n_t = norm(x_t) * gain;   h_t <- sum_j w[j] n_(t - TAPS + 1 + j)
 // x, the norm and the convolution are 32-bit.  A request keeps its last TAPS - 1 rows n in 32-bit, position p in ring row
 // p mod (TAPS - 1); rows ahead of position 0 are zero.
-//
-// One CTA = a strip of rows of one portion (or one single token); the TAPS - 1 rows in front of a strip are normed once more
-// by it, so strips need nothing from one another, which is also why the new residual goes to another buffer.  Strips start at
-// the portion's first row and are at least TAPS - 1 rows long: only the first one reads the ring, and it also writes it, once
-// its own rows are done, norming the portion's last rows itself where they lie in another strip.
+//   * conv_norm_row_kernel      one CTA per row: single tokens, and the norm without a convolution;
+//   * conv_norm_strip_kernel    one CTA per strip of a portion's rows.  A warp per row takes mean and variance while it streams
+//                               the row (chunks of 16 values a lane, merged pairwise, so nothing cancels); then every thread
+//                               slides down its own columns, the last TAPS rows n in registers.
+// The TAPS - 1 rows in front of a strip are taken once more by it, so strips need nothing from one another, which is also why
+// the new residual goes to another buffer.  Strips start at the portion's first row and are at least TAPS - 1 rows long: only
+// the first one reads the ring, and it also writes it, taking the portion's last rows itself where they lie in another strip.
 #include "host_utils.h"
 #include "row_ops.cuh"
 #include <type_traits>
@@ -33,14 +35,51 @@ struct ConvNormParams {
   float mult, eps;
 };
 
+// Residual columns 4i .. 4i + 3 of a row, with what is added to them.
+template <typename T>
+struct CnRow {
+  const T* embed = nullptr;
+  const float* x = nullptr;
+  const T* y = nullptr;
+  __device__ __forceinline__ CnRow(const ConvNormParams<T>& p, long long row, long long src) {
+    if (p.embed) {
+      long long tok = p.tokens[row];
+      tok = tok < 0 ? 0 : (tok >= p.vocab ? p.vocab - 1 : tok);
+      embed = p.embed + tok * p.H;
+    } else {
+      x = p.x + src * p.H;
+    }
+    if (p.y) y = p.y + row * p.H;
+  }
+  __device__ __forceinline__ float4 load(int i, float mult) const {
+    float4 v = embed ? ld4(embed + i * 4) : ld4(x + i * 4);
+    if (y) {
+      const float4 a = ld4(y + i * 4);
+      v.x = fmaf(mult, a.x, v.x); v.y = fmaf(mult, a.y, v.y); v.z = fmaf(mult, a.z, v.z); v.w = fmaf(mult, a.w, v.w);
+    }
+    return v;
+  }
+};
+
+// v minus the mean, zero in the padding.
+__device__ __forceinline__ float4 cn_centred(float4 v, float mean, int c, int H_true) {
+  return make_float4(c < H_true ? v.x - mean : 0.f, c + 1 < H_true ? v.y - mean : 0.f, c + 2 < H_true ? v.z - mean : 0.f,
+                     c + 3 < H_true ? v.w - mean : 0.f);
+}
+__device__ __forceinline__ float4 cn_scaled(float4 v, float f, float4 g) {
+  return make_float4(v.x * f * g.x, v.y * f * g.y, v.z * f * g.z, v.w * f * g.w);
+}
+__device__ __forceinline__ void cn_add(float4& o, float4 w, float4 n) {
+  o.x = fmaf(w.x, n.x, o.x); o.y = fmaf(w.y, n.y, o.y); o.z = fmaf(w.z, n.z, o.z); o.w = fmaf(w.w, n.w, o.w);
+}
+
 // Block-wide sum with one barrier.  Calls alternate between two buffers: a thread that writes one has passed the barrier of the
 // call between, so every thread has read what the buffer held.
-__device__ __forceinline__ float cn_sum(float a, float (*red)[32], int& turn) {
+__device__ __forceinline__ float cn_sum(float a, float (*red)[32], int turn) {
   const int lane = threadIdx.x & 31, w = threadIdx.x >> 5, nw = blockDim.x >> 5;
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) a += __shfl_xor_sync(0xffffffff, a, o);
   float* r = red[turn];
-  turn ^= 1;
   if (lane == 0) r[w] = a;
   __syncthreads();
   a = lane < nw ? r[lane] : 0.f;
@@ -49,185 +88,185 @@ __device__ __forceinline__ float cn_sum(float a, float (*red)[32], int& turn) {
   return a;
 }
 
-// Thread i owns the float4 groups i, i + blockDim, ... (NV of them).  TAPS 1: no convolution.
+// grid: one CTA per row behind the portions.  Thread i owns the float4 groups i, i + blockDim, ... (NV of them).  TAPS 1: no
+// convolution.
 template <typename T, int TAPS, int NV>
-__global__ void __launch_bounds__(TAPS > 4 ? 1024 : 512) conv_norm_kernel(const ConvNormParams<T> p) {
+__global__ void __launch_bounds__(512) conv_norm_row_kernel(const ConvNormParams<T> p) {
   constexpr int W = TAPS - 1;
   __shared__ float red[2][32];
   pdl_launch_dependents();
   pdl_wait();
   const int tid = threadIdx.x, nv = p.H >> 2;
-  int lo, hi, r_beg, r_end, p0 = 0, slot = -1;
-  bool first = false;
-  if (TAPS == 1) {
-    lo = r_beg = blockIdx.x * p.strip;
-    hi = r_end = lo + p.strip < p.rows ? lo + p.strip : p.rows;
-  } else {
-    const int b = blockIdx.x, in_portions = p.n_portions * p.strips;
-    int seg, s = 0;
-    if (b < in_portions) {
-      seg = b / p.strips;
-      s = b - seg * p.strips;
-      r_beg = p.cu[seg];
-      r_end = p.cu[seg + 1];
-    } else {
-      seg = p.n_portions + (b - in_portions);
-      r_beg = p.portion_rows + (b - in_portions);
-      r_end = r_beg + 1;
-    }
-    lo = r_beg + s * p.strip;
-    if (lo >= r_end) return;
-    hi = lo + p.strip < r_end ? lo + p.strip : r_end;
-    first = s == 0;
-    p0 = p.first_pos[seg];
-    slot = p.states[seg];
-  }
-
-  float4 gain[NV], taps[TAPS <= 4 ? TAPS : 1][NV], win[W > 0 ? W : 1][NV];
+  const long long row = (TAPS > 1 ? p.portion_rows : 0) + static_cast<long long>(blockIdx.x);
+  const CnRow<T> src(p, row, TAPS == 1 && p.pick ? p.pick[row] : row);
+  const int seg = p.n_portions + blockIdx.x;
+  const int pos = TAPS > 1 ? p.first_pos[seg] : 0, slot = TAPS > 1 ? p.states[seg] : -1;
+  float4 x[NV];
+  float s = 0.f;
 #pragma unroll
   for (int v = 0; v < NV; ++v) {
     const int i = tid + v * blockDim.x;
-    gain[v] = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (i < nv && p.gain) gain[v] = ld4(p.gain + i * 4);
-    if (TAPS > 1 && TAPS <= 4) {
+    x[v] = i < nv ? src.load(i, p.mult) : make_float4(0.f, 0.f, 0.f, 0.f);
+    if (p.x_out && i < nv) st4(p.x_out + row * p.H + i * 4, x[v]);
+    s += (x[v].x + x[v].y) + (x[v].z + x[v].w);      // columns past H_true are zero
+  }
+  if (!p.h) return;
+  if (p.center) {
+    const float mean = cn_sum(s, red, 0) / p.H_true;
 #pragma unroll
-      for (int j = 0; j < (TAPS <= 4 ? TAPS : 1); ++j)
-        taps[j][v] = i < nv ? ld4(p.taps + static_cast<long long>(j) * p.H + i * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int v = 0; v < NV; ++v) x[v] = cn_centred(x[v], mean, (tid + v * blockDim.x) * 4, p.H_true);
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int v = 0; v < NV; ++v) ss += sq4(x[v]);
+  const float f = 1.f / sqrtf(cn_sum(ss, red, 1) / p.H_true + p.eps);
+#pragma unroll
+  for (int v = 0; v < NV; ++v) {
+    const int i = tid + v * blockDim.x;
+    if (i >= nv) continue;
+    const float4 n = cn_scaled(x[v], f, ld4(p.gain + i * 4));
+    float4 o = n;
+    if (TAPS > 1) {
+      o = make_float4(0.f, 0.f, 0.f, 0.f);
+      float* ring = p.ring + static_cast<long long>(slot < 0 ? 0 : slot) * W * p.H + i * 4;
+#pragma unroll
+      for (int j = 0; j < W; ++j) {
+        const int q = pos - W + j;
+        if (q >= 0 && slot >= 0)
+          cn_add(o, ld4(p.taps + static_cast<long long>(j) * p.H + i * 4), ld4(ring + static_cast<long long>(q % (W > 0 ? W : 1)) * p.H));
+      }
+      cn_add(o, ld4(p.taps + static_cast<long long>(W) * p.H + i * 4), n);
+      if (slot >= 0) st4(ring + static_cast<long long>(pos % (W > 0 ? W : 1)) * p.H, n);
+    }
+    st4(p.h + row * p.H + i * 4, o);
+  }
+}
+
+constexpr int CS_WARPS = 8;
+constexpr int CS_GROUPS = 4;                 // float4 groups a lane takes at a time
+constexpr int CS_MAX_ROWS = CS_WARPS * 4;    // rows of a strip and in front of it
+
+// Number, mean and sum of squared deviations of a set, merged with another's.
+struct CnMoments {
+  float n, mean, m2;
+  __device__ __forceinline__ void merge(float nb, float mb, float sb) {
+    const float all = n + nb;
+    if (nb == 0.f) return;
+    const float d = mb - mean, f = nb / all;
+    mean = fmaf(d, f, mean);
+    m2 += sb + d * d * n * f;
+    n = all;
+  }
+};
+
+// grid: portions x strips.
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(CS_WARPS * 32, TAPS <= 4 ? 3 : 2) conv_norm_strip_kernel(const ConvNormParams<T> p) {
+  constexpr int W = TAPS - 1;
+  __shared__ float s_mean[CS_MAX_ROWS + W], s_rstd[CS_MAX_ROWS + W];   // rows lo - W .. hi - 1, then the portion's last W rows
+  pdl_launch_dependents();
+  pdl_wait();
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nv = p.H >> 2;
+  const int seg = blockIdx.x / p.strips, s = blockIdx.x % p.strips;
+  const int r_beg = p.cu[seg], r_end = p.cu[seg + 1], lo = r_beg + s * p.strip;
+  if (lo >= r_end) return;
+  const int hi = lo + p.strip < r_end ? lo + p.strip : r_end;
+  const int p0 = p.first_pos[seg], slot = p.states[seg];
+  const bool first = s == 0, tail = first && slot >= 0 && hi < r_end;
+  const int front = hi - lo + W;             // rows of the first kind
+  // row behind index k of the statistics
+  auto row_of = [&](int k) { return k < front ? lo - W + k : r_end - W + (k - front); };
+
+  for (int k = warp; k < front + (tail ? W : 0); k += CS_WARPS) {
+    const int r = row_of(k);
+    if (r < r_beg) continue;                 // it is in the ring, or ahead of the sequence
+    const CnRow<T> src(p, r, r);
+    const bool store = r >= lo && r < hi && k < front && p.x_out;
+    CnMoments m = {0.f, 0.f, 0.f};
+    for (int base = 0; base < nv; base += 32 * CS_GROUPS) {
+      float4 v[CS_GROUPS];
+#pragma unroll
+      for (int j = 0; j < CS_GROUPS; ++j) {
+        const int i = base + j * 32 + lane;
+        v[j] = i < nv ? src.load(i, p.mult) : make_float4(0.f, 0.f, 0.f, 0.f);
+      }
+      float sum = 0.f, cnt = 0.f;
+#pragma unroll
+      for (int j = 0; j < CS_GROUPS; ++j) {
+        const int i = base + j * 32 + lane, left = p.H_true - i * 4;
+        if (store && i < nv) st4(p.x_out + static_cast<long long>(r) * p.H + i * 4, v[j]);
+        sum += (v[j].x + v[j].y) + (v[j].z + v[j].w);
+        cnt += left >= 4 ? 4.f : left > 0 ? static_cast<float>(left) : 0.f;
+      }
+      const float mean = p.center && cnt > 0.f ? sum / cnt : 0.f;
+      float ss = 0.f;
+#pragma unroll
+      for (int j = 0; j < CS_GROUPS; ++j) ss += sq4(cn_centred(v[j], mean, (base + j * 32 + lane) * 4, p.H_true));
+      m.merge(cnt, mean, ss);
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float nb = __shfl_xor_sync(0xffffffff, m.n, o), mb = __shfl_xor_sync(0xffffffff, m.mean, o);
+      m.merge(nb, mb, __shfl_xor_sync(0xffffffff, m.m2, o));
+    }
+    if (lane == 0) {
+      s_mean[k] = m.mean;
+      s_rstd[k] = 1.f / sqrtf(m.m2 / p.H_true + p.eps);
     }
   }
+  __syncthreads();                           // also: this CTA's new residual rows are visible to its threads
 
-  // residual of a row, and (y) what is added to it
-  auto load = [&](int r, float4 (&x)[NV], float4 (&y)[NV]) {
-    const T* e = nullptr;
-    const float* xs = nullptr;
-    if (p.embed) {
-      long long tok = p.tokens[r];
-      tok = tok < 0 ? 0 : (tok >= p.vocab ? p.vocab - 1 : tok);
-      e = p.embed + tok * p.H;
-    } else {
-      xs = p.x + (TAPS == 1 && p.pick ? p.pick[r] : static_cast<long long>(r)) * p.H;
-    }
+  for (int i = tid; i < nv; i += CS_WARPS * 32) {
+    const float4 gain = ld4(p.gain + i * 4);
+    float4 taps[TAPS], win[W];
 #pragma unroll
-    for (int v = 0; v < NV; ++v) {
-      const int i = tid + v * blockDim.x;
-      x[v] = y[v] = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (i >= nv) continue;
-      x[v] = e ? ld4(e + i * 4) : ld4(xs + i * 4);
-      if (p.y) y[v] = ld4(p.y + static_cast<long long>(r) * p.H + i * 4);
-    }
-  };
-  int turn = 0;
-  // n of a row whose residual is loaded; x becomes n
-  auto norm = [&](int r, float4 (&x)[NV], const float4 (&y)[NV], bool store) {
-    float s = 0.f;
+    for (int j = 0; j < TAPS; ++j) taps[j] = ld4(p.taps + static_cast<long long>(j) * p.H + i * 4);
+    float* ring = p.ring + static_cast<long long>(slot < 0 ? 0 : slot) * W * p.H + i * 4;
+    auto normed = [&](int k, float4 v) { return cn_scaled(cn_centred(v, s_mean[k], i * 4, p.H_true), s_rstd[k], gain); };
 #pragma unroll
-    for (int v = 0; v < NV; ++v) {
-      const int i = tid + v * blockDim.x;
-      x[v].x = fmaf(p.mult, y[v].x, x[v].x); x[v].y = fmaf(p.mult, y[v].y, x[v].y);
-      x[v].z = fmaf(p.mult, y[v].z, x[v].z); x[v].w = fmaf(p.mult, y[v].w, x[v].w);
-      if (store && i < nv) st4(p.x_out + static_cast<long long>(r) * p.H + i * 4, x[v]);
-      s += (x[v].x + x[v].y) + (x[v].z + x[v].w);      // columns past H_true are zero
+    for (int j = 0; j < W; ++j) {
+      const int r = lo - W + j, q = p0 + (r - r_beg);
+      win[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (r >= r_beg) win[j] = normed(j, CnRow<T>(p, r, r).load(i, p.mult));
+      else if (q >= 0 && slot >= 0) win[j] = ld4(ring + static_cast<long long>(q % W) * p.H);
     }
-    if (!p.h) return;
-    if (p.center) {
-      const float mean = cn_sum(s, red, turn) / p.H_true;
+    constexpr int AHEAD = 4;
+    float4 nx[AHEAD];
+    auto fetch = [&](int r) {
+      if (r >= hi) return make_float4(0.f, 0.f, 0.f, 0.f);
+      return p.x_out ? ld4(p.x_out + static_cast<long long>(r) * p.H + i * 4) : CnRow<T>(p, r, r).load(i, p.mult);
+    };
 #pragma unroll
-      for (int v = 0; v < NV; ++v) {
-        const int c = (tid + v * blockDim.x) * 4;
-        x[v].x = c < p.H_true ? x[v].x - mean : 0.f;
-        x[v].y = c + 1 < p.H_true ? x[v].y - mean : 0.f;
-        x[v].z = c + 2 < p.H_true ? x[v].z - mean : 0.f;
-        x[v].w = c + 3 < p.H_true ? x[v].w - mean : 0.f;
+    for (int a = 0; a < AHEAD; ++a) nx[a] = fetch(lo + a);
+    for (int r0 = lo; r0 < hi; r0 += AHEAD) {
+      float4 cur[AHEAD];
+#pragma unroll
+      for (int a = 0; a < AHEAD; ++a) {
+        cur[a] = nx[a];
+        nx[a] = fetch(r0 + AHEAD + a);       // on their way while these rows are worked on
       }
-    }
-    float ss = 0.f;
 #pragma unroll
-    for (int v = 0; v < NV; ++v) ss += sq4(x[v]);
-    const float f = 1.f / sqrtf(cn_sum(ss, red, turn) / p.H_true + p.eps);
+      for (int a = 0; a < AHEAD; ++a) {
+        const int r = r0 + a;
+        if (r >= hi) break;
+        const float4 n = normed(r - lo + W, cur[a]);
+        float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-    for (int v = 0; v < NV; ++v)
-      x[v] = make_float4(x[v].x * f * gain[v].x, x[v].y * f * gain[v].y, x[v].z * f * gain[v].z, x[v].w * f * gain[v].w);
-  };
-  auto ring_row = [&](int pos) { return p.ring + (static_cast<long long>(slot) * (W > 0 ? W : 1) + pos % (W > 0 ? W : 1)) * p.H; };
-  auto store_ring = [&](int pos, const float4 (&n)[NV]) {
-    float* dst = ring_row(pos);
-#pragma unroll
-    for (int v = 0; v < NV; ++v) {
-      const int i = tid + v * blockDim.x;
-      if (i < nv) st4(dst + i * 4, n[v]);
-    }
-  };
-
-  // the rows in front of the strip
-#pragma unroll
-  for (int k = 0; k < W; ++k) {
-    const int r = lo - W + k;
-    if (r >= r_beg) {
-      float4 y[NV];
-      load(r, win[k], y);
-      norm(r, win[k], y, false);
-    } else {
-      const int pos = p0 + (r - r_beg);
-#pragma unroll
-      for (int v = 0; v < NV; ++v) {
-        const int i = tid + v * blockDim.x;
-        win[k][v] = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (i < nv && pos >= 0 && slot >= 0) win[k][v] = ld4(ring_row(pos) + i * 4);
-      }
-    }
-  }
-
-  float4 x[NV], y[NV];
-  load(lo, x, y);
-  for (int r = lo; r < hi; ++r) {
-    float4 xn[NV], yn[NV];
-    if (r + 1 < hi) {
-      load(r + 1, xn, yn);             // on their way while this row is reduced
-    } else {
-#pragma unroll
-      for (int v = 0; v < NV; ++v) xn[v] = yn[v] = make_float4(0.f, 0.f, 0.f, 0.f);
-    }
-    norm(r, x, y, p.x_out != nullptr);
-    if (p.h) {
-#pragma unroll
-      for (int v = 0; v < NV; ++v) {
-        const int i = tid + v * blockDim.x;
-        if (i >= nv) continue;
-        float4 o = x[v];
-        if (TAPS > 1) {
-          o = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll
-          for (int j = 0; j < TAPS; ++j) {
-            const float4 w = TAPS <= 4 ? taps[TAPS <= 4 ? j : 0][v] : ld4(p.taps + static_cast<long long>(j) * p.H + i * 4);
-            const float4 n = j < W ? win[j < W ? j : 0][v] : x[v];
-            o.x = fmaf(w.x, n.x, o.x); o.y = fmaf(w.y, n.y, o.y); o.z = fmaf(w.z, n.z, o.z); o.w = fmaf(w.w, n.w, o.w);
-          }
-        }
+        for (int j = 0; j < W; ++j) cn_add(o, taps[j], win[j]);
+        cn_add(o, taps[W], n);
         st4(p.h + static_cast<long long>(r) * p.H + i * 4, o);
+#pragma unroll
+        for (int j = 0; j + 1 < W; ++j) win[j] = win[j + 1];
+        win[W - 1] = n;
       }
     }
+    if (first && slot >= 0) {
 #pragma unroll
-    for (int v = 0; v < NV; ++v) {
-#pragma unroll
-      for (int k = 0; k + 1 < W; ++k) win[k][v] = win[k + 1][v];
-      if (W > 0) win[W > 0 ? W - 1 : 0][v] = x[v];
-      x[v] = xn[v];
-      y[v] = yn[v];
-    }
-  }
-
-  if (TAPS > 1 && first && slot >= 0) {
-#pragma unroll
-    for (int k = 0; k < W; ++k) {
-      const int r = r_end - W + k;
-      if (r < r_beg) continue;         // an older row: it is in the ring already
-      if (hi < r_end) {
-        float4 n[NV], z[NV];
-        load(r, n, z);
-        norm(r, n, z, false);
-        store_ring(p0 + (r - r_beg), n);
-      } else {
-        store_ring(p0 + (r - r_beg), win[k]);
+      for (int j = 0; j < W; ++j) {
+        const int r = r_end - W + j;
+        if (r < r_beg) continue;             // an older row: it is in the ring already
+        const float4 n = tail ? normed(front + j, CnRow<T>(p, r, r).load(i, p.mult)) : win[j];
+        st4(ring + static_cast<long long>((p0 + (r - r_beg)) % W) * p.H, n);
       }
     }
   }
@@ -235,37 +274,30 @@ __global__ void __launch_bounds__(TAPS > 4 ? 1024 : 512) conv_norm_kernel(const 
 
 template <typename T, int TAPS>
 int launch_cn(ConvNormParams<T>& p, int max_portion, cudaStream_t st) {
-  const int groups = p.H / 4;
-  int threads, per;
-  if (TAPS > 4) {
-    threads = groups <= 1024 ? (groups + 31) / 32 * 32 : 1024;
-    per = (groups + threads - 1) / threads;
-  } else {
-    per = groups <= 128 ? 1 : 2;
-    threads = ((groups + per - 1) / per + 31) / 32 * 32;
+  if (TAPS > 1 && p.n_portions > 0) {
+    // strips that fill the GPU a few times over; with the rows in front of them they make whole rounds of the CTA's warps
+    constexpr int W = TAPS - 1, LEAST = (2 * W + CS_WARPS - 1) / CS_WARPS;   // at least W rows
+    int rounds = (p.portion_rows / (sm_count() * 4) + W) / CS_WARPS;
+    rounds = rounds < LEAST ? LEAST : rounds > 4 ? 4 : rounds;
+    p.strip = rounds * CS_WARPS - W;
+    p.strips = (max_portion + p.strip - 1) / p.strip;
+    launch_k(conv_norm_strip_kernel<T, (TAPS > 1 ? TAPS : 2)>, dim3(p.n_portions * p.strips), dim3(CS_WARPS * 32), 0, st, p);
+  }
+  const int single = TAPS > 1 ? p.rows - p.portion_rows : p.rows;
+  if (single > 0) {
+    const int groups = p.H / 4;
+    int per = groups <= 128 ? 1 : 2, threads = ((groups + per - 1) / per + 31) / 32 * 32;
     if (threads > 512) {
       threads = 512;
       per = (groups + threads - 1) / threads;
     }
+    const dim3 grid(single), block(threads);
+    if (per <= 1) launch_k(conv_norm_row_kernel<T, TAPS, 1>, grid, block, 0, st, p);
+    else if (per <= 2) launch_k(conv_norm_row_kernel<T, TAPS, 2>, grid, block, 0, st, p);
+    else if (per <= 4) launch_k(conv_norm_row_kernel<T, TAPS, 4>, grid, block, 0, st, p);
+    else if (per <= 8) launch_k(conv_norm_row_kernel<T, TAPS, 8>, grid, block, 0, st, p);
+    else return -2;
   }
-  // strips that fill the GPU a few times over, long enough that the rows in front of them weigh little
-  const int most = TAPS > 4 ? 32 : 16;
-  int strip = p.rows / (sm_count() * 4);
-  strip = strip < 1 ? 1 : strip > most ? most : strip;
-  if (strip < TAPS - 1) strip = TAPS - 1;
-  p.strip = strip;
-  int blocks;
-  if (TAPS == 1) {
-    blocks = (p.rows + strip - 1) / strip;
-  } else {
-    p.strips = (max_portion + strip - 1) / strip;
-    blocks = p.n_portions * p.strips + (p.rows - p.portion_rows);
-  }
-  const dim3 grid(blocks), block(threads);
-  if (per <= 1) launch_k(conv_norm_kernel<T, TAPS, 1>, grid, block, 0, st, p);
-  else if (per <= 2) launch_k(conv_norm_kernel<T, TAPS, 2>, grid, block, 0, st, p);
-  else if (per <= 4 && TAPS <= 4) launch_k(conv_norm_kernel<T, TAPS <= 4 ? TAPS : 1, 4>, grid, block, 0, st, p);
-  else return -2;
   return launch_status();
 }
 
@@ -275,11 +307,11 @@ using namespace gk;
 
 // ptrs: {tokens, embed, x, y, x_out, gain, taps, ring, cu, first_pos, states, pick, h}
 // dims: {rows, H, H_true, n_portions, portion_rows, max_portion, n_taps, vocab, center};  n_taps 0: no convolution, else 2, 3, 4,
-// 8 or 16;  H % 4 == 0, H <= 8192.  x_out must not overlap x.  floats: {mult, eps}
+// 8 or 16;  H % 4 == 0, H <= 16384.  x_out must not overlap x.  floats: {mult, eps}
 GK_EXPORT int gk_conv_norm(int is_fp32, void* const* ptrs, const int* dims, const float* floats, void* stream) {
   const int rows = dims[0], H = dims[1], n_taps = dims[6];
   if (rows == 0) return 0;
-  if (rows < 0 || H <= 0 || H % 4 || dims[2] < 1 || dims[2] > H) return -1;
+  if (rows < 0 || H <= 0 || H % 4 || H > 16384 || dims[2] < 1 || dims[2] > H) return -1;
   if (ptrs[1] ? (!ptrs[0] || dims[7] < 1 || ptrs[11]) : !ptrs[2]) return -1;
   if ((ptrs[2] && ptrs[2] == ptrs[4]) || (ptrs[12] && !ptrs[5]) || (!ptrs[12] && !ptrs[4])) return -1;
   if (n_taps && (!ptrs[6] || !ptrs[7] || !ptrs[9] || !ptrs[10] || !ptrs[12] || ptrs[11])) return -1;
@@ -301,7 +333,7 @@ GK_EXPORT int gk_conv_norm(int is_fp32, void* const* ptrs, const int* dims, cons
     p.pick = static_cast<const long long*>(ptrs[11]);
     p.h = static_cast<T*>(ptrs[12]);
     p.rows = rows; p.H = H; p.H_true = dims[2]; p.n_portions = dims[3]; p.portion_rows = dims[4];
-    p.strips = 0; p.strip = 1; p.vocab = dims[7]; p.center = dims[8];
+    p.strips = 1; p.strip = 1; p.vocab = dims[7]; p.center = dims[8];
     p.mult = floats[0]; p.eps = floats[1];
     cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
     switch (n_taps) {

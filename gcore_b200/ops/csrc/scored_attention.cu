@@ -52,57 +52,119 @@ struct HeadPrepParams {
   float eps;
 };
 
-// One CTA per row, a warp per head.
-template <typename T>
+// Eight elements at a time.
+__device__ __forceinline__ void sa_ld8(const float* p, float (&v)[8]) {
+  const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+__device__ __forceinline__ void sa_ld8(const __nv_bfloat16* p, float (&v)[8]) {
+  const uint4 a = *reinterpret_cast<const uint4*>(p);
+  const uint32_t w[4] = {a.x, a.y, a.z, a.w};
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    v[2 * i] = __uint_as_float(w[i] << 16);
+    v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+  }
+}
+__device__ __forceinline__ void sa_st8(float* p, const float (&v)[8]) {
+  *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
+}
+__device__ __forceinline__ void sa_st8(__nv_bfloat16* p, const float (&v)[8]) {
+  *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]),
+                                            pack_bf16x2(v[6], v[7]));
+}
+
+// One CTA per row; GL lanes (a power of two) per head, each with NU times eight neighbouring elements.
+template <typename T, int GL, int NU>
 __global__ void __launch_bounds__(128) head_prep_kernel(const HeadPrepParams<T> p) {
-  __shared__ float s_cos[SA_MAX_ROT / 2], s_sin[SA_MAX_ROT / 2];
+  __shared__ __align__(16) float s_cos[SA_MAX_ROT / 2], s_sin[SA_MAX_ROT / 2];
   pdl_launch_dependents();
   pdl_wait();
-  const int row = blockIdx.x, tid = threadIdx.x, lane = tid & 31, half = p.rot >> 1;
+  const int row = blockIdx.x, tid = threadIdx.x, half = p.rot >> 1;
   T* pr = p.proj + row * p.ld;
   const int slot = p.slots ? p.slots[row] : -1;
   if (half) {
     const int pos = p.pos[row];
     for (int i = tid; i < half; i += 128) rotation_at(pos, p.turns[i], &s_sin[i], &s_cos[i]);
+    __syncthreads();
   }
-  __syncthreads();
   T* dst_row = p.cache ? p.cache + static_cast<long long>(slot < 0 ? 0 : slot) * (p.NK * p.D + p.VC) : nullptr;
-  const int heads = p.NQ + (p.cache && slot < 0 ? 0 : p.NK), pairs = p.D >> 1;
-  for (int h = tid >> 5; h < heads; h += 4) {
+  const int heads = p.NQ + (p.cache && slot < 0 ? 0 : p.NK), gl = tid % GL;
+  for (int h0 = 0; h0 < heads; h0 += 128 / GL) {            // the same number of rounds for every lane
+    const int h = h0 + tid / GL;
     const bool key = h >= p.NQ;
     const int n = key ? h - p.NQ : h;
     T* src = pr + (key ? p.k_off : p.q_off) + static_cast<long long>(n) * p.D;
     T* dst = key && dst_row ? dst_row + n * p.D : src;
-    float f = 1.f;
-    if (p.true_D) {
-      float ss = 0.f;
-      for (int i = lane; i < pairs; i += 32) {
-        float2 v = sa_ld2(src + 2 * i);
-        if (i < half) v = sa_rotate(v, s_cos[i], s_sin[i]);
-        ss = fmaf(v.x, v.x, fmaf(v.y, v.y, ss));
+    float v[NU][8], ss = 0.f;
+#pragma unroll
+    for (int u = 0; u < NU; ++u) {
+      const int d = (u * GL + gl) * 8;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[u][e] = 0.f;
+      if (h < heads && d < p.D) sa_ld8(src + d, v[u]);
+#pragma unroll
+      for (int e = 0; e < 8; e += 2) {
+        if (d + e < p.rot) {
+          const float2 r = sa_rotate(make_float2(v[u][e], v[u][e + 1]), s_cos[(d + e) >> 1], s_sin[(d + e) >> 1]);
+          v[u][e] = r.x;
+          v[u][e + 1] = r.y;
+        }
+        ss = fmaf(v[u][e], v[u][e], fmaf(v[u][e + 1], v[u][e + 1], ss));
       }
-      f = 1.f / sqrtf(sa_warp_sum(ss) / p.true_D + p.eps);
     }
-    for (int i = lane; i < pairs; i += 32) {
-      float2 v = sa_ld2(src + 2 * i);
-      if (i < half) v = sa_rotate(v, s_cos[i], s_sin[i]);
-      sa_st2(dst + 2 * i, make_float2(v.x * f, v.y * f));
+    if (p.true_D) {
+#pragma unroll
+      for (int o = GL / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffff, ss, o);
+      const float f = 1.f / sqrtf(ss / p.true_D + p.eps);
+#pragma unroll
+      for (int u = 0; u < NU; ++u) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[u][e] *= f;
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < NU; ++u) {
+      const int d = (u * GL + gl) * 8;
+      if (h < heads && d < p.D) sa_st8(dst + d, v[u]);
     }
   }
   if (dst_row && slot >= 0)
-    for (int i = tid; i < p.VC >> 1; i += 128) sa_st2(dst_row + p.NK * p.D + 2 * i, sa_ld2(pr + p.v_off + 2 * i));
+    for (int c = tid * 8; c < p.VC; c += 128 * 8) {
+      float v[8];
+      sa_ld8(pr + p.v_off + c, v);
+      sa_st8(dst_row + p.NK * p.D + c, v);
+    }
 }
 
 template <typename T>
-__global__ void __launch_bounds__(256) silu_columns_kernel(T* __restrict__ proj, long long ld, int off, int pairs, int rows) {
+int launch_head_prep(const HeadPrepParams<T>& p, int rows, cudaStream_t st) {
+  const dim3 grid(rows), block(128);
+  if (p.D <= 32) launch_k(head_prep_kernel<T, 4, 1>, grid, block, 0, st, p);
+  else if (p.D <= 64) launch_k(head_prep_kernel<T, 8, 1>, grid, block, 0, st, p);
+  else if (p.D <= 128) launch_k(head_prep_kernel<T, 16, 1>, grid, block, 0, st, p);
+  else if (p.D <= 256) launch_k(head_prep_kernel<T, 32, 1>, grid, block, 0, st, p);
+  else if (p.D <= 1024) launch_k(head_prep_kernel<T, 32, 4>, grid, block, 0, st, p);
+  else return -2;
+  return launch_status();
+}
+
+// Eight columns a thread: x over the columns, rows blockIdx.y, + gridDim.y, ...
+template <typename T>
+__global__ void __launch_bounds__(256) silu_columns_kernel(T* __restrict__ proj, long long ld, int off, int n, int rows) {
   pdl_launch_dependents();
   pdl_wait();
-  const long long n = static_cast<long long>(rows) * pairs;
-  for (long long i = static_cast<long long>(blockIdx.x) * 256 + threadIdx.x; i < n; i += static_cast<long long>(gridDim.x) * 256) {
-    const long long r = i / pairs;
-    T* at = proj + r * ld + off + 2 * (i - r * pairs);
-    const float2 v = sa_ld2(at);
-    sa_st2(at, make_float2(v.x / (1.f + expf(-v.x)), v.y / (1.f + expf(-v.y))));
+  const int c = (blockIdx.x * 256 + threadIdx.x) * 8;
+  if (c >= n) return;
+  for (int r = blockIdx.y; r < rows; r += gridDim.y) {
+    T* at = proj + r * ld + off + c;
+    float v[8];
+    sa_ld8(at, v);
+#pragma unroll
+    for (int e = 0; e < 8; ++e)
+      v[e] = std::is_same<T, float>::value ? v[e] / (1.f + expf(-v[e])) : __fdividef(v[e], 1.f + __expf(-v[e]));
+    sa_st8(at, v);
   }
 }
 
@@ -574,13 +636,14 @@ using namespace gk;
 
 // ptrs: {proj, turns, pos, slots, cache};  turns: with rot;  cache null: keys in place, slots may be null too
 // dims: {rows, q_off, k_off, v_off, NQ, NK, D, VC, rot, true_D}
-// All offsets and sizes are even; cached rows are NK * D + VC elements.  true_D 0: no norm.
+// Offsets, D and VC are multiples of 8, rot is even; cached rows are NK * D + VC elements.  true_D 0: no norm.
 GK_EXPORT int gk_head_prep(int is_fp32, void* const* ptrs, long long ld, const int* dims, float eps, void* stream) {
   if (dims[0] == 0) return 0;
-  for (int i = 1; i < 9; ++i)
-    if (dims[i] < 0 || (i != 4 && i != 5 && dims[i] % 2)) return -1;
-  if (ld % 2 || dims[8] > dims[6] || dims[8] > SA_MAX_ROT || dims[9] < 0 || dims[9] > dims[6]) return -1;
+  for (int i = 0; i < 10; ++i)
+    if (dims[i] < 0 || ((i == 1 || i == 2 || i == 3 || i == 6 || i == 7) && dims[i] % 8)) return -1;
+  if (ld % 8 || dims[8] % 2 || dims[8] > dims[6] || dims[8] > SA_MAX_ROT || dims[9] > dims[6] || dims[6] < 8) return -1;
   if ((dims[8] && (!ptrs[1] || !ptrs[2])) || (ptrs[4] && !ptrs[3])) return -1;
+  if ((reinterpret_cast<uintptr_t>(ptrs[0]) | reinterpret_cast<uintptr_t>(ptrs[4])) & 15) return -1;
   auto fill = [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
     HeadPrepParams<T> p;
@@ -590,23 +653,22 @@ GK_EXPORT int gk_head_prep(int is_fp32, void* const* ptrs, long long ld, const i
     p.cache = static_cast<T*>(ptrs[4]);
     p.q_off = dims[1]; p.k_off = dims[2]; p.v_off = dims[3]; p.NQ = dims[4]; p.NK = dims[5]; p.D = dims[6]; p.VC = dims[7];
     p.rot = dims[8]; p.true_D = dims[9]; p.eps = eps;
-    launch_k(head_prep_kernel<T>, dim3(dims[0]), dim3(128), 0, reinterpret_cast<cudaStream_t>(stream), p);
-    return launch_status();
+    return launch_head_prep(p, dims[0], reinterpret_cast<cudaStream_t>(stream));
   };
   return is_fp32 ? fill(static_cast<float*>(nullptr)) : fill(static_cast<__nv_bfloat16*>(nullptr));
 }
 
-// Columns off .. off + n (both even) of `rows` rows become their silu.
+// Columns off .. off + n (multiples of 8) of `rows` rows become their silu.
 GK_EXPORT int gk_silu_columns(int is_fp32, void* proj, long long ld, int off, int n, int rows, void* stream) {
   if (rows == 0 || n == 0) return 0;
-  if (rows < 0 || n < 0 || n % 2 || off < 0 || off % 2 || ld % 2 || off + static_cast<long long>(n) > ld) return -1;
-  const long long pairs = static_cast<long long>(rows) * (n / 2);
-  long long blocks = (pairs + 255) / 256;
-  if (blocks > sm_count() * 16) blocks = sm_count() * 16;
-  const dim3 grid(static_cast<unsigned>(blocks)), block(256);
+  if (rows < 0 || n < 0 || n % 8 || off < 0 || off % 8 || ld % 8 || (reinterpret_cast<uintptr_t>(proj) & 15)) return -1;
+  const int x = (n / 8 + 255) / 256;
+  int y = sm_count() * 16 / x;
+  y = y < 1 ? 1 : y > rows ? rows : y;
+  const dim3 grid(x, y), block(256);
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
-  if (is_fp32) launch_k(silu_columns_kernel<float>, grid, block, 0, st, static_cast<float*>(proj), ld, off, n / 2, rows);
-  else launch_k(silu_columns_kernel<__nv_bfloat16>, grid, block, 0, st, static_cast<__nv_bfloat16*>(proj), ld, off, n / 2, rows);
+  if (is_fp32) launch_k(silu_columns_kernel<float>, grid, block, 0, st, static_cast<float*>(proj), ld, off, n, rows);
+  else launch_k(silu_columns_kernel<__nv_bfloat16>, grid, block, 0, st, static_cast<__nv_bfloat16*>(proj), ld, off, n, rows);
   return launch_status();
 }
 

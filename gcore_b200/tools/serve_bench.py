@@ -3,8 +3,9 @@
 For a few real-model layer sizes (random weights) it times, on the device, a prefill step and a captured decode step of an
 engine of the design and of the closest uniform model - for Nafitar a dense grouped-query decoder with the same width,
 heads, window, feed-forward and layer count, for Kedesun and Lobutar a latent-attention decoder with experts
-(``serve_bench_kedesun.py``, ``serve_bench_lobutar.py``) - and then every kernel the design added beside the like kernel of that model: time, the time its bytes or FLOPs would take
-at the measured peaks, and the ratio of the two.  Inputs of every timed launch rotate over buffers larger than L2."""
+(``serve_bench_kedesun.py``, ``serve_bench_lobutar.py``), for Rezulorn both Nafitar and a dense decoder
+(``serve_bench_rezulorn.py``) - and then every kernel the design added beside the like kernel of that model: time, the time its
+bytes or FLOPs would take at the measured peaks, and the ratio of the two.  Inputs of every timed launch rotate over buffers larger than L2."""
 from __future__ import annotations
 
 import json
@@ -56,16 +57,17 @@ def dense_config(s):
 
 
 def build(kind, s, positions, requests, block=64):
-    """Engine of a layer-plan design (``nafitar``, ``kedesun``, ``lobutar``) or of the uniform model it is compared with
-    (``dense``, ``latent``: Kedesun's, ``grouped``: Lobutar's)."""
-    from . import serve_bench_kedesun as sk, serve_bench_lobutar as sl
+    """Engine of a layer-plan design (``nafitar``, ``kedesun``, ``lobutar``, ``rezulorn``) or of the uniform model it is compared
+    with (``dense``, ``latent``: Kedesun's, ``grouped``: Lobutar's, ``mixed``: Rezulorn's dense one)."""
+    from . import serve_bench_kedesun as sk, serve_bench_lobutar as sl, serve_bench_rezulorn as sr
     dev = torch.device("cuda")
-    plans = {"nafitar": lambda: nafitar_conf(s, positions), "kedesun": lambda: sk.conf(s), "lobutar": lambda: sl.conf(s)}
+    plans = {"nafitar": lambda: nafitar_conf(sr.like_sizes(s) if "nff" in s else s, positions), "kedesun": lambda: sk.conf(s),
+             "lobutar": lambda: sl.conf(s), "rezulorn": lambda: sr.conf(s)}
     if kind in plans:
         cfg = from_hf_config(plans[kind]())
         model = build_decoder(cfg, dev).randomize()
     else:
-        cfg = {"dense": dense_config, "latent": sk.latent_config, "grouped": sl.latent_config}[kind](s)
+        cfg = {"dense": dense_config, "latent": sk.latent_config, "grouped": sl.latent_config, "mixed": sr.dense_config}[kind](s)
         model = GPTModel(cfg, recompute="none", device=dev)
     eng = InferEngine(cfg, RolloutWeights.from_model(model), max_running_requests=requests, max_model_len=positions,
                       kv_block_size=block, max_prefill_tokens=1 << 20, device=dev)
@@ -266,14 +268,16 @@ def kernel_table(s, prompts, length, B, ctx, bs=64):
 
 
 def _families():
-    from . import serve_bench_kedesun as sk, serve_bench_lobutar as sl
+    from . import serve_bench_kedesun as sk, serve_bench_lobutar as sl, serve_bench_rezulorn as sr
     active = lambda eng, s, n: n - 2 * VOCAB * s["width"]
     return {"nafitar": dict(like="dense", sizes=SIZES, active=active, table=kernel_table,
                             decode_bytes=lambda kind, s, eng, B, ctx: decode_bytes(kind, s, eng, B, ctx)),
             "kedesun": dict(like="latent", sizes=sk.SIZES, active=sk.active_weights, table=sk.kernel_table,
                             decode_bytes=sk.decode_bytes),
             "lobutar": dict(like="grouped", sizes=sl.SIZES, active=sl.active_weights, table=sl.kernel_table,
-                            decode_bytes=sl.decode_bytes)}
+                            decode_bytes=sl.decode_bytes),
+            "rezulorn": dict(like=("nafitar", "mixed"), sizes=sr.SIZES, active=sr.active_weights, table=sr.kernel_table,
+                             decode_bytes=sr.decode_bytes)}
 
 
 def run(sizes=None, iters=10, design="nafitar"):
@@ -285,7 +289,7 @@ def run(sizes=None, iters=10, design="nafitar"):
     for name in sizes or fam["sizes"]:
         s = fam["sizes"][name]
         rec = {"layer": s, "prefill": {}, "decode": {}}
-        for kind in (design, fam["like"]):
+        for kind in (design, *((fam["like"],) if isinstance(fam["like"], str) else fam["like"])):
             eng = build(kind, s, ctx + 256, 64)
             n_params = sum(t.numel() for t in eng.w.tensors())
             ms = prefill_step(eng, prompts, length, max(3, iters // 2))

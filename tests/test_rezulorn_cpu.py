@@ -70,7 +70,7 @@ def test_specs_refuse_what_no_kernel_computes():
     with pytest.raises(ValueError, match="taps"):
         build_decoder(from_hf_config(ru.uneven_conf(taps=17)))
     with pytest.raises(ValueError, match="width"):
-        build_decoder(from_hf_config(ru.conf([ru.lightning(1, 8, 8, [0.5], None)], 9000, 4)))
+        build_decoder(from_hf_config(ru.conf([ru.lightning(1, 8, 8, [0.5], None)], 17000, 4)))
 
 
 def test_halves_become_neighbours():
