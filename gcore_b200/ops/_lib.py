@@ -244,6 +244,7 @@ def _declare_kernels(lib: ctypes.CDLL):
     d("gk_diff_set_target_ctas", [I], None)
     d("gk_diff_combine", [I, I, P, L, L, P, P, P])
     d("gk_conv_norm", [I, P, P, P, P])
+    d("gk_conv_norm_set_rounds", [I], None)
     d("gk_head_prep", [I, P, L, P, F, P])
     d("gk_silu_columns", [I, P, L, I, I, I, P])
     d("gk_scored_prefill", [P, P, P, P, P])

@@ -101,16 +101,34 @@ __global__ void __launch_bounds__(512) conv_norm_row_kernel(const ConvNormParams
   const CnRow<T> src(p, row, TAPS == 1 && p.pick ? p.pick[row] : row);
   const int seg = p.n_portions + blockIdx.x;
   const int pos = TAPS > 1 ? p.first_pos[seg] : 0, slot = TAPS > 1 ? p.states[seg] : -1;
-  float4 x[NV];
+  float4 x[NV], past[TAPS > 1 ? NV : 1];       // past: the earlier rows' part of the convolution
   float s = 0.f;
 #pragma unroll
   for (int v = 0; v < NV; ++v) {
     const int i = tid + v * blockDim.x;
     x[v] = i < nv ? src.load(i, p.mult) : make_float4(0.f, 0.f, 0.f, 0.f);
+    if (TAPS > 1) past[TAPS > 1 ? v : 0] = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int j = 0; j < W; ++j) {
+      const int q = pos - W + j;
+      if (q >= 0 && slot >= 0 && i < nv)
+        cn_add(past[TAPS > 1 ? v : 0], ld4(p.taps + static_cast<long long>(j) * p.H + i * 4),
+               ld4(p.ring + (static_cast<long long>(slot) * W + q % (W > 0 ? W : 1)) * p.H + i * 4));
+    }
+  }
+#pragma unroll
+  for (int v = 0; v < NV; ++v) {
+    const int i = tid + v * blockDim.x;
     if (p.x_out && i < nv) st4(p.x_out + row * p.H + i * 4, x[v]);
     s += (x[v].x + x[v].y) + (x[v].z + x[v].w);      // columns past H_true are zero
   }
   if (!p.h) return;
+  float4 gain[NV];
+#pragma unroll
+  for (int v = 0; v < NV; ++v) {
+    const int i = tid + v * blockDim.x;
+    gain[v] = i < nv ? ld4(p.gain + i * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
   if (p.center) {
     const float mean = cn_sum(s, red, 0) / p.H_true;
 #pragma unroll
@@ -124,25 +142,20 @@ __global__ void __launch_bounds__(512) conv_norm_row_kernel(const ConvNormParams
   for (int v = 0; v < NV; ++v) {
     const int i = tid + v * blockDim.x;
     if (i >= nv) continue;
-    const float4 n = cn_scaled(x[v], f, ld4(p.gain + i * 4));
+    const float4 n = cn_scaled(x[v], f, gain[v]);
     float4 o = n;
     if (TAPS > 1) {
-      o = make_float4(0.f, 0.f, 0.f, 0.f);
-      float* ring = p.ring + static_cast<long long>(slot < 0 ? 0 : slot) * W * p.H + i * 4;
-#pragma unroll
-      for (int j = 0; j < W; ++j) {
-        const int q = pos - W + j;
-        if (q >= 0 && slot >= 0)
-          cn_add(o, ld4(p.taps + static_cast<long long>(j) * p.H + i * 4), ld4(ring + static_cast<long long>(q % (W > 0 ? W : 1)) * p.H));
-      }
+      o = past[TAPS > 1 ? v : 0];
       cn_add(o, ld4(p.taps + static_cast<long long>(W) * p.H + i * 4), n);
-      if (slot >= 0) st4(ring + static_cast<long long>(pos % (W > 0 ? W : 1)) * p.H, n);
+      if (slot >= 0) st4(p.ring + (static_cast<long long>(slot) * W + pos % (W > 0 ? W : 1)) * p.H + i * 4, n);
     }
     st4(p.h + row * p.H + i * 4, o);
   }
 }
 
 constexpr int CS_WARPS = 8;
+constexpr int CS_CTAS = 4;                   // resident per SM (up to four taps)
+constexpr int CS_AHEAD = 2;                  // rows a thread reads ahead
 constexpr int CS_GROUPS = 4;                 // float4 groups a lane takes at a time
 constexpr int CS_MAX_ROWS = CS_WARPS * 4;    // rows of a strip and in front of it
 
@@ -161,7 +174,7 @@ struct CnMoments {
 
 // grid: portions x strips.
 template <typename T, int TAPS>
-__global__ void __launch_bounds__(CS_WARPS * 32, TAPS <= 4 ? 3 : 2) conv_norm_strip_kernel(const ConvNormParams<T> p) {
+__global__ void __launch_bounds__(CS_WARPS * 32, TAPS <= 4 ? CS_CTAS : 2) conv_norm_strip_kernel(const ConvNormParams<T> p) {
   constexpr int W = TAPS - 1;
   __shared__ float s_mean[CS_MAX_ROWS + W], s_rstd[CS_MAX_ROWS + W];   // rows lo - W .. hi - 1, then the portion's last W rows
   pdl_launch_dependents();
@@ -230,23 +243,22 @@ __global__ void __launch_bounds__(CS_WARPS * 32, TAPS <= 4 ? 3 : 2) conv_norm_st
       if (r >= r_beg) win[j] = normed(j, CnRow<T>(p, r, r).load(i, p.mult));
       else if (q >= 0 && slot >= 0) win[j] = ld4(ring + static_cast<long long>(q % W) * p.H);
     }
-    constexpr int AHEAD = 4;
-    float4 nx[AHEAD];
+    float4 nx[CS_AHEAD];
     auto fetch = [&](int r) {
       if (r >= hi) return make_float4(0.f, 0.f, 0.f, 0.f);
       return p.x_out ? ld4(p.x_out + static_cast<long long>(r) * p.H + i * 4) : CnRow<T>(p, r, r).load(i, p.mult);
     };
 #pragma unroll
-    for (int a = 0; a < AHEAD; ++a) nx[a] = fetch(lo + a);
-    for (int r0 = lo; r0 < hi; r0 += AHEAD) {
-      float4 cur[AHEAD];
+    for (int a = 0; a < CS_AHEAD; ++a) nx[a] = fetch(lo + a);
+    for (int r0 = lo; r0 < hi; r0 += CS_AHEAD) {
+      float4 cur[CS_AHEAD];
 #pragma unroll
-      for (int a = 0; a < AHEAD; ++a) {
+      for (int a = 0; a < CS_AHEAD; ++a) {
         cur[a] = nx[a];
-        nx[a] = fetch(r0 + AHEAD + a);       // on their way while these rows are worked on
+        nx[a] = fetch(r0 + CS_AHEAD + a);       // on their way while these rows are worked on
       }
 #pragma unroll
-      for (int a = 0; a < AHEAD; ++a) {
+      for (int a = 0; a < CS_AHEAD; ++a) {
         const int r = r0 + a;
         if (r >= hi) break;
         const float4 n = normed(r - lo + W, cur[a]);
@@ -272,13 +284,26 @@ __global__ void __launch_bounds__(CS_WARPS * 32, TAPS <= 4 ? 3 : 2) conv_norm_st
   }
 }
 
+inline int& conv_norm_rounds() {           // > 0: fixed
+  static int n = 0;
+  return n;
+}
+
 template <typename T, int TAPS>
 int launch_cn(ConvNormParams<T>& p, int max_portion, cudaStream_t st) {
   if (TAPS > 1 && p.n_portions > 0) {
-    // strips that fill the GPU a few times over; with the rows in front of them they make whole rounds of the CTA's warps
-    constexpr int W = TAPS - 1, LEAST = (2 * W + CS_WARPS - 1) / CS_WARPS;   // at least W rows
-    int rounds = (p.portion_rows / (sm_count() * 4) + W) / CS_WARPS;
-    rounds = rounds < LEAST ? LEAST : rounds > 4 ? 4 : rounds;
+    // with the rows in front of them, strips make whole rounds of the CTA's warps; the length with the fewest rounds over all
+    // waves, one more counted per CTA, and at least W rows
+    constexpr int W = TAPS - 1, LEAST = (2 * W + CS_WARPS - 1) / CS_WARPS;
+    const long long slots = static_cast<long long>(sm_count()) * (TAPS <= 4 ? CS_CTAS : 2);
+    int rounds = LEAST;
+    long long best = 1LL << 60;
+    for (int n = LEAST; n <= 4; ++n) {
+      const int strip = n * CS_WARPS - W;
+      const long long ctas = (p.portion_rows + strip - 1) / strip, cost = (ctas + slots - 1) / slots * (n + 1);
+      if (cost < best) { best = cost; rounds = n; }
+    }
+    if (conv_norm_rounds() >= LEAST) rounds = conv_norm_rounds();
     p.strip = rounds * CS_WARPS - W;
     p.strips = (max_portion + p.strip - 1) / p.strip;
     launch_k(conv_norm_strip_kernel<T, (TAPS > 1 ? TAPS : 2)>, dim3(p.n_portions * p.strips), dim3(CS_WARPS * 32), 0, st, p);
@@ -304,6 +329,8 @@ int launch_cn(ConvNormParams<T>& p, int max_portion, cudaStream_t st) {
 }  // namespace gk
 
 using namespace gk;
+
+GK_EXPORT void gk_conv_norm_set_rounds(int n) { conv_norm_rounds() = n >= 1 && n <= 4 ? n : 0; }
 
 // ptrs: {tokens, embed, x, y, x_out, gain, taps, ring, cu, first_pos, states, pick, h}
 // dims: {rows, H, H_true, n_portions, portion_rows, max_portion, n_taps, vocab, center};  n_taps 0: no convolution, else 2, 3, 4,

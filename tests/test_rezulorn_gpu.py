@@ -343,6 +343,23 @@ def test_convolved_norm_alone(width, pad, taps, dtype):
     assert (bare[:, :width].double().cpu() - oracle.rms(x0.double() + mult * y.double(), eps) * gain).abs().max() < tol
 
 
+def test_strips_of_every_length_agree():
+    """However a long portion is cut, neighbouring strips see the same rows; lengths around the strips' edges."""
+    torch.manual_seed(6)
+    lib, H = _lib.kernels(), 256
+    for stored in (2, 3, 4):
+        segs = [(3, n) for n in (1200, 29, 30, 5, 6, 13, 2)]
+        T = sum(l for _, l in segs)
+        rows = ru.make_rows(segs, 16, 200, 8)
+        x, y, gain, taps = (torch.randn(*s, device="cuda") for s in ((T, H), (T, H), (H,), (stored, H)))
+        start, outs = torch.randn(8, stored - 1, H, device="cuda"), []
+        for n in (1, 2, 3, 4, 0):
+            lib.gk_conv_norm_set_rounds(n)
+            ring = start.clone()
+            outs.append((*cn.conv_add_sublayer(x, y, 0.7, cn.NormSpec(H, 1e-5), gain, rows, taps, ring), ring))
+        assert all(torch.equal(a, b) for o in outs[1:] for a, b in zip(o, outs[0]))
+
+
 # ---------------------------------------------------------------------------------------------------- engine
 @DTYPES
 @pytest.mark.parametrize("which", ["uneven", "round"])
