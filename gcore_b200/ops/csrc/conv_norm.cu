@@ -92,28 +92,42 @@ __device__ __forceinline__ float cn_sum(float a, float (*red)[32], int turn) {
 // convolution.
 template <typename T, int TAPS, int NV>
 __global__ void __launch_bounds__(512) conv_norm_row_kernel(const ConvNormParams<T> p) {
-  constexpr int W = TAPS - 1;
+  constexpr int W = TAPS - 1, HELD = TAPS > 1 && TAPS <= 4 ? TAPS : 1;
   __shared__ float red[2][32];
+  const int tid = threadIdx.x, nv = p.H >> 2;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  // gain and taps are weights: no earlier kernel of the step writes them
+  float4 gain[NV], taps[HELD][NV];
+#pragma unroll
+  for (int v = 0; v < NV; ++v) {
+    const int i = tid + v * blockDim.x;
+    gain[v] = p.gain && i < nv ? ld4(p.gain + i * 4) : zero;
+#pragma unroll
+    for (int j = 0; j < HELD; ++j)
+      taps[j][v] = TAPS > 1 && TAPS <= 4 && i < nv ? ld4(p.taps + static_cast<long long>(j) * p.H + i * 4) : zero;
+  }
+  auto tap = [&](int j, int v, int i) {
+    return TAPS <= 4 ? taps[j < HELD ? j : 0][v] : ld4(p.taps + static_cast<long long>(j) * p.H + i * 4);
+  };
   pdl_launch_dependents();
   pdl_wait();
-  const int tid = threadIdx.x, nv = p.H >> 2;
   const long long row = (TAPS > 1 ? p.portion_rows : 0) + static_cast<long long>(blockIdx.x);
   const CnRow<T> src(p, row, TAPS == 1 && p.pick ? p.pick[row] : row);
   const int seg = p.n_portions + blockIdx.x;
   const int pos = TAPS > 1 ? p.first_pos[seg] : 0, slot = TAPS > 1 ? p.states[seg] : -1;
-  float4 x[NV], past[TAPS > 1 ? NV : 1];       // past: the earlier rows' part of the convolution
+  float* ring = TAPS > 1 ? p.ring + static_cast<long long>(slot < 0 ? 0 : slot) * W * p.H : nullptr;
+  float4 x[NV], past[NV];       // past: the earlier rows' part of the convolution
   float s = 0.f;
 #pragma unroll
   for (int v = 0; v < NV; ++v) {
     const int i = tid + v * blockDim.x;
-    x[v] = i < nv ? src.load(i, p.mult) : make_float4(0.f, 0.f, 0.f, 0.f);
-    if (TAPS > 1) past[TAPS > 1 ? v : 0] = make_float4(0.f, 0.f, 0.f, 0.f);
+    x[v] = i < nv ? src.load(i, p.mult) : zero;
+    past[v] = zero;
 #pragma unroll
     for (int j = 0; j < W; ++j) {
       const int q = pos - W + j;
-      if (q >= 0 && slot >= 0 && i < nv)
-        cn_add(past[TAPS > 1 ? v : 0], ld4(p.taps + static_cast<long long>(j) * p.H + i * 4),
-               ld4(p.ring + (static_cast<long long>(slot) * W + q % (W > 0 ? W : 1)) * p.H + i * 4));
+      const float4 n = i < nv ? ld4(ring + static_cast<long long>((q < 0 ? 0 : q) % (W > 0 ? W : 1)) * p.H + i * 4) : zero;
+      cn_add(past[v], tap(j, v, i < nv ? i : 0), q >= 0 && slot >= 0 ? n : zero);
     }
   }
 #pragma unroll
@@ -123,12 +137,6 @@ __global__ void __launch_bounds__(512) conv_norm_row_kernel(const ConvNormParams
     s += (x[v].x + x[v].y) + (x[v].z + x[v].w);      // columns past H_true are zero
   }
   if (!p.h) return;
-  float4 gain[NV];
-#pragma unroll
-  for (int v = 0; v < NV; ++v) {
-    const int i = tid + v * blockDim.x;
-    gain[v] = i < nv ? ld4(p.gain + i * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
-  }
   if (p.center) {
     const float mean = cn_sum(s, red, 0) / p.H_true;
 #pragma unroll
@@ -145,9 +153,9 @@ __global__ void __launch_bounds__(512) conv_norm_row_kernel(const ConvNormParams
     const float4 n = cn_scaled(x[v], f, gain[v]);
     float4 o = n;
     if (TAPS > 1) {
-      o = past[TAPS > 1 ? v : 0];
-      cn_add(o, ld4(p.taps + static_cast<long long>(W) * p.H + i * 4), n);
-      if (slot >= 0) st4(p.ring + (static_cast<long long>(slot) * W + pos % (W > 0 ? W : 1)) * p.H + i * 4, n);
+      o = past[v];
+      cn_add(o, tap(W, v, i), n);
+      if (slot >= 0) st4(ring + static_cast<long long>(pos % (W > 0 ? W : 1)) * p.H + i * 4, n);
     }
     st4(p.h + row * p.H + i * 4, o);
   }
